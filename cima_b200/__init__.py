@@ -14,7 +14,8 @@ from __future__ import annotations
 
 from typing import List, Optional, Sequence, Union
 
-from .config import (ArchitectureEntry, ConfigError, GisiraxConfig, LipizenConfig, NetezenConfig, Qwen2Config, VunovikConfig, lookup_architecture, read_config_json,
+from .config import (ArchitectureEntry, ConfigError, GisiraxConfig, LipizenConfig, NetezenConfig, PelatarConfig, Qwen2Config, VunovikConfig,
+                     lookup_architecture, read_config_json,
                      register_architecture, registered_architectures)
 from .sampling import GenOptions, OptionError
 
@@ -30,6 +31,9 @@ register_architecture(ArchitectureEntry(name=LipizenConfig.ARCHITECTURE, model_t
 register_architecture(ArchitectureEntry(name=NetezenConfig.ARCHITECTURE, model_type="netezen",
                                         parse=NetezenConfig.from_dict, spec=NetezenConfig.model_spec,
                                         parse_with_shapes=NetezenConfig.from_dict))
+register_architecture(ArchitectureEntry(name=PelatarConfig.ARCHITECTURE, model_type="pelatar",
+                                        parse=PelatarConfig.from_dict, spec=PelatarConfig.model_spec,
+                                        parse_with_shapes=PelatarConfig.from_dict))
 
 __version__ = "0.1.0"
 

@@ -6,8 +6,9 @@ from .vunovik import VunovikConfig
 from .gisirax import GisiraxConfig
 from .lipizen import LipizenConfig
 from .netezen import NetezenConfig
+from .pelatar import PelatarConfig
 from . import shapes
 
 __all__ = ["BlockSpec", "FeedForwardSpec", "MixerSpec", "ModelSpec", "NormSpec", "PositionSpec",
            "ArchitectureEntry", "UnknownArchitecture", "lookup_architecture", "read_config_json",
-           "register_architecture", "registered_architectures", "ConfigError", "Qwen2Config", "VunovikConfig", "GisiraxConfig", "LipizenConfig", "NetezenConfig", "ShortConvSpec", "BigramSpec"]
+           "register_architecture", "registered_architectures", "ConfigError", "Qwen2Config", "VunovikConfig", "GisiraxConfig", "LipizenConfig", "NetezenConfig", "PelatarConfig", "ShortConvSpec", "BigramSpec"]

@@ -94,6 +94,7 @@ class BlockSpec:
                                  # "parallel": h = norm(x); x += mixer(conv(h)) + ffn(h)
                                  # "sandwich": x += m * post(mixer(norm(x))); x += m * post(ffn(norm(x)))
                                  # "postnorm": x = norm(a x + mixer(x)); x = norm(a x + ffn(x)), a = stream_mult
+                                 # "branchnorm": x += norm(mixer(x)); x += norm(ffn(x)), the sublayers read x itself
                                  # "hyper": ``streams`` copies X_s of the stream; a sublayer reads norm(sum_s in[s] X_s) and
                                  #          X_t <- sum_s mix[s, t] X_s + m out[t] y for all t at once, m = residual_mult
     mixer: MixerSpec

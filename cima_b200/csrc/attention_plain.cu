@@ -10,6 +10,8 @@
 // one value head (1: a value head for every key head): value head = key head / v_group, and a row of the step holds
 // nkv / v_group value heads behind its key heads.
 // A head's softmax may hold one more entry without a value: `sink` entries of score 0, or exp(head_sink[h]).
+// `gate_col` > 0: the row's own buffer holds a gate value for every value of the result from that column on (heads of hd
+// values like the queries'); the result leaves times the gate's sigmoid.
 // A row's result depends only on its own sequence: same bits alone or in any batch.
 #include "common.cuh"
 
@@ -19,7 +21,7 @@ k_attention_plain(const TA* __restrict__ qkv, int ld, const TA* __restrict__ cac
                   const int* __restrict__ row_pos, const int* __restrict__ row_seq,
                   const int* __restrict__ seq_slot, const int* __restrict__ seq_first_row,
                   TA* __restrict__ out, int ldo, int T, int nh, int nkv, int hd, float scale, int window, float sink, int keep_first, int v_group,
-                  const float* __restrict__ head_sink) {
+                  const float* __restrict__ head_sink, int gate_col) {
   cima_pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int row = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -81,7 +83,10 @@ k_attention_plain(const TA* __restrict__ qkv, int ld, const TA* __restrict__ cac
 #pragma unroll
   for (int i = 0; i < NI; i++) {
     const int d = lane + 32 * i;
-    if (d < hd) op[d] = cima_from_f32<TA>(acc[i] * inv);
+    if (d < hd) {
+      const float gate = gate_col > 0 ? cima_sigmoid(cima_to_f32<TA>(qkv[(size_t)row * ld + gate_col + (size_t)h * hd + d])) : 1.0f;
+      op[d] = cima_from_f32<TA>(acc[i] * inv * gate);
+    }
   }
 }
 
@@ -91,7 +96,7 @@ extern "C" int cima_attention_plain(const void* qkv, int dtype, int ld, const vo
                                     const int* row_seq, const int* seq_slot, const int* seq_first_row, void* out,
                                     int ldo, int T, int nh, int nkv, int hd, float scale, int window,
                                     int from_cache, int planes, float sink, int keep_first, int v_group, const float* head_sink,
-                                    cudaStream_t stream) {
+                                    int gate_col, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (hd <= 0 || hd > 1024) return cima_fail(CIMA_E_SIZE, "attention_plain: head_dim %d is outside 1..1024", hd);
   if (planes != 1 && planes != 2) return cima_fail(CIMA_E_ARG, "attention_plain: %d planes; pages hold keys | values (2) or one shared vector (1)", planes);
@@ -99,11 +104,12 @@ extern "C" int cima_attention_plain(const void* qkv, int dtype, int ld, const vo
   if (nh > 65535) return cima_fail(CIMA_E_SIZE, "attention_plain: %d heads exceed one launch", nh);
   if (keep_first < 0 || v_group < 1 || nkv % v_group) return cima_fail(CIMA_E_ARG, "attention_plain: keep_first %d must not be negative and %d kv heads be a multiple of v_group %d", keep_first, nkv, v_group);
   if (from_cache && (!cache || !table)) return cima_fail(CIMA_E_ARG, "attention_plain: decoding needs the cache and its block table");
+  if (gate_col < 0 || (gate_col > 0 && gate_col + nh * hd > ld)) return cima_fail(CIMA_E_ARG, "attention_plain: %d gate values from column %d on exceed the rows of %d", nh * hd, gate_col, ld);
   CimaPaged pg{table, table_width, ring, page_size, nkv, hd, planes};
   dim3 grid((T + 3) / 4, nh);
 #define LAUNCH(TA, FC) { int rc_ = hd <= 256 ? LAUNCH_NI(TA, FC, 8) : LAUNCH_NI(TA, FC, 32); if (rc_) return rc_; }
 #define LAUNCH_NI(TA, FC, NI) cima_launch(k_attention_plain<TA, FC, NI>, dim3(grid), dim3(128), (size_t)(0), stream, 1, (const TA*)qkv, ld, (const TA*)cache, pg, \
-    row_pos, row_seq, seq_slot, seq_first_row, (TA*)out, ldo, T, nh, nkv, hd, scale, window, sink, keep_first, v_group, head_sink)
+    row_pos, row_seq, seq_slot, seq_first_row, (TA*)out, ldo, T, nh, nkv, hd, scale, window, sink, keep_first, v_group, head_sink, gate_col)
   if (dtype == CIMA_F32) { if (from_cache) LAUNCH(float, true) else LAUNCH(float, false) }
   else if (dtype == CIMA_BF16) { if (from_cache) LAUNCH(__nv_bfloat16, true) else LAUNCH(__nv_bfloat16, false) }
   else return cima_fail(CIMA_E_DTYPE, "attention_plain: dtype code %d is neither float32 nor bfloat16", dtype);

@@ -66,7 +66,7 @@ k_attention_prefill(const __nv_bfloat16* __restrict__ qkv, int ld, const int* __
                     const __nv_bfloat16* __restrict__ cache, CimaPaged pg, const int* __restrict__ seq_slot,
                     const int* __restrict__ seq_len,
                     __nv_bfloat16* __restrict__ out, int ldo, int T, int nh, int nkv, float scale, int window, float sink, int keep_first, int v_group,
-                    const float* __restrict__ head_sink) {
+                    const float* __restrict__ head_sink, int gate_col) {
   cima_pdl_wait();
   constexpr int ROW = HD + 8;
   constexpr int TILE = BN * ROW;
@@ -276,10 +276,22 @@ k_attention_prefill(const __nv_bfloat16* __restrict__ qkv, int ld, const int* __
 #pragma unroll
   for (int j = 0; j < NTILES; j++) {
     const int d = j * 8 + 2 * t;
+    float g[4] = {1.f, 1.f, 1.f, 1.f};
+    if (gate_col > 0) {                                   // the rows' own gates: the result leaves times their sigmoid
+      const __nv_bfloat16* gp = qkv + (size_t)first * ld + gate_col + (size_t)h * HD + d;
+      if (r0 < len) {
+        const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gp + (size_t)r0 * ld));
+        g[0] = cima_sigmoid(v.x); g[1] = cima_sigmoid(v.y);
+      }
+      if (r1 < len) {
+        const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gp + (size_t)r1 * ld));
+        g[2] = cima_sigmoid(v.x); g[3] = cima_sigmoid(v.y);
+      }
+    }
     if (r0 < len)
-      *reinterpret_cast<uint32_t*>(out + (size_t)(first + r0) * ldo + (size_t)h * HD + d) = pack_bf16(o[j][0] * inv0, o[j][1] * inv0);
+      *reinterpret_cast<uint32_t*>(out + (size_t)(first + r0) * ldo + (size_t)h * HD + d) = pack_bf16(o[j][0] * inv0 * g[0], o[j][1] * inv0 * g[1]);
     if (r1 < len)
-      *reinterpret_cast<uint32_t*>(out + (size_t)(first + r1) * ldo + (size_t)h * HD + d) = pack_bf16(o[j][2] * inv1, o[j][3] * inv1);
+      *reinterpret_cast<uint32_t*>(out + (size_t)(first + r1) * ldo + (size_t)h * HD + d) = pack_bf16(o[j][2] * inv1 * g[2], o[j][3] * inv1 * g[3]);
   }
 }
 
@@ -287,7 +299,7 @@ template <int HD, bool FROM_CACHE>
 int launch_prefill(const void* qkv, int ld, const int* tile_seq, const int* tile_row0, const int* seq_first_row,
                    const void* cache, const CimaPaged& pg, const int* seq_slot, const int* seq_len,
                    void* out, int ldo, int T, int n_tiles, int nh, int nkv, float scale, int window, float sink, int keep_first, int v_group,
-                   const float* head_sink, cudaStream_t stream) {
+                   const float* head_sink, int gate_col, cudaStream_t stream) {
   if ((long long)n_tiles * nh > 0x7fffffffll) return cima_fail(CIMA_E_SIZE, "attention_prefill: %d blocks of rows x %d heads exceed one launch", n_tiles, nh);
   auto kern = k_attention_prefill<HD, FROM_CACHE>;
   const size_t smem = (size_t)2 * 2 * BN * (HD + 8) * sizeof(__nv_bfloat16);
@@ -299,14 +311,15 @@ int launch_prefill(const void* qkv, int ld, const int* tile_seq, const int* tile
   }
   { int rc_ = cima_launch(kern, dim3((unsigned)n_tiles * (unsigned)nh), dim3(WARPS * 32), (size_t)(smem), stream, 1, (const __nv_bfloat16*)qkv, ld, tile_seq, tile_row0, seq_first_row,
                                                         (const __nv_bfloat16*)cache, pg, seq_slot, seq_len,
-                                                        (__nv_bfloat16*)out, ldo, T, nh, nkv, scale, window, sink, keep_first, v_group, head_sink); if (rc_) return rc_; }
+                                                        (__nv_bfloat16*)out, ldo, T, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, gate_col); if (rc_) return rc_; }
   return cima_launch_result();
 }
 
 }  // namespace
 
-static int prefill_checks(const char* who, const void* qkv, int ld, const void* out, int ldo, int hd, int nh, int nkv, int keep_first, int v_group) {
+static int prefill_checks(const char* who, const void* qkv, int ld, const void* out, int ldo, int hd, int nh, int nkv, int keep_first, int v_group, int gate_col) {
   if (keep_first < 0 || v_group < 1 || nkv % v_group) return cima_fail(CIMA_E_ARG, "%s: keep_first %d must not be negative and %d kv heads be a multiple of v_group %d", who, keep_first, nkv, v_group);
+  if (gate_col < 0 || gate_col % 2 || (gate_col > 0 && gate_col + nh * hd > ld)) return cima_fail(CIMA_E_ARG, "%s: %d gate values from column %d (even) on exceed the rows of %d", who, nh * hd, gate_col, ld);
   if (hd % 16 || hd < 16 || hd > 128) return cima_fail(CIMA_E_SIZE, "%s: head_dim %d; this kernel takes multiples of 16 up to 128", who, hd);
   if (nh <= 0 || nkv <= 0 || nh % nkv || nh > 65535) return cima_fail(CIMA_E_SIZE, "%s: %d heads / %d kv heads are not accepted", who, nh, nkv);
   if (ld % 8 || ldo % 2 || ((uintptr_t)qkv & 15) || ((uintptr_t)out & 3))
@@ -318,11 +331,11 @@ static int prefill_checks(const char* who, const void* qkv, int ld, const void* 
 extern "C" int cima_attention_prefill(const void* qkv, int ld, const int* tile_seq, const int* tile_row0,
                                       const int* seq_first_row, void* out, int ldo, int T, int n_tiles, int nh, int nkv,
                                       int hd, float scale, int window, float sink, int keep_first, int v_group, const float* head_sink,
-                                      cudaStream_t stream) {
+                                      int gate_col, cudaStream_t stream) {
   if (T <= 0 || n_tiles <= 0) return 0;
-  if (int rc = prefill_checks("attention_prefill", qkv, ld, out, ldo, hd, nh, nkv, keep_first, v_group)) return rc;
+  if (int rc = prefill_checks("attention_prefill", qkv, ld, out, ldo, hd, nh, nkv, keep_first, v_group, gate_col)) return rc;
   const CimaPaged none{nullptr, 0, 0, BN, nkv, hd};
-#define CASE(H) case H: return launch_prefill<H, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, nullptr, none, nullptr, nullptr, out, ldo, T, n_tiles, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, stream)
+#define CASE(H) case H: return launch_prefill<H, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, nullptr, none, nullptr, nullptr, out, ldo, T, n_tiles, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, gate_col, stream)
   switch (hd) {
     CASE(16); CASE(32); CASE(48); CASE(64); CASE(80); CASE(96); CASE(112); CASE(128);
   }
@@ -336,14 +349,15 @@ extern "C" int cima_attention_extend(const void* qkv, int ld, const int* tile_se
                                      const int* seq_first_row, const void* cache, const int* table, int table_width,
                                      int ring, int page_size, const int* seq_slot, const int* seq_len, void* out, int ldo,
                                      int T, int n_tiles, int nh, int nkv, int hd, float scale, int window,
-                                     int planes, float sink, int keep_first, int v_group, const float* head_sink, cudaStream_t stream) {
+                                     int planes, float sink, int keep_first, int v_group, const float* head_sink, int gate_col,
+                                     cudaStream_t stream) {
   if (T <= 0 || n_tiles <= 0) return 0;
   if (planes != 1 && planes != 2) return cima_fail(CIMA_E_ARG, "attention_extend: %d planes; pages hold keys | values (2) or one shared vector (1)", planes);
-  if (int rc = prefill_checks("attention_extend", qkv, ld, out, ldo, hd, nh, nkv, keep_first, v_group)) return rc;
+  if (int rc = prefill_checks("attention_extend", qkv, ld, out, ldo, hd, nh, nkv, keep_first, v_group, gate_col)) return rc;
   if (page_size != BN) return cima_fail(CIMA_E_SIZE, "attention_extend: page size %d; this kernel takes %d", page_size, BN);
   if (!cache || !table || !seq_slot || !seq_len || ((uintptr_t)cache & 15)) return cima_fail(CIMA_E_ARG, "attention_extend: the cache (16-byte aligned), its block table, slots and lengths are needed");
   const CimaPaged pg{table, table_width, ring, page_size, nkv, hd, planes};
-#define CASE(H) case H: return launch_prefill<H, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, cache, pg, seq_slot, seq_len, out, ldo, T, n_tiles, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, stream)
+#define CASE(H) case H: return launch_prefill<H, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, cache, pg, seq_slot, seq_len, out, ldo, T, n_tiles, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, gate_col, stream)
   switch (hd) {
     CASE(16); CASE(32); CASE(48); CASE(64); CASE(80); CASE(96); CASE(112); CASE(128);
   }

@@ -62,6 +62,8 @@ struct AttnArgs {
   int planes;                   // keys from the cache: 2 = a page holds keys, then values; 1 = one vector serves as both
   float sink;                   // entries of score 0 without a value that join the softmax's denominator (0: none)
   const float* head_sink;       // or null: [nh], head h's denominator also holds exp(head_sink[h]) (instead of `sink`)
+  const __nv_bfloat16* gate;    // or null: the rows' own gates, gate[row * ld_gate + h * HD + d]; the result leaves times their sigmoid
+  int ld_gate;
 };
 
 // Keys of a query block whose rows stand at positions p0 .. (at most p0 + 127, below len): tiles [first, last] of 64.
@@ -332,6 +334,16 @@ k_attention_prefill_tc(const __grid_constant__ CUtensorMap map_qkv, const __grid
           for (int q = 0; q < 4; q++) {
             uint4 t;
             __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&t);
+            if (a.gate) {
+              const uint4 gv = *reinterpret_cast<const uint4*>(a.gate + (size_t)(row_base + r0 + r) * a.ld_gate + (size_t)h * HD + c * 32 + q * 8);
+              const __nv_bfloat162* g2 = reinterpret_cast<const __nv_bfloat162*>(&gv);
+#pragma unroll
+              for (int k = 0; k < 4; k++) {
+                const float2 g = __bfloat1622float2(g2[k]);
+                o[8 * q + 2 * k] *= cima_sigmoid(g.x);
+                o[8 * q + 2 * k + 1] *= cima_sigmoid(g.y);
+              }
+            }
 #pragma unroll
             for (int k = 0; k < 4; k++) h2[k] = __floats2bfloat162_rn(o[8 * q + 2 * k] * inv, o[8 * q + 2 * k + 1] * inv);
             *reinterpret_cast<uint4*>(dst + c * 32 + q * 8) = t;
@@ -359,7 +371,7 @@ struct CacheSource {              // keys and values from a layer's pages; cache
 template <int HD, bool FROM_CACHE>
 int launch_attention_tc(const void* qkv, int ld, const int* tile_seq, const int* tile_row0, const int* seq_first_row,
                         const CacheSource& c, void* out, int ldo, int T, int n_tiles, int nh, int nkv, float scale,
-                        int window, int* error_flag, float sink, const float* head_sink, cudaStream_t stream) {
+                        int window, int* error_flag, float sink, const float* head_sink, int gate_col, cudaStream_t stream) {
   if ((long long)n_tiles * nh > 0x7fffffffll) return cima_fail(CIMA_E_SIZE, "attention_prefill_tc: %d blocks of rows x %d heads exceed one launch", n_tiles, nh);
   CUtensorMap mq, mk;                                  // boxes of 128 rows (Q) and of 64 rows (K and V) by 64 columns
   // (with the keys in the cache only the queries' columns of a row are read, and the row may end there)
@@ -378,7 +390,7 @@ int launch_attention_tc(const void* qkv, int ld, const int* tile_seq, const int*
     raised = true;
   }
   AttnArgs a{tile_seq, tile_row0, seq_first_row, c.seq_len, c.seq_slot, c.table, c.table_width, c.ring,
-             (__nv_bfloat16*)out, ldo, nh, nkv, window, scale, error_flag, c.planes, sink, head_sink};
+             (__nv_bfloat16*)out, ldo, nh, nkv, window, scale, error_flag, c.planes, sink, head_sink, gate_col > 0 ? (const __nv_bfloat16*)qkv + gate_col : nullptr, ld};
   { int rc_ = cima_launch(k_attention_prefill_tc<HD, FROM_CACHE>, dim3((unsigned)n_tiles * (unsigned)nh), dim3(THREADS), smem, stream, 1, mq, mk, a); if (rc_) return rc_; }
   return cima_launch_result();
 }
@@ -386,9 +398,10 @@ int launch_attention_tc(const void* qkv, int ld, const int* tile_seq, const int*
 }  // namespace
 
 static int tc_checks(const char* who, const void* qkv, int ld, const void* out, int ldo, int nh, int nkv, int hd, const int* error_flag,
-                     bool queries_only = false) {
+                     int gate_col, bool queries_only = false) {
   if (hd != 64 && hd != 128) return cima_fail(CIMA_E_SIZE, "%s: head_dim %d; this kernel takes 64 or 128", who, hd);
   if (nh <= 0 || nkv <= 0 || nh % nkv) return cima_fail(CIMA_E_SIZE, "%s: %d heads are not a multiple of %d kv heads", who, nh, nkv);
+  if (gate_col < 0 || gate_col % 8 || (gate_col > 0 && gate_col + nh * hd > ld)) return cima_fail(CIMA_E_ARG, "%s: %d gate values from column %d (a multiple of 8) on exceed the rows of %d", who, nh * hd, gate_col, ld);
   if (ld % 8 || ldo % 8) return cima_fail(CIMA_E_SIZE, "%s: row strides (%d, %d) must be multiples of 8", who, ld, ldo);
   if (ld < (queries_only ? nh : nh + 2 * nkv) * hd) return cima_fail(CIMA_E_SIZE, "%s: row stride %d is smaller than the heads of a row", who, ld);
   if ((((uintptr_t)qkv | (uintptr_t)out) & 15)) return cima_fail(CIMA_E_ARG, "%s: qkv and out must be 16-byte aligned", who);
@@ -403,13 +416,13 @@ static int tc_checks(const char* who, const void* qkv, int ld, const void* out, 
 extern "C" int cima_attention_prefill_tc(const void* qkv, int ld, const int* tile_seq, const int* tile_row0,
                                          const int* seq_first_row, void* out, int ldo, int T, int n_tiles, int nh,
                                          int nkv, int hd, float scale, int window, int* error_flag, float sink, const float* head_sink,
-                                         cudaStream_t stream) {
+                                         int gate_col, cudaStream_t stream) {
   if (T <= 0 || n_tiles <= 0) return 0;
-  if (int rc = tc_checks("attention_prefill_tc", qkv, ld, out, ldo, nh, nkv, hd, error_flag)) return rc;
+  if (int rc = tc_checks("attention_prefill_tc", qkv, ld, out, ldo, nh, nkv, hd, error_flag, gate_col)) return rc;
   const CacheSource none{nullptr, 0, nullptr, nullptr, nullptr, 0, 0};
   if (hd == 64)
-    return launch_attention_tc<64, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, none, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, stream);
-  return launch_attention_tc<128, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, none, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, stream);
+    return launch_attention_tc<64, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, none, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, stream);
+  return launch_attention_tc<128, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, none, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, stream);
 }
 
 // The same for sequences that go on: the rows of sequence s are the positions seq_len[s] - rows .. seq_len[s] - 1, and
@@ -419,16 +432,16 @@ extern "C" int cima_attention_extend_tc(const void* qkv, int ld, const int* tile
                                         int table_width, int ring, int page_size, const int* seq_slot, const int* seq_len,
                                         void* out, int ldo, int T, int n_tiles, int nh, int nkv, int hd, float scale,
                                         int window, int* error_flag, int planes, float sink, const float* head_sink,
-                                        cudaStream_t stream) {
+                                        int gate_col, cudaStream_t stream) {
   if (T <= 0 || n_tiles <= 0) return 0;
   if (planes != 1 && planes != 2) return cima_fail(CIMA_E_ARG, "attention_extend_tc: %d planes; pages hold keys | values (2) or one shared vector (1)", planes);
-  if (int rc = tc_checks("attention_extend_tc", qkv, ld, out, ldo, nh, nkv, hd, error_flag, true)) return rc;
+  if (int rc = tc_checks("attention_extend_tc", qkv, ld, out, ldo, nh, nkv, hd, error_flag, gate_col, true)) return rc;
   if (page_size != BN) return cima_fail(CIMA_E_SIZE, "attention_extend_tc: page size %d; this kernel takes %d", page_size, BN);
   if (!cache || !table || !seq_slot || !seq_len || ((uintptr_t)cache & 15) || n_pages <= 0)
     return cima_fail(CIMA_E_ARG, "attention_extend_tc: the cache (16-byte aligned), its block table, slots and lengths are needed");
   if (n_pages * planes * nkv * BN >= (1ll << 31)) return cima_fail(CIMA_E_SIZE, "attention_extend_tc: %lld pages exceed a tensor map's 32-bit row coordinate", n_pages);
   const CacheSource c{cache, n_pages, table, seq_slot, seq_len, table_width, ring, planes};
   if (hd == 64)
-    return launch_attention_tc<64, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, c, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, stream);
-  return launch_attention_tc<128, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, c, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, stream);
+    return launch_attention_tc<64, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, c, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, stream);
+  return launch_attention_tc<128, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, c, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, stream);
 }

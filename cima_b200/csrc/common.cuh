@@ -65,6 +65,11 @@ __device__ __forceinline__ float cima_gated(float g, float u, int act, float lim
   return cima_gate_act(g, act) * u;
 }
 
+__device__ __forceinline__ float cima_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
+
+// log(1 / (1 + exp(-z))) without overflow in either tail.
+__device__ __forceinline__ float cima_log_sigmoid(float z) { return fminf(z, 0.f) - log1pf(expf(-fabsf(z))); }
+
 // Sum over the threads of a block in a fixed order (warp shuffles, then warp 0 over the warps'
 // partial sums), so that a row's result never depends on what else is launched with it.
 // `red` is shared memory of at least 32 floats.  Every thread gets the total.

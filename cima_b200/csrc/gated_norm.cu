@@ -1,6 +1,8 @@
-// Two small norms behind the recurrent mixers, float32 throughout, one rounding at the store:
-//   group_rmsnorm_gate   out = o / sqrt(mean_group(o^2) + eps) * w * sigmoid(gate)      per group of n values of a row
-//                        (a group = a head's values with one shared weight [n], or the whole row with a weight [G n])
+// Small norms behind the recurrent mixers, float32 throughout, one rounding at the store:
+//   group_rmsnorm_gate   out = o / sqrt(mean_group(o^2) + eps) * w * act(gate)          per group of n values of a row
+//                        (a group = a head's values with one shared weight [n], or the whole row with a weight [G n];
+//                        act the sigmoid or SiLU; with `den` and `low` [T, G] a group is first divided by
+//                        max(|den|, low) + div_eps)
 //   rms_mean             x += (1 / B) * sum_b  y_b / sqrt(mean(y_b^2) + eps) * w_b        B <= 4 branches of one width
 //   scale_add_group_rmsnorm   x <- N(alpha x + y), N the norm in groups with weight w [G n]; also h = x in another dtype
 //                        (the norm behind a sublayer's sum: the stream, the sum and the norm in one pass)
@@ -104,10 +106,18 @@ k_cast_rows(const float* __restrict__ x, TH* __restrict__ h, size_t total) {
   for (size_t j = i; j < total && j < i + 4; j++) h[j] = cima_from_f32<TH>(x[j]);
 }
 
+__device__ __forceinline__ float gate_value(float z, int silu) { return silu ? z / (1.0f + expf(-z)) : 1.0f / (1.0f + expf(-z)); }
+
+// What a group is multiplied by before its norm: 1, or 1 / (max(|den|, low) + div_eps).
+__device__ __forceinline__ float group_factor(const float* den, const float* low, float div_eps, long long unit) {
+  return den ? 1.0f / (fmaxf(fabsf(den[unit]), low[unit]) + div_eps) : 1.0f;
+}
+
 template <typename TG, typename TO>
 __global__ void __launch_bounds__(128)
 k_group_rmsnorm_gate(const float* __restrict__ o, const float* __restrict__ w, const TG* __restrict__ gate, int ldg,
-                     TO* __restrict__ out, long long units, int groups, int n, int shared_w, float eps) {
+                     TO* __restrict__ out, long long units, int groups, int n, int shared_w, float eps, int silu,
+                     const float* __restrict__ den, const float* __restrict__ low, float div_eps) {
   cima_pdl_wait();
   cima_pdl_trigger();        // a short kernel: the next one may be set up while this one runs (it waits for this one's end itself)
   const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -116,16 +126,43 @@ k_group_rmsnorm_gate(const float* __restrict__ o, const float* __restrict__ w, c
   const long long row = unit / groups;
   const int grp = (int)(unit - row * groups);
   const float* src = o + ((size_t)row * groups + grp) * n;
-  float ss = 0.f;
-  for (int i = lane; i < n; i += 32) ss = fmaf(src[i], src[i], ss);
-  for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
-  const float r = 1.0f / sqrtf(ss / (float)n + eps);
   const float* wp = w + (shared_w ? 0 : (size_t)grp * n);
   const TG* gp = gate ? gate + (size_t)row * ldg + (size_t)grp * n : nullptr;
   TO* dst = out + ((size_t)row * groups + grp) * n;
+  const float f = group_factor(den, low, div_eps, unit);
+  if (n <= 256) {                                        // eight values a lane: every load is requested before the first use
+    float v[8], wv[8], gv[8];
+#pragma unroll
+    for (int j = 0; j < 8; j++) {
+      const int i = min(lane + 32 * j, n - 1);           // (beyond the group: its last value, which is then not used)
+      if (32 * j < n) {
+        v[j] = src[i];
+        wv[j] = wp[i];
+        gv[j] = gp ? cima_to_f32<TG>(gp[i]) : 0.f;
+      }
+    }
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; j++)
+      if (lane + 32 * j < n) { v[j] *= f; ss = fmaf(v[j], v[j], ss); }
+    for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+    const float r = 1.0f / sqrtf(ss / (float)n + eps);
+#pragma unroll
+    for (int j = 0; j < 8; j++)
+      if (lane + 32 * j < n) {
+        float y = v[j] * r * wv[j];
+        if (gp) y *= gate_value(gv[j], silu);
+        dst[lane + 32 * j] = cima_from_f32<TO>(y);
+      }
+    return;
+  }
+  float ss = 0.f;
+  for (int i = lane; i < n; i += 32) { const float v = src[i] * f; ss = fmaf(v, v, ss); }
+  for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  const float r = 1.0f / sqrtf(ss / (float)n + eps);
   for (int i = lane; i < n; i += 32) {
-    float y = src[i] * r * wp[i];
-    if (gp) y *= 1.0f / (1.0f + expf(-cima_to_f32<TG>(gp[i])));
+    float y = src[i] * f * r * wp[i];
+    if (gp) y *= gate_value(cima_to_f32<TG>(gp[i]), silu);
     dst[i] = cima_from_f32<TO>(y);
   }
 }
@@ -134,7 +171,8 @@ k_group_rmsnorm_gate(const float* __restrict__ o, const float* __restrict__ w, c
 template <typename TG, typename TO>
 __global__ void __launch_bounds__(256)
 k_group_rmsnorm_gate_wide(const float* __restrict__ o, const float* __restrict__ w, const TG* __restrict__ gate, int ldg,
-                          TO* __restrict__ out, int groups, int n, int shared_w, float eps) {
+                          TO* __restrict__ out, int groups, int n, int shared_w, float eps, int silu,
+                          const float* __restrict__ den, const float* __restrict__ low, float div_eps) {
   cima_pdl_wait();
   cima_pdl_trigger();        // a short kernel: the next one may be set up while this one runs (it waits for this one's end itself)
   __shared__ float red[32];
@@ -142,16 +180,17 @@ k_group_rmsnorm_gate_wide(const float* __restrict__ o, const float* __restrict__
   const long long row = unit / groups;
   const int grp = (int)(unit - row * groups);
   const float* src = o + ((size_t)row * groups + grp) * n;
+  const float f = group_factor(den, low, div_eps, unit);
   float ss = 0.f;
-  for (int i = threadIdx.x; i < n; i += blockDim.x) ss = fmaf(src[i], src[i], ss);
+  for (int i = threadIdx.x; i < n; i += blockDim.x) { const float v = src[i] * f; ss = fmaf(v, v, ss); }
   ss = cima_block_sum(ss, red);
   const float r = 1.0f / sqrtf(ss / (float)n + eps);
   const float* wp = w + (shared_w ? 0 : (size_t)grp * n);
   const TG* gp = gate ? gate + (size_t)row * ldg + (size_t)grp * n : nullptr;
   TO* dst = out + ((size_t)row * groups + grp) * n;
   for (int i = threadIdx.x; i < n; i += blockDim.x) {
-    float y = src[i] * r * wp[i];
-    if (gp) y *= 1.0f / (1.0f + expf(-cima_to_f32<TG>(gp[i])));
+    float y = src[i] * f * r * wp[i];
+    if (gp) y *= gate_value(cima_to_f32<TG>(gp[i]), silu);
     dst[i] = cima_from_f32<TO>(y);
   }
 }
@@ -182,22 +221,24 @@ k_rms_mean(Branches br, float* __restrict__ x, int H, float eps, int assign) {
 }  // namespace
 
 // o [T, groups * n] float32; w [n] (shared_w) or [groups * n]; gate [T, ldg] (gdtype) or null; out [T, groups * n] (odtype).
-extern "C" int cima_group_rmsnorm_gate(const float* o, const float* w, const void* gate, int ldg, void* out, int dtype, int T,
-                                       int groups, int n, int shared_w, float eps, cudaStream_t stream) {
+// silu: the gate's activation (0: the sigmoid).  den, low [T, groups] or null: a group is divided by max(|den|, low) + div_eps first.
+extern "C" int cima_group_rmsnorm_gate(const float* o, const float* w, const void* gate, int ldg, int gdtype, void* out, int odtype, int T,
+                                       int groups, int n, int shared_w, float eps, int silu, const float* den, const float* low,
+                                       float div_eps, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (groups <= 0 || n <= 0) return cima_fail(CIMA_E_SIZE, "group_rmsnorm_gate: %d groups of %d values must be positive", groups, n);
+  if ((den != nullptr) != (low != nullptr)) return cima_fail(CIMA_E_ARG, "group_rmsnorm_gate: the divisors take their lower bounds");
   const long long units = (long long)T * groups;
-  const dim3 grid((unsigned)((units + 3) / 4));
+  const bool wide = n >= 512 && units < 0x7fffffffll;
+  const dim3 grid(wide ? (unsigned)units : (unsigned)((units + 3) / 4));
   int rc;
-  if (n >= 512 && units < 0x7fffffffll) {
-    if (dtype == CIMA_F32) rc = cima_launch(k_group_rmsnorm_gate_wide<float, float>, dim3((unsigned)units), dim3(256), (size_t)0, stream, 1, o, w, (const float*)gate, ldg, (float*)out, groups, n, shared_w, eps);
-    else if (dtype == CIMA_BF16) rc = cima_launch(k_group_rmsnorm_gate_wide<__nv_bfloat16, __nv_bfloat16>, dim3((unsigned)units), dim3(256), (size_t)0, stream, 1, o, w, (const __nv_bfloat16*)gate, ldg, (__nv_bfloat16*)out, groups, n, shared_w, eps);
-    else return cima_fail(CIMA_E_DTYPE, "group_rmsnorm_gate: dtype code %d is neither float32 nor bfloat16", dtype);
-    return rc ? rc : cima_launch_result();
-  }
-  if (dtype == CIMA_F32) rc = cima_launch(k_group_rmsnorm_gate<float, float>, grid, dim3(128), (size_t)0, stream, 1, o, w, (const float*)gate, ldg, (float*)out, units, groups, n, shared_w, eps);
-  else if (dtype == CIMA_BF16) rc = cima_launch(k_group_rmsnorm_gate<__nv_bfloat16, __nv_bfloat16>, grid, dim3(128), (size_t)0, stream, 1, o, w, (const __nv_bfloat16*)gate, ldg, (__nv_bfloat16*)out, units, groups, n, shared_w, eps);
-  else return cima_fail(CIMA_E_DTYPE, "group_rmsnorm_gate: dtype code %d is neither float32 nor bfloat16", dtype);
+#define RUN(TG, TO) rc = wide ? cima_launch(k_group_rmsnorm_gate_wide<TG, TO>, grid, dim3(256), (size_t)0, stream, 1, o, w, (const TG*)gate, ldg, (TO*)out, groups, n, shared_w, eps, silu, den, low, div_eps) \
+                              : cima_launch(k_group_rmsnorm_gate<TG, TO>, grid, dim3(128), (size_t)0, stream, 1, o, w, (const TG*)gate, ldg, (TO*)out, units, groups, n, shared_w, eps, silu, den, low, div_eps)
+  if (gdtype == CIMA_F32 && odtype == CIMA_F32) RUN(float, float);
+  else if (gdtype == CIMA_BF16 && odtype == CIMA_BF16) RUN(__nv_bfloat16, __nv_bfloat16);
+  else if (gdtype == CIMA_F32 && odtype == CIMA_BF16) RUN(float, __nv_bfloat16);
+  else return cima_fail(CIMA_E_DTYPE, "group_rmsnorm_gate: a gate of dtype code %d with an output of %d is not accepted", gdtype, odtype);
+#undef RUN
   return rc ? rc : cima_launch_result();
 }
 

@@ -5,8 +5,12 @@
 //   moe_sort      the (row, choice) pairs ordered by expert: offsets of every expert's pairs and of its row tiles
 //   moe_gemm 0    z[i] = act(W_gate[e] h[row]) * (W_up[e] h[row])      for the sorted pairs i (a tile = 32 pairs of one expert)
 //   moe_gemm 1    y[pair] = W_down[e] z[i]                             float32, back at the pair's own place
+//                 Options: a group's score its best one instead of the sum of two; weights s * scale, not divided by their sum.
 //   moe_combine   x[row] += sum_j weight[row, j] * y[row * top + j]    ascending j, float32; a shared expert's rows (float32), times
-//                 the sigmoid of a gate logit a row where one is given, join the sum behind the chosen experts' 
+//                 the sigmoid of a gate logit a row where one is given, join the sum behind the chosen experts'
+// The router may have more outputs than there are experts with matrices: choices e >= E are identity experts, whose
+// output is the row h itself.  They are routed like the others and take part in no product: the sorts leave their
+// pairs out, and moe_combine reads h[row] for them.
 // A pair's sums run over k in ascending order with one accumulator, so its result does not depend on which other
 // rows share its tile, nor on the order in which the sort placed the pairs of an expert.
 //
@@ -26,7 +30,8 @@ constexpr int BM = 32, BN = 64, BK = 16;
 __device__ __forceinline__ void moe_sort_block(const int* idx, int P, int E, int* offsets, int* tiles, int* perm, int* cnt, int* off) {
   for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&cnt[idx[p]], 1);
+  for (int p = threadIdx.x; p < P; p += blockDim.x)
+    if (idx[p] < E) atomicAdd(&cnt[idx[p]], 1);            // (an identity expert's pair is in no product)
   __syncthreads();
   if (threadIdx.x == 0) {
     int o = 0, t = 0;
@@ -42,7 +47,7 @@ __device__ __forceinline__ void moe_sort_block(const int* idx, int P, int E, int
   __syncthreads();
   for (int p = threadIdx.x; p < P; p += blockDim.x) {
     const int e = idx[p];
-    perm[off[e] + atomicAdd(&cnt[e], 1)] = p;
+    if (e < E) perm[off[e] + atomicAdd(&cnt[e], 1)] = p;
   }
 }
 
@@ -50,10 +55,10 @@ __device__ __forceinline__ void moe_sort_block(const int* idx, int P, int E, int
 // few rows would otherwise walk dependent loads from global memory); with more they stay in the caller's buffer.
 constexpr int ROUTE_THREADS = 64, ROUTE_SMEM_EXPERTS = 128;
 __device__ __forceinline__ void moe_route_row(float* scores, float* local, int row, int E, int ld, int top, int groups, int keep, float scale,
-                                              int softmax, const float* corr, int* idx, float* wgt);
+                                              int softmax, int best_one, int divide, const float* corr, int* idx, float* wgt);
 __global__ void __launch_bounds__(ROUTE_THREADS)
 k_moe_route(float* __restrict__ scores, int T, int E, int ld, int top, int groups, int keep, float scale, int softmax,
-            const float* __restrict__ corr, int* __restrict__ idx,
+            int best_one, int divide, int real, const float* __restrict__ corr, int* __restrict__ idx,
             float* __restrict__ wgt, int* __restrict__ offsets, int* __restrict__ tiles, int* __restrict__ perm) {
   cima_pdl_wait();
   cima_pdl_trigger();        // the next kernel may be set up while this one runs (it waits for this one's end itself)
@@ -61,15 +66,15 @@ k_moe_route(float* __restrict__ scores, int T, int E, int ld, int top, int group
   __shared__ int cnt[MOE_MAX_EXPERTS];
   __shared__ int off[MOE_MAX_EXPERTS + 1];
   const int row = blockIdx.x * blockDim.x + threadIdx.x;
-  if (row < T) moe_route_row(scores, local, row, E, ld, top, groups, keep, scale, softmax, corr, idx, wgt);
+  if (row < T) moe_route_row(scores, local, row, E, ld, top, groups, keep, scale, softmax, best_one, divide, corr, idx, wgt);
   if (offsets) {             // a step of one block's rows: the pairs are ordered by expert here, which saves moe_sort's launch
     __syncthreads();
-    moe_sort_block(idx, T * top, E, offsets, tiles, perm, cnt, off);
+    moe_sort_block(idx, T * top, real, offsets, tiles, perm, cnt, off);
   }
 }
 
 __device__ __forceinline__ void moe_route_row(float* scores, float* local, int row, int E, int ld, int top, int groups, int keep, float scale,
-                                              int softmax, const float* corr, int* idx, float* wgt) {
+                                              int softmax, int best_one, int divide, const float* corr, int* idx, float* wgt) {
   float* s = E <= ROUTE_SMEM_EXPERTS ? local + threadIdx.x * (E + 1) : scores + (size_t)row * ld;
   const float* z = scores + (size_t)row * ld;
   float zmax = -INFINITY;
@@ -107,7 +112,7 @@ __device__ __forceinline__ void moe_route_row(float* scores, float* local, int r
           const float v = s[e] + (corr ? corr[e] : 0.f);
           if (v > a1) { a2 = a1; a1 = v; } else if (v > a2) a2 = v;
         }
-        const float sc = per >= 2 ? a1 + a2 : a1;
+        const float sc = per >= 2 && !best_one ? a1 + a2 : a1;
         if (sc > bs || best < 0) { bs = sc; best = gi; }
       }
       kept |= 1ull << best;
@@ -132,7 +137,7 @@ __device__ __forceinline__ void moe_route_row(float* scores, float* local, int r
     sum += w;
     s[best] = -INFINITY;                                   // taken
   }
-  const float f = scale / (sum + 1e-20f);
+  const float f = divide ? scale / (sum + 1e-20f) : scale;
   for (int c = 0; c < top; c++) wgt[(size_t)row * top + c] *= f;
 }
 
@@ -234,10 +239,13 @@ k_moe_gemm(const TA* __restrict__ A, int lda, const TW* __restrict__ W, void* __
   }
 }
 
-// pos: the row of y that holds pair (row, j), or null where y is kept by pair
+// pos: the row of y that holds pair (row, j), or null where y is kept by pair.  idx (null: no identity experts): the pairs'
+// experts; a pair of an expert >= E has h[row] in place of its row of y.
+template <typename TH>
 __global__ void __launch_bounds__(256)
 k_moe_combine(const float* __restrict__ y, const float* __restrict__ wgt, const int* __restrict__ pos, float* __restrict__ x,
-              int top, int H, int assign, const float* __restrict__ shared, const float* __restrict__ gate, int ldg) {
+              int top, int H, int assign, const float* __restrict__ shared, const float* __restrict__ gate, int ldg,
+              const int* __restrict__ idx, int E, const TH* __restrict__ h) {
   cima_pdl_wait();
   cima_pdl_trigger();        // the next kernel may be set up while this one runs (it waits for this one's end itself)
   const size_t row = blockIdx.x;
@@ -246,7 +254,8 @@ k_moe_combine(const float* __restrict__ y, const float* __restrict__ wgt, const 
     float s = 0.f;
     for (int j = 0; j < top; j++) {
       const size_t p = row * top + j;
-      s = fmaf(wgt[p], y[(pos ? (size_t)pos[p] : p) * H + c], s);
+      const float v = idx && idx[p] >= E ? cima_to_f32<TH>(h[row * H + c]) : y[(pos ? (size_t)pos[p] : p) * H + c];
+      s = fmaf(wgt[p], v, s);
     }
     if (shared) s = fmaf(sg, shared[row * H + c], s);
     x[row * H + c] = assign ? s : x[row * H + c] + s;
@@ -257,20 +266,35 @@ k_moe_combine(const float* __restrict__ y, const float* __restrict__ wgt, const 
 // weights and places fetched once a row, and the rows of all choices requested before the first is used.  The sum runs
 // over j in the same ascending order.
 constexpr int COMBINE_TOP = 8;
+template <typename TH>
+__device__ __forceinline__ float4 moe_row4(const TH* p) {
+  if constexpr (sizeof(TH) == 2) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  } else {
+    return *reinterpret_cast<const float4*>(p);
+  }
+}
+template <typename TH>
 __global__ void __launch_bounds__(128)
 k_moe_combine4(const float* __restrict__ y, const float* __restrict__ wgt, const int* __restrict__ pos, float* __restrict__ x,
-               int top, int H4, int assign, const float* __restrict__ shared, const float* __restrict__ gate, int ldg) {
+               int top, int H4, int assign, const float* __restrict__ shared, const float* __restrict__ gate, int ldg,
+               const int* __restrict__ idx, int E, const TH* __restrict__ h) {
   cima_pdl_wait();
   cima_pdl_trigger();
   const size_t row = blockIdx.x;
   float w[COMBINE_TOP];
+  bool own[COMBINE_TOP];
   const float4* src[COMBINE_TOP];
 #pragma unroll
   for (int j = 0; j < COMBINE_TOP; j++) {
     const size_t p = row * top + (j < top ? j : 0);
     w[j] = j < top ? wgt[p] : 0.f;
-    src[j] = reinterpret_cast<const float4*>(y) + (pos ? (size_t)pos[p] : p) * H4;
+    own[j] = idx && idx[p] >= E;                          // an identity expert: the row itself
+    src[j] = reinterpret_cast<const float4*>(y) + (own[j] ? (size_t)0 : pos ? (size_t)pos[p] : p) * H4;
   }
+  const TH* hr = idx ? h + row * H4 * 4 : nullptr;
   const float sg = shared ? (gate ? 1.0f / (1.0f + expf(-gate[row * (size_t)ldg])) : 1.0f) : 0.f;
   const float4* sh = shared ? reinterpret_cast<const float4*>(shared) + row * H4 : nullptr;
   float4* xr = reinterpret_cast<float4*>(x) + row * H4;
@@ -278,7 +302,7 @@ k_moe_combine4(const float* __restrict__ y, const float* __restrict__ wgt, const
   for (int g = blockIdx.y * blockDim.x + threadIdx.x; g < H4; g += gridDim.y * blockDim.x) {
     float4 v[COMBINE_TOP];
 #pragma unroll
-    for (int j = 0; j < COMBINE_TOP; j++) v[j] = j < top ? src[j][g] : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int j = 0; j < COMBINE_TOP; j++) v[j] = j >= top ? make_float4(0.f, 0.f, 0.f, 0.f) : own[j] ? moe_row4<TH>(hr + 4 * g) : src[j][g];
     const float4 sv = sh ? sh[g] : make_float4(0.f, 0.f, 0.f, 0.f);
     const float4 xo = assign ? make_float4(0.f, 0.f, 0.f, 0.f) : xr[g];
     float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -291,7 +315,7 @@ k_moe_combine4(const float* __restrict__ y, const float* __restrict__ wgt, const
 }
 
 // Every expert's pairs from a multiple of `tile` rows on: pos [P] the place of every pair, tile_expert [n_tiles] the
-// expert of every row tile (-1 beyond the last).  One block.
+// expert of every row tile (-1 beyond the last).  An identity expert's pair (expert >= E) gets the place -1.  One block.
 __global__ void __launch_bounds__(1024)
 k_moe_sort_tiles(const int* __restrict__ idx, int P, int E, int tile, int n_tiles, int* __restrict__ tile_expert, int* __restrict__ pos) {
   cima_pdl_wait();
@@ -300,7 +324,8 @@ k_moe_sort_tiles(const int* __restrict__ idx, int P, int E, int tile, int n_tile
   __shared__ int off[MOE_MAX_EXPERTS + 1];
   for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&cnt[idx[p]], 1);
+  for (int p = threadIdx.x; p < P; p += blockDim.x)
+    if (idx[p] < E) atomicAdd(&cnt[idx[p]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int t = 0;
@@ -322,7 +347,7 @@ k_moe_sort_tiles(const int* __restrict__ idx, int P, int E, int tile, int n_tile
   __syncthreads();
   for (int p = threadIdx.x; p < P; p += blockDim.x) {
     const int e = idx[p];
-    pos[p] = off[e] * tile + atomicAdd(&cnt[e], 1);
+    pos[p] = e < E ? off[e] * tile + atomicAdd(&cnt[e], 1) : -1;      // an identity expert's pair has no place
   }
 }
 
@@ -332,6 +357,7 @@ k_moe_gather_rows(const uint4* __restrict__ src, const int* __restrict__ pos, ui
   cima_pdl_wait();
   cima_pdl_trigger();        // the next kernel may be set up while this one runs (it waits for this one's end itself)
   const size_t p = blockIdx.x;
+  if (pos[p] < 0) return;
   const uint4* s = src + (p / top) * vecs;
   uint4* d = dst + (size_t)pos[p] * vecs;
   for (int v = threadIdx.x; v < vecs; v += blockDim.x) d[v] = s[v];
@@ -442,17 +468,20 @@ k_moe_few(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16* __r
 
 // scores [T, E] float32: the router's logits on entry, scratch afterwards.  idx [T, top] int32, wgt [T, top] float32.
 // offsets, tiles, perm: null, or (at most 64 rows) the outputs of moe_sort, made by the same launch.
+// E: the router's outputs, of which the first `real` have matrices (the rest are identity experts).  best_one: a group's score
+// is its best one instead of the sum of its two best; divide 0: the weights are s * scale as they are.
 extern "C" int cima_moe_route(float* scores, int T, int E, int ld, int top, int groups, int keep, float scale, int softmax,
-                              const float* correction, int* idx, float* wgt,
+                              int best_one, int divide, int real, const float* correction, int* idx, float* wgt,
                               int* offsets, int* tiles, int* perm, cudaStream_t stream) {
   if (T <= 0) return 0;
+  if (real <= 0 || real > E) return cima_fail(CIMA_E_SIZE, "moe_route: %d of %d router outputs have matrices", real, E);
   if (ld < E) return cima_fail(CIMA_E_SIZE, "moe_route: rows of %d scores hold no %d experts", ld, E);
   if (E <= 0 || E > MOE_MAX_EXPERTS || groups <= 0 || groups > 64 || E % groups || keep <= 0 || keep > groups)
     return cima_fail(CIMA_E_SIZE, "moe_route: %d experts in %d groups of which %d stay are not accepted (at most %d experts in at most 64 equal groups)", E, groups, keep, MOE_MAX_EXPERTS);
   if (top <= 0 || top > keep * (E / groups)) return cima_fail(CIMA_E_SIZE, "moe_route: %d choices among %d experts that stay", top, keep * (E / groups));
   if ((offsets || tiles || perm) && (!offsets || !tiles || !perm || T > ROUTE_THREADS))
     return cima_fail(CIMA_E_ARG, "moe_route: ordering the pairs here takes offsets, tiles and perm and at most %d rows (%d given)", ROUTE_THREADS, T);
-  int rc = cima_launch(k_moe_route, dim3((T + ROUTE_THREADS - 1) / ROUTE_THREADS), dim3(ROUTE_THREADS), (size_t)0, stream, 1, scores, T, E, ld, top, groups, keep, scale, softmax, correction, idx, wgt, offsets, tiles, perm);
+  int rc = cima_launch(k_moe_route, dim3((T + ROUTE_THREADS - 1) / ROUTE_THREADS), dim3(ROUTE_THREADS), (size_t)0, stream, 1, scores, T, E, ld, top, groups, keep, scale, softmax, best_one, divide, real, correction, idx, wgt, offsets, tiles, perm);
   return rc ? rc : cima_launch_result();
 }
 
@@ -485,15 +514,20 @@ extern "C" int cima_moe_gemm(const void* a, int adtype, int lda, const void* w, 
 
 // y [pairs or places, H] float32; pos [T * top] the row of y of every pair, or null where y is kept by pair
 // shared (may be null): [T, H] float32 rows added behind the experts', each row times sigmoid(gate[row * ldg]) where gate is given
+// idx (may be null: no identity experts) [T, top] with h [T, H] (hdtype): a pair whose expert is >= E has h[row] as its output
 extern "C" int cima_moe_combine(const float* y, const float* wgt, const int* pos, float* x, int T, int top, int H, int assign,
-                                const float* shared, const float* gate, int ldg, cudaStream_t stream) {
+                                const float* shared, const float* gate, int ldg, const int* idx, int E, const void* h, int hdtype,
+                                cudaStream_t stream) {
   if (T <= 0) return 0;
-  if (top <= COMBINE_TOP && H % 4 == 0 && (((uintptr_t)y | (uintptr_t)x | (uintptr_t)shared) & 15) == 0) {
-    const unsigned parts = (unsigned)((H / 4 + 127) / 128);
-    int rc4 = cima_launch(k_moe_combine4, dim3(T, parts > 65535 ? 65535 : parts), dim3(128), (size_t)0, stream, 1, y, wgt, pos, x, top, H / 4, assign, shared, gate, ldg);
-    return rc4 ? rc4 : cima_launch_result();
-  }
-  int rc = cima_launch(k_moe_combine, dim3(T), dim3(256), (size_t)0, stream, 1, y, wgt, pos, x, top, H, assign, shared, gate, ldg);
+  if (idx && (!h || (hdtype != CIMA_F32 && hdtype != CIMA_BF16))) return cima_fail(CIMA_E_ARG, "moe_combine: identity experts need the rows h in float32 or bfloat16");
+  const bool vec = top <= COMBINE_TOP && H % 4 == 0 && (((uintptr_t)y | (uintptr_t)x | (uintptr_t)shared | (idx ? (uintptr_t)h : (uintptr_t)0)) & 15) == 0;
+  const unsigned parts = (unsigned)((H / 4 + 127) / 128);
+  int rc;
+#define RUN(TH) rc = vec ? cima_launch(k_moe_combine4<TH>, dim3(T, parts > 65535 ? 65535 : parts), dim3(128), (size_t)0, stream, 1, y, wgt, pos, x, top, H / 4, assign, shared, gate, ldg, idx, E, (const TH*)h) \
+                         : cima_launch(k_moe_combine<TH>, dim3(T), dim3(256), (size_t)0, stream, 1, y, wgt, pos, x, top, H, assign, shared, gate, ldg, idx, E, (const TH*)h)
+  if (idx && hdtype == CIMA_BF16) RUN(__nv_bfloat16);
+  else RUN(float);
+#undef RUN
   return rc ? rc : cima_launch_result();
 }
 

@@ -128,7 +128,9 @@ k_rope_append_bf16x8(__nv_bfloat16* __restrict__ qkv, int ld, const float* __res
 
 // The general form: a warp a head of a row.  Before the rotation the first `norm_dim` values of every q and k head are
 // divided by their root mean square (eps inside the root) and multiplied by a weight of `norm_dim` values, one for all
-// q heads and one for all k heads (no norm where the weights are null); and a row holds `nv` value heads behind its key
+// q heads and one for all k heads (without weights for norm_dim > 0 it only divides; no norm where norm_dim is 0); the
+// queries of a row at position p are then multiplied by 1 + temp_coef ln(floor((p + 1) / temp_every) + 1) (temp_every 0: not);
+// and a row holds `nv` value heads behind its key
 // heads (nv <= nkv: neighbouring key heads share a value head), which go to the first nv heads of the pages' value
 // plane.  Sums of squares, the norm, the angle and the rotation are float32; one rounding at the store.
 // VEC 4: a lane takes four neighbouring values at a time (one 8- or 16-byte load and store); the launch chooses it where
@@ -164,7 +166,8 @@ __global__ void __launch_bounds__(128)
 k_norm_rope_append(TA* __restrict__ qkv, int ld, const float* __restrict__ inv_freq, int rotary_dim,
                    const int* __restrict__ row_pos, const int* __restrict__ row_seq, const int* __restrict__ seq_slot,
                    const int* __restrict__ seq_len, TA* __restrict__ cache_in, CimaPaged pg, int nh, int nkv, int nv, int hd,
-                   const float* __restrict__ q_norm, const float* __restrict__ k_norm, int norm_dim, float eps, float amp) {
+                   const float* __restrict__ q_norm, const float* __restrict__ k_norm, int norm_dim, float eps, float amp,
+                   float temp_coef, int temp_every) {
   cima_pdl_wait();
   __shared__ __align__(16) float vals[4][256];
   __shared__ float rot_cos[128], rot_sin[128];
@@ -221,10 +224,15 @@ k_norm_rope_append(TA* __restrict__ qkv, int ld, const float* __restrict__ inv_f
   }
   for (int o = 16; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
   if (VEC == 4) __syncwarp();                          // the norm's loop reads what other lanes wrote
-  if (w) {
+  float temp = 1.0f;
+  if (temp_every > 0 && head < nh) temp = 1.0f + temp_coef * logf((float)((pos + 1) / temp_every + 1));
+  if (norm_dim > 0) {
     const float r = 1.0f / sqrtf(ss / (float)norm_dim + eps);
-    for (int d = lane; d < norm_dim; d += 32) x[d] = x[d] * r * w[d];
+    for (int d = lane; d < norm_dim; d += 32) x[d] = w ? x[d] * r * w[d] : x[d] * r;
   }
+  __syncwarp();
+  if (temp != 1.0f)
+    for (int d = lane; d < hd; d += 32) x[d] *= temp;
   __syncwarp();
   TA* dst = (cache && head >= nh) ? cache + pg.offset(slot, pos, 0, head - nh) : nullptr;
   auto turned = [&](int d) {
@@ -254,36 +262,37 @@ k_norm_rope_append(TA* __restrict__ qkv, int ld, const float* __restrict__ inv_f
 
 // cache may be null (a layer that reads another layer's keys and values writes none).
 // nv: value heads of a row (nkv unless key heads share value heads); q_norm / k_norm (both or neither): the weights of
-// a norm over the first norm_dim values of every q / k head before the rotation.
+// a norm over the first norm_dim values of every q / k head before the rotation (null with norm_dim > 0: a norm without weight).
+// temp_every > 0: the queries' factor by position.
 // seq_len[i] is the length of sequence i after this step.
 extern "C" int cima_rope_append(void* qkv, int dtype, int ld, const float* inv_freq, int rotary_dim,
                                 const int* row_pos, const int* row_seq, const int* seq_slot, const int* seq_len,
                                 void* cache, const int* table, int table_width, int ring, int page_size,
                                 int T, int nh, int nkv, int hd, int nv, const float* q_norm, const float* k_norm, int norm_dim,
-                                float eps, float amp, cudaStream_t stream) {
+                                float eps, float amp, float temp_coef, int temp_every, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (hd <= 0 || hd > 256 || rotary_dim < 0 || rotary_dim > hd || (rotary_dim & 1))
     return cima_fail(CIMA_E_SIZE, "rope_append: head_dim %d (at most 256) and an even rotary_dim %d <= head_dim are needed", hd, rotary_dim);
   if (nv < 0 || nv > nkv || (nv > 0 && nkv % nv)) return cima_fail(CIMA_E_SIZE, "rope_append: %d value heads must divide the %d key heads", nv, nkv);
   if (ld < (nh + nkv + nv) * hd) return cima_fail(CIMA_E_SIZE, "rope_append: row stride %d is smaller than (heads + key heads + value heads) * head_dim = %d", ld, (nh + nkv + nv) * hd);
-  if ((q_norm != nullptr) != (k_norm != nullptr) || (q_norm && (norm_dim <= 0 || norm_dim > hd)))
-    return cima_fail(CIMA_E_ARG, "rope_append: the norm takes weights for q and for k and 1 <= norm_dim %d <= head_dim %d", norm_dim, hd);
+  if ((q_norm != nullptr) != (k_norm != nullptr) || norm_dim < 0 || norm_dim > hd || (q_norm && norm_dim <= 0) || temp_every < 0)
+    return cima_fail(CIMA_E_ARG, "rope_append: the norm takes weights for q and for k (or none) and 1 <= norm_dim %d <= head_dim %d; the temperature's step %d must not be negative", norm_dim, hd, temp_every);
   if (cache && (page_size <= 0 || table_width <= 0)) return cima_fail(CIMA_E_SIZE, "rope_append: page size %d and table width %d must be positive", page_size, table_width);
   CimaPaged pg{table, table_width, ring, page_size, nkv, hd};
-  if (q_norm || nv != nkv) {
+  if (norm_dim > 0 || temp_every > 0 || nv != nkv) {
     const dim3 grid((unsigned)((nh + nkv + nv + 3) / 4), (unsigned)T);
     if (T > 65535) return cima_fail(CIMA_E_SIZE, "rope_append: %d rows exceed one launch of the general kernel; the caller cuts them", T);
     int rc_;
     const size_t bytes = dtype == CIMA_F32 ? 4 : 2;
     const bool vec = hd % 4 == 0 && ld % 4 == 0 && ((uintptr_t)qkv % (4 * bytes)) == 0 && ((uintptr_t)cache % (4 * bytes)) == 0;
     if (vec) {
-      if (dtype == CIMA_F32) rc_ = cima_launch(k_norm_rope_append<float, 4>, grid, dim3(128), (size_t)0, stream, 1, (float*)qkv, ld, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, (float*)cache, pg, nh, nkv, nv, hd, q_norm, k_norm, norm_dim, eps, amp);
-      else if (dtype == CIMA_BF16) rc_ = cima_launch(k_norm_rope_append<__nv_bfloat16, 4>, grid, dim3(128), (size_t)0, stream, 1, (__nv_bfloat16*)qkv, ld, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, (__nv_bfloat16*)cache, pg, nh, nkv, nv, hd, q_norm, k_norm, norm_dim, eps, amp);
+      if (dtype == CIMA_F32) rc_ = cima_launch(k_norm_rope_append<float, 4>, grid, dim3(128), (size_t)0, stream, 1, (float*)qkv, ld, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, (float*)cache, pg, nh, nkv, nv, hd, q_norm, k_norm, norm_dim, eps, amp, temp_coef, temp_every);
+      else if (dtype == CIMA_BF16) rc_ = cima_launch(k_norm_rope_append<__nv_bfloat16, 4>, grid, dim3(128), (size_t)0, stream, 1, (__nv_bfloat16*)qkv, ld, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, (__nv_bfloat16*)cache, pg, nh, nkv, nv, hd, q_norm, k_norm, norm_dim, eps, amp, temp_coef, temp_every);
       else return cima_fail(CIMA_E_DTYPE, "rope_append: dtype code %d is neither float32 nor bfloat16", dtype);
       return rc_ ? rc_ : cima_launch_result();
     }
-    if (dtype == CIMA_F32) rc_ = cima_launch(k_norm_rope_append<float, 1>, grid, dim3(128), (size_t)0, stream, 1, (float*)qkv, ld, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, (float*)cache, pg, nh, nkv, nv, hd, q_norm, k_norm, norm_dim, eps, amp);
-    else if (dtype == CIMA_BF16) rc_ = cima_launch(k_norm_rope_append<__nv_bfloat16, 1>, grid, dim3(128), (size_t)0, stream, 1, (__nv_bfloat16*)qkv, ld, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, (__nv_bfloat16*)cache, pg, nh, nkv, nv, hd, q_norm, k_norm, norm_dim, eps, amp);
+    if (dtype == CIMA_F32) rc_ = cima_launch(k_norm_rope_append<float, 1>, grid, dim3(128), (size_t)0, stream, 1, (float*)qkv, ld, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, (float*)cache, pg, nh, nkv, nv, hd, q_norm, k_norm, norm_dim, eps, amp, temp_coef, temp_every);
+    else if (dtype == CIMA_BF16) rc_ = cima_launch(k_norm_rope_append<__nv_bfloat16, 1>, grid, dim3(128), (size_t)0, stream, 1, (__nv_bfloat16*)qkv, ld, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, (__nv_bfloat16*)cache, pg, nh, nkv, nv, hd, q_norm, k_norm, norm_dim, eps, amp, temp_coef, temp_every);
     else return cima_fail(CIMA_E_DTYPE, "rope_append: dtype code %d is neither float32 nor bfloat16", dtype);
     return rc_ ? rc_ : cima_launch_result();
   }

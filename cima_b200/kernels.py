@@ -15,7 +15,7 @@ import torch
 from .csrc.build import BuildError, library_path
 
 F32, BF16 = 0, 1
-ABI_VERSION = 30
+ABI_VERSION = 31
 SPLIT_BLOCKS = 296          # blocks of the decode attention that one wave holds (two per SM, 148 SMs)
 TC_ATTENTION_MIN_LEN = 256  # prompts from this length on take the tcgen05 attention (head_dim 64 or 128)
 SPLIT_FEW_BLOCKS = 148      # below this many blocks at 8 splits, more splits are taken
@@ -70,14 +70,14 @@ _SIGNATURES = {
     "cima_linear_skinny_norm": [_vp, _vp, _i, _f, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "cima_qkv_rope_skinny": [_vp, _vp, _i, _f, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i,
                              _i, _i, _i, _i, _vp],
-    "cima_rope_append": [_vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _f, _f, _vp],
+    "cima_rope_append": [_vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _f, _f, _f, _i, _vp],
     "cima_attention_plain": [_vp, _i, _i, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i,
-                             _f, _i, _i, _i, _f, _i, _i, _vp, _vp],
-    "cima_attention_decode": [_vp, _i, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _f, _i, _i, _vp, _vp],
-    "cima_attention_prefill": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i, _i, _vp, _vp],
-    "cima_attention_extend": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _f, _i, _i, _vp, _vp],
+                             _f, _i, _i, _i, _f, _i, _i, _vp, _i, _vp],
+    "cima_attention_decode": [_vp, _i, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _f, _i, _i, _vp, _i, _vp],
+    "cima_attention_prefill": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i, _i, _vp, _i, _vp],
+    "cima_attention_extend": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _f, _i, _i, _vp, _i, _vp],
     "cima_attention_extend_tc": [_vp, _i, _vp, _vp, _vp, _vp, ctypes.c_longlong, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
-                                 _f, _i, _vp, _i, _f, _vp, _vp],
+                                 _f, _i, _vp, _i, _f, _vp, _i, _vp],
     "cima_short_conv": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
     "cima_dyt": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "cima_dyt_add": [_vp, _vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
@@ -85,12 +85,12 @@ _SIGNATURES = {
                           _i, _vp],
     "cima_recurrence": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "cima_delta_prepare": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
-    "cima_group_rmsnorm_gate": [_vp, _vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _f, _vp],
+    "cima_group_rmsnorm_gate": [_vp, _vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _f, _i, _vp, _vp, _f, _vp],
     "cima_rms_mean": [_vp, _vp, _i, _vp, _i, _i, _f, _i, _vp],
-    "cima_moe_route": [_vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp],
+    "cima_moe_route": [_vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp],
     "cima_moe_sort": [_vp, _i, _i, _vp, _vp, _vp, _vp],
     "cima_moe_gemm": [_vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
-    "cima_moe_combine": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _i, _vp],
+    "cima_moe_combine": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _i, _vp, _i, _vp, _i, _vp],
     "cima_moe_sort_tiles": [_vp, _i, _i, _i, _i, _vp, _vp, _vp],
     "cima_moe_gather_rows": [_vp, _vp, _vp, _i, _i, _i, _vp],
     "cima_moe_few": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
@@ -106,11 +106,15 @@ _SIGNATURES = {
 
     "cima_head_linear_append": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _f, _vp, _vp, _i, _i, _i, _vp, _vp, _vp,
                                 _i, _vp],
-    "cima_attention_prefill_tc": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _f, _vp, _vp],
+    "cima_attention_prefill_tc": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _f, _vp, _i, _vp],
     "cima_gemm_tcgen05_pair": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp],
     "cima_diff_combine": [_vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _f, _vp],
     "cima_scale_add_group_rmsnorm": [_vp, _vp, _f, _vp, _vp, _i, _i, _i, _i, _f, _vp],
     "cima_cast_rows": [_vp, _vp, _i, _sz, _vp],
+    "cima_memory": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _f, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp],
+    "cima_channel_decay": [_vp, _i, _i, _vp, _i, _vp, _f, _vp, _i, _i, _i, _vp],
+    "cima_scalar_gates": [_vp, _i, _i, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
+    "cima_branch_norm": [_vp, _vp, _vp, _vp, _i, _vp, _i, _i, _f, _f, _vp],
     "cima_softcap": [_vp, _sz, _f, _vp],
     "cima_argmax": [_vp, _i, _i, _i, _vp, _vp],
     "cima_sample": [_vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _vp],
@@ -416,12 +420,13 @@ class Kernels:
     # ------------------------------------------------------------------ attention
     def rope_append(self, qkv: torch.Tensor, inv_freq: torch.Tensor, rotary_dim: int, row_pos, row_seq, seq_slot,
                     seq_len, kv, n_heads: int, n_kv_heads: int, head_dim: int, v_heads: Optional[int] = None,
-                    qk_norm=None, amplitude: float = 1.0) -> None:
+                    qk_norm=None, amplitude: float = 1.0, q_temp=None) -> None:
         """Rotate q and k of ``qkv`` in place and append k, v to the layer's pages (``kv`` a LayerKV or None).
         ``v_heads``: value heads of a row where they are fewer than the key heads (neighbouring key heads share one; the
         pages' value plane holds them in its first heads).  ``qk_norm = (wq, wk, dim, eps)``: before the rotation the first
-        ``dim`` values of every q (k) head are divided by their root mean square and multiplied by wq (wk) [dim].
-        ``amplitude``: a factor of every sine and cosine."""
+        ``dim`` values of every q (k) head are divided by their root mean square and multiplied by wq (wk) [dim]; wq and wk
+        None: only divided.  ``amplitude``: a factor of every sine and cosine.  ``q_temp = (coef, every)``: a row's queries at
+        position p are multiplied by 1 + coef ln(floor((p + 1) / every) + 1)."""
         self._need(qkv, "qkv", None, 2); self._need(inv_freq, "inv_freq", torch.float32, 1)
         for n, t in (("row_pos", row_pos), ("row_seq", row_seq), ("seq_slot", seq_slot), ("seq_len", seq_len)):
             self._need(t, n, torch.int32, 1)
@@ -442,22 +447,25 @@ class Kernels:
         norm = (None, None, 0, 0.0)
         if qk_norm is not None:
             wq, wk, nd, eps = qk_norm
-            self._need(wq, "wq", torch.float32, 1); self._need(wk, "wk", torch.float32, 1)
-            if wq.numel() != nd or wk.numel() != nd:
-                raise KernelError(f"rope_append: the norm's weights have {wq.numel()} and {wk.numel()} values, expected {nd}")
-            norm = (wq.data_ptr(), wk.data_ptr(), int(nd), float(eps))
-        if not self._admit("rope_append", 2 * qkv.numel() * qkv.element_size()): return
-        step = 65535 if (qk_norm is not None or nv != n_kv_heads) else T       # the general kernel takes a row a block of grid.y
+            if wq is not None or wk is not None:
+                self._need(wq, "wq", torch.float32, 1); self._need(wk, "wk", torch.float32, 1)
+                if wq.numel() != nd or wk.numel() != nd:
+                    raise KernelError(f"rope_append: the norm's weights have {wq.numel()} and {wk.numel()} values, expected {nd}")
+            norm = (_ptr(wq), _ptr(wk), int(nd), float(eps))
+        coef, every = (float(q_temp[0]), int(q_temp[1])) if q_temp is not None else (0.0, 0)
+        touched = T * (n_heads + n_kv_heads + nv) * head_dim          # (columns behind the value heads are left alone)
+        if not self._admit("rope_append", 2 * touched * qkv.element_size()): return
+        step = 65535 if (qk_norm is not None or every or nv != n_kv_heads) else T       # the general kernel takes a row a block of grid.y
         for r0 in range(0, T, step):
             r1 = min(T, r0 + step)
             self._check(self.lib.cima_rope_append(qkv[r0:r1].data_ptr(), dtype_code(qkv.dtype), qkv.shape[1], inv_freq.data_ptr(),
                                                   rotary_dim, row_pos[r0:r1].data_ptr(), row_seq[r0:r1].data_ptr(), seq_slot.data_ptr(),
                                                   seq_len.data_ptr(), *args, r1 - r0, n_heads, n_kv_heads, head_dim, nv, *norm,
-                                                  float(amplitude), self._stream()), "rope_append")
+                                                  float(amplitude), coef, every, self._stream()), "rope_append")
 
     def attention_plain(self, qkv: torch.Tensor, kv, row_pos, row_seq, seq_slot, seq_first_row, out: torch.Tensor,
                         n_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int,
-                        from_cache: bool, sink: float = 0.0, keep_first: int = 0, v_group: int = 1, head_sink=None) -> None:
+                        from_cache: bool, sink: float = 0.0, keep_first: int = 0, v_group: int = 1, head_sink=None, gate_col: int = 0) -> None:
         self._need(qkv, "qkv", None, 2); self._need(out, "out", qkv.dtype, 2)
         self._need_head_sink(head_sink, n_heads)
         T = qkv.shape[0]
@@ -477,7 +485,7 @@ class Kernels:
                                                   seq_first_row.data_ptr(), out.data_ptr(), out.shape[1], T,
                                                   n_heads, n_kv_heads, head_dim, scale, window,
                                                   1 if from_cache else 0, planes, sink, keep_first, v_group, _ptr(head_sink),
-                                                  self._stream()), "attention_plain")
+                                                  gate_col, self._stream()), "attention_plain")
 
     def _need_head_sink(self, head_sink, n_heads: int) -> None:
         if head_sink is not None:
@@ -515,7 +523,7 @@ class Kernels:
 
     def attention(self, qkv: torch.Tensor, kv, batch, out: torch.Tensor, n_heads: int, n_kv_heads: int,
                   head_dim: int, scale: float, window: int, from_cache: bool, after_append: bool = False,
-                  sink: float = 0.0, keep_first: int = 0, v_group: int = 1, head_sink=None) -> None:
+                  sink: float = 0.0, keep_first: int = 0, v_group: int = 1, head_sink=None, gate_col: int = 0) -> None:
         """Attention of a step's rows: over the step's own keys (a prompt from position 0) or over the
         cache.  Chooses the kernel; every choice computes the same function.  ``after_append``: the kernel
         launched just before wrote nothing but ``qkv`` and the newest position of each sequence in the cache.
@@ -523,37 +531,38 @@ class Kernels:
         ``keep_first``: with a window, the first so many positions of a sequence stay visible below it.  ``v_group``: that
         many neighbouring key heads share one value head (a step's rows and the pages' value plane hold
         n_kv_heads / v_group value heads).  ``head_sink`` (float32 [n_heads], instead of ``sink``): head h's denominator
-        also holds exp(head_sink[h]), an entry that is not scaled and carries no value."""
+        also holds exp(head_sink[h]), an entry that is not scaled and carries no value.  ``gate_col`` > 0: a row of ``qkv`` holds
+        one gate value for each value of its result from that column on, and the result leaves times their sigmoid."""
         general = keep_first > 0 or v_group > 1        # the tcgen05 kernels take neither
         if (from_cache and qkv.dtype is torch.bfloat16 and kv.page_size == 64 and head_dim % 16 == 0
                 and head_dim <= 128 and batch.n_rows == batch.n_seqs):
             return self.attention_decode(qkv, kv, batch.seq_slot, batch.seq_len, out, n_heads, n_kv_heads, head_dim,
                                          scale, window, batch.max_len, early=after_append, sink=sink,
-                                         keep_first=keep_first, v_group=v_group, head_sink=head_sink)
+                                         keep_first=keep_first, v_group=v_group, head_sink=head_sink, gate_col=gate_col)
         many = (not general and qkv.dtype is torch.bfloat16 and head_dim in (64, 128) and qkv.shape[1] % 8 == 0
                 and getattr(batch, "n_q_tiles_tc", 0) > 0 and getattr(batch, "max_rows", 0) >= TC_ATTENTION_MIN_LEN)
         if from_cache and many and kv.page_size == 64 and kv.storage.numel() // head_dim < 2 ** 31:
             return self.attention_prefill_tc(qkv, batch, out, n_heads, n_kv_heads, head_dim, scale, window, kv=kv, sink=sink,
-                                             head_sink=head_sink)
+                                             head_sink=head_sink, gate_col=gate_col)
         if (from_cache and qkv.dtype is torch.bfloat16 and kv.page_size == 64 and head_dim % 16 == 0
                 and head_dim <= 128 and qkv.shape[1] % 8 == 0 and getattr(batch, "n_q_tiles", 0) > 0):
             return self.attention_extend(qkv, kv, batch, out, n_heads, n_kv_heads, head_dim, scale, window, sink=sink,
-                                         keep_first=keep_first, v_group=v_group, head_sink=head_sink)
+                                         keep_first=keep_first, v_group=v_group, head_sink=head_sink, gate_col=gate_col)
         if not from_cache and many:
             return self.attention_prefill_tc(qkv, batch, out, n_heads, n_kv_heads, head_dim, scale, window, sink=sink,
-                                             head_sink=head_sink)
+                                             head_sink=head_sink, gate_col=gate_col)
         if (not from_cache and qkv.dtype is torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 128
                 and qkv.shape[1] % 8 == 0 and getattr(batch, "n_q_tiles", 0) > 0):
             return self.attention_prefill(qkv, batch.q_tile_seq, batch.q_tile_row0, batch.seq_first_row, out,
                                           n_heads, n_kv_heads, head_dim, scale, window, sink=sink,
-                                          keep_first=keep_first, v_group=v_group, head_sink=head_sink)
+                                          keep_first=keep_first, v_group=v_group, head_sink=head_sink, gate_col=gate_col)
         self.attention_plain(qkv, kv, batch.row_pos, batch.row_seq, batch.seq_slot, batch.seq_first_row, out,
                              n_heads, n_kv_heads, head_dim, scale, window, from_cache, sink=sink, keep_first=keep_first,
-                             v_group=v_group, head_sink=head_sink)
+                             v_group=v_group, head_sink=head_sink, gate_col=gate_col)
 
     def attention_prefill(self, qkv: torch.Tensor, tile_seq, tile_row0, seq_first_row, out: torch.Tensor,
                           n_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int, sink: float = 0.0,
-                          keep_first: int = 0, v_group: int = 1, head_sink=None) -> None:
+                          keep_first: int = 0, v_group: int = 1, head_sink=None, gate_col: int = 0) -> None:
         """Flash attention of ragged prompts that start at position 0 (bf16, head_dim <= 128);
         ``tile_seq``/``tile_row0`` list the blocks of 64 query rows."""
         self._need(qkv, "qkv", torch.bfloat16, 2); self._need(out, "out", torch.bfloat16, 2)
@@ -567,11 +576,11 @@ class Kernels:
         self._check(self.lib.cima_attention_prefill(qkv.data_ptr(), qkv.shape[1], tile_seq.data_ptr(), tile_row0.data_ptr(),
                                                     seq_first_row.data_ptr(), out.data_ptr(), out.shape[1], T,
                                                     tile_seq.numel(), n_heads, n_kv_heads, head_dim, scale, window, sink,
-                                                    keep_first, v_group, _ptr(head_sink), self._stream()), "attention_prefill")
+                                                    keep_first, v_group, _ptr(head_sink), gate_col, self._stream()), "attention_prefill")
 
     def attention_extend(self, qkv: torch.Tensor, kv, batch, out: torch.Tensor, n_heads: int, n_kv_heads: int,
                          head_dim: int, scale: float, window: int, sink: float = 0.0, keep_first: int = 0,
-                         v_group: int = 1, head_sink=None) -> None:
+                         v_group: int = 1, head_sink=None, gate_col: int = 0) -> None:
         """Flash attention of sequences that bring several rows to a cache that already holds keys (bf16, pages of
         64, head_dim <= 128): the rows of sequence s stand at positions seq_len[s] - rows .. seq_len[s] - 1, and all
         keys, the step's own included, are read from the layer's pages.  ``batch`` brings the blocks of 64 rows."""
@@ -587,10 +596,11 @@ class Kernels:
             batch.seq_first_row.data_ptr(), kv.storage.data_ptr(), kv.block_table.data_ptr(), kv.block_table.shape[1],
             kv.ring_pages, kv.page_size, batch.seq_slot.data_ptr(), batch.seq_len.data_ptr(), out.data_ptr(), out.shape[1],
             T, batch.q_tile_seq.numel(), n_heads, n_kv_heads, head_dim, scale, window, kv.planes, sink, keep_first, v_group,
-            _ptr(head_sink), self._stream()), "attention_extend")
+            _ptr(head_sink), gate_col, self._stream()), "attention_extend")
 
     def attention_prefill_tc(self, qkv: torch.Tensor, batch, out: torch.Tensor, n_heads: int, n_kv_heads: int,
-                             head_dim: int, scale: float, window: int, kv=None, sink: float = 0.0, head_sink=None) -> None:
+                             head_dim: int, scale: float, window: int, kv=None, sink: float = 0.0, head_sink=None,
+                             gate_col: int = 0) -> None:
         """Flash attention of ragged prompts on the tcgen05 tensor cores (bf16, head_dim 64 or 128): blocks of 128
         query rows, both products with their results in tensor memory.  ``batch`` brings the blocks
         (``q_tile_tc_*``).  Without ``kv`` the sequences start at position 0 and the keys are the step's own rows;
@@ -611,18 +621,18 @@ class Kernels:
                 batch.seq_first_row.data_ptr(), kv.storage.data_ptr(), kv.storage.shape[0], kv.block_table.data_ptr(),
                 kv.block_table.shape[1], kv.ring_pages, kv.page_size, batch.seq_slot.data_ptr(), batch.seq_len.data_ptr(),
                 out.data_ptr(), out.shape[1], T, batch.n_q_tiles_tc, n_heads, n_kv_heads, head_dim, scale, window,
-                self._error_flag.data_ptr(), kv.planes, sink, _ptr(head_sink), self._stream()), "attention_extend_tc")
+                self._error_flag.data_ptr(), kv.planes, sink, _ptr(head_sink), gate_col, self._stream()), "attention_extend_tc")
             return
         self._check(self.lib.cima_attention_prefill_tc(
             qkv.data_ptr(), qkv.shape[1], batch.q_tile_tc_seq.data_ptr(), batch.q_tile_tc_row0.data_ptr(),
             batch.seq_first_row.data_ptr(), out.data_ptr(),
             out.shape[1], T, batch.n_q_tiles_tc, n_heads, n_kv_heads, head_dim, scale, window,
-            self._error_flag.data_ptr(), sink, _ptr(head_sink), self._stream()), "attention_prefill_tc")
+            self._error_flag.data_ptr(), sink, _ptr(head_sink), gate_col, self._stream()), "attention_prefill_tc")
 
     def attention_decode(self, qkv: torch.Tensor, kv, seq_slot, seq_len, out: torch.Tensor, n_heads: int,
                          n_kv_heads: int, head_dim: int, scale: float, window: int, max_len: int = 0,
                          n_splits: Optional[int] = None, early: bool = False, sink: float = 0.0, keep_first: int = 0,
-                         v_group: int = 1, head_sink=None) -> None:
+                         v_group: int = 1, head_sink=None, gate_col: int = 0) -> None:
         """One query per sequence over the paged cache (bf16, pages of 64, head_dim <= 128), keys split
         over ``n_splits`` blocks per (sequence, kv head).  ``max_len`` (0 = unknown) only bounds the
         number of splits chosen here.  ``early``: the kernel launched just before this one wrote neither
@@ -663,7 +673,7 @@ class Kernels:
             qkv.data_ptr(), qkv.shape[1], kv.storage.data_ptr(), kv.block_table.data_ptr(), kv.block_table.shape[1],
             kv.ring_pages, kv.page_size, seq_slot.data_ptr(), seq_len.data_ptr(), _ptr(part_o), _ptr(part_ml),
             out.data_ptr(), out.shape[1], B, n_heads, n_kv_heads, head_dim, scale, window, n_splits, int(early),
-            kv.planes, sink, keep_first, v_group, _ptr(head_sink), self._stream()), "attention_decode")
+            kv.planes, sink, keep_first, v_group, _ptr(head_sink), gate_col, self._stream()), "attention_decode")
         if n_splits > 1:
             self.launches += 1
 
@@ -1051,22 +1061,33 @@ class Kernels:
                                                 self._stream()), "delta_prepare")
 
     def group_rmsnorm_gate(self, o: torch.Tensor, w: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, groups: int,
-                           eps: float) -> None:
+                           eps: float, silu: bool = False, divisor=None) -> None:
         """out = o / sqrt(mean(o^2) + eps) * w * sigmoid(gate) over each of ``groups`` equal parts of a row: o float32
-        [T, groups * n]; w [n] (one weight for all groups) or [groups * n]; gate [T, groups * n] in out's dtype (rows may
-        be slices) or None."""
+        [T, groups * n]; w [n] (one weight for all groups) or [groups * n]; gate [T, groups * n] in out's dtype or float32 (rows
+        may be slices) or None.  ``silu``: the gate passes z sigmoid(z) instead.  ``divisor = (den, low, e)``, den and low float32
+        [T, groups]: every part is divided by max(|den|, low) + e first."""
         self._need(o, "o", torch.float32, 2); self._need(w, "w", torch.float32, 1); self._need(out, "out", None, 2)
         T, W = o.shape
         if groups <= 0 or W % groups or out.shape != o.shape or w.numel() not in (W // groups, W):
             raise KernelError(f"group_rmsnorm_gate: o {tuple(o.shape)}, w {tuple(w.shape)}, out {tuple(out.shape)}, {groups} groups do not agree")
         n = W // groups
-        if gate is not None and (gate.dim() != 2 or gate.stride(1) != 1 or tuple(gate.shape) != (T, W) or gate.dtype is not out.dtype):
+        if gate is not None and (gate.dim() != 2 or gate.stride(1) != 1 or tuple(gate.shape) != (T, W)
+                                 or gate.dtype not in (out.dtype, torch.float32)):
             raise KernelError(f"group_rmsnorm_gate: the gate {tuple(gate.shape)} {gate.dtype} must match the output")
+        den = low = None
+        div_eps = 0.0
+        if divisor is not None:
+            den, low, div_eps = divisor
+            for name, t in (("den", den), ("low", low)):
+                self._need(t, name, torch.float32, 2)
+                if tuple(t.shape) != (T, groups):
+                    raise KernelError(f"group_rmsnorm_gate: {name} is {tuple(t.shape)}, expected {(T, groups)}")
         shared = int(w.numel() == n and groups > 1)
-        if not self._admit("group_rmsnorm_gate", T * W * (4 + 2 * out.element_size())): return
-        self._check(self.lib.cima_group_rmsnorm_gate(o.data_ptr(), w.data_ptr(), _ptr(gate), gate.stride(0) if gate is not None else 0,
-                                                     out.data_ptr(), dtype_code(out.dtype), T, groups, n, shared, eps,
-                                                     self._stream()), "group_rmsnorm_gate")
+        if not self._admit("group_rmsnorm_gate", T * W * (4 + out.element_size() + (gate.element_size() if gate is not None else 0))): return
+        gd = dtype_code(gate.dtype) if gate is not None else dtype_code(out.dtype)
+        self._check(self.lib.cima_group_rmsnorm_gate(o.data_ptr(), w.data_ptr(), _ptr(gate), gate.stride(0) if gate is not None else 0, gd,
+                                                     out.data_ptr(), dtype_code(out.dtype), T, groups, n, shared, eps, int(bool(silu)),
+                                                     _ptr(den), _ptr(low), float(div_eps), self._stream()), "group_rmsnorm_gate")
 
     def rms_mean(self, ys, ws, x: torch.Tensor, eps: float, assign: bool = False) -> None:
         """x += mean over the branches b of  y_b / sqrt(mean(y_b^2) + eps) * w_b:  y_b float32 [T, H], w_b [H], at most 4.
@@ -1137,11 +1158,110 @@ class Kernels:
         if not self._admit("softcap", logits.numel() * 8): return
         self._check(self.lib.cima_softcap(logits.data_ptr(), logits.numel(), cap, self._stream()), "softcap")
 
+    def branch_norm(self, x: torch.Tensor, y: torch.Tensor, w: torch.Tensor, eps: float, h: Optional[torch.Tensor] = None,
+                    next_norm=None) -> None:
+        """x <- x + y / sqrt(mean(y^2) + eps) * w (x, y float32 [T, W], x in place); ``h`` (either dtype, optional) receives the
+        new rows, or with ``next_norm = (w2, eps2)`` the new rows' RMS norm."""
+        self._need(x, "x", torch.float32, 2); self._need(y, "y", torch.float32, 2); self._need(w, "w", torch.float32, 1)
+        T, W = x.shape
+        if y.shape != x.shape or w.numel() != W:
+            raise KernelError(f"branch_norm: x {tuple(x.shape)}, y {tuple(y.shape)} and w {tuple(w.shape)} do not agree")
+        if h is not None:
+            self._need(h, "h", None, 2)
+            if h.shape != x.shape:
+                raise KernelError(f"branch_norm: h {tuple(h.shape)} is not x's {tuple(x.shape)}")
+        w2, eps2 = (None, 0.0) if next_norm is None else next_norm
+        if w2 is not None:
+            self._need(w2, "w2", torch.float32, 1)
+            if h is None or w2.numel() != W:
+                raise KernelError(f"branch_norm: the second norm takes rows to write to and {W} weights")
+        if not self._admit("branch_norm", T * W * (12 + (h.element_size() if h is not None else 0))): return
+        self._check(self.lib.cima_branch_norm(x.data_ptr(), y.data_ptr(), w.data_ptr(), _ptr(h), dtype_code(h.dtype) if h is not None else F32,
+                                              _ptr(w2), T, W, eps, eps2, self._stream()), "branch_norm")
+
+    # ------------------------------------------------------------------ matrix memories
+    MEMORY_SEGMENT = 256        # tokens of a segment of a long step's recurrence
+
+    def memory_segments(self, batch) -> int:
+        """Into how many segments at most a step's recurrence is cut (1: not at all): a number of the longest sequence's rows."""
+        rows = int(getattr(batch, "max_rows", 0) or 0)
+        return 1 if rows < 2 * self.MEMORY_SEGMENT else -(-rows // self.MEMORY_SEGMENT)
+
+    def memory(self, q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, g: torch.Tensor, state: torch.Tensor, batch, out: torch.Tensor,
+               heads: int, dim: int, vdim: int, qscale: float, norm_state: Optional[torch.Tensor] = None,
+               norm_out: Optional[torch.Tensor] = None) -> None:
+        """A linear recurrence with a matrix a head over the step's rows, the state S [slots, heads, dim, vdim] (float32) carried on.
+        Channel form, g [T, heads * dim]: S <- diag(g) S + k v^T.  Scalar form, g [T, heads, 2] = (a, b): S <- a S + b k v^T, beside
+        it n <- a n + b k in ``norm_state`` [slots, heads, dim], and ``norm_out`` [T, heads] = n . (qscale q).  Both: o = S^T (qscale q),
+        out [T, heads * vdim] float32.  q, k, v of one dtype, column slices of wider matrices as well.  A step of at least two
+        segments' rows in a sequence is cut into segments that run side by side."""
+        scalar = g.dim() == 3
+        self._need(state, "state", torch.float32, 4); self._need(out, "out", torch.float32, 2); self._need(g, "g", torch.float32)
+        T = batch.n_rows
+        for n, t, w in (("q", q, heads * dim), ("k", k, heads * dim), ("v", v, heads * vdim)):
+            if t.dim() != 2 or t.stride(1) != 1 or tuple(t.shape) != (T, w) or not t.is_cuda or t.dtype is not v.dtype:
+                raise KernelError(f"memory: {n} {tuple(t.shape)} {t.dtype} must be GPU rows of the step, {w} values wide, one dtype, unit column stride")
+        want = (T, heads, 2) if scalar else (T, heads * dim)
+        if tuple(state.shape[1:]) != (heads, dim, vdim) or tuple(out.shape) != (T, heads * vdim) or tuple(g.shape) != want:
+            raise KernelError(f"memory: state {tuple(state.shape)}, out {tuple(out.shape)}, g {tuple(g.shape)} do not agree with {heads} heads of {dim} x {vdim}")
+        if scalar:
+            self._need(norm_state, "norm_state", torch.float32, 3); self._need(norm_out, "norm_out", torch.float32, 2)
+            if tuple(norm_state.shape[1:]) != (heads, dim) or tuple(norm_out.shape) != (T, heads):
+                raise KernelError(f"memory: norm_state {tuple(norm_state.shape)} / norm_out {tuple(norm_out.shape)} do not agree with {heads} heads of {dim}")
+        if not self._admit("memory[scalar]" if scalar else "memory[channel]",
+                           batch.n_seqs * heads * dim * vdim * 8 + T * heads * ((2 * dim + vdim) * v.element_size() + vdim * 4 + (8 if scalar else 4 * dim)),
+                           5.0 * T * heads * dim * vdim): return
+        segs = self.memory_segments(batch)
+        buf = nbuf = dbuf = None
+        if segs > 1:
+            units = batch.n_seqs * segs
+            buf = torch.empty(units * heads * dim * vdim, dtype=torch.float32, device=q.device)
+            dbuf = torch.empty(units * heads * (1 if scalar else dim), dtype=torch.float32, device=q.device)
+            if scalar:
+                nbuf = torch.empty(units * heads * dim, dtype=torch.float32, device=q.device)
+        self._check(self.lib.cima_memory(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0), dtype_code(v.dtype),
+                                         g.data_ptr(), int(scalar), state.data_ptr(), _ptr(norm_state), batch.seq_slot.data_ptr(),
+                                         batch.seq_first_row.data_ptr(), out.data_ptr(), _ptr(norm_out), float(qscale), T, batch.n_seqs,
+                                         heads, dim, vdim, self.MEMORY_SEGMENT, segs, _ptr(buf), _ptr(nbuf), _ptr(dbuf), self._stream()), "memory")
+        if segs > 1:
+            self.launches += 2
+
+    def channel_decay(self, a1: torch.Tensor, w2: torch.Tensor, bias: torch.Tensor, tau: float, g: torch.Tensor) -> None:
+        """g = sigmoid(a1 w2^T + bias)^(1 / tau) in float32: a1 [T, rank] (rows may be slices), w2 [channels, rank], g [T, channels]."""
+        self._need(w2, "w2", None, 2); self._need(bias, "bias", torch.float32, 1); self._need(g, "g", torch.float32, 2)
+        T, rank = a1.shape
+        C = w2.shape[0]
+        if a1.stride(1) != 1 or w2.shape[1] != rank or bias.numel() != C or tuple(g.shape) != (T, C) or not a1.is_cuda or tau <= 0:
+            raise KernelError(f"channel_decay: a1 {tuple(a1.shape)}, w2 {tuple(w2.shape)}, bias {tuple(bias.shape)}, g {tuple(g.shape)}, tau {tau} do not agree")
+        if not self._admit("channel_decay", T * (rank * a1.element_size() + C * 4) + w2.numel() * w2.element_size(), 2.0 * T * C * rank): return
+        step = 65535 * 8
+        for r0 in range(0, T, step):
+            r1 = min(T, r0 + step)
+            self._check(self.lib.cima_channel_decay(a1[r0:r1].data_ptr(), dtype_code(a1.dtype), a1.stride(0), w2.data_ptr(), dtype_code(w2.dtype),
+                                                    bias.data_ptr(), 1.0 / tau, g[r0:r1].data_ptr(), r1 - r0, rank, C, self._stream()), "channel_decay")
+
+    def scalar_gates(self, z: torch.Tensor, bi: torch.Tensor, bf: torch.Tensor, cap: float, mstate: torch.Tensor, batch,
+                     ab: torch.Tensor, low: torch.Tensor) -> None:
+        """The scalar form's numbers from the gates' projections z [T, >= 2 heads] (input gates of all heads, then forget gates; rows
+        may be slices): i = cap tanh((zi + bi) / cap), f = log sigmoid(cap tanh((zf + bf) / cap)), m' = max(f + m, i) with m carried in
+        ``mstate`` [slots, heads]; ab [T, heads, 2] = (exp(f + m - m'), exp(i - m')), low [T, heads] = exp(-m')."""
+        self._need(mstate, "mstate", torch.float32, 2); self._need(ab, "ab", torch.float32, 3); self._need(low, "low", torch.float32, 2)
+        self._need(bi, "bi", torch.float32, 1); self._need(bf, "bf", torch.float32, 1)
+        heads, T = bi.numel(), batch.n_rows
+        if (z.dim() != 2 or z.stride(1) != 1 or z.shape[0] != T or z.shape[1] < 2 * heads or bf.numel() != heads or mstate.shape[1] != heads
+                or tuple(ab.shape) != (T, heads, 2) or tuple(low.shape) != (T, heads) or not z.is_cuda):
+            raise KernelError(f"scalar_gates: z {tuple(z.shape)}, ab {tuple(ab.shape)}, low {tuple(low.shape)}, state {tuple(mstate.shape)} do not agree with {heads} heads")
+        if not self._admit("scalar_gates", T * heads * (2 * z.element_size() + 12)): return
+        self._check(self.lib.cima_scalar_gates(z.data_ptr(), dtype_code(z.dtype), z.stride(0), bi.data_ptr(), bf.data_ptr(), float(cap),
+                                               mstate.data_ptr(), batch.seq_slot.data_ptr(), batch.seq_first_row.data_ptr(), ab.data_ptr(),
+                                               low.data_ptr(), T, batch.n_seqs, heads, self._stream()), "scalar_gates")
+
     # ------------------------------------------------------------------ routed feed-forward
     ROUTE_SORT_ROWS = 64        # a step of at most this many rows orders its pairs by expert in the routing launch
 
     def moe_route(self, scores: torch.Tensor, top: int, groups: int, keep: int, scale: float, idx: torch.Tensor,
-                  wgt: torch.Tensor, order: bool = False, experts: Optional[int] = None, softmax: bool = False, correction=None):
+                  wgt: torch.Tensor, order: bool = False, experts: Optional[int] = None, softmax: bool = False, correction=None,
+                  real: Optional[int] = None, best_one: bool = False, divide: bool = True):
         """``scores`` float32 [T, E] holds the router's logits (it is scratch afterwards).  s = sigmoid(logits); the
         experts form ``groups`` equal groups of neighbours, a group's score is the sum of its two best, the best
         ``keep`` groups stay, and the ``top`` best experts among them are chosen: idx [T, top] int32, and their weights
@@ -1149,7 +1269,9 @@ class Kernels:
         same launch also orders the pairs by expert; what it returns goes to ``moe_experts`` as ``ordered``.
         ``experts``: the first so many columns of ``scores`` are the experts' (default: all; further columns are left alone).
         ``softmax``: s = softmax(logits) over the experts instead of the sigmoid.  ``correction`` (float32 [experts]): added to s
-        where groups and experts are compared; the weights are made of s itself."""
+        where groups and experts are compared; the weights are made of s itself.  ``real``: only the first so many experts have
+        matrices (default: all; the rest are identity experts, which ``order`` leaves out).  ``best_one``: a group's score is its
+        largest one.  ``divide`` False: the weights are s * scale, not divided by the sum of the chosen."""
         self._need(scores, "scores", torch.float32, 2); self._need(idx, "idx", torch.int32, 2); self._need(wgt, "wgt", torch.float32, 2)
         T, ld = scores.shape
         E = ld if experts is None else int(experts)
@@ -1161,18 +1283,20 @@ class Kernels:
                 raise KernelError(f"moe_route: the correction has {correction.numel()} values for {E} experts")
         if tuple(idx.shape) != (T, top) or tuple(wgt.shape) != (T, top):
             raise KernelError(f"moe_route: idx {tuple(idx.shape)} / wgt {tuple(wgt.shape)} are not {(T, top)}")
+        R = E if real is None else int(real)
         meta = None
         if order and T <= self.ROUTE_SORT_ROWS:
-            meta = torch.empty(2 * (E + 1) + T * top, dtype=torch.int32, device=scores.device)
+            meta = torch.empty(2 * (R + 1) + T * top, dtype=torch.int32, device=scores.device)
         if not self._admit("moe_route", T * (E * 8 + top * 8)): return meta
-        parts = (meta[:E + 1].data_ptr(), meta[E + 1:2 * (E + 1)].data_ptr(), meta[2 * (E + 1):].data_ptr()) if meta is not None else (None, None, None)
-        self._check(self.lib.cima_moe_route(scores.data_ptr(), T, E, ld, top, groups, keep, scale, int(bool(softmax)), _ptr(correction),
+        parts = (meta[:R + 1].data_ptr(), meta[R + 1:2 * (R + 1)].data_ptr(), meta[2 * (R + 1):].data_ptr()) if meta is not None else (None, None, None)
+        self._check(self.lib.cima_moe_route(scores.data_ptr(), T, E, ld, top, groups, keep, scale, int(bool(softmax)),
+                                            int(bool(best_one)), int(bool(divide)), R, _ptr(correction),
                                             idx.data_ptr(), wgt.data_ptr(), *parts, self._stream()), "moe_route")
         return meta
 
     def moe_experts(self, h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, idx: torch.Tensor, wgt: torch.Tensor,
                     x: torch.Tensor, act: int = 0, assign: bool = False, ordered: Optional[torch.Tensor] = None,
-                    limit: float = 0.0, shared=None) -> None:
+                    limit: float = 0.0, shared=None, identity: bool = False) -> None:
         """x[t] += (with ``assign``: =) sum_j wgt[t, j] * W_down[e] (act(W_gate[e] h[t]) * (W_up[e] h[t])), e = idx[t, j], ascending j.
         gate_up [E, 2 ff, H] (an expert's gate rows, then its up rows), down [E, H, ff]; x float32 [T, H].  Four launches:
         the pairs sorted by expert, the two grouped products over tiles of one expert's pairs, the weighted sum.  The
@@ -1180,7 +1304,8 @@ class Kernels:
         tiles of 256 pairs, a warp a feature for the few pairs of a decode step, or the plain tiles (any dtype and size).
         ``limit`` goes with the clamped form of the middle.  ``shared = (rows, gate, col)``: float32 rows [T, H] (a shared
         expert's output) that join the weighted sum in its launch, each row times sigmoid(gate[t, col]) (gate float32
-        [T, n]; None: unweighted)."""
+        [T, n]; None: unweighted).  ``identity``: indices from E on are identity experts: their pairs are in no product and
+        contribute wgt[t, j] * h[t]."""
         tail = (None, None, 0)
         if shared is not None:
             srows, sgate, scol = shared
@@ -1205,9 +1330,12 @@ class Kernels:
                               f"{tuple(idx.shape)}, x {tuple(x.shape)} do not agree")
         P = T * top
         dev = h.device
+        own = (idx.data_ptr(), E, h.data_ptr(), dtype_code(h.dtype)) if identity else (None, 0, None, F32)
+        if identity and not h.is_contiguous():
+            raise KernelError("moe_experts: the rows of h must be contiguous where identity experts return them")
         bf16 = h.dtype is torch.bfloat16 and gate_up.dtype is torch.bfloat16 and H % 8 == 0 and ff % 8 == 0 and h.stride(0) % 8 == 0
         if bf16 and P >= self.MOE_TC_PAIRS:
-            return self._moe_experts_tc(h, gate_up, down, idx, wgt, x, act, assign, limit, tail)
+            return self._moe_experts_tc(h, gate_up, down, idx, wgt, x, act, assign, limit, tail + own)
         few = bf16 and P <= self.MOE_FEW_PAIRS
         meta = ordered if ordered is not None else torch.empty(2 * (E + 1) + P, dtype=torch.int32, device=dev)
         offsets, tiles, perm = meta[:E + 1], meta[E + 1:2 * (E + 1)], meta[2 * (E + 1):]
@@ -1236,13 +1364,13 @@ class Kernels:
                                                    y.data_ptr(), offsets.data_ptr(), tiles.data_ptr(), perm.data_ptr(), P, E, top,
                                                    H, ff, 1, 0, 0.0, self._stream()), "moe_gemm")
         if self._admit("moe_combine", P * H * 4 + T * H * 8):
-            self._check(self.lib.cima_moe_combine(y.data_ptr(), wgt.data_ptr(), None, x.data_ptr(), T, top, H, int(assign), *tail,
+            self._check(self.lib.cima_moe_combine(y.data_ptr(), wgt.data_ptr(), None, x.data_ptr(), T, top, H, int(assign), *tail, *own,
                                                   self._stream()), "moe_combine")
 
     MOE_TC_PAIRS = 1024      # from this many (row, choice) pairs on, bfloat16 experts run on the tcgen05 tiles of 256 pairs
     MOE_FEW_PAIRS = 128      # up to this many, a warp computes a feature for the pairs of an expert (a decode step)
 
-    def _moe_experts_tc(self, h, gate_up, down, idx, wgt, x, act, assign=False, limit: float = 0.0, tail=(None, None, 0)) -> None:
+    def _moe_experts_tc(self, h, gate_up, down, idx, wgt, x, act, assign=False, limit: float = 0.0, tail=(None, None, 0, None, 0, None, F32)) -> None:
         """Many pairs in bfloat16: every expert's pairs are laid out from a multiple of 256 rows on (the rows of h copied
         there), so that each tile of the tcgen05 product multiplies with one expert's matrix."""
         T, H = h.shape

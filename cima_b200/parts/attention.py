@@ -6,13 +6,19 @@ Formulas and order as the reference's layer loop, steps 2-7 (src/models/transfor
 bias before rotation, rotation before caching, scale = spec.scale, head h reads kv head
 h / (heads / kv_heads), no output bias unless the spec says so.
 
-Every size (heads, kv heads, head_dim, window, scale, bias flags) is a field of the spec.  Two more are ``params``:
+Every size (heads, kv heads, head_dim, window, scale, bias flags) is a field of the spec.  More are ``params``:
 ``v_dim``, a value size that differs from the key size, and ``sink``, a number of entries of score 0 that carry no
 value and join every row's softmax denominator (1: p_j = exp(s_j) / (1 + sum exp(s))); ``keep_first``: with a window, a
 sequence's first so many positions stay visible below it, at their own positions (such a layer keeps every page: a ring
 would hand the first pages on).  A position encoding whose pairs are neighbours (``interleaved``) is served by
 permuting the rows of W_q and W_k at load, alike in every head, which leaves every score as it is; a position
-encoding's ``amplitude`` multiplies sine and cosine in the rotating kernel.  Keys and values live in the
+encoding's ``amplitude`` multiplies sine and cosine in the rotating kernel.  ``qk_norm_eps`` e: every head of q and k is divided
+by its root mean square over its ``head_dim`` values (e inside the root, no weight) before the rotation and the cache;
+``q_temp`` (coef, every): the queries at position p are then multiplied by 1 + coef ln(floor((p + 1) / every) + 1);
+``head_sink``: a stored number a head (tensor "sink") whose exponential joins that head's denominator, neither scaled nor
+attached to a value; ``gate``: the heads' results leave times sigmoid(W_g h), value by value (tensor "g", whose rows stand
+behind q | k | v in the same product, so that a row's gate lies in its own buffer and the attention kernels apply it where
+they finish a row).  ``own_kv`` False goes with ``cache_from``: the layer stores no W_k and W_v.  Keys and values live in the
 cache at one size, the larger of the two rounded up to 16: the rows of W_q, W_k, W_v (and the columns of W_o) that
 pad a head are zero, so scores and outputs are what the unpadded sizes give.
 """
@@ -33,12 +39,22 @@ class Attention:
         self.dim, self.vdim = spec.head_dim, int(spec.params.get("v_dim", spec.head_dim))
         self.sink = float(spec.params.get("sink", 0.0))
         self.keep_first = int(spec.params.get("keep_first", 0)) if spec.window else 0
+        self.qk_eps = spec.params.get("qk_norm_eps")
+        self.q_temp = spec.params.get("q_temp")
+        self.has_sink, self.gated = bool(spec.params.get("head_sink", False)), bool(spec.params.get("gate", False))
+        self.own_kv = bool(spec.params.get("own_kv", True))
+        if not self.own_kv and spec.cache_from is None:
+            raise ValueError("attention: a layer without keys and values of its own names the site whose cache it reads")
+        if self.sink and self.has_sink:
+            raise ValueError("attention: a sink is either a number of entries of score 0 or a stored number a head")
         self.padded = self.dim != self.vdim or self.dim % 16 != 0
         self.hd = -(-max(self.dim, self.vdim) // 16) * 16 if self.padded else self.dim      # a head's size in a step's rows and in the cache
         if min(self.dim, self.vdim) <= 0 or self.hd > 256:
             raise ValueError(f"attention: key size {self.dim} and value size {self.vdim} must be positive, at most 256")
         if spec.n_heads % spec.n_kv_heads:
             raise ValueError(f"attention: {spec.n_heads} heads are not a multiple of {spec.n_kv_heads} kv heads")
+        if (self.gated or not self.own_kv) and (spec.qkv_bias or spec.out_bias):
+            raise ValueError("attention: biases beside an output gate or another layer's keys and values are not implemented")
         if self.padded and (spec.qkv_bias or spec.out_bias):
             raise ValueError(f"attention: head_dim {self.dim} must be a multiple of 16 and equal to the value size {self.vdim} "
                              f"where the projections have biases (heads are padded in the cache only without biases)")
@@ -48,23 +64,39 @@ class Attention:
         self.interleaved = bool(getattr(self.position, "interleaved", False))
         self.amplitude = float(getattr(self.position, "amplitude", 1.0))
         self.qd = spec.n_heads * self.hd
-        self.kvd = spec.n_kv_heads * self.hd
+        self.nk = spec.n_kv_heads if self.own_kv else 0                  # key (and value) heads of a step's rows
+        self.kvd = self.nk * self.hd
+        self.gate_col = self.qd + 2 * self.kvd if self.gated else 0      # where a row's gate begins
         self.qkv = None
         self.out = None
+        self.sinks = None
 
     # ------------------------------------------------------------------ weights
     def plan(self, prefix: str, names: Dict[str, str]) -> Dict[str, TensorSpec]:
         s = self.spec
         sfx = names.get("suffix", ".weight")
         p: Dict[str, TensorSpec] = {}
-        for key, rows in (("q", s.n_heads * self.dim), ("k", s.n_kv_heads * self.dim), ("v", s.n_kv_heads * self.vdim)):
+        for key, heads, size in self._pieces():
+            rows = heads * size
             p[f"{prefix}{names[key]}{sfx}"] = TensorSpec((rows, s.hidden))
             if s.qkv_bias:
                 p[f"{prefix}{names[key]}.bias"] = TensorSpec((rows,))
         p[f"{prefix}{names['o']}{sfx}"] = TensorSpec((s.hidden, s.n_heads * self.vdim))
         if s.out_bias:
             p[f"{prefix}{names['o']}.bias"] = TensorSpec((s.hidden,))
+        if self.has_sink:
+            p[f"{prefix}{names['sink']}{sfx}"] = TensorSpec((s.n_heads,), std=1.0)
         return p
+
+    def _pieces(self):
+        """(key, heads, size of a head) of the matrices that are stacked into the one projection, in its order of rows."""
+        s = self.spec
+        out = [("q", s.n_heads, self.dim)]
+        if self.own_kv:
+            out += [("k", s.n_kv_heads, self.dim), ("v", s.n_kv_heads, self.vdim)]
+        if self.gated:
+            out.append(("g", s.n_heads, self.vdim))
+        return out
 
     def _pad_rows(self, t: torch.Tensor, heads: int, size: int) -> torch.Tensor:
         """[heads * size, K] -> [heads * hd, K]: every head's rows followed by zero rows up to the cache's head size."""
@@ -80,17 +112,18 @@ class Attention:
         bias = None
         if s.qkv_bias:
             bias = torch.cat([tensors[f"{prefix}{names[k]}.bias"].float() for k in ("q", "k", "v")])
-        sizes = {"q": (s.n_heads, self.dim), "k": (s.n_kv_heads, self.dim), "v": (s.n_kv_heads, self.vdim)}
 
-        def rows(k):
+        def rows(k, heads, size):
             t = tensors[f"{prefix}{names[k]}{sfx}"]
-            if k != "v" and self.interleaved:
-                t = t[self.position.to_half_split(sizes[k][0], self.dim).to(t.device)]
-            return self._pad_rows(t, *sizes[k])
+            if k in ("q", "k") and self.interleaved:
+                t = t[self.position.to_half_split(heads, self.dim).to(t.device)]
+            return self._pad_rows(t, heads, size)
 
         if self.interleaved and s.qkv_bias:
             raise ValueError("attention: neighbouring rotary pairs with biases on q and k are not implemented")
-        self.qkv = Linear([rows(k) for k in ("q", "k", "v")], bias, self.rt)
+        self.qkv = Linear([rows(*piece) for piece in self._pieces()], bias, self.rt)
+        if self.has_sink:
+            self.sinks = self.rt.vector(tensors[f"{prefix}{names['sink']}{sfx}"])
         ob = tensors[f"{prefix}{names['o']}.bias"] if s.out_bias else None
         wo = tensors[f"{prefix}{names['o']}{sfx}"]
         if self.vdim != self.hd:
@@ -105,11 +138,11 @@ class Attention:
         out: Dict[str, torch.Tensor] = {}
         s, sfx = self.spec, names.get("suffix", ".weight")
         r = 0
-        for key, rows, heads, size in (("q", self.qd, s.n_heads, self.dim), ("k", self.kvd, s.n_kv_heads, self.dim),
-                                       ("v", self.kvd, s.n_kv_heads, self.vdim)):
+        for key, heads, size in self._pieces():
+            rows = heads * self.hd
             w = self.qkv.weight[r:r + rows]
             w = w if size == self.hd else w.view(heads, self.hd, -1)[:, :size].reshape(heads * size, -1)
-            if key != "v" and self.interleaved:
+            if key in ("q", "k") and self.interleaved:
                 order = self.position.to_half_split(heads, size).to(w.device)
                 back = torch.empty_like(w)
                 back[order] = w
@@ -122,11 +155,13 @@ class Attention:
         out[f"{prefix}{names['o']}{sfx}"] = wo if self.vdim == self.hd else wo.view(-1, s.n_heads, self.hd)[:, :, :self.vdim].reshape(wo.shape[0], -1)
         if self.out.bias is not None:
             out[f"{prefix}{names['o']}.bias"] = self.out.bias
+        if self.has_sink:
+            out[f"{prefix}{names['sink']}{sfx}"] = self.sinks
         return out
 
     def scratch_row(self) -> int:
         """Values of the widest activation row a step of this part holds (its q | k | v row)."""
-        return self.qd + 2 * self.kvd
+        return self.qd * (2 if self.gated else 1) + 2 * self.kvd
 
     graph_safe = True              # a decode step reads nothing of the batch on the host
 
@@ -160,7 +195,8 @@ class Attention:
         writes = s.cache_from is None
         rows = h.shape[0]
         if (not batch.prefill and writes and self.qkv._skinny(rows) and kv.storage.dtype is torch.bfloat16
-                and self.position.rotary_dim == self.hd and self.amplitude == 1.0 and hasattr(K_, "qkv_rope")):
+                and self.position.rotary_dim == self.hd and self.amplitude == 1.0 and not self.qk_eps and not self.q_temp and not self.gated
+                and hasattr(K_, "qkv_rope")):
             # decoding: projection, rotation and the append to the cache as one kernel
             qkv = self.rt.empty(rows, self.qd + 2 * self.kvd)
             if self.qkv._folds(h, rows):
@@ -173,13 +209,15 @@ class Attention:
                             s.n_kv_heads, self.hd)
         else:
             qkv = self.qkv.store(h)
+            opts = {}
             if self.amplitude != 1.0:
-                K_.rope_append(qkv, self.position.inv_freq, self.position.rotary_dim, batch.row_pos, batch.row_seq,
-                               batch.seq_slot, batch.seq_len, kv if writes else None, s.n_heads, s.n_kv_heads, self.hd,
-                               amplitude=self.amplitude)
-            else:
-                K_.rope_append(qkv, self.position.inv_freq, self.position.rotary_dim, batch.row_pos, batch.row_seq,
-                               batch.seq_slot, batch.seq_len, kv if writes else None, s.n_heads, s.n_kv_heads, self.hd)
+                opts["amplitude"] = self.amplitude
+            if self.qk_eps:
+                opts["qk_norm"] = (None, None, self.dim, float(self.qk_eps))
+            if self.q_temp:
+                opts["q_temp"] = self.q_temp
+            K_.rope_append(qkv, self.position.inv_freq, self.position.rotary_dim, batch.row_pos, batch.row_seq,
+                           batch.seq_slot, batch.seq_len, kv if writes else None, s.n_heads, self.nk, self.hd, **opts)
         att = self.rt.empty(h.shape[0], self.qd)
         from_cache = (not batch.prefill) or not writes
         more = {}
@@ -187,6 +225,10 @@ class Attention:
             more["sink"] = self.sink
         if self.keep_first:
             more["keep_first"] = self.keep_first
+        if self.has_sink:
+            more["head_sink"] = self.sinks
+        if self.gated:
+            more["gate_col"] = self.gate_col
         K_.attention(qkv, kv, batch, att, s.n_heads, s.n_kv_heads, self.hd, s.scale, s.window, from_cache,
                      after_append=True, **more)
         return att

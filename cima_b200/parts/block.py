@@ -4,7 +4,8 @@ feeds both sublayers, the mixer optionally through a short causal convolution, t
 ``sandwich``: a norm in front of and behind each sublayer, x += m * post(mixer(norm(x))); x += m * post(ffn(norm(x))) with
 the spec's ``residual_mult`` m; the feed-forward with its two norms may be absent.  ``postnorm``: the norm stands behind
 the sum, x = norm(a x + mixer(x)); x = norm(a x + feed_forward(x)) with the spec's ``stream_mult`` a; the sublayers read the
-stream itself and the feed-forward may be absent.  ``hyper``: the model carries several copies of the stream, and a
+stream itself and the feed-forward may be absent.  ``branchnorm``: the norm stands on a sublayer's output alone,
+x += norm(mixer(x)); x += norm(feed_forward(x)); the sublayers read the stream itself.  ``hyper``: the model carries several copies of the stream, and a
 sublayer reads a weighted sum of them and writes into all of them (``HyperBlock``).  The block builds its parts from the spec through the
 registries; it does not know which kinds they are, nor which model it is in.
 
@@ -293,6 +294,8 @@ class PostNormBlock:
     scaled stream, the sum, the norm and the rows the next sublayer reads are one kernel (the norm's ``close``).  The
     norm is any registered one that offers ``close(x, y, mult)``."""
 
+    CLOSE = "close"            # what the block needs of its norms
+
     def __init__(self, spec, layer: int, rt):
         self.spec, self.layer, self.rt = spec, layer, rt
         self.mult = float(spec.stream_mult)
@@ -301,16 +304,16 @@ class PostNormBlock:
         self.feed_forward = self.ffn_post = None
         if spec.feed_forward is not None:
             if spec.ffn_norm is None:
-                raise ValueError(f"layer {layer}: a postnorm block with a feed-forward needs the norm behind it")
+                raise ValueError(f"layer {layer}: a {spec.kind} block with a feed-forward needs the norm behind it")
             self.feed_forward = build_feed_forward(spec.feed_forward, layer, rt)
             self.ffn_post = build_norm(spec.ffn_norm, rt)
         for part in (self.mixer, self.feed_forward):
             if part is not None and not hasattr(part, "produce"):
-                raise ValueError(f"layer {layer}: {type(part).__name__} offers no produce(); a postnorm block needs a sublayer's "
+                raise ValueError(f"layer {layer}: {type(part).__name__} offers no produce(); a {spec.kind} block needs a sublayer's "
                                  f"output as rows of its own")
         for norm in (self.mixer_post, self.ffn_post):
-            if norm is not None and not hasattr(norm, "close"):
-                raise ValueError(f"layer {layer}: {type(norm).__name__} offers no close(); a postnorm block needs the sum and "
+            if norm is not None and not hasattr(norm, self.CLOSE):
+                raise ValueError(f"layer {layer}: {type(norm).__name__} offers no {self.CLOSE}(); a {spec.kind} block needs the sum and "
                                  f"the norm as one step")
 
     def _named(self):
@@ -354,19 +357,47 @@ class PostNormBlock:
     def nbytes(self) -> int:
         return sum(p.nbytes() for p, _ in self._named())
 
+    def _stream_rows(self, x: torch.Tensor, info) -> torch.Tensor:
+        """The stream in the activations' dtype: what came along in ``info``, x itself in 32-bit, or a copy."""
+        if info is not None and getattr(info, "norm", None) is STREAM_ROWS and info.h is not None:
+            return info.h
+        if self.rt.full_precision:
+            return x
+        h = self.rt.empty(*x.shape)
+        self.rt.kernels.cast_rows(x, h)
+        return h
+
     def forward(self, x: torch.Tensor, batch, cache, site: int, info=None, next_norm=None):
         from .norm import RowsInfo
-        if info is not None and getattr(info, "norm", None) is STREAM_ROWS and info.h is not None:
-            h = info.h                                             # the stream in the activations' dtype came along
-        elif self.rt.full_precision:
-            h = x
-        else:
-            h = self.rt.empty(*x.shape)
-            self.rt.kernels.cast_rows(x, h)
+        h = self._stream_rows(x, info)
         h = self.mixer_post.close(x, self.mixer.produce(h, batch, cache, site), self.mult)
         if self.feed_forward is not None:
             h = self.ffn_post.close(x, self.feed_forward.produce(h, batch), self.mult)
         return RowsInfo(norm=STREAM_ROWS, h=h)
+
+
+class BranchNormBlock(PostNormBlock):
+    """x += norm1(mixer(x)), then x += norm2(feed_forward(x)): the norm stands on what a sublayer adds, in front of the sum,
+    and the stream itself is never normed inside a layer; the sublayers read it in the activations' dtype.  A layer
+    without feed-forward has the first line only.  The norm of a sublayer's output, the sum, and the rows that the next
+    reader takes (the stream in the activations' dtype, or the following norm's rows where one follows) are one kernel (the
+    norm's ``close_branch``)."""
+
+    CLOSE = "close_branch"
+
+    def forward(self, x: torch.Tensor, batch, cache, site: int, info=None, next_norm=None):
+        from .norm import RowsInfo
+        h = self._stream_rows(x, info)
+        if next_norm is not None and (getattr(next_norm, "weight", None) is None or next_norm.spec.kind != "rmsnorm"
+                                      or next_norm.spec.size != x.shape[1]):
+            next_norm = None
+        y = self.mixer.produce(h, batch, cache, site)
+        if self.feed_forward is not None:
+            h = self.mixer_post.close_branch(x, y)
+            h = self.ffn_post.close_branch(x, self.feed_forward.produce(h, batch), next_norm)
+        else:
+            h = self.mixer_post.close_branch(x, y, next_norm)
+        return RowsInfo(norm=STREAM_ROWS if next_norm is None else next_norm, h=h)
 
 
 class HyperConnection:
@@ -522,6 +553,7 @@ STREAM_ROWS = object()      # a RowsInfo whose ``norm`` is this holds the stream
 
 register_block("prenorm", PreNormBlock)
 register_block("postnorm", PostNormBlock)
+register_block("branchnorm", BranchNormBlock)
 register_block("sandwich", SandwichBlock)
 register_block("parallel", ParallelBlock)
 register_block("hyper", HyperBlock)

@@ -7,6 +7,10 @@
     y = sum_e  w_e * W_down[e] (act(W_gate[e] h) * (W_up[e] h))
 
 Options (``params``), each off by default:
+  ``identity`` n: n more router outputs behind the experts', identity experts: they are scored, grouped and chosen like the
+      others, their output is h itself, and they have no tensors;
+  ``group_score`` "best": a group's score is its largest s (with the correction) instead of the sum of its two largest;
+  ``normalize`` False: the weights are s_e * scale, not divided by the sum of the chosen;
   ``scoring`` "softmax": s = softmax(W_router h) over all experts instead of the sigmoid;
   ``correction``: a stored vector (tensor "correction", [experts]) that is added to s where experts are chosen and left
       out of the weights;
@@ -37,6 +41,11 @@ class RoutedExperts:
         from ..kernels import ACTIVATIONS
         p = spec.params
         self.E, self.top = int(p["experts"]), int(p["top"])
+        self.identity = int(p.get("identity", 0))
+        self.n = self.E + self.identity                      # the router's outputs
+        if p.get("group_score", "two") not in ("two", "best"):
+            raise ValueError(f"moe: group_score '{p.get('group_score')}' is neither 'two' nor 'best'")
+        self.best_one, self.normalize = p.get("group_score", "two") == "best", bool(p.get("normalize", True))
         self.groups, self.keep, self.scale = int(p.get("groups", 1)), int(p.get("keep", p.get("groups", 1))), float(p.get("scale", 1.0))
         if spec.activation not in ACTIVATIONS:
             raise ValueError(f"moe: activation '{spec.activation}' is not one of {sorted(ACTIVATIONS)}")
@@ -47,11 +56,11 @@ class RoutedExperts:
         self.has_correction = bool(p.get("correction", False))
         self.shared_spec = p.get("shared")
         self.shared_gate = bool(p.get("shared_gate", False)) and self.shared_spec is not None
-        if self.E <= 0 or self.groups <= 0 or self.E % self.groups or not (0 < self.keep <= self.groups):
-            raise ValueError(f"moe: {self.E} experts in {self.groups} groups of which {self.keep} stay are not a valid routing")
-        if not (0 < self.top <= self.keep * (self.E // self.groups)):
-            raise ValueError(f"moe: {self.top} choices among the {self.keep * (self.E // self.groups)} experts that stay")
-        if self.E > 1024 or self.groups > 64:
+        if self.E <= 0 or self.identity < 0 or self.groups <= 0 or self.n % self.groups or not (0 < self.keep <= self.groups):
+            raise ValueError(f"moe: {self.n} experts in {self.groups} groups of which {self.keep} stay are not a valid routing")
+        if not (0 < self.top <= self.keep * (self.n // self.groups)):
+            raise ValueError(f"moe: {self.top} choices among the {self.keep * (self.n // self.groups)} experts that stay")
+        if self.n > 1024 or self.groups > 64:
             raise ValueError("moe: at most 1024 experts in at most 64 groups")
         self.act = ACTIVATIONS[spec.activation]
         self.spec, self.layer, self.rt = spec, layer, rt
@@ -62,13 +71,13 @@ class RoutedExperts:
 
     def plan(self, prefix: str, names: Dict[str, str]) -> Dict[str, TensorSpec]:
         s = self.spec
-        p = {self._n(prefix, names, "router"): TensorSpec((self.E, s.hidden), std=0.1)}
+        p = {self._n(prefix, names, "router"): TensorSpec((self.n, s.hidden), std=0.1)}
         for j in range(self.E):
             p[self._n(prefix, names, f"e{j}.gate")] = TensorSpec((s.intermediate, s.hidden))
             p[self._n(prefix, names, f"e{j}.up")] = TensorSpec((s.intermediate, s.hidden))
             p[self._n(prefix, names, f"e{j}.down")] = TensorSpec((s.hidden, s.intermediate))
         if self.has_correction:
-            p[self._n(prefix, names, "correction")] = TensorSpec((self.E,), std=0.02)
+            p[self._n(prefix, names, "correction")] = TensorSpec((self.n,), std=0.02)
         if self.shared_spec is not None:
             ffs = int(self.shared_spec["ff"])
             p[self._n(prefix, names, "shared.gate")] = TensorSpec((ffs, s.hidden))
@@ -81,11 +90,12 @@ class RoutedExperts:
     def load(self, tensors, prefix: str, names: Dict[str, str]) -> None:
         s, rt = self.spec, self.rt
         rows = [tensors[self._n(prefix, names, "router")]]
-        if self.shared_gate:
+        if self.shared_gate or self.identity:
             # the gate's row under the router's, then zero rows up to a multiple of 8 outputs (a row of the scores keeps its
             # 16-byte alignment, and the library's product of many rows its fast kernels)
-            rows.append(tensors[self._n(prefix, names, "shared.sg")])
-            pad = -(self.E + 1) % 8
+            if self.shared_gate:
+                rows.append(tensors[self._n(prefix, names, "shared.sg")])
+            pad = -(self.n + int(self.shared_gate)) % 8
             if pad:
                 rows.append(torch.zeros((pad, s.hidden), dtype=rows[0].dtype, device=rows[0].device))
         self.router = Linear(rows, None, rt)
@@ -109,7 +119,7 @@ class RoutedExperts:
 
     def state(self, prefix: str, names: Dict[str, str]) -> Dict[str, torch.Tensor]:
         ff = self.spec.intermediate
-        out = {self._n(prefix, names, "router"): self.router.weight[:self.E]}
+        out = {self._n(prefix, names, "router"): self.router.weight[:self.n]}
         if self.has_correction:
             out[self._n(prefix, names, "correction")] = self.correction
         if self.shared_spec is not None:
@@ -117,7 +127,7 @@ class RoutedExperts:
             out[self._n(prefix, names, "shared.gate")], out[self._n(prefix, names, "shared.up")] = w[:I], w[I:]
             out[self._n(prefix, names, "shared.down")] = self.shared_down.weight
             if self.shared_gate:
-                out[self._n(prefix, names, "shared.sg")] = self.router.weight[self.E:self.E + 1]
+                out[self._n(prefix, names, "shared.sg")] = self.router.weight[self.n:self.n + 1]
         for j in range(self.E):
             out[self._n(prefix, names, f"e{j}.gate")] = self.gate_up[j, :ff]
             out[self._n(prefix, names, f"e{j}.up")] = self.gate_up[j, ff:]
@@ -137,7 +147,7 @@ class RoutedExperts:
 
     def scratch_row(self) -> int:
         shared = 2 * int(self.shared_spec["ff"]) if self.shared_spec is not None else 0
-        return self.top * (2 * self.spec.intermediate + 2 * self.spec.hidden) + self.E + 1 + shared
+        return self.top * (2 * self.spec.intermediate + 2 * self.spec.hidden) + self.n + 8 + shared
 
     graph_safe = True
 
@@ -156,14 +166,22 @@ class RoutedExperts:
         if hasattr(h, "tensor"):
             h = h.tensor()
         rows = h.shape[0]
-        scores = self.router.logits(h)                                # float32 [rows, E (+ 1: the shared expert's gate)]
+        scores = self.router.logits(h)                                # float32 [rows, n (+ 1: the shared expert's gate, + padding)]
         route = {}
         if self.softmax or self.correction is not None:
             route = {"softmax": self.softmax, "correction": self.correction}
+        if self.identity:
+            route["real"] = self.E
+        if self.best_one:
+            route["best_one"] = True
+        if not self.normalize:
+            route["divide"] = False
         if self.limit or self.act >= GATED_ONLY:
             expert = {"limit": self.limit}
         else:
             expert = {}
+        if self.identity:
+            expert["identity"] = True
         idx = rt.empty(rows, self.top, dtype=torch.int32)
         wgt = rt.empty(rows, self.top, dtype=torch.float32)
         # (a decode step's few rows: the routing launch also orders the pairs by expert)
@@ -171,12 +189,12 @@ class RoutedExperts:
         if self.shared_spec is not None:
             # the shared expert's rows (float32) join the chosen experts' weighted sum in its launch, each row times the
             # sigmoid of its gate logit (the last column of the routing product)
-            expert["shared"] = (self.shared_down.logits(self.shared_up.activated(h)), scores if self.shared_gate else None, self.E)
+            expert["shared"] = (self.shared_down.logits(self.shared_up.activated(h)), scores if self.shared_gate else None, self.n)
         if small:
-            ordered = K_.moe_route(scores, self.top, self.groups, self.keep, self.scale, idx, wgt, order=True, experts=self.E, **route)
+            ordered = K_.moe_route(scores, self.top, self.groups, self.keep, self.scale, idx, wgt, order=True, experts=self.n, **route)
             K_.moe_experts(h, self.gate_up, self.down, idx, wgt, x, self.act, assign=assign, ordered=ordered, **expert)
         else:
-            K_.moe_route(scores, self.top, self.groups, self.keep, self.scale, idx, wgt, experts=self.E, **route)
+            K_.moe_route(scores, self.top, self.groups, self.keep, self.scale, idx, wgt, experts=self.n, **route)
             K_.moe_experts(h, self.gate_up, self.down, idx, wgt, x, self.act, assign=assign, **expert)
 
 

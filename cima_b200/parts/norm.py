@@ -69,6 +69,14 @@ class RMSNorm:
     def lazy(self, x: torch.Tensor, ssq=None, xw=None) -> NormedInput:
         return NormedInput(self, x, ssq, xw)
 
+    def close_branch(self, x: torch.Tensor, y: torch.Tensor, next_norm=None) -> torch.Tensor:
+        """x <- x + norm(y) in place (the stream, float32); returns the rows the next reader takes: the new stream in the
+        activations' dtype (x itself where that is float32), or with ``next_norm`` (an ``RMSNorm`` of the same size) its rows."""
+        h = None if self.rt.full_precision and next_norm is None else self.rt.empty(*x.shape)
+        self.rt.kernels.branch_norm(x, y, self.weight, self.spec.eps, h,
+                                    None if next_norm is None else (next_norm.weight, next_norm.spec.eps))
+        return x if h is None else h
+
     def __call__(self, x: torch.Tensor) -> torch.Tensor:
         out = self.rt.empty(*x.shape)
         self.rt.kernels.rmsnorm(x, self.weight, self.spec.eps, out)

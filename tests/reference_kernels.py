@@ -139,7 +139,7 @@ class ReferenceKernels:
         qkv.copy_(y.to(qkv.dtype))
 
     def rope_append(self, qkv, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, kv, n_heads, n_kv_heads, head_dim,
-                    v_heads=None, qk_norm=None, amplitude=1.0):
+                    v_heads=None, qk_norm=None, amplitude=1.0, q_temp=None):
         T = qkv.shape[0]
         half = rotary_dim // 2
         nv = n_kv_heads if v_heads is None else v_heads
@@ -149,9 +149,14 @@ class ReferenceKernels:
             wq, wk, nd, eps = qk_norm
             part = rot[..., :nd]
             part = part / torch.sqrt((part * part).mean(dim=-1, keepdim=True) + eps)
-            part[:, :n_heads] = part[:, :n_heads] * wq.to(self.compute)
-            part[:, n_heads:] = part[:, n_heads:] * wk.to(self.compute)
+            if wq is not None:
+                part[:, :n_heads] = part[:, :n_heads] * wq.to(self.compute)
+                part[:, n_heads:] = part[:, n_heads:] * wk.to(self.compute)
             rot[..., :nd] = part
+        if q_temp is not None:
+            coef, every = q_temp
+            f = 1.0 + coef * torch.log(((row_pos[:T].long() + 1) // every + 1).to(self.compute))
+            rot[:, :n_heads] = rot[:, :n_heads] * f[:, None, None]
         if half:
             ang = (row_pos[:T].to(torch.float32)[:, None] * inv_freq[None, :]).to(self.compute)
             c, s = torch.cos(ang)[:, None, :] * amplitude, torch.sin(ang)[:, None, :] * amplitude
@@ -170,12 +175,12 @@ class ReferenceKernels:
             kv.storage[page, 1, :nv, off, :] = heads[r, n_heads + n_kv_heads:, :]
 
     def attention(self, qkv, kv, batch, out, n_heads, n_kv_heads, head_dim, scale, window, from_cache, after_append=False,
-                  sink=0.0, keep_first=0, v_group=1, head_sink=None):
+                  sink=0.0, keep_first=0, v_group=1, head_sink=None, gate_col=0):
         self.attention_plain(qkv, kv, batch.row_pos, batch.row_seq, batch.seq_slot, batch.seq_first_row, out,
-                             n_heads, n_kv_heads, head_dim, scale, window, from_cache, sink, keep_first, v_group, head_sink)
+                             n_heads, n_kv_heads, head_dim, scale, window, from_cache, sink, keep_first, v_group, head_sink, gate_col)
 
     def attention_plain(self, qkv, kv, row_pos, row_seq, seq_slot, seq_first_row, out, n_heads, n_kv_heads,
-                        head_dim, scale, window, from_cache, sink=0.0, keep_first=0, v_group=1, head_sink=None):
+                        head_dim, scale, window, from_cache, sink=0.0, keep_first=0, v_group=1, head_sink=None, gate_col=0):
         T = qkv.shape[0]
         rep = n_heads // n_kv_heads
         vplane = int(getattr(kv, "planes", 2)) - 1 if from_cache else 1      # one plane: the values are the keys
@@ -214,7 +219,10 @@ class ReferenceKernels:
                     w = e / (e.sum() + sink * torch.exp(-m))
                 else:
                     w = torch.softmax(s, dim=0)
-                out[r, h * head_dim:(h + 1) * head_dim] = (w @ v[:, g // v_group, :]).to(out.dtype)
+                res = w @ v[:, g // v_group, :]
+                if gate_col:                                # the row's own gate, value by value
+                    res = res * torch.sigmoid(qkv[r, gate_col + h * head_dim:gate_col + (h + 1) * head_dim].to(self.compute))
+                out[r, h * head_dim:(h + 1) * head_dim] = res.to(out.dtype)
 
     # ------------------------------------------------------------------ sampling
     def argmax(self, logits, tokens):
@@ -461,14 +469,18 @@ def _delta_prepare(self, qk, a, b, A_log, dt_bias, qn, kn, g, beta, heads, kv_he
     beta.copy_(torch.sigmoid(b.float()))
 
 
-def _group_rmsnorm_gate(self, o, w, gate, out, groups, eps):
+def _group_rmsnorm_gate(self, o, w, gate, out, groups, eps, silu=False, divisor=None):
     T, W = o.shape
     n = W // groups
     z = o.view(T, groups, n)
+    if divisor is not None:
+        den, low, e = divisor
+        z = z / (torch.maximum(den.abs(), low) + e)[:, :, None]
     z = z / torch.sqrt((z * z).mean(-1, keepdim=True) + eps)
     z = z * (w.view(1, 1, n) if w.numel() == n and groups > 1 else w.view(1, groups, n))
     if gate is not None:
-        z = z * torch.sigmoid(gate.float().view(T, groups, n))
+        g = gate.float().reshape(T, groups, n)
+        z = z * (_silu(g) if silu else torch.sigmoid(g))
     out.copy_(z.view(T, W).to(out.dtype))
 
 
@@ -483,30 +495,34 @@ def _rms_mean(self, ys, ws, x, eps, assign=False):
 
 
 # ---------------------------------------------------------------------- routed feed-forward
-def _moe_route(self, scores, top, groups, keep, scale, idx, wgt, experts=None, softmax=False, correction=None):
+def _moe_route(self, scores, top, groups, keep, scale, idx, wgt, experts=None, softmax=False, correction=None, real=None, best_one=False,
+               divide=True):
     T = scores.shape[0]
     E = scores.shape[1] if experts is None else experts
     per = E // groups
     s = torch.softmax(scores[:, :E], dim=-1) if softmax else torch.sigmoid(scores[:, :E])
     cmp = s if correction is None else s + correction
     for t in range(T):
-        gs = [float(cmp[t, gi * per:(gi + 1) * per].topk(min(2, per)).values.sum()) for gi in range(groups)]
+        gs = [float(cmp[t, gi * per:(gi + 1) * per].topk(min(1 if best_one else 2, per)).values.sum()) for gi in range(groups)]
         best = sorted(range(groups), key=lambda gi: (-gs[gi], gi))[:keep]
         allowed = [e for gi in best for e in range(gi * per, (gi + 1) * per)]
         chosen = sorted(allowed, key=lambda e: (-float(cmp[t, e]), e))[:top]
         w = torch.stack([s[t, e] for e in chosen])
         idx[t] = torch.tensor(chosen, dtype=idx.dtype)
-        wgt[t] = w / (w.sum() + 1e-20) * scale
+        wgt[t] = w / (w.sum() + 1e-20) * scale if divide else w * scale
     scores[:, :E] = s
 
 
-def _moe_experts(self, h, gate_up, down, idx, wgt, x, act=0, assign=False, limit=0.0, shared=None):
+def _moe_experts(self, h, gate_up, down, idx, wgt, x, act=0, assign=False, limit=0.0, shared=None, identity=False):
     ff = gate_up.shape[1] // 2
     hf = h.float()
     for t in range(h.shape[0]):
         acc = torch.zeros_like(x[t])
         for j in range(idx.shape[1]):
             e = int(idx[t, j])
+            if identity and e >= gate_up.shape[0]:
+                acc = acc + wgt[t, j] * hf[t]
+                continue
             gu = (gate_up[e].float() @ hf[t]).to(h.dtype).float()
             z = self.gated(gu[:ff], gu[ff:], act, limit).to(h.dtype).float()
             acc = acc + wgt[t, j] * (down[e].float() @ z)
@@ -544,6 +560,64 @@ def _cast_rows(self, x, h):
 def _softcap(self, logits, cap):
     logits.copy_(cap * torch.tanh(logits / cap))
 
+
+# ---------------------------------------------------------------------- matrix memories, the norm on a branch
+def _memory(self, q, k, v, g, state, batch, out, heads, dim, vdim, qscale, norm_state=None, norm_out=None):
+    T = batch.n_rows
+    scalar = g.dim() == 3
+    qf, kf, vf = q.float().reshape(T, heads, dim) * qscale, k.float().reshape(T, heads, dim), v.float().reshape(T, heads, vdim)
+    for s in range(batch.n_seqs):
+        slot = int(batch.seq_slot[s])
+        S = state[slot].clone()
+        n = norm_state[slot].clone() if scalar else None
+        for t in range(int(batch.seq_first_row[s]), int(batch.seq_first_row[s + 1])):
+            if scalar:
+                a, b = g[t, :, 0], g[t, :, 1]
+                S = a[:, None, None] * S + b[:, None, None] * kf[t][:, :, None] * vf[t][:, None, :]
+                n = a[:, None] * n + b[:, None] * kf[t]
+                norm_out[t] = (n * qf[t]).sum(-1)
+            else:
+                S = g[t].view(heads, dim)[:, :, None] * S + kf[t][:, :, None] * vf[t][:, None, :]
+            out[t] = torch.einsum("hdv,hd->hv", S, qf[t]).reshape(-1)
+        state[slot] = S
+        if scalar:
+            norm_state[slot] = n
+
+
+def _log_sigmoid(z):
+    return -torch.nn.functional.softplus(-z)
+
+
+def _channel_decay(self, a1, w2, bias, tau, g):
+    g.copy_(torch.exp(_log_sigmoid(a1.float() @ w2.float().T + bias) / tau))
+
+
+def _scalar_gates(self, z, bi, bf, cap, mstate, batch, ab, low):
+    heads = bi.numel()
+    i = cap * torch.tanh((z[:, :heads].float() + bi) / cap)
+    f = _log_sigmoid(cap * torch.tanh((z[:, heads:2 * heads].float() + bf) / cap))
+    for s in range(batch.n_seqs):
+        slot = int(batch.seq_slot[s])
+        m = mstate[slot].clone()
+        for t in range(int(batch.seq_first_row[s]), int(batch.seq_first_row[s + 1])):
+            new = torch.maximum(f[t] + m, i[t])
+            ab[t, :, 0], ab[t, :, 1], low[t] = torch.exp(f[t] + m - new), torch.exp(i[t] - new), torch.exp(-new)
+            m = new
+        mstate[slot] = m
+
+
+def _branch_norm(self, x, y, w, eps, h=None, next_norm=None):
+    x.add_(y / torch.sqrt((y * y).mean(-1, keepdim=True) + eps) * w)
+    if h is not None:
+        if next_norm is not None:
+            w2, eps2 = next_norm
+            h.copy_((x / torch.sqrt((x * x).mean(-1, keepdim=True) + eps2) * w2).to(h.dtype))
+        else:
+            h.copy_(x.to(h.dtype))
+
+
+for _name, _fn in (("memory", _memory), ("channel_decay", _channel_decay), ("scalar_gates", _scalar_gates), ("branch_norm", _branch_norm)):
+    setattr(ReferenceKernels, _name, _fn)
 
 for _name, _fn in (("diff_combine", _diff_combine), ("scale_add_group_rmsnorm", _scale_add_group_rmsnorm), ("cast_rows", _cast_rows),
                    ("softcap", _softcap)):
