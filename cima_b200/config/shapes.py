@@ -9,6 +9,10 @@ And shapes of the Netezen decoder at those widths: two copies of the stream; lay
 (a position keeps 96 + 32 values) and grouped-query attention with the Qwen2 shape's heads behind a window that keeps first
 positions; the first layer's feed-forward is the ungated one, the others route 3 of 16 clamped experts beside a shared
 one, a token using as many values of a middle as the Qwen2 shape has.
+And shapes of the Pelatar decoder at those widths: of every four layers one runs gated linear attention, one grouped-query
+attention with the Qwen2 shape's heads, one attention on the keys and values of the layer before it, one the mLSTM memory (the
+memories' heads, key and value sizes are the Qwen2 shape's); layers alternate between the dense feed-forward and 12 experts
+beside 4 identity experts, 3 of which a token uses.
 Every entry is a complete config.json; nothing here is read by the model code."""
 
 
@@ -92,13 +96,39 @@ def _netezen(layers, width, heads, kv_heads, dim, ff, vocab, experts=16, top=3, 
             "layers": out}
 
 
-# the Qwen2 shape that a Vunovik, Gisirax, Lipizen or Netezen shape is measured beside
-TWINS = {"netezen-0.5b": "qwen2.5-0.5b", "netezen-1.5b": "qwen2.5-1.5b", "netezen-3b": "qwen2.5-3b", "netezen-7b": "qwen2.5-7b",
+def _pelatar(layers, width, heads, kv_heads, dim, ff, vocab, experts=12, identity=4, top=3, groups=4, keep=2, rank=16, every=8192):
+    """Of every four layers: gated linear attention, attention, attention on its neighbour's keys and values, mLSTM; even layers
+    with the dense feed-forward, odd ones with ``top`` of ``experts`` + ``identity`` experts of ``ff / top`` values each."""
+    moe = {"kind": "moe", "expert": {"ff": -(-ff // top // 64) * 64},
+           "router": {"experts": experts, "identity": identity, "top": top, "groups": {"count": groups, "keep": keep}}}
+    out = []
+    for i in range(layers):
+        mlp = moe if i % 2 else {"kind": "dense", "ff": ff}
+        if i % 4 in (1, 2):
+            mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "q_temp": {"coef": 0.1, "every": every}}
+            if i % 4 == 2:
+                mixer["kv_from"] = i - 1
+            out.append({"type": "attention", "mixer": mixer, "mlp": mlp})
+        else:
+            mixer = {"heads": heads, "dim": dim, "vdim": dim}
+            mixer.update({"tau": 16.0, "rank": rank} if i % 4 == 0 else {"gate_cap": 15.0})
+            out.append({"type": "gla" if i % 4 == 0 else "mlstm", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Pelatar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": out}
+
+
+# the Qwen2 shape that a Vunovik, Gisirax, Lipizen, Netezen or Pelatar shape is measured beside
+TWINS = {"pelatar-0.5b": "qwen2.5-0.5b", "pelatar-1.5b": "qwen2.5-1.5b", "pelatar-3b": "qwen2.5-3b", "pelatar-7b": "qwen2.5-7b",
+         "netezen-0.5b": "qwen2.5-0.5b", "netezen-1.5b": "qwen2.5-1.5b", "netezen-3b": "qwen2.5-3b", "netezen-7b": "qwen2.5-7b",
          "lipizen-0.5b": "qwen2.5-0.5b", "lipizen-1.5b": "qwen2.5-1.5b", "lipizen-3b": "qwen2.5-3b", "lipizen-7b": "qwen2.5-7b",
          "gisirax-0.5b": "qwen2.5-0.5b", "gisirax-1.5b": "qwen2.5-1.5b", "gisirax-3b": "qwen2.5-3b", "gisirax-7b": "qwen2.5-7b",
          "vunovik-0.5b": "qwen2.5-0.5b", "vunovik-1.5b": "qwen2.5-1.5b", "vunovik-3b": "qwen2.5-3b", "vunovik-7b": "qwen2.5-7b"}
 
 SHAPES = {
+    "pelatar-tiny": _pelatar(4, 128, 4, 2, 32, 256, 512, experts=5, identity=3, top=2, groups=4, keep=2, rank=8, every=16),
+    "pelatar-0.5b": _pelatar(24, 896, 14, 2, 64, 4864, 151936),
+    "pelatar-1.5b": _pelatar(28, 1536, 12, 2, 128, 8960, 151936),
+    "pelatar-3b": _pelatar(36, 2048, 16, 2, 128, 11008, 151936),
+    "pelatar-7b": _pelatar(28, 3584, 28, 4, 128, 18944, 152064),
     "netezen-tiny": _netezen(4, 128, 4, 2, 32, 256, 512, experts=6, top=2, window=96, keep_first=4, rank=48, rot=16),
     "netezen-0.5b": _netezen(24, 896, 14, 2, 64, 4864, 151936, rank=96, rot=32),
     "netezen-1.5b": _netezen(28, 1536, 12, 2, 128, 8960, 151936),
