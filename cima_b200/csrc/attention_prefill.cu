@@ -281,11 +281,11 @@ k_attention_prefill(const __nv_bfloat16* __restrict__ qkv, int ld, const int* __
       const __nv_bfloat16* gp = qkv + (size_t)first * ld + gate_col + (size_t)h * HD + d;
       if (r0 < len) {
         const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gp + (size_t)r0 * ld));
-        g[0] = cima_sigmoid(v.x); g[1] = cima_sigmoid(v.y);
+        g[0] = cima_sigmoid_fast(v.x); g[1] = cima_sigmoid_fast(v.y);
       }
       if (r1 < len) {
         const float2 v = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gp + (size_t)r1 * ld));
-        g[2] = cima_sigmoid(v.x); g[3] = cima_sigmoid(v.y);
+        g[2] = cima_sigmoid_fast(v.x); g[3] = cima_sigmoid_fast(v.y);
       }
     }
     if (r0 < len)

@@ -340,8 +340,8 @@ k_attention_prefill_tc(const __grid_constant__ CUtensorMap map_qkv, const __grid
 #pragma unroll
               for (int k = 0; k < 4; k++) {
                 const float2 g = __bfloat1622float2(g2[k]);
-                o[8 * q + 2 * k] *= cima_sigmoid(g.x);
-                o[8 * q + 2 * k + 1] *= cima_sigmoid(g.y);
+                o[8 * q + 2 * k] *= cima_sigmoid_fast(g.x);
+                o[8 * q + 2 * k + 1] *= cima_sigmoid_fast(g.y);
               }
             }
 #pragma unroll

@@ -167,6 +167,72 @@ k_group_rmsnorm_gate(const float* __restrict__ o, const float* __restrict__ w, c
   }
 }
 
+template <typename T> __device__ __forceinline__ float4 read4(const T* p) {
+  if constexpr (sizeof(T) == 2) {
+    const uint2 t = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.x)), b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&t.y));
+    return make_float4(a.x, a.y, b.x, b.y);
+  } else {
+    return *reinterpret_cast<const float4*>(p);
+  }
+}
+
+// The same for groups of at most 512 values whose size and strides are multiples of 4: four neighbouring values a lane at a time.
+template <typename TG, typename TO>
+__global__ void __launch_bounds__(128)
+k_group_rmsnorm_gate4(const float* __restrict__ o, const float* __restrict__ w, const TG* __restrict__ gate, int ldg,
+                      TO* __restrict__ out, long long units, int groups, int n, int shared_w, float eps, int silu,
+                      const float* __restrict__ den, const float* __restrict__ low, float div_eps) {
+  cima_pdl_wait();
+  cima_pdl_trigger();
+  const long long unit = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (unit >= units) return;
+  const int lane = threadIdx.x & 31;
+  const long long row = unit / groups;
+  const int grp = (int)(unit - row * groups);
+  const float* src = o + (size_t)unit * n;
+  const float* wp = w + (shared_w ? 0 : (size_t)grp * n);
+  const TG* gp = gate ? gate + (size_t)row * ldg + (size_t)grp * n : nullptr;
+  float4 v[4], wv[4], gv[4];
+#pragma unroll
+  for (int j = 0; j < 4; j++)
+    if (128 * j < n) {
+      const int i = min(4 * lane + 128 * j, n - 4);      // (beyond the group: its last values, which are then not used)
+      v[j] = read4<float>(src + i);
+      wv[j] = read4<float>(wp + i);
+      gv[j] = gp ? read4<TG>(gp + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+  const float f = group_factor(den, low, div_eps, unit);
+  float ss = 0.f;
+#pragma unroll
+  for (int j = 0; j < 4; j++)
+    if (4 * lane + 128 * j < n) {
+      v[j] = make_float4(v[j].x * f, v[j].y * f, v[j].z * f, v[j].w * f);
+      ss += fmaf(v[j].x, v[j].x, v[j].y * v[j].y) + fmaf(v[j].z, v[j].z, v[j].w * v[j].w);
+    }
+  for (int s = 16; s > 0; s >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, s);
+  const float r = 1.0f / sqrtf(ss / (float)n + eps);
+  TO* dst = out + (size_t)unit * n;
+#pragma unroll
+  for (int j = 0; j < 4; j++)
+    if (4 * lane + 128 * j < n) {
+      float y[4] = {v[j].x * r * wv[j].x, v[j].y * r * wv[j].y, v[j].z * r * wv[j].z, v[j].w * r * wv[j].w};
+      if (gp) {
+        y[0] *= gate_value(gv[j].x, silu); y[1] *= gate_value(gv[j].y, silu);
+        y[2] *= gate_value(gv[j].z, silu); y[3] *= gate_value(gv[j].w, silu);
+      }
+      if constexpr (sizeof(TO) == 2) {
+        uint2 t;
+        __nv_bfloat162* h2 = reinterpret_cast<__nv_bfloat162*>(&t);
+        h2[0] = __floats2bfloat162_rn(y[0], y[1]);
+        h2[1] = __floats2bfloat162_rn(y[2], y[3]);
+        *reinterpret_cast<uint2*>(dst + 4 * lane + 128 * j) = t;
+      } else {
+        *reinterpret_cast<float4*>(dst + 4 * lane + 128 * j) = make_float4(y[0], y[1], y[2], y[3]);
+      }
+    }
+}
+
 // The same for long groups (a whole row of some thousand values): a block a (row, group).
 template <typename TG, typename TO>
 __global__ void __launch_bounds__(256)
@@ -230,10 +296,14 @@ extern "C" int cima_group_rmsnorm_gate(const float* o, const float* w, const voi
   if ((den != nullptr) != (low != nullptr)) return cima_fail(CIMA_E_ARG, "group_rmsnorm_gate: the divisors take their lower bounds");
   const long long units = (long long)T * groups;
   const bool wide = n >= 512 && units < 0x7fffffffll;
+  const size_t gb = gdtype == CIMA_F32 ? 16 : 8, ob = odtype == CIMA_F32 ? 16 : 8;
+  const bool four = !wide && n <= 512 && n % 4 == 0 && ldg % 4 == 0 && (((uintptr_t)o | (uintptr_t)w) & 15) == 0 &&
+                    ((uintptr_t)gate & (gb - 1)) == 0 && ((uintptr_t)out & (ob - 1)) == 0;
   const dim3 grid(wide ? (unsigned)units : (unsigned)((units + 3) / 4));
   int rc;
 #define RUN(TG, TO) rc = wide ? cima_launch(k_group_rmsnorm_gate_wide<TG, TO>, grid, dim3(256), (size_t)0, stream, 1, o, w, (const TG*)gate, ldg, (TO*)out, groups, n, shared_w, eps, silu, den, low, div_eps) \
-                              : cima_launch(k_group_rmsnorm_gate<TG, TO>, grid, dim3(128), (size_t)0, stream, 1, o, w, (const TG*)gate, ldg, (TO*)out, units, groups, n, shared_w, eps, silu, den, low, div_eps)
+               : four ? cima_launch(k_group_rmsnorm_gate4<TG, TO>, grid, dim3(128), (size_t)0, stream, 1, o, w, (const TG*)gate, ldg, (TO*)out, units, groups, n, shared_w, eps, silu, den, low, div_eps) \
+                      : cima_launch(k_group_rmsnorm_gate<TG, TO>, grid, dim3(128), (size_t)0, stream, 1, o, w, (const TG*)gate, ldg, (TO*)out, units, groups, n, shared_w, eps, silu, den, low, div_eps)
   if (gdtype == CIMA_F32 && odtype == CIMA_F32) RUN(float, float);
   else if (gdtype == CIMA_BF16 && odtype == CIMA_BF16) RUN(__nv_bfloat16, __nv_bfloat16);
   else if (gdtype == CIMA_F32 && odtype == CIMA_BF16) RUN(float, __nv_bfloat16);

@@ -5,13 +5,14 @@
 //   scalar form    S <- a_t S + b_t k_t v_t^T;             o_t = S^T (c q_t)        a_t, b_t one number a head
 //                  n <- a_t n + b_t k_t;                   r_t = n . (c q_t)        the normaliser's row beside the matrix
 //
-// with one constant c.  A block owns 32 CPT value channels (columns of S) of one (sequence, head); a column is shared by 8
-// lanes of a warp, each of which keeps an eighth of its rows in registers (rows 32 ii + 4 rg + e of row group rg).  In the
-// scalar form the first block of a head has a ninth warp: it keeps n as one more column whose value is 1.  Tokens are
-// walked in order, 16 (8 for key sizes above 128) at a time: the next ones travel from global memory into registers
-// while the current ones are worked on from shared memory.  No token's read-out feeds the next update, so four tokens
-// are taken together: their updates follow one another row by row, their sums over the lanes run side by side.  A
-// token's own arithmetic is the same wherever it stands among them.  Everything is float32 but the loads of q, k, v.
+// with one constant c.  A block owns 256 CPT / LANES value channels (columns of S) of one (sequence, head): a thread has CPT
+// neighbouring columns, LANES lanes of a warp share them, and each keeps its part of the rows in registers (rows 4 LANES ii +
+// 4 rg + e of row group rg).  In the scalar form the first block of a head has a ninth warp: it keeps n as one more column
+// whose value is 1.  Tokens are walked in order, 16 (8 for key sizes above 128) at a time: the next ones travel from global
+// memory into registers while the current ones are worked on from shared memory.  No token's read-out feeds the next
+// update, so four tokens are taken together: their updates follow one another row by row, and their sums over the lanes
+// are formed in one go.  A token's own arithmetic is the same wherever it stands among them.  Everything is float32 but the
+// loads of q, k, v.
 //
 // Long steps are cut into segments of `seg` tokens that run side by side (three launches):
 //   PHASE 1   every segment but a sequence's last, from S = 0, without read-out: what it adds, E, and the product of its
@@ -41,13 +42,14 @@ struct MemArgs {
   float qscale;
 };
 
-template <typename TA, int DIMP, bool SCALAR, int CPT, int PHASE>
+template <typename TA, int DIMP, bool SCALAR, int CPT, int LANES, int PHASE>
 __global__ void __launch_bounds__(288)
 k_memory(const __grid_constant__ MemArgs a) {
   cima_pdl_wait();
-  constexpr int RP = DIMP / 8;                          // rows of a column that one lane keeps
+  constexpr int RP = DIMP / LANES;                      // rows of a column that one lane keeps
+  constexpr int GW = 32 / LANES;                        // groups of columns of a warp
   constexpr int CH = DIMP > 128 ? 8 : 16;               // tokens staged at a time
-  constexpr int COLS = 32 * CPT;
+  constexpr int COLS = MEM_COL_WARPS * GW * CPT;
   constexpr int NLD = CH * DIMP / 256;                  // values of k (and of q, of g) a thread stages
   constexpr int NLV = (CH * COLS + 255) / 256;
   constexpr bool READ = PHASE != 1;
@@ -71,9 +73,9 @@ k_memory(const __grid_constant__ MemArgs a) {
     n = min(left, a.seg);
   }
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  const int rg = lane >> 2;
+  const int rg = lane / GW;
   const bool extra = warp == MEM_COL_WARPS;             // the ninth warp: the normaliser, or (PHASE 1) the decays' product
-  const int lc = extra ? 0 : warp * 4 + (lane & 3);     // the thread's columns are col0 + lc + 32 x
+  const int lc = extra ? 0 : (warp * GW + lane % GW) * CPT;      // the thread's columns are col0 + lc + x
   const int heads = a.heads, dim = a.dim, vdim = a.vdim;
   const TA* q = static_cast<const TA*>(a.q);
   const TA* k = static_cast<const TA*>(a.k);
@@ -86,10 +88,10 @@ k_memory(const __grid_constant__ MemArgs a) {
   for (int x = 0; x < CPT; x++)
 #pragma unroll
     for (int j = 0; j < RP; j++) {
-      const int row = (j >> 2) * 32 + rg * 4 + (j & 3);
+      const int row = (j >> 2) * (4 * LANES) + rg * 4 + (j & 3);
       float s = 0.f;
       if (READ && row < dim) {
-        if (!extra) { if (col0 + lc + 32 * x < vdim) s = st[(size_t)row * vdim + 32 * x]; }
+        if (!extra) { if (col0 + lc + x < vdim) s = st[(size_t)row * vdim + x]; }
         else if (SCALAR && x == 0) s = nst[row];
       }
       S[x][j] = s;
@@ -150,28 +152,28 @@ k_memory(const __grid_constant__ MemArgs a) {
     const bool works = !extra || (SCALAR && blockIdx.x == 0);
     if (works) {
       for (int tt = 0; tt < nt; tt += TB) {
-        float o[CPT][TB];
+        float o[TB * CPT];                               // [token][column]
 #pragma unroll
         for (int y = 0; y < TB; y++) {
 #pragma unroll
-          for (int x = 0; x < CPT; x++) o[x][y] = 0.f;
+          for (int x = 0; x < CPT; x++) o[y * CPT + x] = 0.f;
           if (tt + y < nt) {
             float u[CPT], f = 1.f;
             if (SCALAR) {
               const float2 ab = sab[tt + y];
               f = ab.x;
 #pragma unroll
-              for (int x = 0; x < CPT; x++) u[x] = (extra ? 1.0f : sv[tt + y][lc + 32 * x]) * ab.y;
+              for (int x = 0; x < CPT; x++) u[x] = (extra ? 1.0f : sv[tt + y][lc + x]) * ab.y;
             } else {
 #pragma unroll
-              for (int x = 0; x < CPT; x++) u[x] = sv[tt + y][lc + 32 * x];
+              for (int x = 0; x < CPT; x++) u[x] = sv[tt + y][lc + x];
             }
             float p[CPT];
 #pragma unroll
             for (int x = 0; x < CPT; x++) p[x] = 0.f;
 #pragma unroll
             for (int j = 0; j < RP; j += 4) {
-              const int i = (j >> 2) * 32 + rg * 4;
+              const int i = (j >> 2) * (4 * LANES) + rg * 4;
               const float4 k4 = *reinterpret_cast<const float4*>(&sk[tt + y][i]);
               float4 g4 = make_float4(f, f, f, f);
               if (!SCALAR) g4 = *reinterpret_cast<const float4*>(&sg[tt + y][i]);
@@ -184,36 +186,43 @@ k_memory(const __grid_constant__ MemArgs a) {
                 S[x][j + 2] = fmaf(k4.z, u[x], g4.z * S[x][j + 2]);
                 S[x][j + 3] = fmaf(k4.w, u[x], g4.w * S[x][j + 3]);
                 if (READ) {
-                  o[x][y] = fmaf(S[x][j], q4.x, o[x][y]); p[x] = fmaf(S[x][j + 1], q4.y, p[x]);
-                  o[x][y] = fmaf(S[x][j + 2], q4.z, o[x][y]); p[x] = fmaf(S[x][j + 3], q4.w, p[x]);
+                  o[y * CPT + x] = fmaf(S[x][j], q4.x, o[y * CPT + x]); p[x] = fmaf(S[x][j + 1], q4.y, p[x]);
+                  o[y * CPT + x] = fmaf(S[x][j + 2], q4.z, o[y * CPT + x]); p[x] = fmaf(S[x][j + 3], q4.w, p[x]);
                 }
               }
             }
             if (READ) {
 #pragma unroll
-              for (int x = 0; x < CPT; x++) o[x][y] += p[x];
+              for (int x = 0; x < CPT; x++) o[y * CPT + x] += p[x];
             }
             if (PHASE == 1 && SCALAR) D[0] *= f;
           }
         }
         if (READ) {
+          // sums over the LANES lanes of a column group, a tree of pairs over the lanes' distance LANES / 2, ..., 1
+          // (as long as a lane has more than one value it keeps one half and hands the other over: in the end it holds one of them)
+          int n_own = TB * CPT, base = 0;
 #pragma unroll
-          for (int s = 4; s < 32; s <<= 1)
+          for (int m = LANES / 2; m > 0; m >>= 1) {
+            if (n_own > 1) {
+              n_own >>= 1;
+              const bool up = (rg & m) != 0;
+              if (up) base += n_own;
 #pragma unroll
-            for (int x = 0; x < CPT; x++)
-#pragma unroll
-              for (int y = 0; y < TB; y++) o[x][y] += __shfl_xor_sync(0xffffffffu, o[x][y], s);
-          if (rg == 0) {
-#pragma unroll
-            for (int y = 0; y < TB; y++)
-              if (tt + y < nt) {
-                if (!extra) {
-#pragma unroll
-                  for (int x = 0; x < CPT; x++) so[tt + y][lc + 32 * x] = o[x][y];
-                } else if (lane == 0) {
-                  so[tt + y][COLS] = o[0][y];
+              for (int i = 0; i < TB * CPT / 2; i++)
+                if (i < n_own) {
+                  const float keep = up ? o[i + n_own] : o[i], give = up ? o[i] : o[i + n_own];
+                  o[i] = keep + __shfl_xor_sync(0xffffffffu, give, m * GW);
                 }
-              }
+            } else {
+              o[0] += __shfl_xor_sync(0xffffffffu, o[0], m * GW);
+            }
+          }
+          static_assert(TB * CPT <= LANES, "a lane ends with one value");
+          const int y = base / CPT, x = base % CPT;
+          if (tt + y < nt) {                              // (lanes with the same value write the same sum)
+            if (!extra) so[tt + y][lc + x] = o[0];
+            else if (x == 0 && lane % GW == 0) so[tt + y][COLS] = o[0];
           }
         }
       }
@@ -242,10 +251,10 @@ k_memory(const __grid_constant__ MemArgs a) {
   for (int x = 0; x < CPT; x++)
 #pragma unroll
     for (int j = 0; j < RP; j++) {
-      const int row = (j >> 2) * 32 + rg * 4 + (j & 3);
+      const int row = (j >> 2) * (4 * LANES) + rg * 4 + (j & 3);
       if (row < dim) {
-        if (!extra) { if (col0 + lc + 32 * x < vdim) st[(size_t)row * vdim + 32 * x] = S[x][j]; }
-        else if (SCALAR && x == 0 && blockIdx.x == 0 && (lane & 3) == 0) nst[row] = S[x][j];
+        if (!extra) { if (col0 + lc + x < vdim) st[(size_t)row * vdim + x] = S[x][j]; }
+        else if (SCALAR && x == 0 && blockIdx.x == 0 && lane % GW == 0) nst[row] = S[x][j];
       }
     }
   if (PHASE == 1 && extra && blockIdx.x == 0) {
@@ -296,11 +305,16 @@ k_memory_combine(const __grid_constant__ MemArgs a) {
   }
 }
 
-template <typename TA, bool SCALAR, int CPT, int PHASE>
+template <typename TA, bool SCALAR, int PHASE>
 int launch_memory(const MemArgs& a, int n_units, cudaStream_t stream) {
-  const dim3 grid((unsigned)((a.vdim + 32 * CPT - 1) / (32 * CPT)), (unsigned)a.heads, (unsigned)n_units);
+  // PHASE 0 (few tokens a sequence, or many sequences): 32 columns a block, so that more blocks share the state's traffic.
+  // Segments: 64 columns, two a thread, so that a read of k, q and g from shared memory serves both (four a thread over 16
+  // lanes measured the same: the kernel issues 0.6 to 0.7 instructions a cycle and scheduler either way).
+  constexpr int CPT = PHASE == 0 ? 1 : 2;
+  constexpr int cols = 32 * CPT;
+  const dim3 grid((unsigned)((a.vdim + cols - 1) / cols), (unsigned)a.heads, (unsigned)n_units);
   const dim3 block(SCALAR || PHASE == 1 ? 288 : 256);
-#define RUN(D) return cima_launch(k_memory<TA, D, SCALAR, CPT, PHASE>, grid, block, (size_t)0, stream, 1, a)
+#define RUN(D) return cima_launch(k_memory<TA, D, SCALAR, CPT, 8, PHASE>, grid, block, (size_t)0, stream, 1, a)
   if (a.dim <= 32) RUN(32);
   if (a.dim <= 64) RUN(64);
   if (a.dim <= 128) RUN(128);
@@ -310,11 +324,11 @@ int launch_memory(const MemArgs& a, int n_units, cudaStream_t stream) {
 
 template <typename TA, bool SCALAR>
 int run_memory(const MemArgs& a, int n_seqs, cudaStream_t stream) {
-  if (a.max_segs <= 1) return launch_memory<TA, SCALAR, 1, 0>(a, n_seqs, stream);
-  if (int rc = launch_memory<TA, SCALAR, 2, 1>(a, n_seqs * a.max_segs, stream)) return rc;
+  if (a.max_segs <= 1) return launch_memory<TA, SCALAR, 0>(a, n_seqs, stream);
+  if (int rc = launch_memory<TA, SCALAR, 1>(a, n_seqs * a.max_segs, stream)) return rc;
   const unsigned blocks = (unsigned)((a.dim * (a.vdim + (SCALAR ? 1 : 0)) + 255) / 256);
   if (int rc = cima_launch(k_memory_combine<SCALAR>, dim3(blocks, (unsigned)a.heads, (unsigned)n_seqs), dim3(256), (size_t)0, stream, 1, a)) return rc;
-  return launch_memory<TA, SCALAR, 2, 2>(a, n_seqs * a.max_segs, stream);
+  return launch_memory<TA, SCALAR, 2>(a, n_seqs * a.max_segs, stream);
 }
 
 // The decays of the channel form from a low-rank projection: g = sigmoid(W2 a + b)^(1 / tau), a thread a channel for
@@ -354,6 +368,42 @@ k_channel_decay(const TA* __restrict__ a1, int lda, const TW* __restrict__ w2, c
 #pragma unroll
   for (int r = 0; r < DECAY_ROWS; r++)
     if (row0 + r < T) g[(size_t)(row0 + r) * channels + c] = expf(cima_log_sigmoid(acc[r] + b) * inv_tau);
+}
+
+// The same for ranks of at most 16: the channel's weights stay in registers, and a block takes DECAY_GROUPS times as many rows.
+constexpr int DECAY_GROUPS = 4;
+template <typename TA, typename TW>
+__global__ void __launch_bounds__(128)
+k_channel_decay16(const TA* __restrict__ a1, int lda, const TW* __restrict__ w2, const float* __restrict__ bias, float inv_tau,
+                  float* __restrict__ g, int T, int rank, int channels, int rows_per_block) {
+  const int c = blockIdx.x * 128 + threadIdx.x;
+  const int cc = min(c, channels - 1);
+  float w[16];                                           // weights and bias do not depend on the kernel in front
+#pragma unroll
+  for (int i = 0; i < 16; i++) w[i] = i < rank ? cima_to_f32<TW>(w2[(size_t)cc * rank + i]) : 0.f;
+  const float b = bias[cc];
+  cima_pdl_wait();
+  cima_pdl_trigger();
+  __shared__ __align__(16) float sa[16][DECAY_ROWS * DECAY_GROUPS];
+  const int row0 = blockIdx.y * rows_per_block, rows = min(rows_per_block, T - row0);
+  for (int idx = threadIdx.x; idx < 16 * rows_per_block; idx += 128) {
+    const int r = idx >> 4, i = idx & 15;
+    sa[i][r] = r < rows && i < rank ? cima_to_f32<TA>(a1[(size_t)(row0 + r) * lda + i]) : 0.f;
+  }
+  __syncthreads();
+  if (c >= channels) return;
+  for (int r0 = 0; r0 < rows; r0 += 4) {
+    float acc[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll
+    for (int i = 0; i < 16; i++) {
+      const float4 x = *reinterpret_cast<const float4*>(&sa[i][r0]);
+      acc[0] = fmaf(w[i], x.x, acc[0]); acc[1] = fmaf(w[i], x.y, acc[1]);
+      acc[2] = fmaf(w[i], x.z, acc[2]); acc[3] = fmaf(w[i], x.w, acc[3]);
+    }
+#pragma unroll
+    for (int r = 0; r < 4; r++)
+      if (r0 + r < rows) g[(size_t)(row0 + r0 + r) * channels + c] = expf(cima_log_sigmoid(acc[r] + b) * inv_tau);
+  }
 }
 
 // The scalar form's numbers from the gates' projections, with a running maximum m a head (state [slots, heads]):
@@ -405,6 +455,60 @@ k_scalar_gates(const TA* __restrict__ z, int ldz, const float* __restrict__ bi, 
   }
   if (lane == 0) *mp = m;
 }
+
+// The same for many tokens a sequence: a block a (sequence, head).  Seven warps make a tile's gates and, two tiles later, its
+// exponentials; between them the first warp walks the chain of maxima, which is the same chain in the same order.
+constexpr int GATE_TILE = 224;
+template <typename TA>
+__global__ void __launch_bounds__(256)
+k_scalar_gates_long(const TA* __restrict__ z, int ldz, const float* __restrict__ bi, const float* __restrict__ bf, float cap,
+                    float* __restrict__ mstate, const int* __restrict__ seq_slot, const int* __restrict__ seq_first_row,
+                    float* __restrict__ ab, float* __restrict__ floor_, int heads) {
+  cima_pdl_wait();
+  cima_pdl_trigger();
+  __shared__ float2 fi[3][GATE_TILE];
+  __shared__ float mm[2][GATE_TILE + 1];
+  const int h = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x;
+  const int first = seq_first_row[seq], n = seq_first_row[seq + 1] - first;
+  const int tiles = (n + GATE_TILE - 1) / GATE_TILE;
+  float* mp = mstate + (size_t)seq_slot[seq] * heads + h;
+  const float b_i = bi[h], b_f = bf[h], inv = 1.0f / cap;
+  float m = *mp;
+  for (int it = 0; it < tiles + 2; it++) {
+    if (tid >= 32) {
+      const int w = tid - 32;
+      if (it < tiles) {
+        const int t = it * GATE_TILE + w;
+        float2 x = make_float2(0.f, -INFINITY);          // behind the end: m stays
+        if (t < n) {
+          const TA* zp = z + (size_t)(first + t) * ldz + h;
+          x.y = cap * tanhf((cima_to_f32<TA>(zp[0]) + b_i) * inv);
+          x.x = cima_log_sigmoid(cap * tanhf((cima_to_f32<TA>(zp[heads]) + b_f) * inv));
+        }
+        fi[it % 3][w] = x;
+      }
+      const int j = it - 2, t = j * GATE_TILE + w;
+      if (j >= 0 && t < n) {
+        const float2 x = fi[j % 3][w];
+        const float before = mm[j & 1][w], after = mm[j & 1][w + 1];
+        const size_t at = (size_t)(first + t) * heads + h;
+        *reinterpret_cast<float2*>(ab + at * 2) = make_float2(expf(x.x + before - after), expf(x.y - after));
+        floor_[at] = expf(-after);
+      }
+    } else if (it >= 1 && it <= tiles) {
+      const int j = it - 1;
+      if (tid == 0) mm[j & 1][0] = m;
+#pragma unroll 16
+      for (int t = 0; t < GATE_TILE; t++) {
+        const float2 x = fi[j % 3][t];
+        m = fmaxf(x.x + m, x.y);
+        if (tid == 0) mm[j & 1][t + 1] = m;
+      }
+    }
+    __syncthreads();
+  }
+  if (tid == 0) *mp = m;
+}
 }  // namespace
 
 // q, k [T, >= heads * dim], v [T, >= heads * vdim] of one dtype (rows of ldq / ldk / ldv values).  scalar 0: g [T, heads * dim] the
@@ -439,7 +543,10 @@ extern "C" int cima_channel_decay(const void* a1, int adtype, int lda, const voi
   const dim3 grid((unsigned)((channels + 127) / 128), (unsigned)((T + DECAY_ROWS - 1) / DECAY_ROWS));
   const size_t smem = (size_t)rank * DECAY_ROWS * sizeof(float);
   int rc;
-#define RUN(TA, TW) rc = cima_launch(k_channel_decay<TA, TW>, grid, dim3(128), smem, stream, 1, (const TA*)a1, lda, (const TW*)w2, bias, inv_tau, g, T, rank, channels)
+  const int per = T <= 64 ? DECAY_ROWS : DECAY_ROWS * DECAY_GROUPS;      // (few rows: more blocks; a row's sum is the same either way)
+  const dim3 grid16(grid.x, (unsigned)((T + per - 1) / per));
+#define RUN(TA, TW) rc = rank <= 16 ? cima_launch(k_channel_decay16<TA, TW>, grid16, dim3(128), (size_t)0, stream, 1, (const TA*)a1, lda, (const TW*)w2, bias, inv_tau, g, T, rank, channels, per) \
+                                    : cima_launch(k_channel_decay<TA, TW>, grid, dim3(128), smem, stream, 1, (const TA*)a1, lda, (const TW*)w2, bias, inv_tau, g, T, rank, channels)
   if (adtype == CIMA_F32 && wdtype == CIMA_F32) RUN(float, float);
   else if (adtype == CIMA_F32 && wdtype == CIMA_BF16) RUN(float, __nv_bfloat16);
   else if (adtype == CIMA_BF16 && wdtype == CIMA_BF16) RUN(__nv_bfloat16, __nv_bfloat16);
@@ -449,14 +556,22 @@ extern "C" int cima_channel_decay(const void* a1, int adtype, int lda, const voi
   return rc ? rc : cima_launch_result();
 }
 
+// max_rows: most rows of a sequence (from 128 on a block walks a head's tokens in tiles; the numbers are the same).
 // z [T, ldz]: the input gates' projections of all heads, then the forget gates'; ab [T, heads, 2] and floor [T, heads] float32.
 extern "C" int cima_scalar_gates(const void* z, int dtype, int ldz, const float* bi, const float* bf, float cap, float* mstate,
                                  const int* seq_slot, const int* seq_first_row, float* ab, float* floor_, int T, int n_seqs, int heads,
-                                 cudaStream_t stream) {
+                                 int max_rows, cudaStream_t stream) {
   if (T <= 0 || n_seqs <= 0) return 0;
   if (heads <= 0 || !(cap > 0.f) || ldz < 2 * heads) return cima_fail(CIMA_E_SIZE, "scalar_gates: %d heads in rows of %d values, cap %g: the cap must be positive and a row hold two values a head", heads, ldz, (double)cap);
   const dim3 grid((unsigned)(((long long)n_seqs * heads + 3) / 4));
   int rc;
+  if (max_rows >= 128 && n_seqs <= 65535) {
+    const dim3 blocks((unsigned)heads, (unsigned)n_seqs);
+    if (dtype == CIMA_F32) rc = cima_launch(k_scalar_gates_long<float>, blocks, dim3(256), (size_t)0, stream, 1, (const float*)z, ldz, bi, bf, cap, mstate, seq_slot, seq_first_row, ab, floor_, heads);
+    else if (dtype == CIMA_BF16) rc = cima_launch(k_scalar_gates_long<__nv_bfloat16>, blocks, dim3(256), (size_t)0, stream, 1, (const __nv_bfloat16*)z, ldz, bi, bf, cap, mstate, seq_slot, seq_first_row, ab, floor_, heads);
+    else return cima_fail(CIMA_E_DTYPE, "scalar_gates: dtype code %d is neither float32 nor bfloat16", dtype);
+    return rc ? rc : cima_launch_result();
+  }
   if (dtype == CIMA_F32) rc = cima_launch(k_scalar_gates<float>, grid, dim3(128), (size_t)0, stream, 1, (const float*)z, ldz, bi, bf, cap, mstate, seq_slot, seq_first_row, ab, floor_, n_seqs, heads);
   else if (dtype == CIMA_BF16) rc = cima_launch(k_scalar_gates<__nv_bfloat16>, grid, dim3(128), (size_t)0, stream, 1, (const __nv_bfloat16*)z, ldz, bi, bf, cap, mstate, seq_slot, seq_first_row, ab, floor_, n_seqs, heads);
   else return cima_fail(CIMA_E_DTYPE, "scalar_gates: dtype code %d is neither float32 nor bfloat16", dtype);

@@ -141,6 +141,128 @@ __device__ __forceinline__ void moe_route_row(float* scores, float* local, int r
   for (int c = 0; c < top; c++) wgt[(size_t)row * top + c] *= f;
 }
 
+// The same with a warp a row, for at most ROUTE_SMEM_EXPERTS experts: the row's scores in registers (four a lane) and shared
+// memory, every choice a tree of comparisons over the lanes (the lowest index among equals, as one thread walking them
+// would take).  A thread a row took 8 us for the 8 rows of a decode step: a chain of some hundred dependent steps.
+constexpr int ROUTE_WARPS = 8, ROUTE_ORDER_WARPS = 32;
+struct RouteBest { float v; int i; };                      // i < 0: nothing
+__device__ __forceinline__ RouteBest route_better(RouteBest a, RouteBest b) {
+  const bool take = b.i >= 0 && (a.i < 0 || b.v > a.v || (b.v == a.v && b.i < a.i));
+  return take ? b : a;
+}
+__device__ __forceinline__ RouteBest route_best_of_warp(RouteBest a) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    RouteBest b;
+    b.v = __shfl_xor_sync(0xffffffffu, a.v, o);
+    b.i = __shfl_xor_sync(0xffffffffu, a.i, o);
+    a = route_better(a, b);
+  }
+  return a;
+}
+
+template <int WARPS>
+__global__ void __launch_bounds__(WARPS * 32)
+k_moe_route_warp(const float* __restrict__ scores, int T, int E, int ld, int top, int groups, int keep, float scale, int softmax,
+                 int best_one, int divide, int real, const float* __restrict__ corr, int* __restrict__ idx, float* __restrict__ wgt,
+                 int* __restrict__ offsets, int* __restrict__ tiles, int* __restrict__ perm) {
+  constexpr int PL = ROUTE_SMEM_EXPERTS / 32;               // scores a lane holds
+  __shared__ float s_choice[WARPS][ROUTE_SMEM_EXPERTS];
+  __shared__ float s_score[WARPS][ROUTE_SMEM_EXPERTS];
+  __shared__ int cnt[MOE_MAX_EXPERTS];
+  __shared__ int off[MOE_MAX_EXPERTS + 1];
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, per = E / groups;
+  float cor[PL];
+#pragma unroll
+  for (int j = 0; j < PL; j++) cor[j] = corr && lane + 32 * j < E ? corr[lane + 32 * j] : 0.f;
+  cima_pdl_wait();
+  cima_pdl_trigger();
+  for (int row = blockIdx.x * WARPS + warp; row < T; row += gridDim.x * WARPS) {
+    float s[PL], c[PL];
+#pragma unroll
+    for (int j = 0; j < PL; j++) s[j] = lane + 32 * j < E ? scores[(size_t)row * ld + lane + 32 * j] : -INFINITY;
+    if (softmax) {
+      float m = s[0];
+#pragma unroll
+      for (int j = 1; j < PL; j++) m = fmaxf(m, s[j]);
+      for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+      float den = 0.f;
+#pragma unroll
+      for (int j = 0; j < PL; j++) {
+        s[j] = lane + 32 * j < E ? expf(s[j] - m) : 0.f;
+        den += s[j];
+      }
+      for (int o = 16; o > 0; o >>= 1) den += __shfl_xor_sync(0xffffffffu, den, o);
+      const float inv = 1.0f / den;
+#pragma unroll
+      for (int j = 0; j < PL; j++) s[j] *= inv;
+    } else {
+#pragma unroll
+      for (int j = 0; j < PL; j++) s[j] = 1.0f / (1.0f + expf(-s[j]));
+    }
+    __syncwarp();
+#pragma unroll
+    for (int j = 0; j < PL; j++) {
+      c[j] = s[j] + cor[j];
+      if (lane + 32 * j < E) { s_choice[warp][lane + 32 * j] = c[j]; s_score[warp][lane + 32 * j] = s[j]; }
+    }
+    __syncwarp();
+    unsigned long long kept = ~0ull;
+    if (keep < groups) {
+      RouteBest g[2];                                       // the lane's groups: lane and lane + 32
+#pragma unroll
+      for (int t = 0; t < 2; t++) {
+        const int gi = lane + 32 * t;
+        float a1 = -INFINITY, a2 = -INFINITY;
+        for (int e = gi * per; gi < groups && e < (gi + 1) * per; e++) {
+          const float v = s_choice[warp][e];
+          if (v > a1) { a2 = a1; a1 = v; } else if (v > a2) a2 = v;
+        }
+        g[t].v = per >= 2 && !best_one ? a1 + a2 : a1;
+        g[t].i = gi < groups ? gi : -1;
+      }
+      kept = 0ull;
+      for (int k = 0; k < keep; k++) {
+        const RouteBest b = route_best_of_warp(route_better(g[0], g[1]));
+        kept |= 1ull << b.i;
+#pragma unroll
+        for (int t = 0; t < 2; t++)
+          if (g[t].i == b.i) g[t].i = -1;
+      }
+    }
+    bool open[PL];
+#pragma unroll
+    for (int j = 0; j < PL; j++) open[j] = lane + 32 * j < E && ((kept >> ((lane + 32 * j) / per)) & 1ull);
+    float sum = 0.f;
+    for (int k = 0; k < top; k++) {
+      RouteBest b{-INFINITY, -1};
+#pragma unroll
+      for (int j = 0; j < PL; j++) b = route_better(b, RouteBest{c[j], open[j] ? lane + 32 * j : -1});
+      b = route_best_of_warp(b);
+#pragma unroll
+      for (int j = 0; j < PL; j++)
+        if (lane + 32 * j == b.i) open[j] = false;
+      const float w = s_score[warp][b.i];
+      sum += w;
+      if (lane == 0) {
+        idx[(size_t)row * top + k] = b.i;
+        if (!divide) wgt[(size_t)row * top + k] = w * scale;
+      }
+      if (divide && lane == 0) s_choice[warp][k] = w;       // (the choice scores are in registers by now: their place holds the weights)
+    }
+    if (divide) {
+      __syncwarp();
+      const float f = scale / (sum + 1e-20f);
+      for (int k = lane; k < top; k += 32) wgt[(size_t)row * top + k] = s_choice[warp][k] * f;
+    }
+    __syncwarp();
+  }
+  if (offsets) {             // a step of one block's rows: the pairs are ordered by expert here, which saves moe_sort's launch
+    __syncthreads();
+    moe_sort_block(idx, T * top, real, offsets, tiles, perm, cnt, off);
+  }
+}
+
 // offsets [E + 1]: first sorted pair of every expert; tiles [E + 1]: first row tile of every expert; perm [P]: the
 // pair at every sorted place.  One block.
 __global__ void __launch_bounds__(1024)
@@ -481,6 +603,12 @@ extern "C" int cima_moe_route(float* scores, int T, int E, int ld, int top, int 
   if (top <= 0 || top > keep * (E / groups)) return cima_fail(CIMA_E_SIZE, "moe_route: %d choices among %d experts that stay", top, keep * (E / groups));
   if ((offsets || tiles || perm) && (!offsets || !tiles || !perm || T > ROUTE_THREADS))
     return cima_fail(CIMA_E_ARG, "moe_route: ordering the pairs here takes offsets, tiles and perm and at most %d rows (%d given)", ROUTE_THREADS, T);
+  if (E <= ROUTE_SMEM_EXPERTS) {
+    int rcw;
+    if (offsets) rcw = cima_launch(k_moe_route_warp<ROUTE_ORDER_WARPS>, dim3(1), dim3(ROUTE_ORDER_WARPS * 32), (size_t)0, stream, 1, scores, T, E, ld, top, groups, keep, scale, softmax, best_one, divide, real, correction, idx, wgt, offsets, tiles, perm);
+    else rcw = cima_launch(k_moe_route_warp<ROUTE_WARPS>, dim3((T + ROUTE_WARPS - 1) / ROUTE_WARPS), dim3(ROUTE_WARPS * 32), (size_t)0, stream, 1, scores, T, E, ld, top, groups, keep, scale, softmax, best_one, divide, real, correction, idx, wgt, offsets, tiles, perm);
+    return rcw ? rcw : cima_launch_result();
+  }
   int rc = cima_launch(k_moe_route, dim3((T + ROUTE_THREADS - 1) / ROUTE_THREADS), dim3(ROUTE_THREADS), (size_t)0, stream, 1, scores, T, E, ld, top, groups, keep, scale, softmax, best_one, divide, real, correction, idx, wgt, offsets, tiles, perm);
   return rc ? rc : cima_launch_result();
 }

@@ -260,6 +260,68 @@ k_norm_rope_append(TA* __restrict__ qkv, int ld, const float* __restrict__ inv_f
   }
 }
 
+// The norm, the queries' factor and the append where nothing rotates, for heads of at most 128 values in multiples of 4: a
+// block a row, a lane four neighbouring values of a head in registers, a warp NORM_HEADS heads at a time with all their loads
+// requested before the first use.
+constexpr int NORM_HEADS = 4;
+template <typename TA>
+__global__ void __launch_bounds__(128)
+k_norm_append(TA* __restrict__ qkv, int ld, const int* __restrict__ row_pos, const int* __restrict__ row_seq,
+              const int* __restrict__ seq_slot, const int* __restrict__ seq_len, TA* __restrict__ cache_in, CimaPaged pg, int nh,
+              int nkv, int hd, const float* __restrict__ q_norm, const float* __restrict__ k_norm, int norm_dim, float eps,
+              float temp_coef, int temp_every) {
+  cima_pdl_wait();
+  const int row = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int heads = nh + 2 * nkv, d = 4 * lane;
+  TA* base = qkv + (size_t)row * ld;
+  const int pos = row_pos[row], seq = row_seq[row];
+  TA* cache = cache_in;
+  if (cache && pg.ring && pos + pg.ring * pg.page_size < seq_len[seq]) cache = nullptr;
+  const int slot = cache ? seq_slot[seq] : 0;
+  const float temp = temp_every > 0 ? 1.0f + temp_coef * logf((float)((pos + 1) / temp_every + 1)) : 1.0f;
+  const bool in = d < hd;
+  for (int h0 = warp; h0 < heads; h0 += 4 * NORM_HEADS) {
+    float v[NORM_HEADS][4];
+#pragma unroll
+    for (int t = 0; t < NORM_HEADS; t++) {
+      const int head = h0 + 4 * t;
+      v[t][0] = v[t][1] = v[t][2] = v[t][3] = 0.f;
+      if (in && head < heads && (head < nh + nkv || cache)) rope_load4<TA>(base + (size_t)head * hd + d, v[t]);
+    }
+    float ss[NORM_HEADS];
+#pragma unroll
+    for (int t = 0; t < NORM_HEADS; t++) {
+      ss[t] = 0.f;
+#pragma unroll
+      for (int e = 0; e < 4; e++)
+        if (d + e < norm_dim) ss[t] = fmaf(v[t][e], v[t][e], ss[t]);
+    }
+    for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+      for (int t = 0; t < NORM_HEADS; t++) ss[t] += __shfl_xor_sync(0xffffffffu, ss[t], o);
+#pragma unroll
+    for (int t = 0; t < NORM_HEADS; t++) {
+      const int head = h0 + 4 * t;
+      if (!in || head >= heads) continue;
+      if (head >= nh + nkv) {                            // a value head: to the pages as it is
+        if (cache) RopePack4<TA>(v[t]).store(cache + pg.offset(slot, pos, 1, head - nh - nkv) + d);
+        continue;
+      }
+      const float* w = head < nh ? q_norm : k_norm;
+      const float f = head < nh ? temp : 1.0f;
+      const float r = norm_dim > 0 ? 1.0f / sqrtf(ss[t] / (float)norm_dim + eps) : 1.0f;
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        if (d + e < norm_dim) v[t][e] = w ? v[t][e] * r * w[d + e] : v[t][e] * r;
+        v[t][e] *= f;
+      }
+      const RopePack4<TA> p(v[t]);
+      p.store(base + (size_t)head * hd + d);
+      if (cache && head >= nh) p.store(cache + pg.offset(slot, pos, 0, head - nh) + d);
+    }
+  }
+}
+
 // cache may be null (a layer that reads another layer's keys and values writes none).
 // nv: value heads of a row (nkv unless key heads share value heads); q_norm / k_norm (both or neither): the weights of
 // a norm over the first norm_dim values of every q / k head before the rotation (null with norm_dim > 0: a norm without weight).
@@ -285,6 +347,12 @@ extern "C" int cima_rope_append(void* qkv, int dtype, int ld, const float* inv_f
     int rc_;
     const size_t bytes = dtype == CIMA_F32 ? 4 : 2;
     const bool vec = hd % 4 == 0 && ld % 4 == 0 && ((uintptr_t)qkv % (4 * bytes)) == 0 && ((uintptr_t)cache % (4 * bytes)) == 0;
+    if (vec && rotary_dim == 0 && hd <= 128 && nv == nkv) {
+      if (dtype == CIMA_F32) rc_ = cima_launch(k_norm_append<float>, dim3(T), dim3(128), (size_t)0, stream, 1, (float*)qkv, ld, row_pos, row_seq, seq_slot, seq_len, (float*)cache, pg, nh, nkv, hd, q_norm, k_norm, norm_dim, eps, temp_coef, temp_every);
+      else if (dtype == CIMA_BF16) rc_ = cima_launch(k_norm_append<__nv_bfloat16>, dim3(T), dim3(128), (size_t)0, stream, 1, (__nv_bfloat16*)qkv, ld, row_pos, row_seq, seq_slot, seq_len, (__nv_bfloat16*)cache, pg, nh, nkv, hd, q_norm, k_norm, norm_dim, eps, temp_coef, temp_every);
+      else return cima_fail(CIMA_E_DTYPE, "rope_append: dtype code %d is neither float32 nor bfloat16", dtype);
+      return rc_ ? rc_ : cima_launch_result();
+    }
     if (vec) {
       if (dtype == CIMA_F32) rc_ = cima_launch(k_norm_rope_append<float, 4>, grid, dim3(128), (size_t)0, stream, 1, (float*)qkv, ld, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, (float*)cache, pg, nh, nkv, nv, hd, q_norm, k_norm, norm_dim, eps, amp, temp_coef, temp_every);
       else if (dtype == CIMA_BF16) rc_ = cima_launch(k_norm_rope_append<__nv_bfloat16, 4>, grid, dim3(128), (size_t)0, stream, 1, (__nv_bfloat16*)qkv, ld, inv_freq, rotary_dim, row_pos, row_seq, seq_slot, seq_len, (__nv_bfloat16*)cache, pg, nh, nkv, nv, hd, q_norm, k_norm, norm_dim, eps, amp, temp_coef, temp_every);

@@ -113,7 +113,7 @@ _SIGNATURES = {
     "cima_cast_rows": [_vp, _vp, _i, _sz, _vp],
     "cima_memory": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _f, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _vp, _vp],
     "cima_channel_decay": [_vp, _i, _i, _vp, _i, _vp, _f, _vp, _i, _i, _i, _vp],
-    "cima_scalar_gates": [_vp, _i, _i, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
+    "cima_scalar_gates": [_vp, _i, _i, _vp, _vp, _f, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
     "cima_branch_norm": [_vp, _vp, _vp, _vp, _i, _vp, _i, _i, _f, _f, _vp],
     "cima_softcap": [_vp, _sz, _f, _vp],
     "cima_argmax": [_vp, _i, _i, _i, _vp, _vp],
@@ -1180,7 +1180,7 @@ class Kernels:
                                               _ptr(w2), T, W, eps, eps2, self._stream()), "branch_norm")
 
     # ------------------------------------------------------------------ matrix memories
-    MEMORY_SEGMENT = 256        # tokens of a segment of a long step's recurrence
+    MEMORY_SEGMENT = 192        # tokens of a segment of a long step's recurrence
 
     def memory_segments(self, batch) -> int:
         """Into how many segments at most a step's recurrence is cut (1: not at all): a number of the longest sequence's rows."""
@@ -1254,7 +1254,8 @@ class Kernels:
         if not self._admit("scalar_gates", T * heads * (2 * z.element_size() + 12)): return
         self._check(self.lib.cima_scalar_gates(z.data_ptr(), dtype_code(z.dtype), z.stride(0), bi.data_ptr(), bf.data_ptr(), float(cap),
                                                mstate.data_ptr(), batch.seq_slot.data_ptr(), batch.seq_first_row.data_ptr(), ab.data_ptr(),
-                                               low.data_ptr(), T, batch.n_seqs, heads, self._stream()), "scalar_gates")
+                                               low.data_ptr(), T, batch.n_seqs, heads, int(getattr(batch, "max_rows", 0) or 0),
+                                               self._stream()), "scalar_gates")
 
     # ------------------------------------------------------------------ routed feed-forward
     ROUTE_SORT_ROWS = 64        # a step of at most this many rows orders its pairs by expert in the routing launch

@@ -89,7 +89,7 @@ def test_heads_normed_and_gated(T, G, n, gate_dtype, out_dtype):
 
 
 @pytest.mark.parametrize("adt,wdt", [("float32", "float32"), ("float32", "bfloat16"), ("bfloat16", "bfloat16")])
-@pytest.mark.parametrize("T,C,rank,tau", [(1, 40, 3, 1.0), (8, 384, 16, 16.0), (300, 129, 5, 4.0), (17, 200, 64, 16.0)])
+@pytest.mark.parametrize("T,C,rank,tau", [(1, 40, 3, 1.0), (8, 384, 16, 16.0), (300, 129, 5, 4.0), (17, 200, 64, 16.0), (100, 130, 8, 16.0), (70, 40, 17, 2.0)])
 def test_channel_decays(T, C, rank, tau, adt, wdt):
     torch.manual_seed(C)
     a1 = (torch.randn(T, rank + 9) * 2).to(DT[adt])
@@ -220,7 +220,7 @@ def test_memories_cut_into_segments(scalar, heads, dim, vdim, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("T,heads,cap", [(1, 3, 5.0), (100, 2, 15.0), (33, 5, 8.0)])
+@pytest.mark.parametrize("T,heads,cap", [(1, 3, 5.0), (100, 2, 15.0), (33, 5, 8.0), (500, 3, 15.0), (448, 2, 6.0)])
 def test_scalar_gates_in_every_cutting(T, heads, cap, dtype):
     torch.manual_seed(T)
     z = (torch.randn(T, 2 * heads + 3) * 6).to(DT[dtype])
@@ -249,7 +249,8 @@ def _cache(hd, nkv=1, dtype=torch.float32, tokens=64 * 12):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("nh,nkv,hd,norm_dim,rot", [(4, 2, 32, 24, 0), (3, 1, 40, 40, 0), (2, 2, 128, 128, 64), (6, 0, 48, 40, 0), (2, 1, 21, 17, 8)])
+@pytest.mark.parametrize("nh,nkv,hd,norm_dim,rot", [(4, 2, 32, 24, 0), (3, 1, 40, 40, 0), (2, 2, 128, 128, 64), (6, 0, 48, 40, 0), (2, 1, 21, 17, 8),
+                                                     (12, 2, 128, 128, 0), (20, 3, 64, 58, 0), (3, 1, 144, 140, 0), (9, 0, 64, 64, 0)])
 def test_weightless_norm_temperature_and_append(nh, nkv, hd, norm_dim, rot, dtype):
     torch.manual_seed(hd)
     dt = DT[dtype]
