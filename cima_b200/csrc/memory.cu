@@ -334,6 +334,8 @@ int run_memory(const MemArgs& a, int n_seqs, cudaStream_t stream) {
 // The decays of the channel form from a low-rank projection: g = sigmoid(W2 a + b)^(1 / tau), a thread a channel for
 // ROWS rows at a time, the row's rank values in shared memory.
 constexpr int DECAY_ROWS = 8;
+// (the logarithm's absolute error decides the factor's relative one, so log(1 + e) serves where log1p would cost twice as much)
+__device__ __forceinline__ float decay_of(float z, float inv_tau) { return expf((fminf(z, 0.f) - logf(1.0f + expf(-fabsf(z)))) * inv_tau); }
 template <typename TA, typename TW>
 __global__ void __launch_bounds__(128)
 k_channel_decay(const TA* __restrict__ a1, int lda, const TW* __restrict__ w2, const float* __restrict__ bias, float inv_tau,
@@ -367,7 +369,7 @@ k_channel_decay(const TA* __restrict__ a1, int lda, const TW* __restrict__ w2, c
   const float b = bias[c];
 #pragma unroll
   for (int r = 0; r < DECAY_ROWS; r++)
-    if (row0 + r < T) g[(size_t)(row0 + r) * channels + c] = expf(cima_log_sigmoid(acc[r] + b) * inv_tau);
+    if (row0 + r < T) g[(size_t)(row0 + r) * channels + c] = decay_of(acc[r] + b, inv_tau);
 }
 
 // The same for ranks of at most 16: the channel's weights stay in registers, and a block takes DECAY_GROUPS times as many rows.
@@ -402,7 +404,7 @@ k_channel_decay16(const TA* __restrict__ a1, int lda, const TW* __restrict__ w2,
     }
 #pragma unroll
     for (int r = 0; r < 4; r++)
-      if (r0 + r < rows) g[(size_t)(row0 + r0 + r) * channels + c] = expf(cima_log_sigmoid(acc[r] + b) * inv_tau);
+      if (r0 + r < rows) g[(size_t)(row0 + r0 + r) * channels + c] = decay_of(acc[r] + b, inv_tau);
   }
 }
 
@@ -498,11 +500,25 @@ k_scalar_gates_long(const TA* __restrict__ z, int ldz, const float* __restrict__
     } else if (it >= 1 && it <= tiles) {
       const int j = it - 1;
       if (tid == 0) mm[j & 1][0] = m;
-#pragma unroll 16
-      for (int t = 0; t < GATE_TILE; t++) {
-        const float2 x = fi[j % 3][t];
-        m = fmaxf(x.x + m, x.y);
-        if (tid == 0) mm[j & 1][t + 1] = m;
+      // sixteen tokens' gates in registers, the next sixteen on their way; a lane keeps its token's maximum
+      constexpr int U = 16;
+      float2 x[U], nx[U];
+#pragma unroll
+      for (int u = 0; u < U; u++) nx[u] = fi[j % 3][u];
+      for (int t = 0; t < GATE_TILE; t += U) {
+#pragma unroll
+        for (int u = 0; u < U; u++) x[u] = nx[u];
+        if (t + U < GATE_TILE) {
+#pragma unroll
+          for (int u = 0; u < U; u++) nx[u] = fi[j % 3][t + U + u];
+        }
+        float mine = m;
+#pragma unroll
+        for (int u = 0; u < U; u++) {
+          m = fmaxf(x[u].x + m, x[u].y);
+          if (u == tid) mine = m;
+        }
+        if (tid < U) mm[j & 1][t + tid + 1] = mine;
       }
     }
     __syncthreads();
