@@ -14,7 +14,7 @@ from __future__ import annotations
 
 from typing import List, Optional, Sequence, Union
 
-from .config import (ArchitectureEntry, ConfigError, GisiraxConfig, LipizenConfig, NetezenConfig, PelatarConfig, Qwen2Config, VunovikConfig,
+from .config import (ArchitectureEntry, ConfigError, GisiraxConfig, GudaraxConfig, LipizenConfig, NetezenConfig, PelatarConfig, Qwen2Config, VunovikConfig,
                      lookup_architecture, read_config_json,
                      register_architecture, registered_architectures)
 from .sampling import GenOptions, OptionError
@@ -34,6 +34,8 @@ register_architecture(ArchitectureEntry(name=NetezenConfig.ARCHITECTURE, model_t
 register_architecture(ArchitectureEntry(name=PelatarConfig.ARCHITECTURE, model_type="pelatar",
                                         parse=PelatarConfig.from_dict, spec=PelatarConfig.model_spec,
                                         parse_with_shapes=PelatarConfig.from_dict))
+register_architecture(ArchitectureEntry(name=GudaraxConfig.ARCHITECTURE, model_type="gudarax",
+                                        parse=GudaraxConfig.from_dict, spec=GudaraxConfig.model_spec))
 
 __version__ = "0.1.0"
 
@@ -149,5 +151,5 @@ def write_random_model(folder: str, config: Union[dict, Qwen2Config], seed: int 
 
 
 __all__ = ["LM", "load", "write_random_model", "eos_ids_of", "GenOptions", "OptionError", "ConfigError",
-           "Qwen2Config", "VunovikConfig", "GisiraxConfig", "LipizenConfig", "NetezenConfig", "register_architecture", "registered_architectures", "lookup_architecture",
+           "Qwen2Config", "VunovikConfig", "GisiraxConfig", "LipizenConfig", "NetezenConfig", "GudaraxConfig", "register_architecture", "registered_architectures", "lookup_architecture",
            "read_config_json", "ArchitectureEntry"]

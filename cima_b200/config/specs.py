@@ -89,6 +89,16 @@ class BigramSpec:
 
 
 @dataclass(frozen=True)
+class TokenSideSpec:
+    """A token's own input to every layer, behind its feed-forward: x += norm(W_proj (act(W_gate x) * e)), e the layer's part
+    (``dim`` values) of the token's row in the side table ``name`` [vocab, layers * dim]; norm an RMS norm with a weight."""
+    name: str
+    dim: int
+    eps: float
+    activation: str = "gelu_tanh"
+
+
+@dataclass(frozen=True)
 class BlockSpec:
     kind: str                    # "prenorm": x += mixer(norm(x)); x += ffn(norm(x))
                                  # "parallel": h = norm(x); x += mixer(conv(h)) + ffn(h)
@@ -98,7 +108,7 @@ class BlockSpec:
                                  # "hyper": ``streams`` copies X_s of the stream; a sublayer reads norm(sum_s in[s] X_s) and
                                  #          X_t <- sum_s mix[s, t] X_s + m out[t] y for all t at once, m = residual_mult
     mixer: MixerSpec
-    feed_forward: Optional[FeedForwardSpec]      # None: the layer has no feed-forward ("parallel" only)
+    feed_forward: Optional[FeedForwardSpec]      # None: the layer has no feed-forward
     mixer_norm: NormSpec
     ffn_norm: Optional[NormSpec]                 # None where one norm serves both sublayers
     prefix: str                  # tensor-name prefix of the layer, e.g. "model.layers.3."
@@ -114,6 +124,8 @@ class BlockSpec:
     residual_mult: float = 1.0
     # "postnorm": the factor of the stream in the sum that the norm behind a sublayer reads
     stream_mult: float = 1.0
+    # "prenorm": what the token itself adds behind the feed-forward (tensors names["side_gate"], ["side_proj"], ["side_norm"])
+    token_side: Optional[TokenSideSpec] = None
     # "hyper": how many copies of the stream the model carries.  With names["mixer_hc"] / names["ffn_hc"] the vectors
     # <stem>.in, <stem>.out [streams] and the matrix <stem>.mix [streams, streams] (indexed [from, to]) of a sublayer are
     # stored tensors; without those names they are ones and the unit matrix (one stream: x += m * sublayer(norm(x)))
@@ -137,6 +149,9 @@ class ModelSpec:
     head_name: str
     embed_scale: float = 1.0
     embed_bigram: Optional[BigramSpec] = None       # a hashed bigram table added to the token embedding
+    embed_positions: Optional[str] = None           # a table [max_position, hidden] whose row p is added (unscaled) at position p
+    token_side: Optional[TokenSideSpec] = None      # the side table that the blocks' token inputs read
+    unread: Tuple[str, ...] = ()                    # glob patterns of names that a checkpoint may hold without the model reading them
     logit_softcap: float = 0.0                      # c > 0: logits <- c * tanh(logits / c)
     # A checkpoint of an untied model that stores no head tensor: the table serves as the head
     # (the reference decides so, src/models/transformer.rs:810, and warns, :839-841).

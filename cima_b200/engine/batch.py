@@ -6,8 +6,8 @@ and its length after the step.  All of it travels to the device in one copy from
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
-from typing import List, Optional, Sequence
+from dataclasses import dataclass, field
+from typing import Any, Dict, List, Optional, Sequence
 
 import numpy as np
 import torch
@@ -51,6 +51,8 @@ class StepBatch:
     host_seq_slot: np.ndarray = None
     host_seq_first_row: np.ndarray = None
     host_seq_len: np.ndarray = None
+    # what a layer leaves for later layers of the same step, by a name of its kind's own (emptied when the step ends)
+    carried: Dict[str, Any] = field(default_factory=dict)
 
 
 def check_entries(entries: Sequence[StepEntry], vocab: Optional[int] = None) -> None:

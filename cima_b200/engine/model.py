@@ -65,10 +65,17 @@ class Model:
                 raise ValueError(f"a depth average needs one vector per site: {len(spec.depth_names)} names for "
                                  f"{len(spec.schedule)} sites")
             self.depth = DepthAverage(spec.depth_names, rt)
+        if (spec.token_side is not None or spec.embed_positions is not None) and (spec.stream != "residual" or spec.embed_bigram is not None):
+            raise ValueError("position vectors and token inputs go with a single stream and without a bigram table")
+        for i, b in enumerate(spec.layers):
+            if b.token_side is not None and (b.kind != "prenorm" or b.token_side != spec.token_side):
+                raise ValueError(f"layer {i}: a token input goes with a block of kind 'prenorm' and the model's own side table")
         self.config = None                                  # set by load_model
         self.step_rows = STEP_ROWS                          # a step of more rows runs in parts
         self.embedding: Optional[torch.Tensor] = None
         self.bigram: Optional[torch.Tensor] = None          # the hashed bigram table, where the spec has one
+        self.positions: Optional[torch.Tensor] = None       # the vectors added at each position, where the spec has a table
+        self.side: Optional[torch.Tensor] = None            # the side table of the blocks' token inputs
         self.head: Optional[Linear] = None
         self.cache: Optional[KVCache] = None
 
@@ -78,6 +85,10 @@ class Model:
         p: Dict[str, TensorSpec] = {s.embed_name: TensorSpec((s.vocab, s.hidden))}
         if s.embed_bigram is not None:
             p[s.embed_bigram.name] = TensorSpec((s.embed_bigram.buckets + 1, s.hidden))
+        if s.embed_positions is not None:
+            p[s.embed_positions] = TensorSpec((s.max_position, s.hidden))
+        if s.token_side is not None:
+            p[s.token_side.name] = TensorSpec((s.vocab, len(s.layers) * s.token_side.dim), std=1.0)
         for b in self.blocks:
             p.update(b.plan())
         if self.depth is not None:
@@ -89,7 +100,7 @@ class Model:
 
     def ignorable(self) -> List[str]:
         """Names a checkpoint may hold without the model reading them."""
-        pats = ["*.rotary_emb.inv_freq"]
+        pats = ["*.rotary_emb.inv_freq", *self.spec.unread]
         if self.spec.tie_head:
             pats.append(self.spec.head_name)
         return pats
@@ -105,8 +116,14 @@ class Model:
         del table
         if s.embed_bigram is not None:
             self.bigram = self.rt.matrix(tensors[s.embed_bigram.name]).to(self.embedding.dtype)
+        if s.embed_positions is not None:
+            self.positions = self.rt.matrix(tensors[s.embed_positions]).to(self.embedding.dtype)
+        if s.token_side is not None:
+            self.side = self.rt.matrix(tensors[s.token_side.name])
         for b in self.blocks:
             b.load(tensors)
+            if getattr(b, "token_side", None) is not None:
+                b.token_side.attach(self.side)
         if self.depth is not None:
             self.depth.load(tensors)
         self.final_norm.load(tensors, s.final_norm_name)
@@ -120,6 +137,10 @@ class Model:
         out: Dict[str, torch.Tensor] = {s.embed_name: self.embedding}
         if self.bigram is not None:
             out[s.embed_bigram.name] = self.bigram
+        if self.positions is not None:
+            out[s.embed_positions] = self.positions
+        if self.side is not None:
+            out[s.token_side.name] = self.side
         for b in self.blocks:
             out.update(b.state())
         if self.depth is not None:
@@ -294,6 +315,12 @@ class Model:
             raise RuntimeError("a kernel's bounded wait ran out (TMA or tensor-core pipeline): results are invalid")
 
     def forward(self, batch: StepBatch) -> torch.Tensor:
+        try:
+            return self._forward(batch)
+        finally:
+            batch.carried.clear()                           # nothing of a step outlives it
+
+    def _forward(self, batch: StepBatch) -> torch.Tensor:
         K_, s = self.rt.kernels, self.spec
         if self.depth is not None:
             return self._forward_depth_average(batch)
@@ -304,6 +331,7 @@ class Model:
         # folded into the products around them (few rows) or run together with the residual add (many rows).
         info = None
         order = [self.blocks[layer] for layer in s.schedule]
+        at = {"positions": self.positions, "row_pos": batch.row_pos} if self.positions is not None else {}
         if s.embed_bigram is not None:
             g = s.embed_bigram
             K_.embed_bigram(batch, self.embedding, self.bigram, x, s.embed_scale, g.buckets, g.mul_prev, g.mul_cur,
@@ -314,13 +342,13 @@ class Model:
             if (getattr(first, "weight", None) is not None and first.spec.kind == "rmsnorm"
                     and first.spec.size == s.hidden):
                 xw = self.rt.empty(batch.n_rows, s.hidden)
-                K_.embed(batch.tokens, self.embedding, x, s.embed_scale, ssq, first.weight, xw)
+                K_.embed(batch.tokens, self.embedding, x, s.embed_scale, ssq, first.weight, xw, **at)
                 info = RowsInfo(ssq=ssq, xw=xw, xw_norm=first)
             else:
-                K_.embed(batch.tokens, self.embedding, x, s.embed_scale, ssq)
+                K_.embed(batch.tokens, self.embedding, x, s.embed_scale, ssq, **at)
                 info = RowsInfo(ssq=ssq)
         else:
-            K_.embed(batch.tokens, self.embedding, x, s.embed_scale)
+            K_.embed(batch.tokens, self.embedding, x, s.embed_scale, **at)
         for site, block in enumerate(order):
             if site + 1 < len(order):
                 nxt = getattr(order[site + 1], "mixer_norm", None)

@@ -18,7 +18,11 @@ by its root mean square over its ``head_dim`` values (e inside the root, no weig
 ``head_sink``: a stored number a head (tensor "sink") whose exponential joins that head's denominator, neither scaled nor
 attached to a value; ``gate``: the heads' results leave times sigmoid(W_g h), value by value (tensor "g", whose rows stand
 behind q | k | v in the same product, so that a row's gate lies in its own buffer and the attention kernels apply it where
-they finish a row).  ``own_kv`` False goes with ``cache_from``: the layer stores no W_k and W_v.  Keys and values live in the
+they finish a row).  ``row_norm_eps`` e: the whole q projection of a row (all its heads at once) is divided by its root mean
+square and multiplied by a weight of its size (tensor "q_norm"), and so is the whole k projection ("k_norm"), before the cache;
+``distance_slopes``, one number a head: m_h (i - j) is taken off the scaled score of position i with position j; ``v_mix``: the
+layer named "first" leaves its values to the later layers of the step, one named "mix" uses (1 - l) v + l v_first with the
+stored number l (tensor "v_mix") and caches that.  ``own_kv`` False goes with ``cache_from``: the layer stores no W_k and W_v.  Keys and values live in the
 cache at one size, the larger of the two rounded up to 16: the rows of W_q, W_k, W_v (and the columns of W_o) that
 pad a head are zero, so scores and outputs are what the unpadded sizes give.
 """
@@ -34,6 +38,9 @@ from .linear import Linear
 from .registry import build_position, register_mixer
 
 
+FIRST_VALUES = "attention.first_values"      # of ``StepBatch.carried``: (rows of values, values of a head there)
+
+
 class Attention:
     def __init__(self, spec, layer: int, rt):
         self.dim, self.vdim = spec.head_dim, int(spec.params.get("v_dim", spec.head_dim))
@@ -43,6 +50,8 @@ class Attention:
         self.q_temp = spec.params.get("q_temp")
         self.has_sink, self.gated = bool(spec.params.get("head_sink", False)), bool(spec.params.get("gate", False))
         self.own_kv = bool(spec.params.get("own_kv", True))
+        self.row_eps, self.v_mix = spec.params.get("row_norm_eps"), spec.params.get("v_mix")
+        self.slopes_host = spec.params.get("distance_slopes")
         if not self.own_kv and spec.cache_from is None:
             raise ValueError("attention: a layer without keys and values of its own names the site whose cache it reads")
         if self.sink and self.has_sink:
@@ -55,9 +64,16 @@ class Attention:
             raise ValueError(f"attention: {spec.n_heads} heads are not a multiple of {spec.n_kv_heads} kv heads")
         if (self.gated or not self.own_kv) and (spec.qkv_bias or spec.out_bias):
             raise ValueError("attention: biases beside an output gate or another layer's keys and values are not implemented")
-        if self.padded and (spec.qkv_bias or spec.out_bias):
-            raise ValueError(f"attention: head_dim {self.dim} must be a multiple of 16 and equal to the value size {self.vdim} "
-                             f"where the projections have biases (heads are padded in the cache only without biases)")
+        if self.v_mix not in (None, "first", "mix"):
+            raise ValueError(f"attention: v_mix '{self.v_mix}' is neither 'first' nor 'mix'")
+        if self.slopes_host is not None and len(self.slopes_host) != spec.n_heads:
+            raise ValueError(f"attention: {len(self.slopes_host)} distance slopes for {spec.n_heads} heads")
+        if self.row_eps is not None or self.v_mix is not None:
+            if spec.cache_from is not None or self.qk_eps or self.q_temp or self.gated or (spec.position is not None and spec.position.rotary_dim):
+                raise ValueError("attention: a norm over the whole projection and mixed values go with keys and values of the layer's own and "
+                                 "without rotation, head norms, query temperature or gate")
+            if self.row_eps is None:
+                raise ValueError("attention: mixed values go with the norm over the whole projection (one kernel does both)")
         self.spec, self.layer, self.rt = spec, layer, rt
         self.position = build_position(spec.position, rt)
         # (a position part registered elsewhere may offer neither: half-split pairs, amplitude 1)
@@ -69,7 +85,7 @@ class Attention:
         self.gate_col = self.qd + 2 * self.kvd if self.gated else 0      # where a row's gate begins
         self.qkv = None
         self.out = None
-        self.sinks = None
+        self.sinks = self.slopes = self.q_weight = self.k_weight = self.mix = None
 
     # ------------------------------------------------------------------ weights
     def plan(self, prefix: str, names: Dict[str, str]) -> Dict[str, TensorSpec]:
@@ -80,13 +96,22 @@ class Attention:
             rows = heads * size
             p[f"{prefix}{names[key]}{sfx}"] = TensorSpec((rows, s.hidden))
             if s.qkv_bias:
-                p[f"{prefix}{names[key]}.bias"] = TensorSpec((rows,))
+                p[f"{prefix}{names[key]}{self._bias(names)}"] = TensorSpec((rows,))
+        if self.row_eps is not None:
+            p[f"{prefix}{names['q_norm']}{sfx}"] = TensorSpec((s.n_heads * self.dim,), init="ones_normal")
+            p[f"{prefix}{names['k_norm']}{sfx}"] = TensorSpec((s.n_kv_heads * self.dim,), init="ones_normal")
+        if self.v_mix == "mix":
+            p[f"{prefix}{names['v_mix']}{sfx}"] = TensorSpec((), std=0.5)
         p[f"{prefix}{names['o']}{sfx}"] = TensorSpec((s.hidden, s.n_heads * self.vdim))
         if s.out_bias:
-            p[f"{prefix}{names['o']}.bias"] = TensorSpec((s.hidden,))
+            p[f"{prefix}{names['o']}{self._bias(names)}"] = TensorSpec((s.hidden,))
         if self.has_sink:
             p[f"{prefix}{names['sink']}{sfx}"] = TensorSpec((s.n_heads,), std=1.0)
         return p
+
+    @staticmethod
+    def _bias(names: Dict[str, str]) -> str:
+        return names.get("bias_suffix", ".bias")
 
     def _pieces(self):
         """(key, heads, size of a head) of the matrices that are stacked into the one projection, in its order of rows."""
@@ -111,7 +136,8 @@ class Attention:
         sfx = names.get("suffix", ".weight")
         bias = None
         if s.qkv_bias:
-            bias = torch.cat([tensors[f"{prefix}{names[k]}.bias"].float() for k in ("q", "k", "v")])
+            bias = torch.cat([self._pad_rows(tensors[f"{prefix}{names[k]}{self._bias(names)}"].float()[:, None], heads, size)[:, 0]
+                              for k, heads, size in self._pieces()])
 
         def rows(k, heads, size):
             t = tensors[f"{prefix}{names[k]}{sfx}"]
@@ -124,7 +150,14 @@ class Attention:
         self.qkv = Linear([rows(*piece) for piece in self._pieces()], bias, self.rt)
         if self.has_sink:
             self.sinks = self.rt.vector(tensors[f"{prefix}{names['sink']}{sfx}"])
-        ob = tensors[f"{prefix}{names['o']}.bias"] if s.out_bias else None
+        if self.row_eps is not None:                  # a head's padding is zero in q and k; its weights stay zero as well
+            self.q_weight = self.rt.vector(self._pad_rows(tensors[f"{prefix}{names['q_norm']}{sfx}"].float()[:, None], s.n_heads, self.dim)[:, 0])
+            self.k_weight = self.rt.vector(self._pad_rows(tensors[f"{prefix}{names['k_norm']}{sfx}"].float()[:, None], s.n_kv_heads, self.dim)[:, 0])
+        if self.v_mix == "mix":
+            self.mix = self.rt.vector(tensors[f"{prefix}{names['v_mix']}{sfx}"]).reshape(1)
+        if self.slopes_host is not None:
+            self.slopes = torch.tensor([float(m) for m in self.slopes_host], dtype=torch.float32, device=self.rt.device)
+        ob = tensors[f"{prefix}{names['o']}{self._bias(names)}"] if s.out_bias else None
         wo = tensors[f"{prefix}{names['o']}{sfx}"]
         if self.vdim != self.hd:
             wo = self._pad_rows(wo.t().contiguous(), s.n_heads, self.vdim).t().contiguous()
@@ -149,12 +182,18 @@ class Attention:
                 w = back
             out[f"{prefix}{names[key]}{sfx}"] = w
             if self.qkv.bias is not None:
-                out[f"{prefix}{names[key]}.bias"] = self.qkv.bias[r:r + rows]
+                b = self.qkv.bias[r:r + rows]
+                out[f"{prefix}{names[key]}{self._bias(names)}"] = b if size == self.hd else b.view(heads, self.hd)[:, :size].reshape(-1)
             r += rows
+        if self.row_eps is not None:
+            out[f"{prefix}{names['q_norm']}{sfx}"] = self.q_weight.view(s.n_heads, self.hd)[:, :self.dim].reshape(-1)
+            out[f"{prefix}{names['k_norm']}{sfx}"] = self.k_weight.view(s.n_kv_heads, self.hd)[:, :self.dim].reshape(-1)
+        if self.v_mix == "mix":
+            out[f"{prefix}{names['v_mix']}{sfx}"] = self.mix.reshape(())
         wo = self.out.weight
         out[f"{prefix}{names['o']}{sfx}"] = wo if self.vdim == self.hd else wo.view(-1, s.n_heads, self.hd)[:, :, :self.vdim].reshape(wo.shape[0], -1)
         if self.out.bias is not None:
-            out[f"{prefix}{names['o']}.bias"] = self.out.bias
+            out[f"{prefix}{names['o']}{self._bias(names)}"] = self.out.bias
         if self.has_sink:
             out[f"{prefix}{names['sink']}{sfx}"] = self.sinks
         return out
@@ -196,7 +235,7 @@ class Attention:
         rows = h.shape[0]
         if (not batch.prefill and writes and self.qkv._skinny(rows) and kv.storage.dtype is torch.bfloat16
                 and self.position.rotary_dim == self.hd and self.amplitude == 1.0 and not self.qk_eps and not self.q_temp and not self.gated
-                and hasattr(K_, "qkv_rope")):
+                and self.row_eps is None and hasattr(K_, "qkv_rope")):
             # decoding: projection, rotation and the append to the cache as one kernel
             qkv = self.rt.empty(rows, self.qd + 2 * self.kvd)
             if self.qkv._folds(h, rows):
@@ -207,6 +246,13 @@ class Attention:
                 K_.qkv_rope(h.tensor() if hasattr(h, "tensor") else h, self.qkv.weight, self.qkv.bias, qkv,
                             self.position.inv_freq, batch.row_pos, batch.row_seq, batch.seq_slot, kv, s.n_heads,
                             s.n_kv_heads, self.hd)
+        elif self.row_eps is not None:
+            qkv = self.qkv.store(h)
+            mix = (self.mix, *batch.carried[FIRST_VALUES]) if self.v_mix == "mix" else None
+            K_.row_norm_append(qkv, (self.q_weight, self.k_weight, self.dim, float(self.row_eps)), batch, kv, s.n_heads, s.n_kv_heads,
+                               self.hd, self.vdim, mix)
+            if self.v_mix == "first":                 # (the layer's own columns of its step's buffer, which nothing writes again)
+                batch.carried[FIRST_VALUES] = (qkv[:, self.qd + self.kvd:], self.hd)
         else:
             qkv = self.qkv.store(h)
             opts = {}
@@ -229,6 +275,8 @@ class Attention:
             more["head_sink"] = self.sinks
         if self.gated:
             more["gate_col"] = self.gate_col
+        if self.slopes is not None:
+            more["slopes"] = self.slopes
         K_.attention(qkv, kv, batch, att, s.n_heads, s.n_kv_heads, self.hd, s.scale, s.window, from_cache,
                      after_append=True, **more)
         return att

@@ -1,5 +1,6 @@
 """Arrangement of a layer's parts.  ``prenorm``: x += mixer(norm(x)); x += feed_forward(norm(x))
-(src/models/transformer.rs:1024-1319).  ``parallel``: h = norm(x); x += mixer(conv(h)) + feed_forward(h): one norm
+(src/models/transformer.rs:1024-1319); the feed-forward may be absent, and behind it the token's own input may join the
+stream (``TokenSide``).  ``parallel``: h = norm(x); x += mixer(conv(h)) + feed_forward(h): one norm
 feeds both sublayers, the mixer optionally through a short causal convolution, the feed-forward optionally absent.
 ``sandwich``: a norm in front of and behind each sublayer, x += m * post(mixer(norm(x))); x += m * post(ffn(norm(x))) with
 the spec's ``residual_mult`` m; the feed-forward with its two norms may be absent.  ``postnorm``: the norm stands behind
@@ -28,24 +29,34 @@ class PreNormBlock:
         self.spec, self.layer, self.rt = spec, layer, rt
         self.mixer_norm = build_norm(spec.mixer_norm, rt)
         self.mixer = build_mixer(spec.mixer, layer, rt)
-        self.ffn_norm = build_norm(spec.ffn_norm, rt)
-        self.feed_forward = build_feed_forward(spec.feed_forward, layer, rt)
+        self.ffn_norm = self.feed_forward = self.token_side = None
+        if spec.feed_forward is not None:
+            self.ffn_norm = build_norm(spec.ffn_norm, rt)
+            self.feed_forward = build_feed_forward(spec.feed_forward, layer, rt)
+        if spec.token_side is not None:
+            from .token_side import TokenSide
+            self.token_side = TokenSide(spec.token_side, layer, spec.mixer.hidden, rt)
+
+    def _named(self):
+        """(part, the arguments of its plan / load / state) for every part that owns tensors."""
+        s = self.spec
+        sfx = s.names.get("suffix", ".weight")
+        out = [(self.mixer_norm, (f"{s.prefix}{s.names['mixer_norm']}{sfx}",)), (self.mixer, (s.prefix, s.names))]
+        if self.feed_forward is not None:
+            out += [(self.ffn_norm, (f"{s.prefix}{s.names['ffn_norm']}{sfx}",)), (self.feed_forward, (s.prefix, s.names))]
+        if self.token_side is not None:
+            out.append((self.token_side, (s.prefix, s.names)))
+        return out
 
     def plan(self) -> Dict[str, TensorSpec]:
-        s = self.spec
         p: Dict[str, TensorSpec] = {}
-        p.update(self.mixer_norm.plan(f"{s.prefix}{s.names['mixer_norm']}.weight"))
-        p.update(self.mixer.plan(s.prefix, s.names))
-        p.update(self.ffn_norm.plan(f"{s.prefix}{s.names['ffn_norm']}.weight"))
-        p.update(self.feed_forward.plan(s.prefix, s.names))
+        for part, args in self._named():
+            p.update(part.plan(*args))
         return p
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
-        s = self.spec
-        self.mixer_norm.load(tensors, f"{s.prefix}{s.names['mixer_norm']}.weight")
-        self.mixer.load(tensors, s.prefix, s.names)
-        self.ffn_norm.load(tensors, f"{s.prefix}{s.names['ffn_norm']}.weight")
-        self.feed_forward.load(tensors, s.prefix, s.names)
+        for part, args in self._named():
+            part.load(tensors, *args)
 
     def cache_requests(self, site: int) -> List[object]:
         return list(self.mixer.cache_requests(site))
@@ -53,10 +64,8 @@ class PreNormBlock:
     def state(self) -> Dict[str, torch.Tensor]:
         """The layer's tensors by name as they are kept on the device (the inverse of ``load``).  A part offers
         ``state`` with the arguments of its ``plan``; one that does not cannot be written out."""
-        s = self.spec
         out: Dict[str, torch.Tensor] = {}
-        for part, args in ((self.mixer_norm, (f"{s.prefix}{s.names['mixer_norm']}.weight",)), (self.mixer, (s.prefix, s.names)),
-                           (self.ffn_norm, (f"{s.prefix}{s.names['ffn_norm']}.weight",)), (self.feed_forward, (s.prefix, s.names))):
+        for part, args in self._named():
             if not hasattr(part, "state"):
                 raise NotImplementedError(f"{type(part).__name__} of layer {self.layer} offers no state(): its tensors "
                                           f"cannot be given back by name")
@@ -65,17 +74,17 @@ class PreNormBlock:
 
     def scratch_row(self) -> int:
         """Values of the widest activation row that a step holds inside this layer (sizes the memory forecast)."""
-        return max(int(getattr(p, "scratch_row", lambda: 0)()) for p in (self.mixer, self.feed_forward))
+        return max(int(getattr(p, "scratch_row", lambda: 0)()) for p in (self.mixer, self.feed_forward, self.token_side) if p is not None)
 
     @property
     def graph_safe(self) -> bool:
         """Whether a decode step of this layer may be recorded as a CUDA graph: every part says so itself
         (``graph_safe = True``: it reads nothing of the batch on the host and keeps its buffers' addresses); a part
         that says nothing is taken as unfit, and the stepper then decodes step by step."""
-        return all(getattr(p, "graph_safe", False) for p in (self.mixer_norm, self.mixer, self.ffn_norm, self.feed_forward))
+        return all(getattr(p, "graph_safe", False) for p, _ in self._named())
 
     def nbytes(self) -> int:
-        return self.mixer_norm.nbytes() + self.mixer.nbytes() + self.ffn_norm.nbytes() + self.feed_forward.nbytes()
+        return sum(p.nbytes() for p, _ in self._named())
 
     def forward(self, x: torch.Tensor, batch, cache, site: int, info=None, next_norm=None):
         """``info`` (a ``RowsInfo`` or None): what the kernel that last wrote x left behind; the same for the
@@ -84,8 +93,13 @@ class PreNormBlock:
         its first product; one that declares ``takes_next_norm`` is told which norm follows it and may produce
         it with its last product.  Any other part gets the normalised tensor, and what it returns is
         ignored."""
-        info = self._run(self.mixer, self.mixer_norm, info, self.ffn_norm, x, (batch, cache, site))
-        return self._run(self.feed_forward, self.ffn_norm, info, next_norm, x, (batch,))
+        after = None if self.token_side is not None else next_norm       # the norm that reads x behind the sublayers
+        info = self._run(self.mixer, self.mixer_norm, info, self.ffn_norm if self.feed_forward is not None else after, x, (batch, cache, site))
+        if self.feed_forward is not None:
+            info = self._run(self.feed_forward, self.ffn_norm, info, after, x, (batch,))
+        if self.token_side is not None:
+            info = self.token_side.forward(x, batch, next_norm)
+        return info
 
     @staticmethod
     def _run(part, norm, info, next_norm, x, args):

@@ -1,4 +1,4 @@
-"""The gated delta rule with one decay a key channel (mixer kind ``channel_delta``).
+"""The gated delta rule with one decay a key channel (mixer kind ``channel_delta``), and with one decay a head (kind ``delta``).
 
     q, k = silu(conv(W_q h)), silu(conv(W_k h))  [kv_heads, dim];   v = silu(conv(W_v h))  [heads, v_dim]
            conv: a causal convolution over time on each channel (``taps`` taps, zeros before the start, no bias)
@@ -13,6 +13,11 @@ convolution's newest ``taps - 1`` inputs (two ``StateRequest``s, zeroed when a s
 before the start).  Unit norms, decays, step sizes and the recurrence are float32; projections and the convolution
 with its activation run in the activations' dtype.  The ranks of the two low-rank pairs (a1/a2, g1/g2) are
 ``a_rank`` and ``g_rank``.
+
+Kind ``delta`` is the same but for two lines,
+    g     = exp(-exp(A_log[h]) * softplus(W_a h + dt_bias))               one a head
+    y     = W_o ( rms(o over a head's values) * w * silu(W_g h) )
+and its projections q | k | v | g | b | a are one product.
 """
 from __future__ import annotations
 
@@ -139,4 +144,107 @@ class ChannelDelta:
         return gated
 
 
+class HeadDelta:
+    def __init__(self, spec, layer: int, rt):
+        from ..kernels import ACTIVATIONS
+        p = spec.params
+        self.heads, self.kv_heads, self.dim, self.vdim = spec.n_heads, spec.n_kv_heads, spec.head_dim, int(p["v_dim"])
+        self.taps, self.eps = int(p["taps"]), float(p["eps"])
+        if min(self.heads, self.kv_heads, self.dim, self.vdim) <= 0 or self.dim > 256:
+            raise ValueError("delta: heads, key heads, key size (at most 256) and value size must be positive")
+        if self.heads % self.kv_heads:
+            raise ValueError(f"delta: {self.heads} heads are not a multiple of {self.kv_heads} key heads")
+        self.spec, self.layer, self.rt = spec, layer, rt
+        self.kd, self.vd = self.kv_heads * self.dim, self.heads * self.vdim
+        self.channels = 2 * self.kd + self.vd
+        self.conv = ShortConv(ShortConvSpec(channels=self.channels, taps=self.taps), rt)
+        self.silu = ACTIVATIONS["silu"]
+        self.proj = self.out = self.A_log = self.dt_bias = self.norm = None
+
+    _n = staticmethod(ChannelDelta._n)
+
+    def _pieces(self):
+        """(key, rows) of the matrices stacked into the one projection, in its order."""
+        return (("q", self.kd), ("k", self.kd), ("v", self.vd), ("g", self.vd), ("b", self.heads), ("a", self.heads))
+
+    def plan(self, prefix: str, names: Dict[str, str]) -> Dict[str, TensorSpec]:
+        H = self.spec.hidden
+        p = {self._n(prefix, names, k): TensorSpec((rows, H)) for k, rows in self._pieces()}
+        for k, rows in self._pieces()[:3]:
+            p[self._n(prefix, names, k, ".conv")] = TensorSpec((rows, self.taps), std=0.3)
+        p[self._n(prefix, names, "A_log")] = TensorSpec((self.heads,), std=0.5)
+        p[self._n(prefix, names, "dt_bias")] = TensorSpec((self.heads,), std=0.5)
+        p[self._n(prefix, names, "norm")] = TensorSpec((self.vdim,), init="ones_normal")
+        p[self._n(prefix, names, "o")] = TensorSpec((H, self.vd))
+        return p
+
+    def load(self, tensors, prefix: str, names: Dict[str, str]) -> None:
+        rt = self.rt
+        mats = [tensors[self._n(prefix, names, k)] for k, _ in self._pieces()]
+        pad = -sum(m.shape[0] for m in mats) % 8                # zero rows up to a multiple of 8 outputs: rows keep their alignment
+        if pad:
+            mats.append(torch.zeros((pad, self.spec.hidden), dtype=mats[0].dtype, device=mats[0].device))
+        self.proj = Linear(mats, None, rt)
+        del mats
+        self.out = Linear(tensors[self._n(prefix, names, "o")], None, rt)
+        self.conv.load({"w": torch.cat([tensors[self._n(prefix, names, k, ".conv")].float() for k, _ in self._pieces()[:3]])}, "w")
+        self.A_log, self.dt_bias, self.norm = (rt.vector(tensors[self._n(prefix, names, k)]) for k in ("A_log", "dt_bias", "norm"))
+
+    def state(self, prefix: str, names: Dict[str, str]) -> Dict[str, torch.Tensor]:
+        out, r = {}, 0
+        taps = self.conv.weight.t()
+        for i, (k, rows) in enumerate(self._pieces()):
+            out[self._n(prefix, names, k)] = self.proj.weight[r:r + rows]
+            if i < 3:
+                out[self._n(prefix, names, k, ".conv")] = taps[r:r + rows]
+            r += rows
+        out[self._n(prefix, names, "o")] = self.out.weight
+        for k in ("A_log", "dt_bias", "norm"):
+            out[self._n(prefix, names, k)] = getattr(self, k)
+        return out
+
+    def nbytes(self) -> int:
+        return self.proj.nbytes() + self.out.nbytes() + self.conv.nbytes() + (2 * self.heads + self.vdim) * 4
+
+    def scratch_row(self) -> int:
+        return 2 * self.channels + 4 * self.kd + 4 * self.vd + 8 * self.heads
+
+    graph_safe = True
+    takes_pending_norm = True
+    takes_next_norm = True
+
+    @staticmethod
+    def state_name(site: int) -> str:
+        return f"delta.{site}"
+
+    def cache_requests(self, site: int) -> List[object]:
+        return [StateRequest(self.state_name(site), (self.heads, self.dim, self.vdim), torch.float32)] + self.conv.cache_requests(site)
+
+    def forward(self, h, x: torch.Tensor, batch, cache, site: int, next_norm=None):
+        return self.out.accumulate(self._gated(h, batch, cache, site), x, next_norm)
+
+    def produce(self, h, batch, cache, site: int) -> torch.Tensor:
+        """The mixer's output as float32 rows of its own (what ``forward`` adds into x)."""
+        return self.out.logits(self._gated(h, batch, cache, site))
+
+    def _gated(self, h, batch, cache, site: int) -> torch.Tensor:
+        K_, rt = self.rt.kernels, self.rt
+        rows, kd, C, H = h.shape[0], self.kd, self.channels, self.heads
+        p = self.proj.store(h)                                        # [rows, q | k | v | g | b | a]
+        gate, b, a = p[:, C:C + self.vd], p[:, C + self.vd:C + self.vd + H], p[:, C + self.vd + H:C + self.vd + 2 * H]
+        c = rt.empty(rows, C)
+        K_.short_conv(p[:, :C], self.conv.weight, cache.state[self.conv.state_name(site)] if self.taps > 1 else None, batch, c,
+                      add_input=False, act=self.silu)
+        f32 = torch.float32
+        qn, kn = rt.empty(rows, kd, dtype=f32), rt.empty(rows, kd, dtype=f32)
+        g, beta = rt.empty(rows, H, dtype=f32), rt.empty(rows, H, dtype=f32)
+        K_.delta_prepare(c, a, b, self.A_log, self.dt_bias, qn, kn, g, beta, H, self.kv_heads, self.dim)
+        o = rt.empty(rows, self.vd, dtype=f32)
+        K_.recurrence(qn, kn, c[:, 2 * kd:], cache.state[self.state_name(site)], batch, o, H, self.kv_heads, self.dim, self.vdim, g=g, beta=beta)
+        gated = rt.empty(rows, self.vd)
+        K_.group_rmsnorm_gate(o, self.norm, gate, gated, H, self.eps, silu=True)
+        return gated
+
+
 register_mixer("channel_delta", ChannelDelta)
+register_mixer("delta", HeadDelta)

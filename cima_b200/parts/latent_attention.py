@@ -18,7 +18,7 @@ own W_uk and W_uv.  Scores and softmax are float32 in every attention kernel; th
 
 Sizes and constants (heads, head_dim, v_dim, kv_rank, scale, the latent norm's eps) are the spec's.
 
-Four options, each off by default (``params``):
+Five options, each off by default (``params``):
   ``rot_dim`` r > 0 (with the spec's ``position`` of r rotary dims): the latent projection has r more rows; their output,
       rotated at the row's position, is one key part for all heads and is cached behind the latent (a position keeps
       kv_rank + r values).  A query head is [head_dim plain | r rotated] and its score q_plain . k_plain + q_rot . k_rot.
@@ -28,6 +28,8 @@ Four options, each off by default (``params``):
       matrix with the latent projection, and one kernel norms both latents, rotates the key part and appends.
   the spec's ``window`` w > 0: a row sees itself and the w - 1 positions before it; the pages form a ring.
   ``head_sink``: a stored number a head (tensor "sink") whose exponential joins the softmax's denominator without a value.
+  ``gate``: the concatenated heads leave times sigmoid(W_g u), value by value (tensor "g", whose rows stand behind the latent's
+      in the first matrix, so that the gates come with the first product; the product by W_uv applies them).
 """
 from __future__ import annotations
 
@@ -50,11 +52,12 @@ class LatentAttention:
             raise ValueError(f"latent_attention: heads {self.heads}, head_dim {self.dim}, v_dim {self.vdim} and kv_rank "
                              f"{self.rank} must be positive")
         self.rot, self.q_rank, self.has_sink = int(p.get("rot_dim", 0)), int(p.get("q_rank", 0)), bool(p.get("head_sink", False))
+        self.gated = bool(p.get("gate", False))
         self.spec, self.layer, self.rt = spec, layer, rt
         self.own = spec.cache_from is None
-        self.extended = bool(self.rot or self.q_rank or self.has_sink or spec.window)
+        self.extended = bool(self.rot or self.q_rank or self.has_sink or self.gated or spec.window)
         if self.extended and not self.own:
-            raise ValueError("latent_attention: a layer that reads another's latents takes no rotated part, query latent, window or sink")
+            raise ValueError("latent_attention: a layer that reads another's latents takes no rotated part, query latent, window, sink or gate")
         self.position = build_position(spec.position, rt) if self.rot else None
         if self.rot and self.position.rotary_dim != self.rot:
             raise ValueError(f"latent_attention: the rotated part has {self.rot} values, its position encoding turns {self.position.rotary_dim}")
@@ -86,6 +89,8 @@ class LatentAttention:
             p[self._n(prefix, names, "latent_norm")] = TensorSpec((self.rank,), init="ones_normal")
         p[self._n(prefix, names, "k_up")] = TensorSpec((self.heads * self.dim, self.rank), std=self.rank ** -0.5)
         p[self._n(prefix, names, "v_up")] = TensorSpec((self.od, self.rank), std=self.rank ** -0.5)
+        if self.gated:
+            p[self._n(prefix, names, "g")] = TensorSpec((self.od, s.hidden))
         if self.has_sink:
             p[self._n(prefix, names, "sink")] = TensorSpec((self.heads,), std=1.0)
         p[self._n(prefix, names, "o")] = TensorSpec((s.hidden, self.od))
@@ -102,6 +107,12 @@ class LatentAttention:
         if self.own:
             mats.append(tensors[self._n(prefix, names, "latent")])
             self.latent_norm = rt.vector(tensors[self._n(prefix, names, "latent_norm")])
+        if self.gated:
+            # (zero rows before the gates: they begin at a multiple of 8 values)
+            pad = -(sum(m.shape[0] for m in mats)) % 8
+            if pad:
+                mats.append(torch.zeros((pad, self.spec.hidden), dtype=mats[0].dtype, device=mats[0].device))
+            mats.append(tensors[self._n(prefix, names, "g")])
         if self.has_sink:
             self.sink = rt.vector(tensors[self._n(prefix, names, "sink")])
         self.q_latent = Linear(mats, None, rt)
@@ -123,10 +134,12 @@ class LatentAttention:
         else:
             out = {self._n(prefix, names, "q"): self.q_latent.weight[:first]}
         if self.own:
-            out[self._n(prefix, names, "latent")] = self.q_latent.weight[first:]
+            out[self._n(prefix, names, "latent")] = self.q_latent.weight[first:first + self.kd]
             out[self._n(prefix, names, "latent_norm")] = self.latent_norm
         out[self._n(prefix, names, "k_up")] = self.k_up_t.transpose(1, 2).reshape(self.heads * self.dim, self.rank)
         out[self._n(prefix, names, "v_up")] = self.v_up.reshape(self.od, self.rank)
+        if self.gated:
+            out[self._n(prefix, names, "g")] = self.q_latent.weight[self.q_latent.N - self.od:]
         if self.has_sink:
             out[self._n(prefix, names, "sink")] = self.sink
         out[self._n(prefix, names, "o")] = self.out.weight
@@ -138,7 +151,7 @@ class LatentAttention:
                 + (self.latent_norm.numel() * 4 if self.own else 0) + (self.q_up.nbytes() + self.q_rank * 4 if self.q_rank else 0))
 
     def scratch_row(self) -> int:
-        return self.qd + self.q_rank + self.kd + 2 * self.heads * self.kd + self.od
+        return self.qd + self.q_rank + self.kd + 2 * self.heads * self.kd + (2 if self.gated else 1) * self.od
 
     graph_safe = True
 
@@ -154,6 +167,12 @@ class LatentAttention:
         return [KVRequest(n_kv_heads=1, head_dim=self.kd, window=int(self.spec.window), planes=1)]
 
     # ------------------------------------------------------------------ step
+    @property
+    def takes_pending_norm(self) -> bool:
+        return self.extended            # u may be a NormedInput: the first product folds the norm in when it can
+
+    takes_next_norm = True
+
     def forward(self, u, x: torch.Tensor, batch, cache, site: int, next_norm=None):
         if self.extended:
             return self.out.accumulate(self._attend(u, batch, cache, site), x, next_norm)
@@ -185,12 +204,10 @@ class LatentAttention:
     def _attend(self, u, batch, cache, site: int) -> torch.Tensor:
         """The road of the options: [rows, heads * v_dim] in front of W_o."""
         K_, rt, s = self.rt.kernels, self.rt, self.spec
-        if hasattr(u, "tensor"):
-            u = u.tensor()
         rows = u.shape[0]
         kv = cache.layer_kv(site)
         first = self.q_rank or self.qd
-        ql = self.q_latent.store(u)                                  # [rows, (q latent or q) | latent | key part to rotate]
+        ql = self.q_latent.store(u)                                  # [rows, (q latent or q) | latent | key part to rotate (| gates)]
         cq = rt.empty(rows, self.q_rank) if self.q_rank else None
         pos = self.position
         # A prompt that starts reads its own rows (a window's ring of pages does not hold a long prompt): the moved
@@ -212,7 +229,8 @@ class LatentAttention:
         more = {"head_sink": self.sink} if self.sink is not None else {}
         K_.attention(qa, kv, batch, ol, self.heads, 1, self.kd, s.scale, int(s.window), not own_rows, **more)
         att = rt.empty(rows, self.od)
-        K_.head_linear(ol, self.v_up, att, a_head=self.kd, out_head=self.vdim)
+        gate = {"gate": (ql, self.q_latent.N - self.od)} if self.gated else {}
+        K_.head_linear(ol, self.v_up, att, a_head=self.kd, out_head=self.vdim, **gate)
         return att
 
 

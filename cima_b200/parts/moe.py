@@ -7,6 +7,9 @@
     y = sum_e  w_e * W_down[e] (act(W_gate[e] h) * (W_up[e] h))
 
 Options (``params``), each off by default:
+  ``gated`` False: an expert has no gate, y_e = W_down[e] act(W_up[e] h), act one of ``kernels.UNGATED_ACTIVATIONS`` (tensors
+      "e<j>.up", "e<j>.down" only);
+  ``weight_on`` "input": the weight multiplies what an expert reads, not what it gives: y = sum_e expert_e(w_e h);
   ``identity`` n: n more router outputs behind the experts', identity experts: they are scored, grouped and chosen like the
       others, their output is h itself, and they have no tensors;
   ``group_score`` "best": a group's score is its largest s (with the correction) instead of the sum of its two largest;
@@ -19,7 +22,7 @@ Options (``params``), each off by default:
       "shared.up", "shared.down"), added unweighted, or with ``shared_gate`` times sigmoid(w_sg . h) (tensor "shared.sg",
       [1, hidden]; its row stands under the router's in one matrix, so the routing product gives its logit too).
 
-The experts' matrices are kept stacked, [E, 2 ff, H] (an expert's gate rows, then its up rows) and [E, H, ff]; a step
+The experts' matrices are kept stacked, [E, 2 ff, H] (an expert's gate rows, then its up rows; ungated: [E, ff, H]) and [E, H, ff]; a step
 sorts its (row, choice) pairs by expert on the device and runs two grouped products over tiles of one expert's pairs,
 so nothing of the routing is read on the host.  Tensors: ``router`` and, per expert j, ``e<j>.gate``, ``e<j>.up``,
 ``e<j>.down`` under the feed-forward's stem (names["experts"]).
@@ -38,7 +41,7 @@ from .registry import register_feed_forward
 
 class RoutedExperts:
     def __init__(self, spec, layer: int, rt):
-        from ..kernels import ACTIVATIONS
+        from ..kernels import ACTIVATIONS, UNGATED_ACTIVATIONS
         p = spec.params
         self.E, self.top = int(p["experts"]), int(p["top"])
         self.identity = int(p.get("identity", 0))
@@ -47,8 +50,12 @@ class RoutedExperts:
             raise ValueError(f"moe: group_score '{p.get('group_score')}' is neither 'two' nor 'best'")
         self.best_one, self.normalize = p.get("group_score", "two") == "best", bool(p.get("normalize", True))
         self.groups, self.keep, self.scale = int(p.get("groups", 1)), int(p.get("keep", p.get("groups", 1))), float(p.get("scale", 1.0))
-        if spec.activation not in ACTIVATIONS:
-            raise ValueError(f"moe: activation '{spec.activation}' is not one of {sorted(ACTIVATIONS)}")
+        self.gated, self.weigh_input = bool(p.get("gated", True)), p.get("weight_on", "output") == "input"
+        if p.get("weight_on", "output") not in ("output", "input"):
+            raise ValueError(f"moe: weight_on '{p.get('weight_on')}' is neither 'output' nor 'input'")
+        table = ACTIVATIONS if self.gated else UNGATED_ACTIVATIONS
+        if spec.activation not in table:
+            raise ValueError(f"moe: activation '{spec.activation}' is not one of {sorted(table)}")
         self.limit = float(p.get("limit", 0.0))
         self.softmax = p.get("scoring", "sigmoid") == "softmax"
         if p.get("scoring", "sigmoid") not in ("sigmoid", "softmax"):
@@ -62,7 +69,9 @@ class RoutedExperts:
             raise ValueError(f"moe: {self.top} choices among the {self.keep * (self.n // self.groups)} experts that stay")
         if self.n > 1024 or self.groups > 64:
             raise ValueError("moe: at most 1024 experts in at most 64 groups")
-        self.act = ACTIVATIONS[spec.activation]
+        if (self.weigh_input or not self.gated) and (self.identity or self.shared_spec is not None):
+            raise ValueError("moe: weights on the experts' inputs and ungated experts beside identity or shared experts are not implemented")
+        self.act = table[spec.activation]
         self.spec, self.layer, self.rt = spec, layer, rt
         self.router = self.gate_up = self.down = self.correction = self.shared_up = self.shared_down = None
 
@@ -73,7 +82,8 @@ class RoutedExperts:
         s = self.spec
         p = {self._n(prefix, names, "router"): TensorSpec((self.n, s.hidden), std=0.1)}
         for j in range(self.E):
-            p[self._n(prefix, names, f"e{j}.gate")] = TensorSpec((s.intermediate, s.hidden))
+            if self.gated:
+                p[self._n(prefix, names, f"e{j}.gate")] = TensorSpec((s.intermediate, s.hidden))
             p[self._n(prefix, names, f"e{j}.up")] = TensorSpec((s.intermediate, s.hidden))
             p[self._n(prefix, names, f"e{j}.down")] = TensorSpec((s.hidden, s.intermediate))
         if self.has_correction:
@@ -90,7 +100,7 @@ class RoutedExperts:
     def load(self, tensors, prefix: str, names: Dict[str, str]) -> None:
         s, rt = self.spec, self.rt
         rows = [tensors[self._n(prefix, names, "router")]]
-        if self.shared_gate or self.identity:
+        if self.shared_gate or self.identity or not self.gated:
             # the gate's row under the router's, then zero rows up to a multiple of 8 outputs (a row of the scores keeps its
             # 16-byte alignment, and the library's product of many rows its fast kernels)
             if self.shared_gate:
@@ -109,12 +119,14 @@ class RoutedExperts:
                                              rt, sh.get("activation", s.activation), limit=float(sh.get("limit", 0.0)))
             self.shared_down = Linear(tensors[self._n(prefix, names, "shared.down")], None, rt)
         ff, H = s.intermediate, s.hidden
-        first = rt.matrix(tensors[self._n(prefix, names, "e0.gate")])
-        self.gate_up = torch.empty((self.E, 2 * ff, H), dtype=first.dtype, device=rt.device)
+        key = "gate" if self.gated else "up"
+        first = rt.matrix(tensors[self._n(prefix, names, f"e0.{key}")])
+        self.gate_up = torch.empty((self.E, (2 if self.gated else 1) * ff, H), dtype=first.dtype, device=rt.device)
         self.down = torch.empty((self.E, H, ff), dtype=first.dtype, device=rt.device)
         for j in range(self.E):
-            self.gate_up[j, :ff].copy_(first if j == 0 else tensors[self._n(prefix, names, f"e{j}.gate")])
-            self.gate_up[j, ff:].copy_(tensors[self._n(prefix, names, f"e{j}.up")])
+            self.gate_up[j, :ff].copy_(first if j == 0 else tensors[self._n(prefix, names, f"e{j}.{key}")])
+            if self.gated:
+                self.gate_up[j, ff:].copy_(tensors[self._n(prefix, names, f"e{j}.up")])
             self.down[j].copy_(tensors[self._n(prefix, names, f"e{j}.down")])
 
     def state(self, prefix: str, names: Dict[str, str]) -> Dict[str, torch.Tensor]:
@@ -129,8 +141,9 @@ class RoutedExperts:
             if self.shared_gate:
                 out[self._n(prefix, names, "shared.sg")] = self.router.weight[self.n:self.n + 1]
         for j in range(self.E):
-            out[self._n(prefix, names, f"e{j}.gate")] = self.gate_up[j, :ff]
-            out[self._n(prefix, names, f"e{j}.up")] = self.gate_up[j, ff:]
+            if self.gated:
+                out[self._n(prefix, names, f"e{j}.gate")] = self.gate_up[j, :ff]
+            out[self._n(prefix, names, f"e{j}.up")] = self.gate_up[j, -ff:]
             out[self._n(prefix, names, f"e{j}.down")] = self.down[j]
         return out
 
@@ -176,10 +189,13 @@ class RoutedExperts:
             route["best_one"] = True
         if not self.normalize:
             route["divide"] = False
-        if self.limit or self.act >= GATED_ONLY:
-            expert = {"limit": self.limit}
-        else:
-            expert = {}
+        expert = {}
+        if self.gated and (self.limit or self.act >= GATED_ONLY):
+            expert["limit"] = self.limit
+        if not self.gated:
+            expert["gated"] = False
+        if self.weigh_input:
+            expert["weigh_input"] = True
         if self.identity:
             expert["identity"] = True
         idx = rt.empty(rows, self.top, dtype=torch.int32)

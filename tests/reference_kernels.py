@@ -34,8 +34,10 @@ class ReferenceKernels:
         self.launches = 0
 
     # ------------------------------------------------------------------ elementwise
-    def embed(self, ids, table, x, scale=1.0, ssq=None, w_next=None, xw=None):
+    def embed(self, ids, table, x, scale=1.0, ssq=None, w_next=None, xw=None, positions=None, row_pos=None):
         x.copy_(table[ids.long()].float() * scale)
+        if positions is not None:
+            x.add_(positions[row_pos[:ids.numel()].long()].float())
         if ssq is not None:
             ssq.copy_((x.double() ** 2).sum(dim=1, keepdim=True).float())
         if xw is not None:
@@ -65,6 +67,11 @@ class ReferenceKernels:
             u = torch.clamp(u, min=-limit, max=limit)
             return g * torch.sigmoid(1.702 * g) * (u + 1.0)
         return cls.gate_act(g, act) * u
+
+    @classmethod
+    def ungated(cls, z, act):
+        """An ungated middle by its code: the gate activations, or (5) the square of ReLU."""
+        return torch.clamp(z, min=0.0) ** 2 if act == 5 else cls.gate_act(z, act)
 
     def swiglu(self, gate_up, out, act=0, limit=0.0):
         I = gate_up.shape[1] // 2
@@ -175,12 +182,12 @@ class ReferenceKernels:
             kv.storage[page, 1, :nv, off, :] = heads[r, n_heads + n_kv_heads:, :]
 
     def attention(self, qkv, kv, batch, out, n_heads, n_kv_heads, head_dim, scale, window, from_cache, after_append=False,
-                  sink=0.0, keep_first=0, v_group=1, head_sink=None, gate_col=0):
+                  sink=0.0, keep_first=0, v_group=1, head_sink=None, gate_col=0, slopes=None):
         self.attention_plain(qkv, kv, batch.row_pos, batch.row_seq, batch.seq_slot, batch.seq_first_row, out,
-                             n_heads, n_kv_heads, head_dim, scale, window, from_cache, sink, keep_first, v_group, head_sink, gate_col)
+                             n_heads, n_kv_heads, head_dim, scale, window, from_cache, sink, keep_first, v_group, head_sink, gate_col, slopes)
 
     def attention_plain(self, qkv, kv, row_pos, row_seq, seq_slot, seq_first_row, out, n_heads, n_kv_heads,
-                        head_dim, scale, window, from_cache, sink=0.0, keep_first=0, v_group=1, head_sink=None, gate_col=0):
+                        head_dim, scale, window, from_cache, sink=0.0, keep_first=0, v_group=1, head_sink=None, gate_col=0, slopes=None):
         T = qkv.shape[0]
         rep = n_heads // n_kv_heads
         vplane = int(getattr(kv, "planes", 2)) - 1 if from_cache else 1      # one plane: the values are the keys
@@ -208,6 +215,8 @@ class ReferenceKernels:
             for h in range(n_heads):
                 g = h // rep
                 s = (k[:, g, :] @ q[h]) * scale
+                if slopes is not None:                      # a bias by distance
+                    s = s - slopes[h].to(self.compute) * (pos - torch.tensor(seen)).to(self.compute)
                 if head_sink is not None:                   # one entry of the head's own score without a value
                     z = head_sink[h].to(self.compute)
                     m = torch.maximum(s.max(), z)
@@ -300,14 +309,18 @@ def _latent_append(self, raw, g, eps, kv, batch):
         kv.storage[page, 0, 0, off, :] = c[t].to(kv.storage.dtype)
 
 
-def _head_linear(self, a, w, out, append=None, a_head=None, out_head=None):
+def _head_linear(self, a, w, out, append=None, a_head=None, out_head=None, gate=None):
     if append is not None:
         self.latent_append(*append)
     heads, N, K = w.shape
     ha, ho = a_head or K, out_head or N
     T = a.shape[0]
     av = torch.stack([a[:, h * ha:h * ha + K] for h in range(heads)], dim=1)
-    y = torch.einsum("thk,hnk->thn", av.to(self.compute), w.to(self.compute)).to(out.dtype)
+    y = torch.einsum("thk,hnk->thn", av.to(self.compute), w.to(self.compute))
+    if gate is not None:
+        rows, col = gate
+        y = y * torch.sigmoid(rows[:, col:col + heads * N].to(self.compute)).view(T, heads, N)
+    y = y.to(out.dtype)
     for h in range(heads):
         out[:, h * ho:h * ho + N] = y[:, h]
 
@@ -375,8 +388,7 @@ def _hyper_connect(self, xs, y, C, b, mult, a_next, w_next, eps, h, spread=False
 
 
 def _activate(self, z, act):
-    f = z.float()
-    z.copy_((torch.clamp(f, min=0.0) ** 2 if act == 5 else self.gate_act(f, act)).to(z.dtype))
+    z.copy_(self.ungated(z.float(), act).to(z.dtype))
 
 
 ReferenceKernels.short_conv = _short_conv
@@ -448,7 +460,7 @@ def _recurrence(self, q, k, v, state, batch, out, heads, kv_heads, dim, vdim, g=
             S = state[slot, h].clone()
             for t in range(lo, hi):
                 if delta:
-                    S = g[t].view(heads, dim)[h][:, None] * S
+                    S = (g[t].view(heads, dim)[h][:, None] if g.shape[1] == heads * dim else g[t, h]) * S
                     u = beta[t, h] * (vf[t, h] - S.T @ kf[t, c])
                 else:
                     S = decay[h] * S
@@ -464,8 +476,8 @@ def _delta_prepare(self, qk, a, b, A_log, dt_bias, qn, kn, g, beta, heads, kv_he
     qf, kf = qk[:, :kd].float().view(T, kv_heads, dim), qk[:, kd:2 * kd].float().view(T, kv_heads, dim)
     qn.copy_((qf / torch.sqrt((qf * qf).sum(-1, keepdim=True) + 1e-6) * dim ** -0.5).view(T, kd))
     kn.copy_((kf / torch.sqrt((kf * kf).sum(-1, keepdim=True) + 1e-6)).view(T, kd))
-    step = torch.nn.functional.softplus(a.float() + dt_bias).view(T, heads, dim)
-    g.copy_(torch.exp(-torch.exp(A_log)[None, :, None] * step).view(T, heads * dim))
+    step = torch.nn.functional.softplus(a.float() + dt_bias).view(T, heads, -1)         # a decay a key channel, or one a head
+    g.copy_(torch.exp(-torch.exp(A_log)[None, :, None] * step).view(T, -1))
     beta.copy_(torch.sigmoid(b.float()))
 
 
@@ -513,8 +525,8 @@ def _moe_route(self, scores, top, groups, keep, scale, idx, wgt, experts=None, s
     scores[:, :E] = s
 
 
-def _moe_experts(self, h, gate_up, down, idx, wgt, x, act=0, assign=False, limit=0.0, shared=None, identity=False):
-    ff = gate_up.shape[1] // 2
+def _moe_experts(self, h, gate_up, down, idx, wgt, x, act=0, assign=False, limit=0.0, shared=None, identity=False, gated=True, weigh_input=False):
+    ff = gate_up.shape[1] // 2 if gated else gate_up.shape[1]
     hf = h.float()
     for t in range(h.shape[0]):
         acc = torch.zeros_like(x[t])
@@ -523,9 +535,11 @@ def _moe_experts(self, h, gate_up, down, idx, wgt, x, act=0, assign=False, limit
             if identity and e >= gate_up.shape[0]:
                 acc = acc + wgt[t, j] * hf[t]
                 continue
-            gu = (gate_up[e].float() @ hf[t]).to(h.dtype).float()
-            z = self.gated(gu[:ff], gu[ff:], act, limit).to(h.dtype).float()
-            acc = acc + wgt[t, j] * (down[e].float() @ z)
+            gu = gate_up[e].float() @ hf[t]
+            gu = ((gu * wgt[t, j]) if weigh_input else gu).to(h.dtype).float()
+            z = (self.gated(gu[:ff], gu[ff:], act, limit) if gated else self.ungated(gu, act)).to(h.dtype).float()
+            y = down[e].float() @ z
+            acc = acc + (y if weigh_input else wgt[t, j] * y)
         if shared is not None:
             rows, gate, col = shared
             acc = acc + (torch.sigmoid(gate[t, col]) if gate is not None else 1.0) * rows[t]
@@ -626,4 +640,41 @@ for _name, _fn in (("diff_combine", _diff_combine), ("scale_add_group_rmsnorm", 
 for _name, _fn in (("dyt", _dyt), ("dyt_add", _dyt_add), ("embed_bigram", _embed_bigram), ("recurrence", _recurrence),
                    ("delta_prepare", _delta_prepare), ("group_rmsnorm_gate", _group_rmsnorm_gate), ("rms_mean", _rms_mean),
                    ("moe_route", _moe_route), ("moe_experts", _moe_experts)):
+    setattr(ReferenceKernels, _name, _fn)
+
+
+# ---------------------------------------------------------------------- a token's own input, the norm over whole projections
+def _row_norm_append(self, qkv, norm, batch, kv, n_heads, n_kv_heads, head_dim, v_dim, mix=None):
+    wq, wk, dim, eps = norm
+    T = qkv.shape[0]
+    qd, kvd = n_heads * head_dim, n_kv_heads * head_dim
+    for lo, hi, w, heads in ((0, qd, wq, n_heads), (qd, qd + kvd, wk, n_kv_heads)):
+        z = qkv[:, lo:hi].to(self.compute)
+        z = z / torch.sqrt((z * z).sum(-1, keepdim=True) / (heads * dim) + eps) * w.to(self.compute)
+        qkv[:, lo:hi] = z.to(qkv.dtype)
+    if mix is not None:
+        lam, first, first_hd = mix
+        v = qkv[:, qd + kvd:qd + 2 * kvd].view(T, n_kv_heads, head_dim)
+        f = first[:, :n_kv_heads * first_hd].view(T, n_kv_heads, first_hd)
+        v[..., :v_dim] = ((1.0 - lam) * v[..., :v_dim].to(self.compute) + lam * f[..., :v_dim].to(self.compute)).to(qkv.dtype)
+    for t in range(T):
+        seq, pos = int(batch.row_seq[t]), int(batch.row_pos[t])
+        if kv.ring_pages and pos + kv.ring_pages * kv.page_size < int(batch.seq_len[seq]):
+            continue
+        page, off = _page_offset(kv, int(batch.seq_slot[seq]), pos)
+        kv.storage[page, 0, :, off, :] = qkv[t, qd:qd + kvd].view(n_kv_heads, head_dim)
+        kv.storage[page, 1, :, off, :] = qkv[t, qd + kvd:qd + 2 * kvd].view(n_kv_heads, head_dim)
+
+
+def _token_side_apply(self, z, table, tokens, col, act):
+    e = table[tokens[:z.shape[0]].long(), col:col + z.shape[1]].float()
+    z.copy_((self.gate_act(z.float(), act) * e).to(z.dtype))
+
+
+def _token_side_few(self, x, w, table, tokens, col, z, act):
+    e = table[tokens[:z.shape[0]].long(), col:col + z.shape[1]].float()
+    z.copy_((self.gate_act(x.float() @ w.float().t(), act) * e).to(z.dtype))
+
+
+for _name, _fn in (("row_norm_append", _row_norm_append), ("token_side_apply", _token_side_apply), ("token_side_few", _token_side_few)):
     setattr(ReferenceKernels, _name, _fn)
