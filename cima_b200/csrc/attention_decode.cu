@@ -17,7 +17,8 @@
 // Accepts head_dim in {16, 32, ..., 128}, page_size 64, any group size (16 heads per m-tile), any
 // window; other sizes are refused with a sentence and the caller takes the plain kernel.  With `keep_first` f > 0 the
 // first f positions stay visible below the window: their pages head the list of pages that the splits share.
-// `v_group` neighbouring key heads share one value head (value head = key head / v_group).
+// `v_group` neighbouring key heads share one value head (value head = key head / v_group).  With `slopes`, one number a head,
+// slopes[h] * (distance back to the key) is taken off the scaled score.
 #include "common.cuh"
 
 namespace {
@@ -86,7 +87,7 @@ k_attention_decode(const __nv_bfloat16* __restrict__ qkv, int ld, const __nv_bfl
                    CimaPaged pg, const int* __restrict__ seq_slot, const int* __restrict__ seq_len,
                    float* __restrict__ part_o, float* __restrict__ part_ml, __nv_bfloat16* __restrict__ out, int ldo,
                    int nh, int nkv, int mtiles, float scale, int window, int n_splits, int early, float sink, int keep_first, int v_group,
-                   const float* __restrict__ head_sink, int gate_col) {
+                   const float* __restrict__ head_sink, int gate_col, const float* __restrict__ slopes) {
   if (!early) cima_pdl_wait();
   constexpr int ROW = HD + 8;                         // padded row of a tile, in elements (16 bytes of padding)
   constexpr int TILE = PS * ROW;                      // elements of one K or V tile
@@ -179,6 +180,11 @@ k_attention_decode(const __nv_bfloat16* __restrict__ qkv, int ld, const __nv_bfl
 #pragma unroll
     for (int e = 0; e < 4; e++) o[j][e] = 0.f;
   float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};
+  float sl2[2] = {0.f, 0.f};                          // the two rows' slopes (0 without: the bias is then 0)
+  if (slopes) {
+    if (g < rows) sl2[0] = slopes[h0 + g] * 1.4426950408889634f;
+    if (g + 8 < rows) sl2[1] = slopes[h0 + g + 8] * 1.4426950408889634f;
+  }
 
   for (int p = p0; p < p1; p++) {
     const int stage = (p - p0) % STAGES;
@@ -208,7 +214,7 @@ k_attention_decode(const __nv_bfloat16* __restrict__ qkv, int ld, const __nv_bfl
 #pragma unroll
       for (int e = 0; e < 4; e++) {
         const int key = key0 + j * 8 + 2 * t + (e & 1);
-        const float v = ((key >= lo || key < keep_first) && key < len) ? s[j][e] * sc2 : -INFINITY;
+        const float v = ((key >= lo || key < keep_first) && key < len) ? fmaf(sl2[e >> 1], (float)(key - len + 1), s[j][e] * sc2) : -INFINITY;
         s[j][e] = v;
         mx[e >> 1] = fmaxf(mx[e >> 1], v);
       }
@@ -361,7 +367,7 @@ k_attention_combine(const float* __restrict__ part_o, const float* __restrict__ 
 template <int HD, int PLANES>
 int launch_decode(const void* qkv, int ld, const void* cache, CimaPaged pg, const int* seq_slot, const int* seq_len,
                   float* part_o, float* part_ml, void* out, int ldo, int B, int nh, int nkv, float scale, int window,
-                  int n_splits, int early, float sink, int keep_first, int v_group, const float* head_sink, int gate_col, cudaStream_t stream) {
+                  int n_splits, int early, float sink, int keep_first, int v_group, const float* head_sink, int gate_col, const float* slopes, cudaStream_t stream) {
   auto kern = k_attention_decode<HD, PLANES>;
   constexpr int STAGES = decode_stages(HD, PLANES);
   const size_t tiles = (size_t)STAGES * PLANES * PS * (HD + 8) * sizeof(__nv_bfloat16);
@@ -377,7 +383,7 @@ int launch_decode(const void* qkv, int ld, const void* cache, CimaPaged pg, cons
   dim3 grid(n_splits, nkv * mtiles, B);
   { int rc_ = cima_launch(kern, dim3(grid), dim3(WARPS * 32), (size_t)(smem), stream, 1, (const __nv_bfloat16*)qkv, ld, (const __nv_bfloat16*)cache, pg, seq_slot,
                                            seq_len, part_o, part_ml, (__nv_bfloat16*)out, ldo, nh, nkv, mtiles, scale,
-                                           window, n_splits, early, sink, keep_first, v_group, head_sink, gate_col); if (rc_) return rc_; }
+                                           window, n_splits, early, sink, keep_first, v_group, head_sink, gate_col, slopes); if (rc_) return rc_; }
   int rc = cima_launch_result();
   if (rc || n_splits == 1) return rc;
   { int rc_ = cima_launch(k_attention_combine, dim3(dim3(nh, B)), dim3(128), (size_t)(0), stream, 1, part_o, part_ml, seq_len, (__nv_bfloat16*)out, ldo, nh, HD, window, n_splits, sink, keep_first, head_sink, (const __nv_bfloat16*)qkv, ld, gate_col); if (rc_) return rc_; }
@@ -396,7 +402,7 @@ extern "C" int cima_attention_decode(const void* qkv, int ld, const void* cache,
                                      int ring, int page_size, const int* seq_slot, const int* seq_len, float* part_o,
                                      float* part_ml, void* out, int ldo, int B, int nh, int nkv, int hd, float scale,
                                      int window, int n_splits, int early, int planes, float sink, int keep_first, int v_group,
-                                     const float* head_sink, int gate_col, cudaStream_t stream) {
+                                     const float* head_sink, int gate_col, const float* slopes, cudaStream_t stream) {
   if (B <= 0) return 0;
   if (planes != 1 && planes != 2) return cima_fail(CIMA_E_ARG, "attention_decode: %d planes; pages hold keys | values (2) or one shared vector (1)", planes);
   if (page_size != PS) return cima_fail(CIMA_E_SIZE, "attention_decode: page size %d; this kernel takes 64", page_size);
@@ -408,8 +414,8 @@ extern "C" int cima_attention_decode(const void* qkv, int ld, const void* cache,
   if (ld % 2 || ((uintptr_t)qkv & 3) || ((uintptr_t)cache & 15)) return cima_fail(CIMA_E_ARG, "attention_decode: qkv rows must be 4-byte and the cache 16-byte aligned");
   if (gate_col < 0 || (gate_col > 0 && gate_col + nh * hd > ld)) return cima_fail(CIMA_E_ARG, "attention_decode: %d gate values from column %d on exceed the rows of %d", nh * hd, gate_col, ld);
   CimaPaged pg{table, table_width, ring, page_size, nkv, hd, planes};
-#define CASE(H) case H: return planes == 2 ? launch_decode<H, 2>(qkv, ld, cache, pg, seq_slot, seq_len, part_o, part_ml, out, ldo, B, nh, nkv, scale, window, n_splits, early != 0, sink, keep_first, v_group, head_sink, gate_col, stream) \
-                                          : launch_decode<H, 1>(qkv, ld, cache, pg, seq_slot, seq_len, part_o, part_ml, out, ldo, B, nh, nkv, scale, window, n_splits, early != 0, sink, keep_first, v_group, head_sink, gate_col, stream)
+#define CASE(H) case H: return planes == 2 ? launch_decode<H, 2>(qkv, ld, cache, pg, seq_slot, seq_len, part_o, part_ml, out, ldo, B, nh, nkv, scale, window, n_splits, early != 0, sink, keep_first, v_group, head_sink, gate_col, slopes, stream) \
+                                          : launch_decode<H, 1>(qkv, ld, cache, pg, seq_slot, seq_len, part_o, part_ml, out, ldo, B, nh, nkv, scale, window, n_splits, early != 0, sink, keep_first, v_group, head_sink, gate_col, slopes, stream)
   switch (hd) {
     CASE(16); CASE(32); CASE(48); CASE(64); CASE(80); CASE(96); CASE(112); CASE(128);
   }
@@ -464,5 +470,5 @@ extern "C" int cima_attention_decode_static(const void* qkv, int ld, const void*
   float* part_o = scratch;                       // [B, nh, n_splits, hd]
   float* part_ml = scratch + cells * hd;         // [B, nh, n_splits, 2]
   return cima_attention_decode(qkv, ld, cache, table, table_width, ring, page_size, seq_slot, seq_len, part_o, part_ml,
-                               out, ldo, B, nh, nkv, hd, scale, window, n_splits, 0, 2, 0.f, 0, 1, nullptr, 0, stream);
+                               out, ldo, B, nh, nkv, hd, scale, window, n_splits, 0, 2, 0.f, 0, 1, nullptr, 0, nullptr, stream);
 }

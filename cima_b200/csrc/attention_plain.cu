@@ -12,6 +12,7 @@
 // A head's softmax may hold one more entry without a value: `sink` entries of score 0, or exp(head_sink[h]).
 // `gate_col` > 0: the row's own buffer holds a gate value for every value of the result from that column on (heads of hd
 // values like the queries'); the result leaves times the gate's sigmoid.
+// `slopes` (or null), one number a head: slopes[h] * (p - j) is taken off the scaled score of key j for a query at position p.
 // A row's result depends only on its own sequence: same bits alone or in any batch.
 #include "common.cuh"
 
@@ -21,7 +22,7 @@ k_attention_plain(const TA* __restrict__ qkv, int ld, const TA* __restrict__ cac
                   const int* __restrict__ row_pos, const int* __restrict__ row_seq,
                   const int* __restrict__ seq_slot, const int* __restrict__ seq_first_row,
                   TA* __restrict__ out, int ldo, int T, int nh, int nkv, int hd, float scale, int window, float sink, int keep_first, int v_group,
-                  const float* __restrict__ head_sink, int gate_col) {
+                  const float* __restrict__ head_sink, int gate_col, const float* __restrict__ slopes) {
   cima_pdl_wait();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int row = blockIdx.x * (blockDim.x >> 5) + warp;
@@ -43,6 +44,7 @@ k_attention_plain(const TA* __restrict__ qkv, int ld, const TA* __restrict__ cac
     q[i] = d < hd ? cima_to_f32<TA>(qp[d]) : 0.f;
     acc[i] = 0.f;
   }
+  const float slope = slopes ? slopes[h] : 0.f;
   float m = -1e30f, l = 0.f;
   const int lo = (window > 0 && pos + 1 > window) ? pos + 1 - window : 0;
   const int kept = min(keep_first, lo);         // the first positions that stay visible below the window
@@ -64,7 +66,7 @@ k_attention_plain(const TA* __restrict__ qkv, int ld, const TA* __restrict__ cac
     }
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) s += __shfl_xor_sync(0xffffffffu, s, o);
-    s *= scale;
+    s = s * scale - slope * (float)(pos - j);
     const float m2 = fmaxf(m, s);
     const float corr = expf(m - m2), p = expf(s - m2);
 #pragma unroll
@@ -96,7 +98,7 @@ extern "C" int cima_attention_plain(const void* qkv, int dtype, int ld, const vo
                                     const int* row_seq, const int* seq_slot, const int* seq_first_row, void* out,
                                     int ldo, int T, int nh, int nkv, int hd, float scale, int window,
                                     int from_cache, int planes, float sink, int keep_first, int v_group, const float* head_sink,
-                                    int gate_col, cudaStream_t stream) {
+                                    int gate_col, const float* slopes, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (hd <= 0 || hd > 1024) return cima_fail(CIMA_E_SIZE, "attention_plain: head_dim %d is outside 1..1024", hd);
   if (planes != 1 && planes != 2) return cima_fail(CIMA_E_ARG, "attention_plain: %d planes; pages hold keys | values (2) or one shared vector (1)", planes);
@@ -109,7 +111,7 @@ extern "C" int cima_attention_plain(const void* qkv, int dtype, int ld, const vo
   dim3 grid((T + 3) / 4, nh);
 #define LAUNCH(TA, FC) { int rc_ = hd <= 256 ? LAUNCH_NI(TA, FC, 8) : LAUNCH_NI(TA, FC, 32); if (rc_) return rc_; }
 #define LAUNCH_NI(TA, FC, NI) cima_launch(k_attention_plain<TA, FC, NI>, dim3(grid), dim3(128), (size_t)(0), stream, 1, (const TA*)qkv, ld, (const TA*)cache, pg, \
-    row_pos, row_seq, seq_slot, seq_first_row, (TA*)out, ldo, T, nh, nkv, hd, scale, window, sink, keep_first, v_group, head_sink, gate_col)
+    row_pos, row_seq, seq_slot, seq_first_row, (TA*)out, ldo, T, nh, nkv, hd, scale, window, sink, keep_first, v_group, head_sink, gate_col, slopes)
   if (dtype == CIMA_F32) { if (from_cache) LAUNCH(float, true) else LAUNCH(float, false) }
   else if (dtype == CIMA_BF16) { if (from_cache) LAUNCH(__nv_bfloat16, true) else LAUNCH(__nv_bfloat16, false) }
   else return cima_fail(CIMA_E_DTYPE, "attention_plain: dtype code %d is neither float32 nor bfloat16", dtype);

@@ -12,7 +12,8 @@
 // the bfloat16 rounding of P);
 // P is rounded to bfloat16 only as the operand of P V.  Key tiles wholly above the
 // diagonal or wholly below the window are skipped.  With `keep_first` f > 0 the first f positions stay visible below
-// the window: their tiles are visited first.  `v_group` neighbouring key heads share one value head.  The list of (sequence, first row) of the blocks
+// the window: their tiles are visited first.  With `slopes`, one number a head, slopes[h] * (distance from the query back to the
+// key) is taken off the scaled score.  `v_group` neighbouring key heads share one value head.  The list of (sequence, first row) of the blocks
 // comes from the host, heaviest first.
 //
 // Counterpart in the reference: k_attn_prefill_tiled (src/kernels.cu:659-753), one warp per query
@@ -66,7 +67,7 @@ k_attention_prefill(const __nv_bfloat16* __restrict__ qkv, int ld, const int* __
                     const __nv_bfloat16* __restrict__ cache, CimaPaged pg, const int* __restrict__ seq_slot,
                     const int* __restrict__ seq_len,
                     __nv_bfloat16* __restrict__ out, int ldo, int T, int nh, int nkv, float scale, int window, float sink, int keep_first, int v_group,
-                    const float* __restrict__ head_sink, int gate_col) {
+                    const float* __restrict__ head_sink, int gate_col, const float* __restrict__ slopes) {
   cima_pdl_wait();
   constexpr int ROW = HD + 8;
   constexpr int TILE = BN * ROW;
@@ -88,7 +89,9 @@ k_attention_prefill(const __nv_bfloat16* __restrict__ qkv, int ld, const int* __
   const int g = lane >> 2, t = lane & 3;
   const int vh = kvh / v_group;
   const int kcol = (nh + kvh) * HD, vcol = (nh + nkv + vh) * HD;
-  const float sc2 = scale * 1.4426950408889634f;       // scores are kept in the base-2 domain
+  const float sc_in = scale * 1.4426950408889634f;     // scores are kept in the base-2 domain
+  const float sl2 = slopes ? slopes[h] * 1.4426950408889634f : 0.f;
+  const float sc2 = slopes ? 1.0f : sc_in;             // with a distance bias the scores are scaled where it is added
 
   // this thread's two query rows (among the sequence's rows; their positions are start + row)
   const int r0 = q0 + warp * 16 + g, r1 = r0 + 8;
@@ -194,6 +197,13 @@ k_attention_prefill(const __nv_bfloat16* __restrict__ qkv, int ld, const int* __
     const int wr0 = start + q0 + warp * 16;            // this warp's first query position
     const bool masked = key_base + BN - 1 > wr0 || (window > 0 && wr0 + 15 - key_base >= window);
     float mx[2] = {-INFINITY, -INFINITY};
+    if (slopes) {
+      const float d0 = (float)(key_base + 2 * t - (start + r0)), d1 = d0 - 8.0f;        // minus the distance, of the lane's first key
+#pragma unroll
+      for (int j = 0; j < 8; j++)
+#pragma unroll
+        for (int e = 0; e < 4; e++) s[j][e] = fmaf(sl2, ((e >> 1) ? d1 : d0) + (float)(j * 8 + (e & 1)), s[j][e] * sc_in);
+    }
     if (masked) {
 #pragma unroll
       for (int j = 0; j < 8; j++)
@@ -299,7 +309,7 @@ template <int HD, bool FROM_CACHE>
 int launch_prefill(const void* qkv, int ld, const int* tile_seq, const int* tile_row0, const int* seq_first_row,
                    const void* cache, const CimaPaged& pg, const int* seq_slot, const int* seq_len,
                    void* out, int ldo, int T, int n_tiles, int nh, int nkv, float scale, int window, float sink, int keep_first, int v_group,
-                   const float* head_sink, int gate_col, cudaStream_t stream) {
+                   const float* head_sink, int gate_col, const float* slopes, cudaStream_t stream) {
   if ((long long)n_tiles * nh > 0x7fffffffll) return cima_fail(CIMA_E_SIZE, "attention_prefill: %d blocks of rows x %d heads exceed one launch", n_tiles, nh);
   auto kern = k_attention_prefill<HD, FROM_CACHE>;
   const size_t smem = (size_t)2 * 2 * BN * (HD + 8) * sizeof(__nv_bfloat16);
@@ -311,7 +321,7 @@ int launch_prefill(const void* qkv, int ld, const int* tile_seq, const int* tile
   }
   { int rc_ = cima_launch(kern, dim3((unsigned)n_tiles * (unsigned)nh), dim3(WARPS * 32), (size_t)(smem), stream, 1, (const __nv_bfloat16*)qkv, ld, tile_seq, tile_row0, seq_first_row,
                                                         (const __nv_bfloat16*)cache, pg, seq_slot, seq_len,
-                                                        (__nv_bfloat16*)out, ldo, T, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, gate_col); if (rc_) return rc_; }
+                                                        (__nv_bfloat16*)out, ldo, T, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, gate_col, slopes); if (rc_) return rc_; }
   return cima_launch_result();
 }
 
@@ -331,11 +341,11 @@ static int prefill_checks(const char* who, const void* qkv, int ld, const void* 
 extern "C" int cima_attention_prefill(const void* qkv, int ld, const int* tile_seq, const int* tile_row0,
                                       const int* seq_first_row, void* out, int ldo, int T, int n_tiles, int nh, int nkv,
                                       int hd, float scale, int window, float sink, int keep_first, int v_group, const float* head_sink,
-                                      int gate_col, cudaStream_t stream) {
+                                      int gate_col, const float* slopes, cudaStream_t stream) {
   if (T <= 0 || n_tiles <= 0) return 0;
   if (int rc = prefill_checks("attention_prefill", qkv, ld, out, ldo, hd, nh, nkv, keep_first, v_group, gate_col)) return rc;
   const CimaPaged none{nullptr, 0, 0, BN, nkv, hd};
-#define CASE(H) case H: return launch_prefill<H, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, nullptr, none, nullptr, nullptr, out, ldo, T, n_tiles, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, gate_col, stream)
+#define CASE(H) case H: return launch_prefill<H, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, nullptr, none, nullptr, nullptr, out, ldo, T, n_tiles, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, gate_col, slopes, stream)
   switch (hd) {
     CASE(16); CASE(32); CASE(48); CASE(64); CASE(80); CASE(96); CASE(112); CASE(128);
   }
@@ -350,14 +360,14 @@ extern "C" int cima_attention_extend(const void* qkv, int ld, const int* tile_se
                                      int ring, int page_size, const int* seq_slot, const int* seq_len, void* out, int ldo,
                                      int T, int n_tiles, int nh, int nkv, int hd, float scale, int window,
                                      int planes, float sink, int keep_first, int v_group, const float* head_sink, int gate_col,
-                                     cudaStream_t stream) {
+                                     const float* slopes, cudaStream_t stream) {
   if (T <= 0 || n_tiles <= 0) return 0;
   if (planes != 1 && planes != 2) return cima_fail(CIMA_E_ARG, "attention_extend: %d planes; pages hold keys | values (2) or one shared vector (1)", planes);
   if (int rc = prefill_checks("attention_extend", qkv, ld, out, ldo, hd, nh, nkv, keep_first, v_group, gate_col)) return rc;
   if (page_size != BN) return cima_fail(CIMA_E_SIZE, "attention_extend: page size %d; this kernel takes %d", page_size, BN);
   if (!cache || !table || !seq_slot || !seq_len || ((uintptr_t)cache & 15)) return cima_fail(CIMA_E_ARG, "attention_extend: the cache (16-byte aligned), its block table, slots and lengths are needed");
   const CimaPaged pg{table, table_width, ring, page_size, nkv, hd, planes};
-#define CASE(H) case H: return launch_prefill<H, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, cache, pg, seq_slot, seq_len, out, ldo, T, n_tiles, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, gate_col, stream)
+#define CASE(H) case H: return launch_prefill<H, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, cache, pg, seq_slot, seq_len, out, ldo, T, n_tiles, nh, nkv, scale, window, sink, keep_first, v_group, head_sink, gate_col, slopes, stream)
   switch (hd) {
     CASE(16); CASE(32); CASE(48); CASE(64); CASE(80); CASE(96); CASE(112); CASE(128);
   }

@@ -64,6 +64,7 @@ struct AttnArgs {
   const float* head_sink;       // or null: [nh], head h's denominator also holds exp(head_sink[h]) (instead of `sink`)
   const __nv_bfloat16* gate;    // or null: the rows' own gates, gate[row * ld_gate + h * HD + d]; the result leaves times their sigmoid
   int ld_gate;
+  const float* slopes;          // or null: [nh], slopes[h] * (distance from the query back to the key) is taken off the scaled score
 };
 
 // Keys of a query block whose rows stand at positions p0 .. (at most p0 + 127, below len): tiles [first, last] of 64.
@@ -220,7 +221,9 @@ k_attention_prefill_tc(const __grid_constant__ CUtensorMap map_qkv, const __grid
     const int r = warp * 32 + lane;                     // row of the block = TMEM lane
     const int pos = q0 + r;                             // its position in the sequence
     const unsigned lane_off = (unsigned)(warp * 32) << 16;
-    const float sc2 = a.scale * 1.4426950408889634f;
+    const float sc_in = a.scale * 1.4426950408889634f;
+    const float sl2 = a.slopes ? a.slopes[h] * 1.4426950408889634f : 0.f;
+    const float sc2 = a.slopes ? 1.0f : sc_in;          // with a distance bias the scores are scaled where it is added
     float m_run = -INFINITY, l_run = 0.f;
     bool ok = true;
     for (int j = 0; j < n && ok; j++) {
@@ -238,6 +241,14 @@ k_attention_prefill_tc(const __grid_constant__ CUtensorMap map_qkv, const __grid
 #pragma unroll
       for (int c = 0; c < NC; c++) tmem_ld32_issue(tm_s[s] + lane_off + (unsigned)(c * 32), raw[c]);
       tmem_ld_wait();
+      if (a.slopes) {                                   // s * scale + slope * (key - position), in the base-2 domain
+        const float far = sl2 * (float)(k0 - pos);
+#pragma unroll
+        for (int c = 0; c < NC; c++)
+#pragma unroll
+          for (int e = 0; e < 32; e++)
+            raw[c][e] = __float_as_uint(fmaf(__uint_as_float(raw[c][e]), sc_in, fmaf(sl2, (float)(c * 32 + e), far)));
+      }
       // maxima of the raw scores (the scale is positive): four chains instead of one
       float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
       if (masked) {
@@ -371,7 +382,7 @@ struct CacheSource {              // keys and values from a layer's pages; cache
 template <int HD, bool FROM_CACHE>
 int launch_attention_tc(const void* qkv, int ld, const int* tile_seq, const int* tile_row0, const int* seq_first_row,
                         const CacheSource& c, void* out, int ldo, int T, int n_tiles, int nh, int nkv, float scale,
-                        int window, int* error_flag, float sink, const float* head_sink, int gate_col, cudaStream_t stream) {
+                        int window, int* error_flag, float sink, const float* head_sink, int gate_col, const float* slopes, cudaStream_t stream) {
   if ((long long)n_tiles * nh > 0x7fffffffll) return cima_fail(CIMA_E_SIZE, "attention_prefill_tc: %d blocks of rows x %d heads exceed one launch", n_tiles, nh);
   CUtensorMap mq, mk;                                  // boxes of 128 rows (Q) and of 64 rows (K and V) by 64 columns
   // (with the keys in the cache only the queries' columns of a row are read, and the row may end there)
@@ -390,7 +401,7 @@ int launch_attention_tc(const void* qkv, int ld, const int* tile_seq, const int*
     raised = true;
   }
   AttnArgs a{tile_seq, tile_row0, seq_first_row, c.seq_len, c.seq_slot, c.table, c.table_width, c.ring,
-             (__nv_bfloat16*)out, ldo, nh, nkv, window, scale, error_flag, c.planes, sink, head_sink, gate_col > 0 ? (const __nv_bfloat16*)qkv + gate_col : nullptr, ld};
+             (__nv_bfloat16*)out, ldo, nh, nkv, window, scale, error_flag, c.planes, sink, head_sink, gate_col > 0 ? (const __nv_bfloat16*)qkv + gate_col : nullptr, ld, slopes};
   { int rc_ = cima_launch(k_attention_prefill_tc<HD, FROM_CACHE>, dim3((unsigned)n_tiles * (unsigned)nh), dim3(THREADS), smem, stream, 1, mq, mk, a); if (rc_) return rc_; }
   return cima_launch_result();
 }
@@ -416,13 +427,13 @@ static int tc_checks(const char* who, const void* qkv, int ld, const void* out, 
 extern "C" int cima_attention_prefill_tc(const void* qkv, int ld, const int* tile_seq, const int* tile_row0,
                                          const int* seq_first_row, void* out, int ldo, int T, int n_tiles, int nh,
                                          int nkv, int hd, float scale, int window, int* error_flag, float sink, const float* head_sink,
-                                         int gate_col, cudaStream_t stream) {
+                                         int gate_col, const float* slopes, cudaStream_t stream) {
   if (T <= 0 || n_tiles <= 0) return 0;
   if (int rc = tc_checks("attention_prefill_tc", qkv, ld, out, ldo, nh, nkv, hd, error_flag, gate_col)) return rc;
   const CacheSource none{nullptr, 0, nullptr, nullptr, nullptr, 0, 0};
   if (hd == 64)
-    return launch_attention_tc<64, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, none, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, stream);
-  return launch_attention_tc<128, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, none, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, stream);
+    return launch_attention_tc<64, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, none, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, slopes, stream);
+  return launch_attention_tc<128, false>(qkv, ld, tile_seq, tile_row0, seq_first_row, none, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, slopes, stream);
 }
 
 // The same for sequences that go on: the rows of sequence s are the positions seq_len[s] - rows .. seq_len[s] - 1, and
@@ -432,7 +443,7 @@ extern "C" int cima_attention_extend_tc(const void* qkv, int ld, const int* tile
                                         int table_width, int ring, int page_size, const int* seq_slot, const int* seq_len,
                                         void* out, int ldo, int T, int n_tiles, int nh, int nkv, int hd, float scale,
                                         int window, int* error_flag, int planes, float sink, const float* head_sink,
-                                        int gate_col, cudaStream_t stream) {
+                                        int gate_col, const float* slopes, cudaStream_t stream) {
   if (T <= 0 || n_tiles <= 0) return 0;
   if (planes != 1 && planes != 2) return cima_fail(CIMA_E_ARG, "attention_extend_tc: %d planes; pages hold keys | values (2) or one shared vector (1)", planes);
   if (int rc = tc_checks("attention_extend_tc", qkv, ld, out, ldo, nh, nkv, hd, error_flag, gate_col, true)) return rc;
@@ -442,6 +453,6 @@ extern "C" int cima_attention_extend_tc(const void* qkv, int ld, const int* tile
   if (n_pages * planes * nkv * BN >= (1ll << 31)) return cima_fail(CIMA_E_SIZE, "attention_extend_tc: %lld pages exceed a tensor map's 32-bit row coordinate", n_pages);
   const CacheSource c{cache, n_pages, table, seq_slot, seq_len, table_width, ring, planes};
   if (hd == 64)
-    return launch_attention_tc<64, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, c, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, stream);
-  return launch_attention_tc<128, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, c, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, stream);
+    return launch_attention_tc<64, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, c, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, slopes, stream);
+  return launch_attention_tc<128, true>(qkv, ld, tile_seq, tile_row0, seq_first_row, c, out, ldo, T, n_tiles, nh, nkv, scale, window, error_flag, sink, head_sink, gate_col, slopes, stream);
 }

@@ -65,6 +65,17 @@ __device__ __forceinline__ float cima_gated(float g, float u, int act, float lim
   return cima_gate_act(g, act) * u;
 }
 
+// An ungated feed-forward's middle: the activations above, or the square of ReLU.
+enum { CIMA_UNGATED_RELU2 = 5 };
+static inline bool cima_ungated_known(int act) { return (act >= 0 && act < CIMA_ACT_COUNT) || act == CIMA_UNGATED_RELU2; }
+__device__ __forceinline__ float cima_ungated_act(float z, int act) {
+  if (act == CIMA_UNGATED_RELU2) {
+    const float r = fmaxf(z, 0.f);
+    return r * r;
+  }
+  return cima_gate_act(z, act);
+}
+
 __device__ __forceinline__ float cima_sigmoid(float z) { return 1.0f / (1.0f + expf(-z)); }
 
 // The same with the fast exponential and division (a few ulp), for results that leave in bfloat16.

@@ -11,7 +11,7 @@
 template <typename TW>
 __global__ void k_embed(const int* __restrict__ ids, const TW* __restrict__ table, float* __restrict__ x,
                         int H, int V, float scale, float* __restrict__ ssq, const float* __restrict__ w_next,
-                        __nv_bfloat16* __restrict__ xw) {
+                        __nv_bfloat16* __restrict__ xw, const TW* __restrict__ ptable, const int* __restrict__ row_pos, int n_pos) {
   cima_pdl_wait();
   __shared__ float red[32];
   const int row = blockIdx.x;
@@ -19,9 +19,15 @@ __global__ void k_embed(const int* __restrict__ ids, const TW* __restrict__ tabl
   id = id < 0 ? 0 : (id >= V ? V - 1 : id);    // ids are checked on the host; never read outside the table
   const TW* src = table + (size_t)id * H;
   float* dst = x + (size_t)row * H;
+  const TW* pv = nullptr;                      // the position's own vector, where the model has such a table
+  if (ptable) {
+    const int p = row_pos[row];
+    pv = ptable + (size_t)(p < 0 ? 0 : (p >= n_pos ? n_pos - 1 : p)) * H;      // (rows that pad a recorded prompt may stand beyond the table)
+  }
   float acc = 0.f;
   for (int i = threadIdx.x; i < H; i += blockDim.x) {
-    const float v = cima_to_f32<TW>(src[i]) * scale;
+    float v = cima_to_f32<TW>(src[i]) * scale;
+    if (pv) v += cima_to_f32<TW>(pv[i]);
     dst[i] = v;
     if (xw) xw[(size_t)row * H + i] = __float2bfloat16_rn(v * w_next[i]);      // for a norm folded into the next product
     acc += v * v;
@@ -33,13 +39,16 @@ __global__ void k_embed(const int* __restrict__ ids, const TW* __restrict__ tabl
 }
 
 // ssq (may be null): [T] sum of squares of each row written.  w_next / xw (may be null): weight [H] of the norm
-// that follows and where to put bf16(row * weight), [T, H].
+// that follows and where to put bf16(row * weight), [T, H].  ptable (may be null): [n_pos, H] in the table's dtype, row p of
+// which is added (unscaled) to a row at position p.
 extern "C" int cima_embed(const int* ids, const void* table, int table_dtype, float* x, int T, int H, int V,
-                          float scale, float* ssq, const float* w_next, void* xw, cudaStream_t stream) {
+                          float scale, float* ssq, const float* w_next, void* xw, const void* ptable, const int* row_pos,
+                          int n_pos, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (H <= 0 || V <= 0) return cima_fail(CIMA_E_SIZE, "embed: hidden %d and vocab %d must be positive", H, V);
-  if (table_dtype == CIMA_F32) { int rc_ = cima_launch(k_embed<float>, dim3(T), dim3(256), (size_t)(0), stream, 1, ids, (const float*)table, x, H, V, scale, ssq, w_next, (__nv_bfloat16*)xw); if (rc_) return rc_; }
-  else if (table_dtype == CIMA_BF16) { int rc_ = cima_launch(k_embed<__nv_bfloat16>, dim3(T), dim3(256), (size_t)(0), stream, 1, ids, (const __nv_bfloat16*)table, x, H, V, scale, ssq, w_next, (__nv_bfloat16*)xw); if (rc_) return rc_; }
+  if (ptable && (!row_pos || n_pos <= 0)) return cima_fail(CIMA_E_ARG, "embed: the table of %d positions needs the rows' positions", n_pos);
+  if (table_dtype == CIMA_F32) { int rc_ = cima_launch(k_embed<float>, dim3(T), dim3(256), (size_t)(0), stream, 1, ids, (const float*)table, x, H, V, scale, ssq, w_next, (__nv_bfloat16*)xw, (const float*)ptable, row_pos, n_pos); if (rc_) return rc_; }
+  else if (table_dtype == CIMA_BF16) { int rc_ = cima_launch(k_embed<__nv_bfloat16>, dim3(T), dim3(256), (size_t)(0), stream, 1, ids, (const __nv_bfloat16*)table, x, H, V, scale, ssq, w_next, (__nv_bfloat16*)xw, (const __nv_bfloat16*)ptable, row_pos, n_pos); if (rc_) return rc_; }
   else return cima_fail(CIMA_E_DTYPE, "embed: table dtype code %d is neither float32 nor bfloat16", table_dtype);
   return cima_launch_result();
 }

@@ -35,7 +35,7 @@ constexpr int BK = 64;           // k per stage: 64 bf16 = 128 bytes = one swizz
 constexpr int UMMA_K = 16;
 constexpr int THREADS = 192;
 
-enum { EPI_STORE = 0, EPI_ACCUM = 1, EPI_SWIGLU = 2, EPI_STORE_F32 = 3 };
+enum { EPI_STORE = 0, EPI_ACCUM = 1, EPI_SWIGLU = 2, EPI_STORE_F32 = 3, EPI_ACT = 4 };      // EPI_ACT: an ungated activation, bfloat16 store
 
 __device__ __forceinline__ unsigned cluster_addr(const void* p, unsigned rank) {      // address of p in block `rank`
   unsigned a = smem_u32(p), r;
@@ -213,6 +213,15 @@ k_gemm_tcgen05_pair(const __grid_constant__ CUtensorMap map_p, const __grid_cons
             for (int e = 0; e < 32; e++) v[e] = cima_gated(v[e], u[e], a.act, a.act_limit);
           }
         }
+        if (EPI == EPI_ACT) {
+          if (a.act == CIMA_UNGATED_RELU2) {
+#pragma unroll
+            for (int e = 0; e < 32; e++) { const float r = fmaxf(v[e], 0.f); v[e] = r * r; }
+          } else {
+#pragma unroll
+            for (int e = 0; e < 32; e++) v[e] = cima_ungated_act(v[e], a.act);
+          }
+        }
         if (i >= p_first && i < a.p_rows) {
           const int jmax = GATED ? a.up_offset : a.q_rows;
           const int j0 = q0 + c0;
@@ -334,17 +343,17 @@ extern "C" int cima_gemm_tcgen05_pair(const void* P, const void* Q, const float*
 
 // The grouped product: Q = [E][q_rows, K], P [p_rows, K] with p_rows a multiple of 256, tile_expert [p_rows / 256] names
 // the matrix of every row tile (-1: the tile has no rows).  Epilogues 2 (gated: a matrix of Q is [gate | up],
-// q_rows = 2 * up_offset) and 3 (float32 store); out [p_rows, ldo].
+// q_rows = 2 * up_offset), 3 (float32 store) and 4 (an ungated activation, bfloat16 store); out [p_rows, ldo].
 extern "C" int cima_gemm_tcgen05_pair_grouped(const void* P, const void* Q, void* out, int epi, int p_rows, int q_rows, int E,
                                               int K, int ldo, int up_offset, int act, float act_limit, const int* tile_expert,
                                               int* error_flag, cudaStream_t stream) {
   if (p_rows <= 0 || q_rows <= 0 || E <= 0) return 0;
-  if (act < 0 || act >= CIMA_GATED_COUNT) return cima_fail(CIMA_E_ARG, "gemm_tcgen05_pair_grouped: activation code %d is not one of 0..%d", act, CIMA_GATED_COUNT - 1);
+  if (epi == EPI_ACT ? !cima_ungated_known(act) : (act < 0 || act >= CIMA_GATED_COUNT)) return cima_fail(CIMA_E_ARG, "gemm_tcgen05_pair_grouped: activation code %d is unknown to epilogue %d", act, epi);
   if (K <= 0 || K % 8) return cima_fail(CIMA_E_SIZE, "gemm_tcgen05_pair_grouped: K %d must be a positive multiple of 8", K);
   if (p_rows % (2 * BM)) return cima_fail(CIMA_E_SIZE, "gemm_tcgen05_pair_grouped: %d rows are not whole tiles of %d", p_rows, 2 * BM);
   if (((uintptr_t)P | (uintptr_t)Q) & 15) return cima_fail(CIMA_E_ARG, "gemm_tcgen05_pair_grouped: P and Q must be 16-byte aligned");
   if (!error_flag || !tile_expert) return cima_fail(CIMA_E_ARG, "gemm_tcgen05_pair_grouped: the tiles' experts and an error flag on the device are needed");
-  if (epi != EPI_SWIGLU && epi != EPI_STORE_F32) return cima_fail(CIMA_E_ARG, "gemm_tcgen05_pair_grouped: epilogue %d is neither 2 (gated) nor 3 (float32)", epi);
+  if (epi != EPI_SWIGLU && epi != EPI_STORE_F32 && epi != EPI_ACT) return cima_fail(CIMA_E_ARG, "gemm_tcgen05_pair_grouped: epilogue %d is none of 2 (gated), 3 (float32), 4 (activation)", epi);
   if (epi == EPI_SWIGLU && (up_offset <= 0 || q_rows != 2 * up_offset)) return cima_fail(CIMA_E_SIZE, "gemm_tcgen05_pair_grouped: the gated epilogue needs q_rows = 2 * up_offset");
   if ((long long)E * q_rows >= (1ll << 31)) return cima_fail(CIMA_E_SIZE, "gemm_tcgen05_pair_grouped: %d matrices of %d rows exceed a tensor map's coordinate", E, q_rows);
   constexpr int BN = 256;
@@ -359,5 +368,6 @@ extern "C" int cima_gemm_tcgen05_pair_grouped(const void* P, const void* Q, void
   if (rc) return rc;
   PairArgs a{p_rows, q_rows, K, up_offset, nullptr, out, ldo, error_flag, act, tile_expert, q_rows, act_limit};
   if (epi == EPI_SWIGLU) return launch<BN, 6, EPI_SWIGLU>(mp, mq, a, p_tiles, tiles_q, stream);
+  if (epi == EPI_ACT) return launch<BN, 6, EPI_ACT>(mp, mq, a, p_tiles, tiles_q, stream);
   return launch<BN, 6, EPI_STORE_F32>(mp, mq, a, p_tiles, tiles_q, stream);
 }

@@ -210,16 +210,11 @@ static int launch_hyper4(float* X, const float* y, const float* C, const float* 
   }
 }
 
-__device__ __forceinline__ float ungated_act(float z, int act) {
-  if (act == 5) { const float r = fmaxf(z, 0.f); return r * r; }
-  return cima_gate_act(z, act);
-}
-
 template <typename TA>
 __global__ void k_activate(TA* __restrict__ z, size_t total, int act) {
   cima_pdl_wait();
   for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x)
-    z[i] = cima_from_f32<TA>(ungated_act(cima_to_f32<TA>(z[i]), act));
+    z[i] = cima_from_f32<TA>(cima_ungated_act(cima_to_f32<TA>(z[i]), act));
 }
 
 __global__ void k_activate_bf16x8(__nv_bfloat16* __restrict__ z, size_t groups, int act) {
@@ -230,7 +225,7 @@ __global__ void k_activate_bf16x8(__nv_bfloat16* __restrict__ z, size_t groups, 
 #pragma unroll
     for (int e = 0; e < 4; e++) {
       const float2 f = __bfloat1622float2(p[e]);
-      p[e] = __floats2bfloat162_rn(ungated_act(f.x, act), ungated_act(f.y, act));
+      p[e] = __floats2bfloat162_rn(cima_ungated_act(f.x, act), cima_ungated_act(f.y, act));
     }
     *reinterpret_cast<uint4*>(z + i * 8) = v;
   }
@@ -264,7 +259,7 @@ extern "C" int cima_hyper_connect(float* X, const float* y, const float* C, cons
 
 extern "C" int cima_activate(void* z, int dtype, size_t total, int act, cudaStream_t stream) {
   if (total == 0) return 0;
-  if (!((act >= 0 && act < CIMA_ACT_COUNT) || act == 5)) return cima_fail(CIMA_E_ARG, "activate: activation code %d is unknown", act);
+  if (!cima_ungated_known(act)) return cima_fail(CIMA_E_ARG, "activate: activation code %d is unknown", act);
   int rc;
   if (dtype == CIMA_BF16 && total % 8 == 0 && ((uintptr_t)z & 15) == 0) {
     const size_t groups = total / 8;

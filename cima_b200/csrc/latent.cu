@@ -8,6 +8,7 @@
 // head_linear: the same small matrix product for every head,
 //   out[t, h, n] = sum_k a[t, h, k] * w[h, n, k]        a: [T, heads, K] in rows of lda; out: [T, heads, N] in rows of ldo
 // (a head of a row may be wider than K or N: `ha` and `ho` values lie between one head's start and the next in a and out)
+// with a gate row beside a's (`gate`, null: none), the output leaves times sigmoid(gate[t, h * N + n]);
 // which moves a query into the latents' space (w = the key projection's head, transposed) and an attention
 // result out of it (w = the value projection's head).  FFMA with one float32 accumulator per output in ascending
 // k: the same bits for a row whatever comes with it.  It serves the 32-bit path at every size and the
@@ -53,7 +54,7 @@ extern "C" int cima_latent_append(const void* raw, int dtype, int ld, const floa
 template <typename TA>
 __global__ void __launch_bounds__(256)
 k_head_linear(const TA* __restrict__ A, const TA* __restrict__ W, TA* __restrict__ out, int M, int N, int K, int lda, int ldo,
-              int ha, int ho) {
+              int ha, int ho, const TA* __restrict__ gate, int ldg) {
   cima_pdl_wait();
   constexpr int BM = 64, BN = 64, BK = 16;
   __shared__ float As[BK][BM + 4];
@@ -105,7 +106,10 @@ k_head_linear(const TA* __restrict__ A, const TA* __restrict__ W, TA* __restrict
 #pragma unroll
     for (int j = 0; j < 4; j++) {
       const int n = n0 + tx * 4 + j;
-      if (n < N) out[(size_t)m * ldo + n] = cima_from_f32<TA>(acc[i][j]);
+      if (n < N) {
+        const float f = gate ? cima_sigmoid(cima_to_f32<TA>(gate[(size_t)m * ldg + (size_t)head * N + n])) : 1.0f;
+        out[(size_t)m * ldo + n] = cima_from_f32<TA>(acc[i][j] * f);
+      }
     }
   }
 }
@@ -140,7 +144,7 @@ struct LatentJob {
 template <typename TA>
 __global__ void __launch_bounds__(32 * HL_FEW_ROWS)
 k_head_linear_few(const TA* __restrict__ A, const TA* __restrict__ W, TA* __restrict__ out, int M, int N, int K, int lda, int ldo,
-                  int ha, int ho, int vec, LatentJob<TA> job) {
+                  int ha, int ho, int vec, LatentJob<TA> job, const TA* __restrict__ gate, int ldg) {
   extern __shared__ __align__(16) float a_sh[];         // [M][Kp], Kp = K rounded up to 4
   const int Kp = (K + 3) & ~3;
   const int head = blockIdx.y;
@@ -184,6 +188,7 @@ k_head_linear_few(const TA* __restrict__ A, const TA* __restrict__ W, TA* __rest
   }
   __syncthreads();
   const float* ar = a_sh + m * Kp;
+  const float f = gate && live ? cima_sigmoid(cima_to_f32<TA>(gate[(size_t)m * ldg + (size_t)head * N + n])) : 1.0f;
   float acc = 0.f;
   for (int k0 = 0; k0 < K; k0 += HL_FEW_K) {
     const int kn = min(HL_FEW_K, K - k0);
@@ -213,7 +218,55 @@ k_head_linear_few(const TA* __restrict__ A, const TA* __restrict__ W, TA* __rest
       }
     }
   }
-  if (live) out[(size_t)m * ldo + (size_t)head * ho + n] = cima_from_f32<TA>(acc);
+  if (live) out[(size_t)m * ldo + (size_t)head * ho + n] = cima_from_f32<TA>(acc * f);
+}
+
+// The gate alone, behind a product that the library made: src [heads, T, N] contiguous -> out[t, h * ho + n] times the sigmoid.
+template <typename TA, int V>
+__global__ void __launch_bounds__(256)
+k_gate_heads(const TA* __restrict__ src, const TA* __restrict__ gate, int ldg, TA* __restrict__ out, int ldo, int ho, int T, int heads, int N) {
+  cima_pdl_wait();
+  cima_pdl_trigger();
+  const size_t total = (size_t)T * heads * (N / V);
+  for (size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x; i < total; i += (size_t)gridDim.x * blockDim.x) {
+    const int n = (int)(i % (N / V)) * V;
+    const size_t th = i / (N / V);
+    const int h = (int)(th % heads);
+    const size_t t = th / heads;
+    const TA* s = src + ((size_t)h * T + t) * N + n;
+    const TA* g = gate + t * ldg + (size_t)h * N + n;
+    TA* o = out + t * ldo + (size_t)h * ho + n;
+    if constexpr (V == 8) {                                   // eight bfloat16: 16 bytes
+      const uint4 sv = *reinterpret_cast<const uint4*>(s), gv = *reinterpret_cast<const uint4*>(g);
+      uint4 ov;
+      const __nv_bfloat162 *sp = reinterpret_cast<const __nv_bfloat162*>(&sv), *gp = reinterpret_cast<const __nv_bfloat162*>(&gv);
+      __nv_bfloat162* op = reinterpret_cast<__nv_bfloat162*>(&ov);
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const float2 a = __bfloat1622float2(sp[e]), b = __bfloat1622float2(gp[e]);
+        op[e] = __floats2bfloat162_rn(a.x * cima_sigmoid_fast(b.x), a.y * cima_sigmoid_fast(b.y));
+      }
+      *reinterpret_cast<uint4*>(o) = ov;
+    } else {
+      o[0] = cima_from_f32<TA>(cima_to_f32<TA>(s[0]) * cima_sigmoid(cima_to_f32<TA>(g[0])));
+    }
+  }
+}
+
+extern "C" int cima_gate_heads(const void* src, const void* gate, int ldg, void* out, int ldo, int ho, int dtype, int T, int heads, int N,
+                               cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (heads <= 0 || N <= 0 || ho < N || ldo < (heads - 1) * ho + N || ldg < heads * N)
+    return cima_fail(CIMA_E_SIZE, "gate_heads: rows of (%d, %d) do not hold %d heads of %d values", ldo, ldg, heads, N);
+  const bool vec = dtype == CIMA_BF16 && N % 8 == 0 && ldg % 8 == 0 && ldo % 8 == 0 && ho % 8 == 0 && (((uintptr_t)src | (uintptr_t)gate | (uintptr_t)out) & 15) == 0;
+  const size_t work = (size_t)T * heads * (vec ? N / 8 : N);
+  const unsigned grid = (unsigned)((work + 255) / 256 > 148 * 16 ? 148 * 16 : (work + 255) / 256);
+  int rc;
+  if (vec) rc = cima_launch(k_gate_heads<__nv_bfloat16, 8>, dim3(grid), dim3(256), (size_t)0, stream, 1, (const __nv_bfloat16*)src, (const __nv_bfloat16*)gate, ldg, (__nv_bfloat16*)out, ldo, ho, T, heads, N);
+  else if (dtype == CIMA_BF16) rc = cima_launch(k_gate_heads<__nv_bfloat16, 1>, dim3(grid), dim3(256), (size_t)0, stream, 1, (const __nv_bfloat16*)src, (const __nv_bfloat16*)gate, ldg, (__nv_bfloat16*)out, ldo, ho, T, heads, N);
+  else if (dtype == CIMA_F32) rc = cima_launch(k_gate_heads<float, 1>, dim3(grid), dim3(256), (size_t)0, stream, 1, (const float*)src, (const float*)gate, ldg, (float*)out, ldo, ho, T, heads, N);
+  else return cima_fail(CIMA_E_DTYPE, "gate_heads: dtype code %d is neither float32 nor bfloat16", dtype);
+  return rc ? rc : cima_launch_result();
 }
 
 // a [M, heads, K] in rows of lda, w [heads, N, K] contiguous, out [M, heads, N] in rows of ldo; all of `dtype`.
@@ -222,12 +275,13 @@ k_head_linear_few(const TA* __restrict__ A, const TA* __restrict__ W, TA* __rest
 static int head_linear_impl(const void* a, const void* w, void* out, int dtype, int M, int heads, int N, int K, int lda,
                             int ldo, int ha, int ho, const void* raw, int ld_raw, const float* g, float eps, void* cache, const int* table,
                             int table_width, int ring, int page_size, const int* row_pos, const int* row_seq,
-                            const int* seq_slot, int R, cudaStream_t stream);
+                            const int* seq_slot, int R, const void* gate, int ldg, cudaStream_t stream);
 
 extern "C" int cima_head_linear(const void* a, const void* w, void* out, int dtype, int M, int heads, int N, int K, int lda,
-                                int ldo, int ha, int ho, cudaStream_t stream) {
+                                int ldo, int ha, int ho, const void* gate, int ldg, cudaStream_t stream) {
+  if (gate && ldg < heads * N) return cima_fail(CIMA_E_SIZE, "head_linear: gate rows of %d values do not hold %d heads of %d", ldg, heads, N);
   return head_linear_impl(a, w, out, dtype, M, heads, N, K, lda, ldo, ha, ho, nullptr, 0, nullptr, 0.f, nullptr, nullptr, 0, 0, 0,
-                          nullptr, nullptr, nullptr, 0, stream);
+                          nullptr, nullptr, nullptr, 0, gate, ldg, stream);
 }
 
 extern "C" int cima_head_linear_append(const void* a, const void* w, void* out, int dtype, int M, int heads, int N, int K, int lda,
@@ -239,13 +293,13 @@ extern "C" int cima_head_linear_append(const void* a, const void* w, void* out, 
   if (!raw || !g || !cache || !table || R <= 0 || ld_raw < R)
     return cima_fail(CIMA_E_ARG, "head_linear_append: the compressed rows (%d values in rows of %d), the norm's weight, the pages and their table are needed", R, ld_raw);
   return head_linear_impl(a, w, out, dtype, M, heads, N, K, lda, ldo, K, N, raw, ld_raw, g, eps, cache, table, table_width, ring,
-                          page_size, row_pos, row_seq, seq_slot, R, stream);
+                          page_size, row_pos, row_seq, seq_slot, R, nullptr, 0, stream);
 }
 
 static int head_linear_impl(const void* a, const void* w, void* out, int dtype, int M, int heads, int N, int K, int lda,
                             int ldo, int ha, int ho, const void* raw, int ld_raw, const float* g, float eps, void* cache, const int* table,
                             int table_width, int ring, int page_size, const int* row_pos, const int* row_seq,
-                            const int* seq_slot, int R, cudaStream_t stream) {
+                            const int* seq_slot, int R, const void* gate, int ldg, cudaStream_t stream) {
   if (M <= 0) return 0;
   if (heads <= 0 || N <= 0 || K <= 0) return cima_fail(CIMA_E_SIZE, "head_linear: %d heads, N %d and K %d must be positive", heads, N, K);
   if (ha < K || ho < N || lda < (heads - 1) * ha + K || ldo < (heads - 1) * ho + N)
@@ -259,16 +313,16 @@ static int head_linear_impl(const void* a, const void* w, void* out, int dtype, 
     const int esz = dtype == CIMA_F32 ? 4 : 2;
     const int vec = (((uintptr_t)w & 15) == 0 && ((size_t)K * esz) % 16 == 0) ? 1 : 0;      // every row of w starts on 16 bytes
     if (dtype == CIMA_F32) rc = cima_launch(k_head_linear_few<float>, grid, dim3(32 * M), smem, stream, 1, (const float*)a, (const float*)w, (float*)out, M, N, K, lda, ldo, ha, ho, vec,
-                                                LatentJob<float>{(const float*)raw, ld_raw, g, eps, (float*)cache, pg, row_pos, row_seq, seq_slot, R});
+                                                LatentJob<float>{(const float*)raw, ld_raw, g, eps, (float*)cache, pg, row_pos, row_seq, seq_slot, R}, (const float*)gate, ldg);
     else if (dtype == CIMA_BF16) rc = cima_launch(k_head_linear_few<__nv_bfloat16>, grid, dim3(32 * M), smem, stream, 1, (const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, M, N, K, lda, ldo, ha, ho, vec,
-                                                  LatentJob<__nv_bfloat16>{(const __nv_bfloat16*)raw, ld_raw, g, eps, (__nv_bfloat16*)cache, pg, row_pos, row_seq, seq_slot, R});
+                                                  LatentJob<__nv_bfloat16>{(const __nv_bfloat16*)raw, ld_raw, g, eps, (__nv_bfloat16*)cache, pg, row_pos, row_seq, seq_slot, R}, (const __nv_bfloat16*)gate, ldg);
     else return cima_fail(CIMA_E_DTYPE, "head_linear: dtype code %d is neither float32 nor bfloat16", dtype);
   } else if (dtype == CIMA_BF16) {
     const dim3 grid((N + 63) / 64, (M + 63) / 64, heads);
-    rc = cima_launch(k_head_linear<__nv_bfloat16>, grid, dim3(256), (size_t)0, stream, 1, (const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, M, N, K, lda, ldo, ha, ho);
+    rc = cima_launch(k_head_linear<__nv_bfloat16>, grid, dim3(256), (size_t)0, stream, 1, (const __nv_bfloat16*)a, (const __nv_bfloat16*)w, (__nv_bfloat16*)out, M, N, K, lda, ldo, ha, ho, (const __nv_bfloat16*)gate, ldg);
   } else if (dtype == CIMA_F32) {
     const dim3 grid((N + 63) / 64, (M + 63) / 64, heads);
-    rc = cima_launch(k_head_linear<float>, grid, dim3(256), (size_t)0, stream, 1, (const float*)a, (const float*)w, (float*)out, M, N, K, lda, ldo, ha, ho);
+    rc = cima_launch(k_head_linear<float>, grid, dim3(256), (size_t)0, stream, 1, (const float*)a, (const float*)w, (float*)out, M, N, K, lda, ldo, ha, ho, (const float*)gate, ldg);
   } else return cima_fail(CIMA_E_DTYPE, "head_linear: dtype code %d is neither float32 nor bfloat16", dtype);
   if (rc) return rc;
   return cima_launch_result();

@@ -4,6 +4,8 @@
 //                 (float32).  With a correction vector c the comparisons use s + c, the weights s.
 //   moe_sort      the (row, choice) pairs ordered by expert: offsets of every expert's pairs and of its row tiles
 //   moe_gemm 0    z[i] = act(W_gate[e] h[row]) * (W_up[e] h[row])      for the sorted pairs i (a tile = 32 pairs of one expert)
+//                 moe_gemm 2 is the form without gates, z[i] = act(W_up[e] h[row]).  With `weigh` the pair's weight multiplies
+//                 what the expert reads (the product's sums, in front of their rounding and the activation) instead of y.
 //   moe_gemm 1    y[pair] = W_down[e] z[i]                             float32, back at the pair's own place
 //                 Options: a group's score its best one instead of the sum of two; weights s * scale, not divided by their sum.
 //   moe_combine   x[row] += sum_j weight[row, j] * y[row * top + j]    ascending j, float32; a shared expert's rows (float32), times
@@ -275,11 +277,13 @@ k_moe_sort(const int* __restrict__ idx, int P, int E, int* __restrict__ offsets,
 }
 
 // MODE 0: A = h [T, K] gathered by row = perm[i] / top; W = [E, 2 N, K] (gate rows, then up rows); out z [P, N] (TA) at i.
+// MODE 2: the same with W = [E, N, K] and an ungated activation.  weigh (modes 0 and 2, may be null): [P] factors by pair.
 // MODE 1: A = z [P, K] at i; W = [E, N, K]; out y [P, N] float32 at perm[i].
 template <typename TA, typename TW, int MODE>
 __global__ void __launch_bounds__(256)
 k_moe_gemm(const TA* __restrict__ A, int lda, const TW* __restrict__ W, void* __restrict__ out, const int* __restrict__ offsets,
-           const int* __restrict__ tiles, const int* __restrict__ perm, int E, int top, int N, int K, int act, float limit) {
+           const int* __restrict__ tiles, const int* __restrict__ perm, int E, int top, int N, int K, int act, float limit,
+           const float* __restrict__ weigh) {
   cima_pdl_wait();
   __shared__ float As[BK][BM + 1];
   __shared__ float Bs[MODE == 0 ? 2 : 1][BK][BN + 1];
@@ -305,7 +309,7 @@ k_moe_gemm(const TA* __restrict__ A, int lda, const TW* __restrict__ W, void* __
   const int i0 = s_i0, nrows = s_n;
   if (threadIdx.x < BM) {
     const int r = threadIdx.x;
-    s_row[r] = r < nrows ? (MODE == 0 ? perm[i0 + r] / top : i0 + r) : -1;
+    s_row[r] = r < nrows ? (MODE != 1 ? perm[i0 + r] / top : i0 + r) : -1;
   }
   __syncthreads();
   const int n0 = blockIdx.y * BN;
@@ -346,14 +350,17 @@ k_moe_gemm(const TA* __restrict__ A, int lda, const TW* __restrict__ W, void* __
   for (int i = 0; i < 2; i++) {
     const int r = ty * 2 + i;
     if (r >= nrows) continue;
+    const float f = MODE != 1 && weigh ? weigh[perm[i0 + r]] : 1.0f;
 #pragma unroll
     for (int j = 0; j < 4; j++) {
       const int c = n0 + tx * 4 + j;
       if (c >= N) continue;
       if (MODE == 0) {
         // the gate is rounded to the activations' dtype before its activation, as a stored projection would be
-        const float gt = cima_to_f32<TA>(cima_from_f32<TA>(acc[i][j])), up = cima_to_f32<TA>(cima_from_f32<TA>(acc2[i][j]));
+        const float gt = cima_to_f32<TA>(cima_from_f32<TA>(acc[i][j] * f)), up = cima_to_f32<TA>(cima_from_f32<TA>(acc2[i][j] * f));
         reinterpret_cast<TA*>(out)[(size_t)(i0 + r) * N + c] = cima_from_f32<TA>(cima_gated(gt, up, act, limit));
+      } else if (MODE == 2) {
+        reinterpret_cast<TA*>(out)[(size_t)(i0 + r) * N + c] = cima_from_f32<TA>(cima_ungated_act(cima_to_f32<TA>(cima_from_f32<TA>(acc[i][j] * f)), act));
       } else {
         reinterpret_cast<float*>(out)[(size_t)perm[i0 + r] * N + c] = acc[i][j];
       }
@@ -377,7 +384,7 @@ k_moe_combine(const float* __restrict__ y, const float* __restrict__ wgt, const 
     for (int j = 0; j < top; j++) {
       const size_t p = row * top + j;
       const float v = idx && idx[p] >= E ? cima_to_f32<TH>(h[row * H + c]) : y[(pos ? (size_t)pos[p] : p) * H + c];
-      s = fmaf(wgt[p], v, s);
+      s = fmaf(wgt ? wgt[p] : 1.0f, v, s);
     }
     if (shared) s = fmaf(sg, shared[row * H + c], s);
     x[row * H + c] = assign ? s : x[row * H + c] + s;
@@ -412,7 +419,7 @@ k_moe_combine4(const float* __restrict__ y, const float* __restrict__ wgt, const
 #pragma unroll
   for (int j = 0; j < COMBINE_TOP; j++) {
     const size_t p = row * top + (j < top ? j : 0);
-    w[j] = j < top ? wgt[p] : 0.f;
+    w[j] = j < top ? (wgt ? wgt[p] : 1.0f) : 0.f;
     own[j] = idx && idx[p] >= E;                          // an identity expert: the row itself
     src[j] = reinterpret_cast<const float4*>(y) + (own[j] ? (size_t)0 : pos ? (size_t)pos[p] : p) * H4;
   }
@@ -473,15 +480,30 @@ k_moe_sort_tiles(const int* __restrict__ idx, int P, int E, int tile, int n_tile
   }
 }
 
-// dst[pos[p]] = src[p / top]: rows of K values, 16 bytes a thread
+// dst[pos[p]] = src[p / top]: rows of K values, 16 bytes a thread; with `weigh` a row of bfloat16 times its pair's factor
 __global__ void __launch_bounds__(256)
-k_moe_gather_rows(const uint4* __restrict__ src, const int* __restrict__ pos, uint4* __restrict__ dst, int top, int vecs) {
+k_moe_gather_rows(const uint4* __restrict__ src, const int* __restrict__ pos, uint4* __restrict__ dst, int top, int vecs,
+                  const float* __restrict__ weigh) {
   cima_pdl_wait();
   cima_pdl_trigger();        // the next kernel may be set up while this one runs (it waits for this one's end itself)
   const size_t p = blockIdx.x;
   if (pos[p] < 0) return;
   const uint4* s = src + (p / top) * vecs;
   uint4* d = dst + (size_t)pos[p] * vecs;
+  if (weigh) {
+    const float f = weigh[p];
+    for (int v = threadIdx.x; v < vecs; v += blockDim.x) {
+      uint4 t = s[v];
+      __nv_bfloat162* q = reinterpret_cast<__nv_bfloat162*>(&t);
+#pragma unroll
+      for (int e = 0; e < 4; e++) {
+        const float2 a = __bfloat1622float2(q[e]);
+        q[e] = __floats2bfloat162_rn(a.x * f, a.y * f);
+      }
+      d[v] = t;
+    }
+    return;
+  }
   for (int v = threadIdx.x; v < vecs; v += blockDim.x) d[v] = s[v];
 }
 
@@ -494,7 +516,7 @@ template <int MODE>
 __global__ void __launch_bounds__(256)
 k_moe_few(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16* __restrict__ W, void* __restrict__ out,
           const int* __restrict__ offsets, const int* __restrict__ tiles, const int* __restrict__ perm, int E, int top, int N,
-          int K, int act, float limit) {
+          int K, int act, float limit, const float* __restrict__ weigh) {
   cima_pdl_wait();
   __shared__ int s_row[BM];
   __shared__ int s_e, s_i0, s_n;
@@ -516,7 +538,11 @@ k_moe_few(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16* __r
   if (e < 0) return;
   const int i0 = s_i0, nrows = s_n;
   const int tid = (int)threadIdx.x;
-  if (tid < BM) s_row[tid] = tid < nrows ? (MODE == 0 ? perm[i0 + tid] / top : i0 + tid) : -1;
+  __shared__ float s_w[BM];
+  if (tid < BM) {
+    s_row[tid] = tid < nrows ? (MODE != 1 ? perm[i0 + tid] / top : i0 + tid) : -1;
+    s_w[tid] = MODE != 1 && weigh && tid < nrows ? weigh[perm[i0 + tid]] : 1.0f;
+  }
   __syncthreads();
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   // A warp streams FEW_ROWS rows of weights at once, so that enough loads are in flight: a feature's gate and up rows
@@ -574,9 +600,12 @@ k_moe_few(const __nv_bfloat16* __restrict__ A, int lda, const __nv_bfloat16* __r
 #pragma unroll
         for (int f = 0; f < FEATS; f++) {
           if (!valid[f]) continue;
-          if (MODE == 0) {
+          if (MODE == 2) {
+            const float z = __bfloat162float(__float2bfloat16_rn(acc[f][r] * s_w[r0 + r]));
+            reinterpret_cast<__nv_bfloat16*>(out)[(size_t)(i0 + r0 + r) * N + n + 8 * f] = __float2bfloat16_rn(cima_ungated_act(z, act));
+          } else if (MODE == 0) {
             // gate and up are rounded to bfloat16 before the activation, as stored projections would be
-            const float gt = __bfloat162float(__float2bfloat16_rn(acc[2 * f][r])), uv = __bfloat162float(__float2bfloat16_rn(acc[2 * f + 1][r]));
+            const float gt = __bfloat162float(__float2bfloat16_rn(acc[2 * f][r] * s_w[r0 + r])), uv = __bfloat162float(__float2bfloat16_rn(acc[2 * f + 1][r] * s_w[r0 + r]));
             reinterpret_cast<__nv_bfloat16*>(out)[(size_t)(i0 + r0 + r) * N + n + 8 * f] = __float2bfloat16_rn(cima_gated(gt, uv, act, limit));
           } else {
             reinterpret_cast<float*>(out)[(size_t)perm[i0 + r0 + r] * N + n + 8 * f] = acc[f][r];
@@ -620,27 +649,29 @@ extern "C" int cima_moe_sort(const int* idx, int P, int E, int* offsets, int* ti
   return rc ? rc : cima_launch_result();
 }
 
-// mode 0: a [T, lda] (adtype), w [E, 2 N, K] (wdtype), out [P, N] (adtype); mode 1: a [P, lda], w [E, N, K], out [P, N] float32.
+// mode 0: a [T, lda] (adtype), w [E, 2 N, K] (wdtype), out [P, N] (adtype); mode 2: the same with w [E, N, K]; mode 1: a [P, lda], w [E, N, K], out [P, N] float32.
 extern "C" int cima_moe_gemm(const void* a, int adtype, int lda, const void* w, int wdtype, void* out, const int* offsets,
                              const int* tiles, const int* perm, int P, int E, int top, int N, int K, int mode, int act, float limit,
-                             cudaStream_t stream) {
+                             const float* weigh, cudaStream_t stream) {
   if (P <= 0) return 0;
   if (N <= 0 || K <= 0 || E <= 0 || top <= 0) return cima_fail(CIMA_E_SIZE, "moe_gemm: sizes must be positive");
-  if (mode != 0 && mode != 1) return cima_fail(CIMA_E_ARG, "moe_gemm: mode %d is neither 0 (gate | up) nor 1 (down)", mode);
-  if (act < 0 || act >= CIMA_GATED_COUNT) return cima_fail(CIMA_E_ARG, "moe_gemm: activation code %d is unknown", act);
+  if (mode < 0 || mode > 2) return cima_fail(CIMA_E_ARG, "moe_gemm: mode %d is none of 0 (gate | up), 1 (down), 2 (up without gates)", mode);
+  if (mode == 2 ? !cima_ungated_known(act) : (act < 0 || act >= CIMA_GATED_COUNT)) return cima_fail(CIMA_E_ARG, "moe_gemm: activation code %d is unknown", act);
   const dim3 grid((unsigned)((P + BM - 1) / BM + E), (unsigned)((N + BN - 1) / BN));
   if (grid.y > 65535) return cima_fail(CIMA_E_SIZE, "moe_gemm: %d outputs exceed one launch", N);
   int rc;
-#define RUN(TA, TW, M) rc = cima_launch(k_moe_gemm<TA, TW, M>, grid, dim3(256), (size_t)0, stream, 1, (const TA*)a, lda, (const TW*)w, out, offsets, tiles, perm, E, top, N, K, act, limit)
-  if (adtype == CIMA_F32 && wdtype == CIMA_F32) { if (mode == 0) RUN(float, float, 0); else RUN(float, float, 1); }
-  else if (adtype == CIMA_BF16 && wdtype == CIMA_BF16) { if (mode == 0) RUN(__nv_bfloat16, __nv_bfloat16, 0); else RUN(__nv_bfloat16, __nv_bfloat16, 1); }
-  else if (adtype == CIMA_BF16 && wdtype == CIMA_F32) { if (mode == 0) RUN(__nv_bfloat16, float, 0); else RUN(__nv_bfloat16, float, 1); }
+#define RUN(TA, TW, M) rc = cima_launch(k_moe_gemm<TA, TW, M>, grid, dim3(256), (size_t)0, stream, 1, (const TA*)a, lda, (const TW*)w, out, offsets, tiles, perm, E, top, N, K, act, limit, weigh)
+#define MODES(TA, TW) { if (mode == 0) RUN(TA, TW, 0); else if (mode == 1) RUN(TA, TW, 1); else RUN(TA, TW, 2); }
+  if (adtype == CIMA_F32 && wdtype == CIMA_F32) MODES(float, float)
+  else if (adtype == CIMA_BF16 && wdtype == CIMA_BF16) MODES(__nv_bfloat16, __nv_bfloat16)
+  else if (adtype == CIMA_BF16 && wdtype == CIMA_F32) MODES(__nv_bfloat16, float)
   else return cima_fail(CIMA_E_DTYPE, "moe_gemm: activations of dtype %d with weights of dtype %d are not accepted", adtype, wdtype);
+#undef MODES
 #undef RUN
   return rc ? rc : cima_launch_result();
 }
 
-// y [pairs or places, H] float32; pos [T * top] the row of y of every pair, or null where y is kept by pair
+// y [pairs or places, H] float32; wgt [T * top], or null where the rows of y are summed as they are; pos [T * top] the row of y of every pair, or null where y is kept by pair
 // shared (may be null): [T, H] float32 rows added behind the experts', each row times sigmoid(gate[row * ldg]) where gate is given
 // idx (may be null: no identity experts) [T, top] with h [T, H] (hdtype): a pair whose expert is >= E has h[row] as its output
 extern "C" int cima_moe_combine(const float* y, const float* wgt, const int* pos, float* x, int T, int top, int H, int assign,
@@ -668,28 +699,31 @@ extern "C" int cima_moe_sort_tiles(const int* idx, int P, int E, int tile, int n
   return rc ? rc : cima_launch_result();
 }
 
-// dst[pos[p]] = src[p / top] for the P pairs: rows of `row_bytes` bytes (a multiple of 16, both 16-byte aligned)
-extern "C" int cima_moe_gather_rows(const void* src, const int* pos, void* dst, int P, int top, int row_bytes, cudaStream_t stream) {
+// dst[pos[p]] = src[p / top] for the P pairs: rows of `row_bytes` bytes (a multiple of 16, both 16-byte aligned); with weigh [P]
+// the rows are bfloat16 and leave times their pair's factor
+extern "C" int cima_moe_gather_rows(const void* src, const int* pos, void* dst, int P, int top, int row_bytes, const float* weigh, cudaStream_t stream) {
   if (P <= 0) return 0;
   if (row_bytes <= 0 || row_bytes % 16 || (((uintptr_t)src | (uintptr_t)dst) & 15))
     return cima_fail(CIMA_E_ARG, "moe_gather_rows: rows of %d bytes must be multiples of 16 bytes at 16-byte aligned addresses", row_bytes);
-  int rc = cima_launch(k_moe_gather_rows, dim3(P), dim3(256), (size_t)0, stream, 1, (const uint4*)src, pos, (uint4*)dst, top, row_bytes / 16);
+  int rc = cima_launch(k_moe_gather_rows, dim3(P), dim3(256), (size_t)0, stream, 1, (const uint4*)src, pos, (uint4*)dst, top, row_bytes / 16, weigh);
   return rc ? rc : cima_launch_result();
 }
 
 // The products of moe_gemm for few pairs, bfloat16 activations and weights, K a multiple of 8, 16-byte aligned rows.
 extern "C" int cima_moe_few(const void* a, int lda, const void* w, void* out, const int* offsets, const int* tiles,
-                            const int* perm, int P, int E, int top, int N, int K, int mode, int act, float limit, cudaStream_t stream) {
+                            const int* perm, int P, int E, int top, int N, int K, int mode, int act, float limit, const float* weigh,
+                             cudaStream_t stream) {
   if (P <= 0) return 0;
   if (N <= 0 || K <= 0 || K % 8 || lda % 8 || E <= 0 || top <= 0 || (((uintptr_t)a | (uintptr_t)w) & 15))
     return cima_fail(CIMA_E_SIZE, "moe_few: K %d and the row stride %d must be multiples of 8 and the operands 16-byte aligned", K, lda);
-  if (mode != 0 && mode != 1) return cima_fail(CIMA_E_ARG, "moe_few: mode %d is neither 0 (gate | up) nor 1 (down)", mode);
-  if (act < 0 || act >= CIMA_GATED_COUNT) return cima_fail(CIMA_E_ARG, "moe_few: activation code %d is unknown", act);
+  if (mode < 0 || mode > 2) return cima_fail(CIMA_E_ARG, "moe_few: mode %d is none of 0 (gate | up), 1 (down), 2 (up without gates)", mode);
+  if (mode == 2 ? !cima_ungated_known(act) : (act < 0 || act >= CIMA_GATED_COUNT)) return cima_fail(CIMA_E_ARG, "moe_few: activation code %d is unknown", act);
   const int per_block = 8 * (mode == 0 ? FEW_ROWS / 2 : FEW_ROWS);          // features of a block: its 8 warps' 
   const dim3 grid((unsigned)((P + BM - 1) / BM + E), (unsigned)((N + per_block - 1) / per_block));
   if (grid.y > 65535) return cima_fail(CIMA_E_SIZE, "moe_few: %d outputs exceed one launch", N);
   int rc;
-  if (mode == 0) rc = cima_launch(k_moe_few<0>, grid, dim3(256), (size_t)0, stream, 1, (const __nv_bfloat16*)a, lda, (const __nv_bfloat16*)w, out, offsets, tiles, perm, E, top, N, K, act, limit);
-  else rc = cima_launch(k_moe_few<1>, grid, dim3(256), (size_t)0, stream, 1, (const __nv_bfloat16*)a, lda, (const __nv_bfloat16*)w, out, offsets, tiles, perm, E, top, N, K, act, limit);
+  if (mode == 0) rc = cima_launch(k_moe_few<0>, grid, dim3(256), (size_t)0, stream, 1, (const __nv_bfloat16*)a, lda, (const __nv_bfloat16*)w, out, offsets, tiles, perm, E, top, N, K, act, limit, weigh);
+  else if (mode == 2) rc = cima_launch(k_moe_few<2>, grid, dim3(256), (size_t)0, stream, 1, (const __nv_bfloat16*)a, lda, (const __nv_bfloat16*)w, out, offsets, tiles, perm, E, top, N, K, act, limit, weigh);
+  else rc = cima_launch(k_moe_few<1>, grid, dim3(256), (size_t)0, stream, 1, (const __nv_bfloat16*)a, lda, (const __nv_bfloat16*)w, out, offsets, tiles, perm, E, top, N, K, act, limit, weigh);
   return rc ? rc : cima_launch_result();
 }

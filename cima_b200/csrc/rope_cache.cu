@@ -322,6 +322,115 @@ k_norm_append(TA* __restrict__ qkv, int ld, const int* __restrict__ row_pos, con
   }
 }
 
+// The norm over whole projections with the append, where nothing rotates: of a row [q heads | k heads | v heads] (heads of hd
+// values, what pads a head being zero) all of q is divided by its root mean square over q_count values and multiplied by q_w
+// [nh * hd], all of k likewise with k_w; with `mix` the values become (1 - l) v + l f, l = *mix and f the same row's values in
+// `first` (heads of first_hd values), on the first v_dim values of a head; k and v go to the row's place in the pages.  A block
+// a row, four neighbouring values a thread at a time, NV of them kept in registers between the sums and the stores with every
+// load requested before the first use.  Float32 inside, sums in a fixed order, one rounding at the store.
+template <typename TA, int NV, int THREADS>
+__global__ void __launch_bounds__(THREADS)
+k_row_norm_append(TA* __restrict__ qkv, int ld, const int* __restrict__ row_pos, const int* __restrict__ row_seq,
+                  const int* __restrict__ seq_slot, const int* __restrict__ seq_len, TA* __restrict__ cache_in, CimaPaged pg, int nh,
+                  int nkv, int hd, const float* __restrict__ q_w, const float* __restrict__ k_w, float q_count, float k_count, float eps,
+                  const float* __restrict__ mix, const TA* __restrict__ first, int ld_first, int first_hd, int v_dim) {
+  __shared__ float red[32];
+  const int nq4 = nh * hd / 4, nqk4 = (nh + nkv) * hd / 4, all4 = (nh + 2 * nkv) * hd / 4;
+  float4 w[NV];
+  // (the norms' weights depend on no kernel: they are fetched before the wait)
+#pragma unroll
+  for (int j = 0; j < NV; j++) {
+    const int i = threadIdx.x + j * THREADS;
+    w[j] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i < nqk4) w[j] = i < nq4 ? reinterpret_cast<const float4*>(q_w)[i] : reinterpret_cast<const float4*>(k_w)[i - nq4];
+  }
+  const float lam = mix ? *mix : 0.f;
+  cima_pdl_wait();
+  const int row = blockIdx.x;
+  TA* base = qkv + (size_t)row * ld;
+  const int pos = row_pos[row], seq = row_seq[row];
+  float v[NV][4];
+#pragma unroll
+  for (int j = 0; j < NV; j++) {
+    const int i = threadIdx.x + j * THREADS;
+    v[j][0] = v[j][1] = v[j][2] = v[j][3] = 0.f;
+    if (i < all4) rope_load4<TA>(base + 4 * i, v[j]);
+  }
+  TA* cache = cache_in;
+  if (pg.ring && pos + pg.ring * pg.page_size < seq_len[seq]) cache = nullptr;      // a later row of the step takes the place
+  const int slot = seq_slot[seq];
+  float sq = 0.f, sk = 0.f;
+#pragma unroll
+  for (int j = 0; j < NV; j++) {
+    const int i = threadIdx.x + j * THREADS;
+    const float s = fmaf(v[j][0], v[j][0], v[j][1] * v[j][1]) + fmaf(v[j][2], v[j][2], v[j][3] * v[j][3]);
+    if (i < nq4) sq += s;
+    else if (i < nqk4) sk += s;
+  }
+  sq = cima_block_sum(sq, red);
+  sk = cima_block_sum(sk, red);
+  const float rq = 1.0f / sqrtf(sq / q_count + eps), rk = 1.0f / sqrtf(sk / k_count + eps);
+#pragma unroll
+  for (int j = 0; j < NV; j++) {
+    const int i = threadIdx.x + j * THREADS;
+    if (i >= all4) continue;
+    if (i < nqk4) {
+      const float r = i < nq4 ? rq : rk;
+      v[j][0] *= r * w[j].x; v[j][1] *= r * w[j].y; v[j][2] *= r * w[j].z; v[j][3] *= r * w[j].w;
+      const RopePack4<TA> p(v[j]);
+      p.store(base + 4 * i);
+      if (cache && i >= nq4) {
+        const int c = 4 * (i - nq4), head = c / hd;
+        p.store(cache + pg.offset(slot, pos, 0, head) + (c - head * hd));
+      }
+    } else {
+      const int c = 4 * (i - nqk4), head = c / hd, d = c - head * hd;
+      if (mix && d < v_dim) {
+        float f[4];
+        rope_load4<TA>(first + (size_t)row * ld_first + (size_t)head * first_hd + d, f);
+#pragma unroll
+        for (int e = 0; e < 4; e++)
+          if (d + e < v_dim) v[j][e] = (1.0f - lam) * v[j][e] + lam * f[e];
+      }
+      const RopePack4<TA> p(v[j]);
+      if (mix) p.store(base + 4 * i);
+      if (cache) p.store(cache + pg.offset(slot, pos, 1, head) + d);
+    }
+  }
+}
+
+// qkv [T, ld]: rows of nh + 2 nkv heads of hd values (hd, ld and first's strides multiples of 4, pointers on 4 values); q_w, k_w
+// float32 [nh * hd], [nkv * hd]; q_count and k_count: the values that the norms average over (padding left out).  mix (may be
+// null): one float32 on the device, with first [T, ld_first].  The cache is the layer's pages (two planes).
+extern "C" int cima_row_norm_append(void* qkv, int dtype, int ld, const int* row_pos, const int* row_seq, const int* seq_slot,
+                                    const int* seq_len, void* cache, const int* table, int table_width, int ring, int page_size, int T,
+                                    int nh, int nkv, int hd, const float* q_w, const float* k_w, int q_count, int k_count, float eps,
+                                    const float* mix, const void* first, int ld_first, int first_hd, int v_dim, cudaStream_t stream) {
+  if (T <= 0) return 0;
+  if (nh <= 0 || nkv <= 0 || hd <= 0 || hd % 4 || ld % 4 || ld < (nh + 2 * nkv) * hd)
+    return cima_fail(CIMA_E_SIZE, "row_norm_append: %d + 2 x %d heads of %d values (a multiple of 4) in rows of %d are not accepted", nh, nkv, hd, ld);
+  if (!q_w || !k_w || q_count <= 0 || k_count <= 0) return cima_fail(CIMA_E_ARG, "row_norm_append: the norms' weights and the values they average over are needed");
+  if (!cache || !table || page_size <= 0 || table_width <= 0) return cima_fail(CIMA_E_ARG, "row_norm_append: the layer's pages and their block table are needed");
+  if (mix && (!first || first_hd % 4 || ld_first % 4 || v_dim <= 0 || v_dim > hd || v_dim > first_hd || ld_first < nkv * first_hd))
+    return cima_fail(CIMA_E_ARG, "row_norm_append: the values to mix in, heads of %d in rows of %d, do not fit %d heads of %d", first_hd, ld_first, nkv, v_dim);
+  const size_t bytes = dtype == CIMA_F32 ? 16 : 8;
+  if ((((uintptr_t)qkv | (uintptr_t)cache | (uintptr_t)first) & (bytes - 1)) || (((uintptr_t)q_w | (uintptr_t)k_w) & 15))
+    return cima_fail(CIMA_E_ARG, "row_norm_append: rows, pages and weights must start on four values");
+  const CimaPaged pg{table, table_width, ring, page_size, nkv, hd};
+  const int all4 = (nh + 2 * nkv) * hd / 4;
+  int rc;
+#define RUN(TA, NV, B) rc = cima_launch(k_row_norm_append<TA, NV, B>, dim3(T), dim3(B), (size_t)0, stream, 1, (TA*)qkv, ld, row_pos, row_seq, seq_slot, seq_len, (TA*)cache, pg, nh, nkv, hd, q_w, k_w, (float)q_count, (float)k_count, eps, mix, (const TA*)first, ld_first, first_hd, v_dim)
+#define PICK(TA) { if (all4 <= 256) RUN(TA, 2, 128); else if (all4 <= 512) RUN(TA, 2, 256); else if (all4 <= 1024) RUN(TA, 4, 256); \
+                   else if (all4 <= 2048) RUN(TA, 4, 512); else if (all4 <= 4096) RUN(TA, 4, 1024); \
+                   else return cima_fail(CIMA_E_SIZE, "row_norm_append: rows of %d values exceed one block (16384)", 4 * all4); }
+  if (dtype == CIMA_F32) PICK(float)
+  else if (dtype == CIMA_BF16) PICK(__nv_bfloat16)
+  else return cima_fail(CIMA_E_DTYPE, "row_norm_append: dtype code %d is neither float32 nor bfloat16", dtype);
+#undef PICK
+#undef RUN
+  return rc ? rc : cima_launch_result();
+}
+
 // cache may be null (a layer that reads another layer's keys and values writes none).
 // nv: value heads of a row (nkv unless key heads share value heads); q_norm / k_norm (both or neither): the weights of
 // a norm over the first norm_dim values of every q / k head before the rotation (null with norm_dim > 0: a norm without weight).

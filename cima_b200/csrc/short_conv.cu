@@ -19,7 +19,7 @@ template <typename TA, bool ONE_ROW>
 __global__ void __launch_bounds__(CONV_THREADS)
 k_short_conv(const TA* __restrict__ h, const float* __restrict__ w, TA* __restrict__ state,
              const int* __restrict__ row_seq, const int* __restrict__ seq_slot, const int* __restrict__ seq_first_row,
-             TA* __restrict__ u, int C, int taps, int add_input, int act) {
+             TA* __restrict__ u, int ldh, int C, int taps, int add_input, int act) {
   cima_pdl_wait();
   const int row = blockIdx.x;
   const int c = blockIdx.y * CONV_THREADS + threadIdx.x;
@@ -28,7 +28,7 @@ k_short_conv(const TA* __restrict__ h, const float* __restrict__ w, TA* __restri
   const int k = ONE_ROW ? 0 : row - seq_first_row[seq];          // index of the row among the step's rows of its sequence
   const int slot = seq_slot[seq];
   TA* st = state + (size_t)slot * (taps - 1) * C + c;
-  const float cur = cima_to_f32<TA>(h[(size_t)row * C + c]);
+  const float cur = cima_to_f32<TA>(h[(size_t)row * ldh + c]);
   float acc = add_input ? cur : 0.f;
   float old[CONV_MAX_TAPS];
 #pragma unroll
@@ -37,7 +37,7 @@ k_short_conv(const TA* __restrict__ h, const float* __restrict__ w, TA* __restri
     const int back = taps - 1 - j;                                // positions back from this row
     float v;
     if (back == 0) v = cur;
-    else if (back <= k) v = cima_to_f32<TA>(h[(size_t)(row - back) * C + c]);
+    else if (back <= k) v = cima_to_f32<TA>(h[(size_t)(row - back) * ldh + c]);
     else v = cima_to_f32<TA>(st[(size_t)(taps - 1 - (back - k)) * C]);
     old[j] = v;
     acc = fmaf(w[(size_t)j * C + c], v, acc);
@@ -65,7 +65,7 @@ template <typename TA>
 __global__ void __launch_bounds__(CONV_THREADS)
 k_short_conv_wide(const TA* __restrict__ h, const float* __restrict__ w, const TA* __restrict__ state,
                   const int* __restrict__ row_seq, const int* __restrict__ seq_slot, const int* __restrict__ seq_first_row,
-                  TA* __restrict__ u, int C, int taps, int add_input, int act) {
+                  TA* __restrict__ u, int ldh, int C, int taps, int add_input, int act) {
   cima_pdl_wait();
   constexpr int V = ConvVec<TA>::N;
   const int row = blockIdx.x;
@@ -76,7 +76,7 @@ k_short_conv_wide(const TA* __restrict__ h, const float* __restrict__ w, const T
   const TA* st = state + (size_t)seq_slot[seq] * (taps - 1) * C + c;
   float acc[V], cur[V];
   {
-    const uint4 raw = *reinterpret_cast<const uint4*>(h + (size_t)row * C + c);
+    const uint4 raw = *reinterpret_cast<const uint4*>(h + (size_t)row * ldh + c);
     const TA* e = reinterpret_cast<const TA*>(&raw);
 #pragma unroll
     for (int i = 0; i < V; i++) { cur[i] = cima_to_f32<TA>(e[i]); acc[i] = add_input ? cur[i] : 0.f; }
@@ -88,7 +88,7 @@ k_short_conv_wide(const TA* __restrict__ h, const float* __restrict__ w, const T
 #pragma unroll
       for (int i = 0; i < V; i++) v[i] = cur[i];
     } else {
-      const TA* src = back <= k ? h + (size_t)(row - back) * C + c : st + (size_t)(taps - 1 - (back - k)) * C;
+      const TA* src = back <= k ? h + (size_t)(row - back) * ldh + c : st + (size_t)(taps - 1 - (back - k)) * C;
       const uint4 raw = *reinterpret_cast<const uint4*>(src);
       const TA* e = reinterpret_cast<const TA*>(&raw);
 #pragma unroll
@@ -121,7 +121,7 @@ template <typename TA, int CONV_ROWS>
 __global__ void __launch_bounds__(CONV_THREADS)
 k_short_conv_rows(const TA* __restrict__ h, const float* __restrict__ w, const TA* __restrict__ state,
                   const int* __restrict__ row_seq, const int* __restrict__ seq_slot, const int* __restrict__ seq_first_row,
-                  TA* __restrict__ u, int T, int C, int taps, int add_input, int act) {
+                  TA* __restrict__ u, int T, int ldh, int C, int taps, int add_input, int act) {
   cima_pdl_wait();
   constexpr int V = ConvVec<TA>::N;
   const int c = (blockIdx.y * CONV_THREADS + threadIdx.x) * V;
@@ -143,10 +143,10 @@ k_short_conv_rows(const TA* __restrict__ h, const float* __restrict__ w, const T
   int seqs[CONV_ROWS], ks[CONV_ROWS];
 #pragma unroll
   for (int r = 0; r < CONV_ROWS; r++)
-    if (r0 + r < r1) rows[r] = *reinterpret_cast<const uint4*>(h + (size_t)(r0 + r) * C + c);
+    if (r0 + r < r1) rows[r] = *reinterpret_cast<const uint4*>(h + (size_t)(r0 + r) * ldh + c);
 #pragma unroll
   for (int b = 1; b < CONV_FEW_TAPS; b++)
-    if (b < taps && r0 - b >= 0) halo[b - 1] = *reinterpret_cast<const uint4*>(h + (size_t)(r0 - b) * C + c);
+    if (b < taps && r0 - b >= 0) halo[b - 1] = *reinterpret_cast<const uint4*>(h + (size_t)(r0 - b) * ldh + c);
 #pragma unroll
   for (int r = 0; r < CONV_ROWS; r++) seqs[r] = r0 + r < r1 ? row_seq[r0 + r] : 0;
 #pragma unroll
@@ -172,7 +172,7 @@ k_short_conv_rows(const TA* __restrict__ h, const float* __restrict__ w, const T
         if (b < taps) {
           uint4 raw;
           if (r == 0 && b <= k) raw = halo[b - 1];
-          else raw = *reinterpret_cast<const uint4*>(b <= k ? h + (size_t)(row - b) * C + c : st + (size_t)(taps - 1 - (b - k)) * C);
+          else raw = *reinterpret_cast<const uint4*>(b <= k ? h + (size_t)(row - b) * ldh + c : st + (size_t)(taps - 1 - (b - k)) * C);
           const TA* e = reinterpret_cast<const TA*>(&raw);
 #pragma unroll
           for (int i = 0; i < V; i++) past[b - 1][i] = cima_to_f32<TA>(e[i]);
@@ -213,7 +213,7 @@ k_short_conv_rows(const TA* __restrict__ h, const float* __restrict__ w, const T
 template <typename TA>
 __global__ void __launch_bounds__(CONV_THREADS)
 k_short_conv_state(const TA* __restrict__ h, TA* __restrict__ state, const int* __restrict__ seq_slot,
-                   const int* __restrict__ seq_first_row, int C, int taps) {
+                   const int* __restrict__ seq_first_row, int ldh, int C, int taps) {
   cima_pdl_wait();
   const int seq = blockIdx.x;
   const int c = blockIdx.y * CONV_THREADS + threadIdx.x;
@@ -225,7 +225,7 @@ k_short_conv_state(const TA* __restrict__ h, TA* __restrict__ state, const int* 
   for (int k = 0; k < CONV_MAX_TAPS - 1; k++) {
     if (k >= taps - 1) break;
     const int i = n - (taps - 1) + k;                             // the step's row that becomes entry k, if it is one
-    v[k] = i >= 0 ? h[(size_t)(first + i) * C + c] : st[(size_t)(k + n) * C];
+    v[k] = i >= 0 ? h[(size_t)(first + i) * ldh + c] : st[(size_t)(k + n) * C];
   }
 #pragma unroll
   for (int k = 0; k < CONV_MAX_TAPS - 1; k++) {
@@ -235,22 +235,23 @@ k_short_conv_state(const TA* __restrict__ h, TA* __restrict__ state, const int* 
 }
 
 // add_input 0 leaves the input out of the sum (a plain convolution); act >= 0 applies that activation (CIMA_ACT_*) to the sum.
-// h, u [T, C] and state [slots, taps - 1, C] of one dtype; w [taps, C] float32.  one_row != 0: row r is sequence r's only row.
+// h [T, C] in rows of ldh values; u [T, C] and state [slots, taps - 1, C] of one dtype; w [taps, C] float32.  one_row != 0: row r is sequence r's only row.
 // rows_per_thread: 0, or how many consecutive rows a thread of the many-row kernel walks (the result does not depend on it).
-extern "C" int cima_short_conv(const void* h, int dtype, const float* w, void* state, const int* row_seq, const int* seq_slot,
+extern "C" int cima_short_conv(const void* h, int dtype, int ldh, const float* w, void* state, const int* row_seq, const int* seq_slot,
                                const int* seq_first_row, void* u, int T, int n_seqs, int C, int taps, int one_row,
                                int rows_per_thread, int add_input, int act, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (act >= CIMA_ACT_COUNT) return cima_fail(CIMA_E_ARG, "short_conv: activation code %d is unknown", act);
   if (taps < 1 || taps > CONV_MAX_TAPS) return cima_fail(CIMA_E_SIZE, "short_conv: %d taps are outside 1..%d", taps, CONV_MAX_TAPS);
   if (C <= 0 || n_seqs <= 0) return cima_fail(CIMA_E_SIZE, "short_conv: %d channels and %d sequences must be positive", C, n_seqs);
+  if (ldh < C) return cima_fail(CIMA_E_SIZE, "short_conv: rows of %d values hold no %d channels", ldh, C);
   if (one_row && T != n_seqs) return cima_fail(CIMA_E_ARG, "short_conv: %d rows are not one for each of %d sequences", T, n_seqs);
   if (taps > 1 && !state) return cima_fail(CIMA_E_ARG, "short_conv: more than one tap needs the sequences' state");
   const dim3 block(CONV_THREADS);
   const unsigned cy = (unsigned)((C + CONV_THREADS - 1) / CONV_THREADS);
   // 16-byte accesses: the rows of h, u and the state must all start on 16 bytes
   const int per16 = dtype == CIMA_F32 ? 4 : 8;
-  const bool wide = C % per16 == 0 && (((uintptr_t)h | (uintptr_t)u | (uintptr_t)state | (uintptr_t)w) & 15) == 0;
+  const bool wide = C % per16 == 0 && ldh % per16 == 0 && (((uintptr_t)h | (uintptr_t)u | (uintptr_t)state | (uintptr_t)w) & 15) == 0;
   // rows a thread walks: 8 where that still leaves the SMs a few hundred thousand threads; else one (the kernel above)
   const long long cells = (long long)T * (C / per16);
   // (measured inside a 2,048-row step at 3,584 channels: 8 rows a thread 14 to 16 us, one row 18 to 19, two rows 22; at
@@ -260,14 +261,14 @@ extern "C" int cima_short_conv(const void* h, int dtype, const float* w, void* s
   else if (rows_per_thread != 0) return cima_fail(CIMA_E_ARG, "short_conv: %d rows a thread; 0 (chosen here), 1, 2, 4 or 8 are possible", rows_per_thread);
 #define RUN(TA) { \
     int rc_; \
-    if (one_row) rc_ = cima_launch(k_short_conv<TA, true>, dim3(T, cy), block, (size_t)0, stream, 1, (const TA*)h, w, (TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, C, taps, add_input, act); \
-    else if (wide && taps <= CONV_FEW_TAPS && rows_each == 8) rc_ = cima_launch(k_short_conv_rows<TA, 8>, dim3((T + 7) / 8, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, T, C, taps, add_input, act); \
-    else if (wide && taps <= CONV_FEW_TAPS && rows_each == 4) rc_ = cima_launch(k_short_conv_rows<TA, 4>, dim3((T + 3) / 4, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, T, C, taps, add_input, act); \
-    else if (wide && taps <= CONV_FEW_TAPS && rows_each == 2) rc_ = cima_launch(k_short_conv_rows<TA, 2>, dim3((T + 1) / 2, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, T, C, taps, add_input, act); \
-    else if (wide) rc_ = cima_launch(k_short_conv_wide<TA>, dim3(T, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, C, taps, add_input, act); \
-    else rc_ = cima_launch(k_short_conv<TA, false>, dim3(T, cy), block, (size_t)0, stream, 1, (const TA*)h, w, (TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, C, taps, add_input, act); \
+    if (one_row) rc_ = cima_launch(k_short_conv<TA, true>, dim3(T, cy), block, (size_t)0, stream, 1, (const TA*)h, w, (TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, ldh, C, taps, add_input, act); \
+    else if (wide && taps <= CONV_FEW_TAPS && rows_each == 8) rc_ = cima_launch(k_short_conv_rows<TA, 8>, dim3((T + 7) / 8, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, T, ldh, C, taps, add_input, act); \
+    else if (wide && taps <= CONV_FEW_TAPS && rows_each == 4) rc_ = cima_launch(k_short_conv_rows<TA, 4>, dim3((T + 3) / 4, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, T, ldh, C, taps, add_input, act); \
+    else if (wide && taps <= CONV_FEW_TAPS && rows_each == 2) rc_ = cima_launch(k_short_conv_rows<TA, 2>, dim3((T + 1) / 2, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, T, ldh, C, taps, add_input, act); \
+    else if (wide) rc_ = cima_launch(k_short_conv_wide<TA>, dim3(T, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, ldh, C, taps, add_input, act); \
+    else rc_ = cima_launch(k_short_conv<TA, false>, dim3(T, cy), block, (size_t)0, stream, 1, (const TA*)h, w, (TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, ldh, C, taps, add_input, act); \
     if (rc_) return rc_; \
-    if (!one_row && taps > 1) { rc_ = cima_launch(k_short_conv_state<TA>, dim3(n_seqs, cy), block, (size_t)0, stream, 1, (const TA*)h, (TA*)state, seq_slot, seq_first_row, C, taps); if (rc_) return rc_; } }
+    if (!one_row && taps > 1) { rc_ = cima_launch(k_short_conv_state<TA>, dim3(n_seqs, cy), block, (size_t)0, stream, 1, (const TA*)h, (TA*)state, seq_slot, seq_first_row, ldh, C, taps); if (rc_) return rc_; } }
   if (dtype == CIMA_F32) RUN(float)
   else if (dtype == CIMA_BF16) RUN(__nv_bfloat16)
   else return cima_fail(CIMA_E_DTYPE, "short_conv: dtype code %d is neither float32 nor bfloat16", dtype);

@@ -15,7 +15,7 @@ import torch
 from .csrc.build import BuildError, library_path
 
 F32, BF16 = 0, 1
-ABI_VERSION = 31
+ABI_VERSION = 32
 SPLIT_BLOCKS = 296          # blocks of the decode attention that one wave holds (two per SM, 148 SMs)
 TC_ATTENTION_MIN_LEN = 256  # prompts from this length on take the tcgen05 attention (head_dim 64 or 128)
 SPLIT_FEW_BLOCKS = 148      # below this many blocks at 8 splits, more splits are taken
@@ -34,6 +34,7 @@ def short_context(head_dim: int) -> int:
 
 # epilogues of the skinny product
 SK_STORE, SK_ACCUM, SK_SWIGLU, SK_STORE_F32 = 0, 1, 2, 3
+EPI_ACT = 4                 # grouped tcgen05 product only: an ungated activation, bfloat16 store
 # activations of a gated feed-forward's gate (CIMA_ACT_* of csrc/common.cuh), by the names config files use
 ACTIVATIONS = {"silu": 0, "swish": 0, "gelu_pytorch_tanh": 1, "gelu_tanh": 1, "gelu_new": 1, "gelu": 2, "relu": 3,
                # min(g, L) * sigmoid(1.702 min(g, L)) * (clamp(u, -L, L) + 1): the kernels that take it take the limit L beside the code
@@ -58,7 +59,7 @@ def dtype_code(dt: torch.dtype) -> int:
 _vp, _i, _f, _sz = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_size_t
 
 _SIGNATURES = {
-    "cima_embed": [_vp, _vp, _i, _vp, _i, _i, _i, _f, _vp, _vp, _vp, _vp],
+    "cima_embed": [_vp, _vp, _i, _vp, _i, _i, _i, _f, _vp, _vp, _vp, _vp, _vp, _i, _vp],
     "cima_rmsnorm": [_vp, _vp, _vp, _i, _i, _i, _f, _vp],
     "cima_swiglu": [_vp, _vp, _i, _i, _i, _i, _f, _vp],
     "cima_add_residual": [_vp, _vp, _i, _sz, _vp],
@@ -72,32 +73,36 @@ _SIGNATURES = {
                              _i, _i, _i, _i, _vp],
     "cima_rope_append": [_vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _f, _f, _f, _i, _vp],
     "cima_attention_plain": [_vp, _i, _i, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i,
-                             _f, _i, _i, _i, _f, _i, _i, _vp, _i, _vp],
-    "cima_attention_decode": [_vp, _i, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _f, _i, _i, _vp, _i, _vp],
-    "cima_attention_prefill": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i, _i, _vp, _i, _vp],
-    "cima_attention_extend": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _f, _i, _i, _vp, _i, _vp],
+                             _f, _i, _i, _i, _f, _i, _i, _vp, _i, _vp, _vp],
+    "cima_attention_decode": [_vp, _i, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _f, _i, _i, _vp, _i, _vp, _vp],
+    "cima_attention_prefill": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _f, _i, _i, _vp, _i, _vp, _vp],
+    "cima_attention_extend": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _f, _i, _i, _vp, _i, _vp, _vp],
     "cima_attention_extend_tc": [_vp, _i, _vp, _vp, _vp, _vp, ctypes.c_longlong, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i,
-                                 _f, _i, _vp, _i, _f, _vp, _i, _vp],
-    "cima_short_conv": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
+                                 _f, _i, _vp, _i, _f, _vp, _i, _vp, _vp],
+    "cima_row_norm_append": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _vp, _i, _i, _f, _vp, _vp, _i, _i, _i, _vp],
+    "cima_token_side_few": [_vp, _vp, _i, _vp, _i, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _vp],
+    "cima_token_side_apply": [_vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _vp],
+    "cima_gate_heads": [_vp, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _vp],
+    "cima_short_conv": [_vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
     "cima_dyt": [_vp, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "cima_dyt_add": [_vp, _vp, _vp, _vp, _vp, _f, _vp, _vp, _vp, _vp, _i, _i, _i, _vp],
     "cima_embed_bigram": [_vp, _vp, _vp, _i, _vp, _i, _i, _i, _f, _i, ctypes.c_longlong, ctypes.c_longlong, _vp, _vp, _vp, _vp, _vp,
                           _i, _vp],
     "cima_recurrence": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
-    "cima_delta_prepare": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    "cima_delta_prepare": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
     "cima_group_rmsnorm_gate": [_vp, _vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _f, _i, _vp, _vp, _f, _vp],
     "cima_rms_mean": [_vp, _vp, _i, _vp, _i, _i, _f, _i, _vp],
     "cima_moe_route": [_vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp],
     "cima_moe_sort": [_vp, _i, _i, _vp, _vp, _vp, _vp],
-    "cima_moe_gemm": [_vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
+    "cima_moe_gemm": [_vp, _i, _i, _vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp],
     "cima_moe_combine": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp, _vp, _i, _vp, _i, _vp, _i, _vp],
     "cima_moe_sort_tiles": [_vp, _i, _i, _i, _i, _vp, _vp, _vp],
-    "cima_moe_gather_rows": [_vp, _vp, _vp, _i, _i, _i, _vp],
-    "cima_moe_few": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp],
+    "cima_moe_gather_rows": [_vp, _vp, _vp, _i, _i, _i, _vp, _vp],
+    "cima_moe_few": [_vp, _i, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp],
     "cima_gemm_tcgen05_pair_grouped": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp, _vp],
     "cima_depth_average": [_vp, ctypes.c_longlong, _vp, _i, _vp, _vp, _vp, _i, _i, _i, _f, _vp, _i, _vp, _vp, _vp, _vp],
     "cima_latent_append": [_vp, _i, _i, _vp, _f, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _i, _i, _vp],
-    "cima_head_linear": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp],
+    "cima_head_linear": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _i, _i, _vp, _i, _vp],
     "cima_latent_prepare": [_vp, _i, _i, _i, _vp, _vp, _i, _vp, _f, _i, _i, _vp, _f, _i, _vp, _vp, _i, _i, _i, _vp, _vp, _vp, _vp,
                             _vp, _i, _i, _i, _vp],
     "cima_rope_rows": [_vp, _i, _i, _i, _i, _vp, _i, _i, _i, _i, _i, _vp, _f, _i, _vp, _i, _vp],
@@ -106,7 +111,7 @@ _SIGNATURES = {
 
     "cima_head_linear_append": [_vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp, _i, _vp, _f, _vp, _vp, _i, _i, _i, _vp, _vp, _vp,
                                 _i, _vp],
-    "cima_attention_prefill_tc": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _f, _vp, _i, _vp],
+    "cima_attention_prefill_tc": [_vp, _i, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _f, _i, _vp, _f, _vp, _i, _vp, _vp],
     "cima_gemm_tcgen05_pair": [_vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _f, _vp, _vp],
     "cima_diff_combine": [_vp, _i, _vp, _i, _vp, _i, _i, _i, _i, _i, _i, _f, _f, _f, _vp],
     "cima_scale_add_group_rmsnorm": [_vp, _vp, _f, _vp, _vp, _i, _i, _i, _i, _f, _vp],
@@ -193,8 +198,8 @@ class Kernels:
     # ------------------------------------------------------------------ elementwise
     def embed(self, ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, scale: float = 1.0,
               ssq: Optional[torch.Tensor] = None, w_next: Optional[torch.Tensor] = None,
-              xw: Optional[torch.Tensor] = None) -> None:
-        """x[t] = scale * table[ids[t]]; ``ssq`` [T, 1] (optional) receives each row's sum of squares, ``xw``
+              xw: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None, row_pos: Optional[torch.Tensor] = None) -> None:
+        """x[t] = scale * table[ids[t]] (+ positions[row_pos[t]], a table of the same dtype); ``ssq`` [T, 1] (optional) receives each row's sum of squares, ``xw``
         [T, H] bf16 (optional) the rows times ``w_next`` (the weight of the norm that follows)."""
         self._need(ids, "ids", torch.int32, 1); self._need(table, "table", None, 2); self._need(x, "x", torch.float32, 2)
         T, (V, H) = ids.numel(), table.shape
@@ -208,9 +213,15 @@ class Kernels:
             self._need(xw, "xw", torch.bfloat16, 2); self._need(w_next, "w_next", torch.float32, 1)
             if tuple(xw.shape) != (T, H) or w_next.numel() != H:
                 raise KernelError(f"embed: xw {tuple(xw.shape)} / w_next {tuple(w_next.shape)} do not fit {(T, H)}")
-        if not self._admit("embed", T * H * (table.element_size() + 4)): return
+        at = (None, None, 0)
+        if positions is not None:
+            self._need(positions, "positions", table.dtype, 2); self._need(row_pos, "row_pos", torch.int32, 1)
+            if positions.shape[1] != H or row_pos.numel() < T:
+                raise KernelError(f"embed: the positions' table {tuple(positions.shape)} does not fit {T} rows of {H}")
+            at = (positions.data_ptr(), row_pos.data_ptr(), positions.shape[0])
+        if not self._admit("embed", T * H * ((2 if positions is not None else 1) * table.element_size() + 4)): return
         self._check(self.lib.cima_embed(ids.data_ptr(), table.data_ptr(), dtype_code(table.dtype), x.data_ptr(),
-                                        T, H, V, scale, _ptr(ssq), _ptr(w_next) if xw is not None else None, _ptr(xw),
+                                        T, H, V, scale, _ptr(ssq), _ptr(w_next) if xw is not None else None, _ptr(xw), *at,
                                         self._stream()), "embed")
 
     def rmsnorm(self, x: torch.Tensor, w: torch.Tensor, eps: float, out: torch.Tensor) -> None:
@@ -465,9 +476,10 @@ class Kernels:
 
     def attention_plain(self, qkv: torch.Tensor, kv, row_pos, row_seq, seq_slot, seq_first_row, out: torch.Tensor,
                         n_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int,
-                        from_cache: bool, sink: float = 0.0, keep_first: int = 0, v_group: int = 1, head_sink=None, gate_col: int = 0) -> None:
+                        from_cache: bool, sink: float = 0.0, keep_first: int = 0, v_group: int = 1, head_sink=None, gate_col: int = 0,
+                        slopes=None) -> None:
         self._need(qkv, "qkv", None, 2); self._need(out, "out", qkv.dtype, 2)
-        self._need_head_sink(head_sink, n_heads)
+        self._need_head_sink(head_sink, n_heads, slopes)
         T = qkv.shape[0]
         if tuple(out.shape) != (T, n_heads * head_dim):
             raise KernelError(f"attention: out is {tuple(out.shape)}, expected {(T, n_heads * head_dim)}")
@@ -485,9 +497,13 @@ class Kernels:
                                                   seq_first_row.data_ptr(), out.data_ptr(), out.shape[1], T,
                                                   n_heads, n_kv_heads, head_dim, scale, window,
                                                   1 if from_cache else 0, planes, sink, keep_first, v_group, _ptr(head_sink),
-                                                  gate_col, self._stream()), "attention_plain")
+                                                  gate_col, _ptr(slopes), self._stream()), "attention_plain")
 
-    def _need_head_sink(self, head_sink, n_heads: int) -> None:
+    def _need_head_sink(self, head_sink, n_heads: int, slopes=None) -> None:
+        if slopes is not None:
+            self._need(slopes, "slopes", torch.float32, 1)
+            if slopes.numel() != n_heads:
+                raise KernelError(f"attention: {slopes.numel()} distance slopes, expected one for each of {n_heads} heads")
         if head_sink is not None:
             self._need(head_sink, "head_sink", torch.float32, 1)
             if head_sink.numel() != n_heads:
@@ -523,7 +539,7 @@ class Kernels:
 
     def attention(self, qkv: torch.Tensor, kv, batch, out: torch.Tensor, n_heads: int, n_kv_heads: int,
                   head_dim: int, scale: float, window: int, from_cache: bool, after_append: bool = False,
-                  sink: float = 0.0, keep_first: int = 0, v_group: int = 1, head_sink=None, gate_col: int = 0) -> None:
+                  sink: float = 0.0, keep_first: int = 0, v_group: int = 1, head_sink=None, gate_col: int = 0, slopes=None) -> None:
         """Attention of a step's rows: over the step's own keys (a prompt from position 0) or over the
         cache.  Chooses the kernel; every choice computes the same function.  ``after_append``: the kernel
         launched just before wrote nothing but ``qkv`` and the newest position of each sequence in the cache.
@@ -532,62 +548,63 @@ class Kernels:
         many neighbouring key heads share one value head (a step's rows and the pages' value plane hold
         n_kv_heads / v_group value heads).  ``head_sink`` (float32 [n_heads], instead of ``sink``): head h's denominator
         also holds exp(head_sink[h]), an entry that is not scaled and carries no value.  ``gate_col`` > 0: a row of ``qkv`` holds
-        one gate value for each value of its result from that column on, and the result leaves times their sigmoid."""
+        one gate value for each value of its result from that column on, and the result leaves times their sigmoid.  ``slopes`` (float32 [n_heads]): slopes[h] * (i - j) is taken
+        off the scaled score of the query at position i with the key at j."""
         general = keep_first > 0 or v_group > 1        # the tcgen05 kernels take neither
         if (from_cache and qkv.dtype is torch.bfloat16 and kv.page_size == 64 and head_dim % 16 == 0
                 and head_dim <= 128 and batch.n_rows == batch.n_seqs):
             return self.attention_decode(qkv, kv, batch.seq_slot, batch.seq_len, out, n_heads, n_kv_heads, head_dim,
                                          scale, window, batch.max_len, early=after_append, sink=sink,
-                                         keep_first=keep_first, v_group=v_group, head_sink=head_sink, gate_col=gate_col)
+                                         keep_first=keep_first, v_group=v_group, head_sink=head_sink, gate_col=gate_col, slopes=slopes)
         many = (not general and qkv.dtype is torch.bfloat16 and head_dim in (64, 128) and qkv.shape[1] % 8 == 0
                 and getattr(batch, "n_q_tiles_tc", 0) > 0 and getattr(batch, "max_rows", 0) >= TC_ATTENTION_MIN_LEN)
         if from_cache and many and kv.page_size == 64 and kv.storage.numel() // head_dim < 2 ** 31:
             return self.attention_prefill_tc(qkv, batch, out, n_heads, n_kv_heads, head_dim, scale, window, kv=kv, sink=sink,
-                                             head_sink=head_sink, gate_col=gate_col)
+                                             head_sink=head_sink, gate_col=gate_col, slopes=slopes)
         if (from_cache and qkv.dtype is torch.bfloat16 and kv.page_size == 64 and head_dim % 16 == 0
                 and head_dim <= 128 and qkv.shape[1] % 8 == 0 and getattr(batch, "n_q_tiles", 0) > 0):
             return self.attention_extend(qkv, kv, batch, out, n_heads, n_kv_heads, head_dim, scale, window, sink=sink,
-                                         keep_first=keep_first, v_group=v_group, head_sink=head_sink, gate_col=gate_col)
+                                         keep_first=keep_first, v_group=v_group, head_sink=head_sink, gate_col=gate_col, slopes=slopes)
         if not from_cache and many:
             return self.attention_prefill_tc(qkv, batch, out, n_heads, n_kv_heads, head_dim, scale, window, sink=sink,
-                                             head_sink=head_sink, gate_col=gate_col)
+                                             head_sink=head_sink, gate_col=gate_col, slopes=slopes)
         if (not from_cache and qkv.dtype is torch.bfloat16 and head_dim % 16 == 0 and head_dim <= 128
                 and qkv.shape[1] % 8 == 0 and getattr(batch, "n_q_tiles", 0) > 0):
             return self.attention_prefill(qkv, batch.q_tile_seq, batch.q_tile_row0, batch.seq_first_row, out,
                                           n_heads, n_kv_heads, head_dim, scale, window, sink=sink,
-                                          keep_first=keep_first, v_group=v_group, head_sink=head_sink, gate_col=gate_col)
+                                          keep_first=keep_first, v_group=v_group, head_sink=head_sink, gate_col=gate_col, slopes=slopes)
         self.attention_plain(qkv, kv, batch.row_pos, batch.row_seq, batch.seq_slot, batch.seq_first_row, out,
                              n_heads, n_kv_heads, head_dim, scale, window, from_cache, sink=sink, keep_first=keep_first,
-                             v_group=v_group, head_sink=head_sink, gate_col=gate_col)
+                             v_group=v_group, head_sink=head_sink, gate_col=gate_col, slopes=slopes)
 
     def attention_prefill(self, qkv: torch.Tensor, tile_seq, tile_row0, seq_first_row, out: torch.Tensor,
                           n_heads: int, n_kv_heads: int, head_dim: int, scale: float, window: int, sink: float = 0.0,
-                          keep_first: int = 0, v_group: int = 1, head_sink=None, gate_col: int = 0) -> None:
+                          keep_first: int = 0, v_group: int = 1, head_sink=None, gate_col: int = 0, slopes=None) -> None:
         """Flash attention of ragged prompts that start at position 0 (bf16, head_dim <= 128);
         ``tile_seq``/``tile_row0`` list the blocks of 64 query rows."""
         self._need(qkv, "qkv", torch.bfloat16, 2); self._need(out, "out", torch.bfloat16, 2)
         for n, t in (("tile_seq", tile_seq), ("tile_row0", tile_row0), ("seq_first_row", seq_first_row)):
             self._need(t, n, torch.int32, 1)
         T = qkv.shape[0]
-        self._need_head_sink(head_sink, n_heads)
+        self._need_head_sink(head_sink, n_heads, slopes)
         if tuple(out.shape) != (T, n_heads * head_dim) or tile_seq.numel() != tile_row0.numel():
             raise KernelError(f"attention_prefill: out {tuple(out.shape)} or the block list do not fit")
         if not self._admit("attention_prefill", *self._attention_work(qkv, n_heads, n_kv_heads, head_dim)): return
         self._check(self.lib.cima_attention_prefill(qkv.data_ptr(), qkv.shape[1], tile_seq.data_ptr(), tile_row0.data_ptr(),
                                                     seq_first_row.data_ptr(), out.data_ptr(), out.shape[1], T,
                                                     tile_seq.numel(), n_heads, n_kv_heads, head_dim, scale, window, sink,
-                                                    keep_first, v_group, _ptr(head_sink), gate_col, self._stream()), "attention_prefill")
+                                                    keep_first, v_group, _ptr(head_sink), gate_col, _ptr(slopes), self._stream()), "attention_prefill")
 
     def attention_extend(self, qkv: torch.Tensor, kv, batch, out: torch.Tensor, n_heads: int, n_kv_heads: int,
                          head_dim: int, scale: float, window: int, sink: float = 0.0, keep_first: int = 0,
-                         v_group: int = 1, head_sink=None, gate_col: int = 0) -> None:
+                         v_group: int = 1, head_sink=None, gate_col: int = 0, slopes=None) -> None:
         """Flash attention of sequences that bring several rows to a cache that already holds keys (bf16, pages of
         64, head_dim <= 128): the rows of sequence s stand at positions seq_len[s] - rows .. seq_len[s] - 1, and all
         keys, the step's own included, are read from the layer's pages.  ``batch`` brings the blocks of 64 rows."""
         self._need(qkv, "qkv", torch.bfloat16, 2); self._need(out, "out", torch.bfloat16, 2)
         self._need(kv.storage, "cache", torch.bfloat16, 5); self._need(kv.block_table, "block_table", torch.int32, 2)
         T = qkv.shape[0]
-        self._need_head_sink(head_sink, n_heads)
+        self._need_head_sink(head_sink, n_heads, slopes)
         if tuple(out.shape) != (T, n_heads * head_dim) or batch.q_tile_seq.numel() != batch.q_tile_row0.numel():
             raise KernelError(f"attention_extend: out {tuple(out.shape)} or the block list do not fit")
         if not self._admit("attention_extend", *self._attention_work(qkv, n_heads, n_kv_heads, head_dim, kv.planes)): return
@@ -596,11 +613,11 @@ class Kernels:
             batch.seq_first_row.data_ptr(), kv.storage.data_ptr(), kv.block_table.data_ptr(), kv.block_table.shape[1],
             kv.ring_pages, kv.page_size, batch.seq_slot.data_ptr(), batch.seq_len.data_ptr(), out.data_ptr(), out.shape[1],
             T, batch.q_tile_seq.numel(), n_heads, n_kv_heads, head_dim, scale, window, kv.planes, sink, keep_first, v_group,
-            _ptr(head_sink), gate_col, self._stream()), "attention_extend")
+            _ptr(head_sink), gate_col, _ptr(slopes), self._stream()), "attention_extend")
 
     def attention_prefill_tc(self, qkv: torch.Tensor, batch, out: torch.Tensor, n_heads: int, n_kv_heads: int,
                              head_dim: int, scale: float, window: int, kv=None, sink: float = 0.0, head_sink=None,
-                             gate_col: int = 0) -> None:
+                             gate_col: int = 0, slopes=None) -> None:
         """Flash attention of ragged prompts on the tcgen05 tensor cores (bf16, head_dim 64 or 128): blocks of 128
         query rows, both products with their results in tensor memory.  ``batch`` brings the blocks
         (``q_tile_tc_*``).  Without ``kv`` the sequences start at position 0 and the keys are the step's own rows;
@@ -608,7 +625,7 @@ class Kernels:
         seq_len[s] - rows .. seq_len[s] - 1 and all keys come from the pages."""
         self._need(qkv, "qkv", torch.bfloat16, 2); self._need(out, "out", torch.bfloat16, 2)
         T = qkv.shape[0]
-        self._need_head_sink(head_sink, n_heads)
+        self._need_head_sink(head_sink, n_heads, slopes)
         if tuple(out.shape) != (T, n_heads * head_dim) or batch.n_q_tiles_tc <= 0:
             raise KernelError(f"attention_prefill_tc: out {tuple(out.shape)} or the block list do not fit")
         if self._error_flag is None:
@@ -621,18 +638,18 @@ class Kernels:
                 batch.seq_first_row.data_ptr(), kv.storage.data_ptr(), kv.storage.shape[0], kv.block_table.data_ptr(),
                 kv.block_table.shape[1], kv.ring_pages, kv.page_size, batch.seq_slot.data_ptr(), batch.seq_len.data_ptr(),
                 out.data_ptr(), out.shape[1], T, batch.n_q_tiles_tc, n_heads, n_kv_heads, head_dim, scale, window,
-                self._error_flag.data_ptr(), kv.planes, sink, _ptr(head_sink), gate_col, self._stream()), "attention_extend_tc")
+                self._error_flag.data_ptr(), kv.planes, sink, _ptr(head_sink), gate_col, _ptr(slopes), self._stream()), "attention_extend_tc")
             return
         self._check(self.lib.cima_attention_prefill_tc(
             qkv.data_ptr(), qkv.shape[1], batch.q_tile_tc_seq.data_ptr(), batch.q_tile_tc_row0.data_ptr(),
             batch.seq_first_row.data_ptr(), out.data_ptr(),
             out.shape[1], T, batch.n_q_tiles_tc, n_heads, n_kv_heads, head_dim, scale, window,
-            self._error_flag.data_ptr(), sink, _ptr(head_sink), gate_col, self._stream()), "attention_prefill_tc")
+            self._error_flag.data_ptr(), sink, _ptr(head_sink), gate_col, _ptr(slopes), self._stream()), "attention_prefill_tc")
 
     def attention_decode(self, qkv: torch.Tensor, kv, seq_slot, seq_len, out: torch.Tensor, n_heads: int,
                          n_kv_heads: int, head_dim: int, scale: float, window: int, max_len: int = 0,
                          n_splits: Optional[int] = None, early: bool = False, sink: float = 0.0, keep_first: int = 0,
-                         v_group: int = 1, head_sink=None, gate_col: int = 0) -> None:
+                         v_group: int = 1, head_sink=None, gate_col: int = 0, slopes=None) -> None:
         """One query per sequence over the paged cache (bf16, pages of 64, head_dim <= 128), keys split
         over ``n_splits`` blocks per (sequence, kv head).  ``max_len`` (0 = unknown) only bounds the
         number of splits chosen here.  ``early``: the kernel launched just before this one wrote neither
@@ -641,7 +658,7 @@ class Kernels:
         self._need(qkv, "qkv", torch.bfloat16, 2); self._need(out, "out", torch.bfloat16, 2)
         self._need(kv.storage, "cache", torch.bfloat16, 5); self._need(kv.block_table, "block_table", torch.int32, 2)
         B = qkv.shape[0]
-        self._need_head_sink(head_sink, n_heads)
+        self._need_head_sink(head_sink, n_heads, slopes)
         if tuple(out.shape) != (B, n_heads * head_dim) or seq_slot.numel() < B or seq_len.numel() < B:
             raise KernelError(f"attention_decode: out {tuple(out.shape)} / sequences do not fit {B} rows")
         if n_splits is None:
@@ -673,7 +690,7 @@ class Kernels:
             qkv.data_ptr(), qkv.shape[1], kv.storage.data_ptr(), kv.block_table.data_ptr(), kv.block_table.shape[1],
             kv.ring_pages, kv.page_size, seq_slot.data_ptr(), seq_len.data_ptr(), _ptr(part_o), _ptr(part_ml),
             out.data_ptr(), out.shape[1], B, n_heads, n_kv_heads, head_dim, scale, window, n_splits, int(early),
-            kv.planes, sink, keep_first, v_group, _ptr(head_sink), gate_col, self._stream()), "attention_decode")
+            kv.planes, sink, keep_first, v_group, _ptr(head_sink), gate_col, _ptr(slopes), self._stream()), "attention_decode")
         if n_splits > 1:
             self.launches += 1
 
@@ -695,8 +712,10 @@ class Kernels:
         step; what lies before the step's rows comes from ``state`` [slots, taps - 1, C] (the sequences' last
         inputs), which is brought up to date.  ``w`` [taps, C] float32 (tap by tap); h, out, state of one dtype.
         ``add_input`` False leaves h[t] out of the sum (a plain convolution); ``act`` >= 0 applies that entry of
-        ``ACTIVATIONS`` to the sum."""
-        self._need(h, "h", None, 2); self._need(w, "w", torch.float32, 2); self._need(out, "out", h.dtype, 2)
+        ``ACTIVATIONS`` to the sum.  h may be a column slice of wider rows."""
+        if h.dim() != 2 or h.stride(1) != 1 or not h.is_cuda:
+            raise KernelError(f"short_conv: h {tuple(h.shape)} must be GPU rows with unit column stride")
+        self._need(w, "w", torch.float32, 2); self._need(out, "out", h.dtype, 2)
         T, C = h.shape
         taps = w.shape[0]
         if w.shape[1] != C or out.shape != h.shape:
@@ -707,7 +726,7 @@ class Kernels:
                 raise KernelError(f"short_conv: state is {tuple(state.shape)}, expected [slots, {taps - 1}, {C}]")
         one_row = batch.n_rows == batch.n_seqs
         if not self._admit("short_conv", 2 * T * C * h.element_size()): return
-        self._check(self.lib.cima_short_conv(h.data_ptr(), dtype_code(h.dtype), w.data_ptr(), _ptr(state if taps > 1 else None),
+        self._check(self.lib.cima_short_conv(h.data_ptr(), dtype_code(h.dtype), h.stride(0), w.data_ptr(), _ptr(state if taps > 1 else None),
                                              batch.row_seq.data_ptr(), batch.seq_slot.data_ptr(), batch.seq_first_row.data_ptr(),
                                              out.data_ptr(), T, batch.n_seqs, C, taps, int(one_row), rows_per_thread,
                                              int(add_input), act, self._stream()), "short_conv")
@@ -764,15 +783,16 @@ class Kernels:
     FUSED_APPEND_ROWS = 8       # a step of at most this many rows appends its latents in the launch of its first head product
 
     def head_linear(self, a: torch.Tensor, w: torch.Tensor, out: torch.Tensor, append=None, a_head: Optional[int] = None,
-                    out_head: Optional[int] = None) -> None:
+                    out_head: Optional[int] = None, gate=None) -> None:
         """out[t, h, :] = a[t, h, :] @ w[h].T for every head: a [T, heads * K] (rows may be slices of a wider
         matrix), w [heads, N, K], out [T, heads * N]; one dtype.  ``append = (raw, g, eps, kv, batch)``: the arguments
         of ``latent_append`` for the same rows, done by the same launch (a decode step's few rows) or, for more rows,
         by a launch of its own first.  ``a_head`` / ``out_head``: values from one head's start to the next in a row of
         ``a`` / ``out`` where a head there is wider than K / N (the product reads a head's first K values and writes its
-        first N; what lies behind them is left alone)."""
-        if a_head is not None or out_head is not None:
-            return self._head_linear_strided(a, w, out, int(a_head or w.shape[2]), int(out_head or w.shape[1]))
+        first N; what lies behind them is left alone).  ``gate = (rows, col)``: the output leaves times
+        sigmoid(rows[t, col + h * N + n]), rows [T, >= col + heads * N] of a's dtype."""
+        if a_head is not None or out_head is not None or gate is not None:
+            return self._head_linear_strided(a, w, out, int(a_head or w.shape[2]), int(out_head or w.shape[1]), gate)
         if append is not None and (a.shape[0] > self.FUSED_APPEND_ROWS or a.shape[0] * (w.shape[2] + 3) * 4 > 48 * 1024):
             self.latent_append(*append)
             append = None
@@ -802,9 +822,9 @@ class Kernels:
                 batch.seq_slot.data_ptr(), R, self._stream()), "head_linear_append")
             return
         self._check(self.lib.cima_head_linear(a.data_ptr(), w.data_ptr(), out.data_ptr(), dtype_code(a.dtype), T, heads, N, K,
-                                              a.stride(0), out.stride(0), K, N, self._stream()), "head_linear")
+                                              a.stride(0), out.stride(0), K, N, None, 0, self._stream()), "head_linear")
 
-    def _head_linear_strided(self, a, w, out, a_head: int, out_head: int) -> None:
+    def _head_linear_strided(self, a, w, out, a_head: int, out_head: int, gate=None) -> None:
         self._need(w, "w", a.dtype, 3)
         heads, N, K = w.shape
         T = a.shape[0]
@@ -812,16 +832,27 @@ class Kernels:
                 or a_head < K or out_head < N or a.shape[1] < (heads - 1) * a_head + K or out.shape[1] < (heads - 1) * out_head + N):
             raise KernelError(f"head_linear: a {tuple(a.shape)} in heads of {a_head}, w {tuple(w.shape)}, out {tuple(out.shape)} in heads "
                               f"of {out_head} do not agree")
-        if not self._admit("head_linear", (w.numel() + T * heads * (K + N)) * a.element_size(), 2.0 * T * heads * N * K): return
+        gp, ldg = None, 0
+        if gate is not None:
+            rows, col = gate
+            if rows.dim() != 2 or rows.stride(1) != 1 or rows.shape[0] != T or rows.dtype is not a.dtype or col < 0 or rows.shape[1] < col + heads * N:
+                raise KernelError(f"head_linear: the gate {tuple(rows.shape)} from column {col} on does not fit {heads} heads of {N}")
+            gp, ldg = rows[:, col:].data_ptr(), rows.stride(0)
+        if not self._admit("head_linear", (w.numel() + T * heads * (K + (2 if gate else 1) * N)) * a.element_size(), 2.0 * T * heads * N * K): return
         if a.dtype is torch.bfloat16 and T > 8:
             # many bfloat16 rows: the library's batched product over the heads' columns
             self.library_launches += 1
             av = torch.as_strided(a, (heads, T, K), (a_head, a.stride(0), 1))
+            if gate is not None:
+                made = torch.bmm(av, w.transpose(1, 2))
+                self._check(self.lib.cima_gate_heads(made.data_ptr(), gp, ldg, out.data_ptr(), out.stride(0), out_head, dtype_code(a.dtype), T,
+                                                     heads, N, self._stream()), "gate_heads")
+                return
             ov = torch.as_strided(out, (heads, T, N), (out_head, out.stride(0), 1))
             ov.copy_(torch.bmm(av, w.transpose(1, 2)))
             return
         self._check(self.lib.cima_head_linear(a.data_ptr(), w.data_ptr(), out.data_ptr(), dtype_code(a.dtype), T, heads, N, K,
-                                              a.stride(0), out.stride(0), a_head, out_head, self._stream()), "head_linear")
+                                              a.stride(0), out.stride(0), a_head, out_head, gp, ldg, self._stream()), "head_linear")
 
     def latent_prepare(self, ql: torch.Tensor, first: int, q_norm, cq, c_norm: torch.Tensor, eps: float, rank: int, rot: int,
                        inv_freq, amplitude: float, interleaved: bool, kv, batch, step_rows=None) -> None:
@@ -982,7 +1013,7 @@ class Kernels:
                    beta: Optional[torch.Tensor] = None, decay: Optional[torch.Tensor] = None, gate=None) -> None:
         """A linear recurrence over the step's rows, sequence by sequence, with the state S [slots, heads, dim, vdim]
         (float32) carried on.  With ``decay`` [heads]: S <- d S + k v^T, o = S^T q, and q, k, v (one dtype) pass SiLU.
-        With ``g`` [T, heads * dim] and ``beta`` [T, heads]: the gated delta rule on prepared float32 q and k
+        With ``g`` [T, heads * dim] (a decay a key channel) or [T, heads] (one a head) and ``beta`` [T, heads]: the gated delta rule on prepared float32 q and k
         ([T, kv_heads * dim]).  With ``gate`` = (bias, lower), both float32 [heads * dim]: the gate rule, S <- diag(f) S +
         (1 - f) v^T with f = lower + (1 - lower) * sigmoid(k + bias) made from the projection that ``k`` holds, o = S^T silu(q),
         v as it is (q, k, v of one dtype, kv_heads = heads).  q, k, v may be column slices of wider matrices; out
@@ -1001,20 +1032,22 @@ class Kernels:
                               f"out {tuple(out.shape)} do not agree with {heads} heads on {kv_heads} of {dim} x {vdim}")
         if delta:
             self._need(g, "g", torch.float32, 2); self._need(beta, "beta", torch.float32, 2)
-            if q.dtype is not torch.float32 or tuple(g.shape) != (T, heads * dim) or tuple(beta.shape) != (T, heads):
-                raise KernelError("recurrence: the delta rule takes float32 q and k, g [T, heads * dim] and beta [T, heads]")
+            if q.dtype is not torch.float32 or tuple(g.shape) not in ((T, heads * dim), (T, heads)) or tuple(beta.shape) != (T, heads):
+                raise KernelError("recurrence: the delta rule takes float32 q and k, g [T, heads * dim] or [T, heads], and beta [T, heads]")
+            per_head = g.shape[1] == heads and dim > 1
         else:
             self._need(decay, "decay", torch.float32, 1)
             if decay.numel() != heads or q.dtype is not v.dtype:
                 raise KernelError("recurrence: the decay rule takes q, k, v of one dtype and one decay a head")
-        if not self._admit("recurrence[delta]" if delta else "recurrence[decay]",
+        mode = 0 if not delta else (3 if per_head else 1)
+        if not self._admit(("recurrence[delta, a decay a head]" if mode == 3 else "recurrence[delta]") if delta else "recurrence[decay]",
                            batch.n_seqs * heads * dim * vdim * 8 + T * (2 * kv_heads * dim * q.element_size() + heads * vdim * (4 + v.element_size())
-                                                                        + (heads * dim * 4 if delta else 0)),
+                                                                        + (g.shape[1] * 4 if delta else 0)),
                            (8.0 if delta else 5.0) * T * heads * dim * vdim): return
         self._check(self.lib.cima_recurrence(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0),
                                              dtype_code(v.dtype), _ptr(g), _ptr(beta), _ptr(decay), state.data_ptr(),
                                              batch.seq_slot.data_ptr(), batch.seq_first_row.data_ptr(), out.data_ptr(), T,
-                                             batch.n_seqs, heads, kv_heads, dim, vdim, int(delta), self._stream()), "recurrence")
+                                             batch.n_seqs, heads, kv_heads, dim, vdim, mode, self._stream()), "recurrence")
 
     def _recurrence_gate(self, q, k, v, state, batch, out, heads, kv_heads, dim, vdim, bias, lower) -> None:
         self._need(state, "state", torch.float32, 4); self._need(out, "out", torch.float32, 2)
@@ -1039,26 +1072,30 @@ class Kernels:
                       qn: torch.Tensor, kn: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, heads: int, kv_heads: int,
                       dim: int) -> None:
         """What the gated delta rule needs of a token besides v, in float32: q and k as unit vectors per head (q also
-        times dim^-1/2), g = exp(-exp(A_log[h]) * softplus(a + dt_bias)) per head and key channel, beta = sigmoid(b).
+        times dim^-1/2), g = exp(-exp(A_log[h]) * softplus(a + dt_bias)) per head and key channel (or, with a [T, heads] and
+        as many biases, per head), beta = sigmoid(b).
         ``qk`` [T, >= 2 * kv_heads * dim] holds q's heads and then k's; qk, a, b of one dtype, rows may be slices."""
         T = qk.shape[0]
         for n, t in (("qk", qk), ("a", a), ("b", b)):
             if t.dim() != 2 or t.stride(1) != 1 or t.shape[0] != T or t.dtype is not qk.dtype or not t.is_cuda:
                 raise KernelError(f"delta_prepare: {n} {tuple(t.shape)} {t.dtype} must be GPU rows of one dtype with unit column stride")
-        for n, t, shape in (("qn", qn, (T, kv_heads * dim)), ("kn", kn, (T, kv_heads * dim)), ("g", g, (T, heads * dim)),
+        gdim = 1 if a.shape[1] == heads else dim                  # decays a head
+        for n, t, shape in (("qn", qn, (T, kv_heads * dim)), ("kn", kn, (T, kv_heads * dim)), ("g", g, (T, heads * gdim)),
                             ("beta", beta, (T, heads))):
             self._need(t, n, torch.float32, 2)
             if tuple(t.shape) != shape:
                 raise KernelError(f"delta_prepare: {n} is {tuple(t.shape)}, expected {shape}")
         self._need(A_log, "A_log", torch.float32, 1); self._need(dt_bias, "dt_bias", torch.float32, 1)
-        if (qk.shape[1] < 2 * kv_heads * dim or a.shape[1] != heads * dim or b.shape[1] != heads or A_log.numel() != heads
-                or dt_bias.numel() != heads * dim):
+        if (qk.shape[1] < 2 * kv_heads * dim or a.shape[1] != heads * gdim or b.shape[1] != heads or A_log.numel() != heads
+                or dt_bias.numel() != heads * gdim):
             raise KernelError("delta_prepare: the inputs' widths do not agree with the heads and the key size")
-        if not self._admit("delta_prepare", T * (2 * kv_heads * dim + heads * dim + heads) * (4 + qk.element_size())): return
-        self._check(self.lib.cima_delta_prepare(qk.data_ptr(), qk.stride(0), a.data_ptr(), a.stride(0), b.data_ptr(), b.stride(0),
-                                                dtype_code(qk.dtype), A_log.data_ptr(), dt_bias.data_ptr(), qn.data_ptr(),
-                                                kn.data_ptr(), g.data_ptr(), beta.data_ptr(), T, heads, kv_heads, dim,
-                                                self._stream()), "delta_prepare")
+        if not self._admit("delta_prepare", T * (2 * kv_heads * dim + heads * gdim + heads) * (4 + qk.element_size())): return
+        for r0 in range(0, T, 65535):                             # a row a block of grid.y
+            r1 = min(T, r0 + 65535)
+            self._check(self.lib.cima_delta_prepare(qk[r0:r1].data_ptr(), qk.stride(0), a[r0:r1].data_ptr(), a.stride(0), b[r0:r1].data_ptr(),
+                                                    b.stride(0), dtype_code(qk.dtype), A_log.data_ptr(), dt_bias.data_ptr(), qn[r0:r1].data_ptr(),
+                                                    kn[r0:r1].data_ptr(), g[r0:r1].data_ptr(), beta[r0:r1].data_ptr(), r1 - r0, heads, kv_heads,
+                                                    dim, gdim, self._stream()), "delta_prepare")
 
     def group_rmsnorm_gate(self, o: torch.Tensor, w: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, groups: int,
                            eps: float, silu: bool = False, divisor=None) -> None:
@@ -1179,6 +1216,64 @@ class Kernels:
         self._check(self.lib.cima_branch_norm(x.data_ptr(), y.data_ptr(), w.data_ptr(), _ptr(h), dtype_code(h.dtype) if h is not None else F32,
                                               _ptr(w2), T, W, eps, eps2, self._stream()), "branch_norm")
 
+    # ------------------------------------------------------------------ a token's own input, the norm over whole projections
+    SIDE_FEW_ROWS = 8           # up to this many rows the gated middle of a token's input is one launch
+
+    def _need_side(self, table, tokens, col: int, rows: int, dim: int, dtype) -> None:
+        self._need(table, "table", dtype, 2); self._need(tokens, "tokens", torch.int32, 1)
+        if tokens.numel() < rows or col < 0 or table.shape[1] < col + dim:
+            raise KernelError(f"token_side: table {tuple(table.shape)} / tokens {tuple(tokens.shape)} do not fit {rows} rows of {dim} values from column {col} on")
+
+    def token_side_few(self, x: torch.Tensor, w: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, col: int, z: torch.Tensor, act: int) -> None:
+        """z[t, j] = act(x[t] . w[j]) * table[tokens[t], col + j]: x float32 [T, W] with at most ``SIDE_FEW_ROWS`` rows, w [dim, W], z
+        [T, dim] and the table of one dtype."""
+        self._need(x, "x", torch.float32, 2); self._need(w, "w", None, 2); self._need(z, "z", None, 2)
+        (T, W), dim = x.shape, w.shape[0]
+        if w.shape[1] != W or tuple(z.shape) != (T, dim):
+            raise KernelError(f"token_side_few: x {tuple(x.shape)}, w {tuple(w.shape)}, z {tuple(z.shape)} do not agree")
+        self._need_side(table, tokens, col, T, dim, z.dtype)
+        if not self._admit("token_side_few", w.numel() * w.element_size() + T * W * 4 + 2 * z.numel() * z.element_size(), 2.0 * T * W * dim): return
+        self._check(self.lib.cima_token_side_few(x.data_ptr(), w.data_ptr(), dtype_code(w.dtype), table.data_ptr(), table.shape[1], dtype_code(z.dtype),
+                                                 tokens.data_ptr(), int(col), z.data_ptr(), T, dim, W, table.shape[0], int(act), self._stream()), "token_side_few")
+
+    def token_side_apply(self, z: torch.Tensor, table: torch.Tensor, tokens: torch.Tensor, col: int, act: int) -> None:
+        """z[t, j] <- act(z[t, j]) * table[tokens[t], col + j] in place (z and the table of one dtype; float32 inside)."""
+        self._need(z, "z", None, 2)
+        T, dim = z.shape
+        self._need_side(table, tokens, col, T, dim, z.dtype)
+        if not self._admit("token_side_apply", 3 * z.numel() * z.element_size()): return
+        self._check(self.lib.cima_token_side_apply(z.data_ptr(), table.data_ptr(), table.shape[1], dtype_code(z.dtype), tokens.data_ptr(), int(col), T, dim,
+                                                   table.shape[0], int(act), self._stream()), "token_side_apply")
+
+    def row_norm_append(self, qkv: torch.Tensor, norm, batch, kv, n_heads: int, n_kv_heads: int, head_dim: int, v_dim: int, mix=None) -> None:
+        """A step's rows [q heads | k heads | v heads] of ``head_dim`` values, in place: all of a row's q (and all of its k) divided by
+        their root mean square and multiplied by a weight; k and v to the rows' places in the layer's pages.  ``norm = (wq, wk, dim,
+        eps)``: the weights float32 [n_heads * head_dim] and [n_kv_heads * head_dim]; a head's values from ``dim`` on are padding (zero,
+        not counted).  ``mix = (l, first, first_head)``: v <- (1 - l) v + l first on a head's first ``v_dim`` values, l one float32 on the
+        device, first [T, >= n_kv_heads * first_head] the values to mix in (rows may be slices)."""
+        wq, wk, dim, eps = norm
+        self._need(qkv, "qkv", None, 2); self._need(wq, "wq", torch.float32, 1); self._need(wk, "wk", torch.float32, 1)
+        T, ld = qkv.shape
+        self._need(kv.storage, "cache", qkv.dtype, 5); self._need(kv.block_table, "block_table", torch.int32, 2)
+        if (wq.numel() != n_heads * head_dim or wk.numel() != n_kv_heads * head_dim or not (0 < dim <= head_dim)
+                or tuple(kv.storage.shape[1:]) != (2, n_kv_heads, kv.page_size, head_dim) or batch.row_pos.numel() < T):
+            raise KernelError(f"row_norm_append: weights {tuple(wq.shape)} / {tuple(wk.shape)} or pages {tuple(kv.storage.shape)} do not fit {n_heads} + 2 x "
+                              f"{n_kv_heads} heads of {head_dim}")
+        more = (None, None, 0, 0)
+        if mix is not None:
+            lam, first, first_head = mix
+            self._need(lam, "lambda", torch.float32)
+            if (first.dim() != 2 or first.stride(1) != 1 or first.dtype is not qkv.dtype or first.shape[0] != T or not first.is_cuda
+                    or first.shape[1] < n_kv_heads * first_head):
+                raise KernelError(f"row_norm_append: the values to mix in are {tuple(first.shape)} {first.dtype}, expected {T} rows of {n_kv_heads} heads of {first_head}")
+            more = (lam.data_ptr(), first.data_ptr(), first.stride(0), int(first_head))
+        width = (n_heads + 2 * n_kv_heads) * head_dim
+        if not self._admit("row_norm_append", 2 * T * width * qkv.element_size()): return
+        self._check(self.lib.cima_row_norm_append(
+            qkv.data_ptr(), dtype_code(qkv.dtype), ld, batch.row_pos.data_ptr(), batch.row_seq.data_ptr(), batch.seq_slot.data_ptr(), batch.seq_len.data_ptr(),
+            kv.storage.data_ptr(), kv.block_table.data_ptr(), kv.block_table.shape[1], kv.ring_pages, kv.page_size, T, n_heads, n_kv_heads, head_dim,
+            wq.data_ptr(), wk.data_ptr(), n_heads * dim, n_kv_heads * dim, float(eps), *more, int(v_dim), self._stream()), "row_norm_append")
+
     # ------------------------------------------------------------------ matrix memories
     MEMORY_SEGMENT = 192        # tokens of a segment of a long step's recurrence
 
@@ -1297,7 +1392,7 @@ class Kernels:
 
     def moe_experts(self, h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, idx: torch.Tensor, wgt: torch.Tensor,
                     x: torch.Tensor, act: int = 0, assign: bool = False, ordered: Optional[torch.Tensor] = None,
-                    limit: float = 0.0, shared=None, identity: bool = False) -> None:
+                    limit: float = 0.0, shared=None, identity: bool = False, gated: bool = True, weigh_input: bool = False) -> None:
         """x[t] += (with ``assign``: =) sum_j wgt[t, j] * W_down[e] (act(W_gate[e] h[t]) * (W_up[e] h[t])), e = idx[t, j], ascending j.
         gate_up [E, 2 ff, H] (an expert's gate rows, then its up rows), down [E, H, ff]; x float32 [T, H].  Four launches:
         the pairs sorted by expert, the two grouped products over tiles of one expert's pairs, the weighted sum.  The
@@ -1306,7 +1401,8 @@ class Kernels:
         ``limit`` goes with the clamped form of the middle.  ``shared = (rows, gate, col)``: float32 rows [T, H] (a shared
         expert's output) that join the weighted sum in its launch, each row times sigmoid(gate[t, col]) (gate float32
         [T, n]; None: unweighted).  ``identity``: indices from E on are identity experts: their pairs are in no product and
-        contribute wgt[t, j] * h[t]."""
+        contribute wgt[t, j] * h[t].  ``gated`` False: experts W_down act(W_up h) with gate_up [E, ff, H] and an entry of
+        ``UNGATED_ACTIVATIONS``.  ``weigh_input``: an expert reads wgt[t, j] * h[t] and what it gives is summed as it is."""
         tail = (None, None, 0)
         if shared is not None:
             srows, sgate, scol = shared
@@ -1324,7 +1420,11 @@ class Kernels:
         self._need(idx, "idx", torch.int32, 2); self._need(wgt, "wgt", torch.float32, 2); self._need(x, "x", torch.float32, 2)
         T, H = h.shape
         E, ff2, _ = gate_up.shape
-        ff, top = ff2 // 2, idx.shape[1]
+        ff, top = (ff2 // 2 if gated else ff2), idx.shape[1]
+        if (weigh_input or not gated) and (identity or shared is not None):
+            raise KernelError("moe_experts: ungated experts and weights on their inputs go without identity and shared experts")
+        weigh, given = (wgt.data_ptr(), None) if weigh_input else (None, wgt.data_ptr())
+        mode, mats = (0, 2) if gated else (2, 1)               # the first product's form, and the matrices of an expert in it
         if (gate_up.shape[2] != H or tuple(down.shape) != (E, H, ff) or idx.shape[0] != T or wgt.shape != idx.shape
                 or tuple(x.shape) != (T, H)):
             raise KernelError(f"moe_experts: h {tuple(h.shape)}, gate_up {tuple(gate_up.shape)}, down {tuple(down.shape)}, idx "
@@ -1336,7 +1436,7 @@ class Kernels:
             raise KernelError("moe_experts: the rows of h must be contiguous where identity experts return them")
         bf16 = h.dtype is torch.bfloat16 and gate_up.dtype is torch.bfloat16 and H % 8 == 0 and ff % 8 == 0 and h.stride(0) % 8 == 0
         if bf16 and P >= self.MOE_TC_PAIRS:
-            return self._moe_experts_tc(h, gate_up, down, idx, wgt, x, act, assign, limit, tail + own)
+            return self._moe_experts_tc(h, gate_up, down, idx, wgt, x, act, assign, limit, tail + own, gated, weigh_input)
         few = bf16 and P <= self.MOE_FEW_PAIRS
         meta = ordered if ordered is not None else torch.empty(2 * (E + 1) + P, dtype=torch.int32, device=dev)
         offsets, tiles, perm = meta[:E + 1], meta[E + 1:2 * (E + 1)], meta[2 * (E + 1):]
@@ -1348,35 +1448,36 @@ class Kernels:
             self._check(self.lib.cima_moe_sort(idx.data_ptr(), P, E, offsets.data_ptr(), tiles.data_ptr(), perm.data_ptr(),
                                                self._stream()), "moe_sort")
         name = "moe_few" if few else "moe_gemm"
-        if self._admit(f"{name}[gate|up]", touched * 2 * ff * H * wb + P * (H + ff) * h.element_size(), 4.0 * P * ff * H):
+        if self._admit(f"{name}[gate|up]" if gated else f"{name}[up]", touched * mats * ff * H * wb + P * (H + ff) * h.element_size(), 2.0 * mats * P * ff * H):
             if few:
                 self._check(self.lib.cima_moe_few(h.data_ptr(), h.stride(0), gate_up.data_ptr(), z.data_ptr(), offsets.data_ptr(),
-                                                  tiles.data_ptr(), perm.data_ptr(), P, E, top, ff, H, 0, act, limit, self._stream()), "moe_few")
+                                                  tiles.data_ptr(), perm.data_ptr(), P, E, top, ff, H, mode, act, limit, weigh, self._stream()), "moe_few")
             else:
                 self._check(self.lib.cima_moe_gemm(h.data_ptr(), dtype_code(h.dtype), h.stride(0), gate_up.data_ptr(),
                                                    dtype_code(gate_up.dtype), z.data_ptr(), offsets.data_ptr(), tiles.data_ptr(),
-                                                   perm.data_ptr(), P, E, top, ff, H, 0, act, limit, self._stream()), "moe_gemm")
+                                                   perm.data_ptr(), P, E, top, ff, H, mode, act, limit, weigh, self._stream()), "moe_gemm")
         if self._admit(f"{name}[down]", touched * ff * H * wb + P * (ff * h.element_size() + H * 4), 2.0 * P * ff * H):
             if few:
                 self._check(self.lib.cima_moe_few(z.data_ptr(), ff, down.data_ptr(), y.data_ptr(), offsets.data_ptr(),
-                                                  tiles.data_ptr(), perm.data_ptr(), P, E, top, H, ff, 1, 0, 0.0, self._stream()), "moe_few")
+                                                  tiles.data_ptr(), perm.data_ptr(), P, E, top, H, ff, 1, 0, 0.0, None, self._stream()), "moe_few")
             else:
                 self._check(self.lib.cima_moe_gemm(z.data_ptr(), dtype_code(z.dtype), ff, down.data_ptr(), dtype_code(down.dtype),
                                                    y.data_ptr(), offsets.data_ptr(), tiles.data_ptr(), perm.data_ptr(), P, E, top,
-                                                   H, ff, 1, 0, 0.0, self._stream()), "moe_gemm")
+                                                   H, ff, 1, 0, 0.0, None, self._stream()), "moe_gemm")
         if self._admit("moe_combine", P * H * 4 + T * H * 8):
-            self._check(self.lib.cima_moe_combine(y.data_ptr(), wgt.data_ptr(), None, x.data_ptr(), T, top, H, int(assign), *tail, *own,
+            self._check(self.lib.cima_moe_combine(y.data_ptr(), given, None, x.data_ptr(), T, top, H, int(assign), *tail, *own,
                                                   self._stream()), "moe_combine")
 
     MOE_TC_PAIRS = 1024      # from this many (row, choice) pairs on, bfloat16 experts run on the tcgen05 tiles of 256 pairs
     MOE_FEW_PAIRS = 128      # up to this many, a warp computes a feature for the pairs of an expert (a decode step)
 
-    def _moe_experts_tc(self, h, gate_up, down, idx, wgt, x, act, assign=False, limit: float = 0.0, tail=(None, None, 0, None, 0, None, F32)) -> None:
+    def _moe_experts_tc(self, h, gate_up, down, idx, wgt, x, act, assign=False, limit: float = 0.0, tail=(None, None, 0, None, 0, None, F32),
+                        gated: bool = True, weigh_input: bool = False) -> None:
         """Many pairs in bfloat16: every expert's pairs are laid out from a multiple of 256 rows on (the rows of h copied
         there), so that each tile of the tcgen05 product multiplies with one expert's matrix."""
         T, H = h.shape
         E, ff2, _ = gate_up.shape
-        ff, top = ff2 // 2, idx.shape[1]
+        ff, top = (ff2 // 2 if gated else ff2), idx.shape[1]
         P, dev, TILE = T * top, h.device, 256
         n_tiles = -(-P // TILE) + E
         meta = torch.empty(n_tiles + P, dtype=torch.int32, device=dev)
@@ -1391,18 +1492,20 @@ class Kernels:
             self._check(self.lib.cima_moe_sort_tiles(idx.data_ptr(), P, E, TILE, n_tiles, tile_expert.data_ptr(), pos.data_ptr(),
                                                      self._stream()), "moe_sort_tiles")
         if self._admit("moe_gather_rows", 2 * P * H * 2):
-            self._check(self.lib.cima_moe_gather_rows(h.data_ptr(), pos.data_ptr(), hs.data_ptr(), P, top, H * 2, self._stream()),
+            self._check(self.lib.cima_moe_gather_rows(h.data_ptr(), pos.data_ptr(), hs.data_ptr(), P, top, H * 2,
+                                                      wgt.data_ptr() if weigh_input else None, self._stream()),
                         "moe_gather_rows")
-        if self._admit("gemm_tcgen05_pair_grouped[gate|up]", E * 2 * ff * H * 2 + P * (H + ff) * 2, 4.0 * P * ff * H):
-            self._check(self.lib.cima_gemm_tcgen05_pair_grouped(hs.data_ptr(), gate_up.data_ptr(), z.data_ptr(), SK_SWIGLU,
-                                                                n_tiles * TILE, 2 * ff, E, H, ff, ff, act, limit, tile_expert.data_ptr(),
+        if self._admit("gemm_tcgen05_pair_grouped[gate|up]" if gated else "gemm_tcgen05_pair_grouped[up]", E * ff2 * H * 2 + P * (H + ff) * 2,
+                       2.0 * P * ff2 * H):
+            self._check(self.lib.cima_gemm_tcgen05_pair_grouped(hs.data_ptr(), gate_up.data_ptr(), z.data_ptr(), SK_SWIGLU if gated else EPI_ACT,
+                                                                n_tiles * TILE, ff2, E, H, ff, ff if gated else 0, act, limit, tile_expert.data_ptr(),
                                                                 flag.data_ptr(), self._stream()), "gemm_tcgen05_pair_grouped")
         if self._admit("gemm_tcgen05_pair_grouped[down]", E * ff * H * 2 + P * (ff * 2 + H * 4), 2.0 * P * ff * H):
             self._check(self.lib.cima_gemm_tcgen05_pair_grouped(z.data_ptr(), down.data_ptr(), y.data_ptr(), SK_STORE_F32,
                                                                 n_tiles * TILE, H, E, ff, H, 0, 0, 0.0, tile_expert.data_ptr(),
                                                                 flag.data_ptr(), self._stream()), "gemm_tcgen05_pair_grouped")
         if self._admit("moe_combine", P * H * 4 + T * H * 8):
-            self._check(self.lib.cima_moe_combine(y.data_ptr(), wgt.data_ptr(), pos.data_ptr(), x.data_ptr(), T, top, H,
+            self._check(self.lib.cima_moe_combine(y.data_ptr(), None if weigh_input else wgt.data_ptr(), pos.data_ptr(), x.data_ptr(), T, top, H,
                                                   int(assign), *tail, self._stream()), "moe_combine")
 
     # ------------------------------------------------------------------ sampling
