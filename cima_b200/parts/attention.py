@@ -64,6 +64,9 @@ class Attention:
             raise ValueError(f"attention: {spec.n_heads} heads are not a multiple of {spec.n_kv_heads} kv heads")
         if (self.gated or not self.own_kv) and (spec.qkv_bias or spec.out_bias):
             raise ValueError("attention: biases beside an output gate or another layer's keys and values are not implemented")
+        if self.padded and (spec.qkv_bias or spec.out_bias) and spec.position.rotary_dim:
+            raise ValueError(f"attention: head_dim {self.dim} must be a multiple of 16 and equal to the value size {self.vdim} "
+                             f"where biased projections rotate (their heads are padded in the cache only without rotation)")
         if self.v_mix not in (None, "first", "mix"):
             raise ValueError(f"attention: v_mix '{self.v_mix}' is neither 'first' nor 'mix'")
         if self.slopes_host is not None and len(self.slopes_host) != spec.n_heads:

@@ -123,7 +123,7 @@ def plain_attention(h, W, m: dict, eps: float, first_values=None, weights_out=No
     q = (plain_rms(h @ W["q"].T + W["q.b"], eps) * W["q.norm"]).reshape(T, H, dim)
     k = (plain_rms(h @ W["k"].T + W["k.b"], eps) * W["k.norm"]).reshape(T, G, dim)
     own = h @ W["v"].T + W["v.b"]
-    v = (plain_mixed_values(own, first_values, W["vmix"]) if m.get("v_mix") else own).reshape(T, G, vdim)
+    v = (plain_mixed_values(own, first_values, W.get("vmix")) if m.get("v_mix") else own).reshape(T, G, vdim)
     P = torch.zeros((H, T, T), dtype=h.dtype)
     out = torch.zeros((T, H, vdim), dtype=h.dtype)
     for a, slope in enumerate(plain_slopes(H)):
