@@ -93,6 +93,8 @@ def _milder(cfg: dict) -> dict:
     for L in c["layers"]:
         if "scale" in L["mixer"]:
             L["mixer"]["scale"] /= 3.0
+        if (L["mlp"] or {}).get("kind") == "moe":
+            L["mlp"]["router"]["top"] = L["mlp"]["router"]["experts"]
     return c
 
 
@@ -101,8 +103,9 @@ _FOLDERS = {}
 
 def write_folder(d: str, cfg: dict, seed: int = 0, sharp: bool = True) -> str:
     """A model folder of ``cfg``; ``sharp`` False divides the attentions' scales by 3 (queries and keys are normed, so the scale
-    alone decides how sharp a map is): with sharp maps the rounding of a query in bfloat16 decides which key carries a row,
-    so bfloat16 runs are compared on the milder configuration."""
+    alone decides how sharp a map is) and lets every token use all experts: with sharp maps and close calls between experts
+    the rounding of a row in bfloat16 decides which key carries it or which expert it takes, so bfloat16 runs are compared on
+    the milder configuration."""
     from safetensors.torch import load_file, save_file
     cima_b200.write_random_model(d, cfg if sharp else _milder(cfg), seed=seed)
     path = os.path.join(d, "model.safetensors")

@@ -355,8 +355,8 @@ def agrees(got, want, dtype, what=""):
     if dtype == "float32":
         assert e.max() < TOL[dtype], (what, float(e.max()))
     else:
-        # in bfloat16 a row whose router scores two experts nearly alike may take the other one; such rows are rare and the
-        # 32-bit runs compare every row sharply
+        # a head of the delta rule is divided by its own size: where its read-out nearly cancels (q almost orthogonal to all that
+        # is stored) bfloat16's rounding decides its direction; such rows are rare and the 32-bit runs compare every row sharply
         over = int((e >= 3 * TOL[dtype]).sum())
         assert e.median() < TOL[dtype] / 2 and over <= max(1, len(e) // 20) and e.max() < 1.0, (what, float(e.median()), float(e.max()), over)
 
@@ -439,7 +439,7 @@ def test_batch_composition_and_slot_do_not_change_a_row(dtype):
     if dtype == "float32":
         assert e.max() < 2e-5, float(e.max())
     else:
-        assert e.median() < 2e-2 and int((e > 0.1).sum()) <= 5, (float(e.median()), float(e.max()))
+        assert e.median() < 2e-2 and e.max() < 0.1, (float(e.median()), float(e.max()))
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
@@ -455,17 +455,17 @@ def test_a_key_at_a_windows_edge(dtype, tmp_path):
     from safetensors.torch import load_file, save_file
     path = os.path.join(d, "model.safetensors")
     t = load_file(path)
-    E = torch.randn(64, 64, generator=torch.Generator().manual_seed(0))
-    E[1, :32], E[1, 32:] = 3.0, 0.0                                # the query's token
-    E[2, :32], E[2, 32:] = 0.0, 3.0                                # the key's token
+    gen = torch.Generator().manual_seed(0)
+    rand = lambda *shape: torch.randn(*shape, generator=gen)
+    E = rand(64, 64)
+    E[:, 62:] = 0.0
+    E[1], E[2] = 0.0, 0.0
+    E[1, 62], E[2, 63] = 8.0, 8.0                                  # the query's token and the key's token: a column of their own each
     t["embed"], t["pos"] = E.to(torch.bfloat16), torch.zeros_like(t["pos"])
-    u = torch.randn(32, generator=torch.Generator().manual_seed(1))
-    u = u / u.norm() * 32 ** 0.5
-    W = torch.zeros(64, 64)
-    W[:32, :32] = torch.outer(u, torch.ones(32)) / 32              # head 0 of the query's token looks for u ...
-    W[32:, :32] = W[:32, :32]
-    t["l0.mix.q"] = (W + 0.02 * torch.randn(64, 64)).to(torch.bfloat16)
-    t["l0.mix.k"] = torch.cat([torch.zeros(32, 32), torch.outer(u, torch.ones(32)) / 32], 1).to(torch.bfloat16) + (0.02 * torch.randn(32, 64)).to(torch.bfloat16)
+    u = rand(32)
+    Wq, Wk = rand(64, 64), rand(32, 64)
+    Wq[:, 62], Wk[:, 63] = torch.cat([u, u]), u                    # both heads of the one look for what the other has
+    t["l0.mix.q"], t["l0.mix.k"] = Wq.to(torch.bfloat16), Wk.to(torch.bfloat16)
     for n in ("l0.mix.q.b", "l0.mix.k.b"):
         t[n] = torch.zeros_like(t[n])
     save_file({n: x.contiguous() for n, x in t.items()}, path)
@@ -500,7 +500,7 @@ def test_greedy_generation_through_the_entry_point(dtype):
             spread = float((lg - lg.mean()).pow(2).mean().sqrt())
             off += int(lg[t] < lg.max() - (1e-4 if dtype == "float32" else 0.2 * spread))
             seq.append(t)
-        assert off <= (0 if dtype == "float32" else 1)              # (a close call between experts may fall the other way)
+        assert off == 0
     assert lm.model.cache.slots.held == 0
     again = lm.generate(prompts[:2], temperature=0, repeat_penalty=1.0, max_tokens=12)     # on used slots, pages and states
     if dtype == "float32":
