@@ -13,6 +13,9 @@ And shapes of the Pelatar decoder at those widths: of every four layers one runs
 attention with the Qwen2 shape's heads, one attention on the keys and values of the layer before it, one the mLSTM memory (the
 memories' heads, key and value sizes are the Qwen2 shape's); layers alternate between the dense feed-forward and 12 experts
 beside 4 identity experts, 3 of which a token uses.
+And shapes of the Gudarax decoder at those widths: of every three layers one runs attention with the Qwen2 shape's heads behind
+a window, one the delta rule, one latent attention; every fourth layer has the dense feed-forward, the others 16 ungated
+experts of which a token uses 3 (as many parameters a token as the dense one); every layer takes a token input.
 Every entry is a complete config.json; nothing here is read by the model code."""
 
 
@@ -116,14 +119,39 @@ def _pelatar(layers, width, heads, kv_heads, dim, ff, vocab, experts=12, identit
     return {"architecture": "Pelatar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "layers": out}
 
 
-# the Qwen2 shape that a Vunovik, Gisirax, Lipizen, Netezen or Pelatar shape is measured beside
-TWINS = {"pelatar-0.5b": "qwen2.5-0.5b", "pelatar-1.5b": "qwen2.5-1.5b", "pelatar-3b": "qwen2.5-3b", "pelatar-7b": "qwen2.5-7b",
+def _gudarax(layers, width, heads, kv_heads, dim, ff, vocab, experts=16, top=3, window=1024, rank=128, taps=4, side=256, positions=32768):
+    """Layers 0, 3, ... run attention with mixed values, layers 1, 4, ... the delta rule, layers 2, 5, ... latent attention; an expert
+    has two matrices where the dense feed-forward has three, so ``top`` experts of ``3 ff / (2 top)`` values stand for it."""
+    moe = {"kind": "moe", "expert": {"ff": -(-3 * ff // (2 * top) // 64) * 64}, "router": {"experts": experts, "top": top}}
+    out = []
+    for i in range(layers):
+        mlp = {"kind": "dense", "ff": ff} if i % 4 == 0 else moe
+        if i % 3 == 0:
+            out.append({"type": "attention", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                                                                   "v_mix": True, "mask": {"size": window}}})
+        elif i % 3 == 1:
+            out.append({"type": "delta", "mlp": mlp, "mixer": {"heads": heads, "kv_heads": heads, "dim": dim, "vdim": dim, "conv": taps}})
+        else:
+            out.append({"type": "latent_attention", "mlp": mlp, "mixer": {"heads": heads, "dim": dim, "vdim": dim, "kv_rank": rank,
+                                                                          "q_rank": max(64, width // 4 // 64 * 64), "scale": dim ** -0.5}})
+    return {"architecture": "Gudarax", "vocab": vocab, "width": width, "max_positions": positions, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 1.0}, "token_side": {"dim": side}, "layers": out}
+
+
+# the Qwen2 shape that a Vunovik, Gisirax, Lipizen, Netezen, Pelatar or Gudarax shape is measured beside
+TWINS = {"gudarax-0.5b": "qwen2.5-0.5b", "gudarax-1.5b": "qwen2.5-1.5b", "gudarax-3b": "qwen2.5-3b", "gudarax-7b": "qwen2.5-7b",
+         "pelatar-0.5b": "qwen2.5-0.5b", "pelatar-1.5b": "qwen2.5-1.5b", "pelatar-3b": "qwen2.5-3b", "pelatar-7b": "qwen2.5-7b",
          "netezen-0.5b": "qwen2.5-0.5b", "netezen-1.5b": "qwen2.5-1.5b", "netezen-3b": "qwen2.5-3b", "netezen-7b": "qwen2.5-7b",
          "lipizen-0.5b": "qwen2.5-0.5b", "lipizen-1.5b": "qwen2.5-1.5b", "lipizen-3b": "qwen2.5-3b", "lipizen-7b": "qwen2.5-7b",
          "gisirax-0.5b": "qwen2.5-0.5b", "gisirax-1.5b": "qwen2.5-1.5b", "gisirax-3b": "qwen2.5-3b", "gisirax-7b": "qwen2.5-7b",
          "vunovik-0.5b": "qwen2.5-0.5b", "vunovik-1.5b": "qwen2.5-1.5b", "vunovik-3b": "qwen2.5-3b", "vunovik-7b": "qwen2.5-7b"}
 
 SHAPES = {
+    "gudarax-tiny": _gudarax(4, 128, 4, 2, 32, 256, 512, experts=6, top=2, window=80, rank=48, taps=3, side=8, positions=512),
+    "gudarax-0.5b": _gudarax(24, 896, 14, 2, 64, 4864, 151936, rank=64, side=128),
+    "gudarax-1.5b": _gudarax(28, 1536, 12, 2, 128, 8960, 151936),
+    "gudarax-3b": _gudarax(36, 2048, 16, 2, 128, 11008, 151936),
+    "gudarax-7b": _gudarax(28, 3584, 28, 4, 128, 18944, 152064),
     "pelatar-tiny": _pelatar(4, 128, 4, 2, 32, 256, 512, experts=5, identity=3, top=2, groups=4, keep=2, rank=8, every=16),
     "pelatar-0.5b": _pelatar(24, 896, 14, 2, 64, 4864, 151936),
     "pelatar-1.5b": _pelatar(28, 1536, 12, 2, 128, 8960, 151936),

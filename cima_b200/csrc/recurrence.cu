@@ -4,7 +4,6 @@
 //   decay rule   S <- d_h S + k v^T;                       o = S^T q       d_h one constant a head; q, k, v through SiLU
 //   delta rule   S <- diag(g_t) S;  u = beta_t (v - S^T k);  S <- S + k u^T;  o = S^T q
 //                g_t one decay a key channel and token, beta_t one scalar a token; the read-out sees the token's write
-//                with one decay a head (g_t a scalar a token):  u = beta_t (v - g_t (S^T k));  S <- g_t S + k u^T
 //   gate rule    S <- diag(f_t) S + (1 - f_t) v^T;          o = S^T q       f_t = l + (1 - l) sigmoid(z_t + b) one forget gate
 //                a key channel and token, made here from the projection z, a bias b and a lower bound l (both
 //                [heads * dim]); what the gate forgets is what it lets in; q through SiLU, v as it is
@@ -36,15 +35,14 @@ __device__ __forceinline__ float rec_sum_over_lanes(float v) {        // over th
 // CPT: columns a thread owns (its columns stand 32 apart).  With two, every read of k, q and g from shared memory serves
 // both, but a block covers 64 columns and a sequence gets half as many blocks: measured slower for one prompt (1.2 ms
 // against 0.97 ms a layer of 2,048 tokens at key and value size 128), so the launch takes one.
-// MODE: 0 the decay rule, 1 the delta rule, 2 the gate rule, 3 the delta rule with one decay a head.
+// MODE: 0 the decay rule, 1 the delta rule, 2 the gate rule.
 template <typename TQ, typename TV, int DIMP, int MODE, int CPT>
 __global__ void __launch_bounds__(REC_THREADS)
 k_recurrence(const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k, int ldk, const TV* __restrict__ v, int ldv,
              const float* __restrict__ g, const float* __restrict__ beta, const float* __restrict__ decay,
              float* __restrict__ state, const int* __restrict__ seq_slot, const int* __restrict__ seq_first_row,
              float* __restrict__ out, int heads, int kv_heads, int dim, int vdim) {
-  constexpr bool DELTA = MODE == 1 || MODE == 3, GATE = MODE == 2, HEAD = MODE == 3;
-  constexpr bool CHANNEL = MODE == 1 || GATE;           // a decay a key channel and token
+  constexpr bool DELTA = MODE == 1, GATE = MODE == 2, CHANNEL = MODE != 0;      // CHANNEL: a decay a key channel and token
   cima_pdl_wait();
   constexpr int RP = DIMP / REC_SPLIT;                  // rows of a column that one lane keeps
   constexpr int CH = DIMP > 128 ? 8 : 16;               // tokens staged at a time
@@ -54,7 +52,7 @@ k_recurrence(const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k, int ld
   __shared__ __align__(16) float sg[CHANNEL ? CH : 1][DIMP];
   __shared__ float sv[CH][COLS];
   __shared__ float so[CH][COLS];
-  __shared__ float sb[CH], sd[HEAD ? CH : 1];
+  __shared__ float sb[CH];
   const int seq = blockIdx.z, h = blockIdx.y, col0 = blockIdx.x * COLS;
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int rg = lane >> 2, lc = warp * 4 + (lane & 3);  // row group; the thread's columns are col0 + lc + 32 x
@@ -69,7 +67,7 @@ k_recurrence(const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k, int ld
       const int row = (j >> 2) * 32 + rg * 4 + (j & 3);
       S[x][j] = (col0 + lc + 32 * x < vdim && row < dim) ? st[(size_t)row * vdim + 32 * x] : 0.f;
     }
-  const float dh = MODE == 0 ? decay[h] : 1.f;
+  const float dh = CHANNEL ? 1.f : decay[h];
   const int ldo = heads * vdim;
 
   // The next tokens' k, q, g, v and beta travel from global memory into registers while the current ones are worked on
@@ -79,7 +77,7 @@ k_recurrence(const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k, int ld
   // They wait there as they were loaded: a conversion in front of the work would wait for the load it converts.
   TQ rk[NLD], rq[NLD];
   TV rv[NLV];
-  float rgt[CHANNEL && DELTA ? NLD : 1], rb = 0.f, rd = 1.f;
+  float rgt[DELTA ? NLD : 1], rb = 0.f;
   const TQ zero_q = cima_from_f32<TQ>(0.f);
   const TV zero_v = cima_from_f32<TV>(0.f);
   // The gate rule: k holds the gate's projection z, g its bias and decay its lower bound (the same for every token: a
@@ -103,7 +101,7 @@ k_recurrence(const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k, int ld
       const bool ok = tt < nt && i < dim;
       rk[r] = ok ? k[row * ldk + (size_t)kvh * dim + i] : zero_q;
       rq[r] = ok ? q[row * ldq + (size_t)kvh * dim + i] : zero_q;
-      if (CHANNEL && DELTA) rgt[r] = ok ? g[(row * heads + h) * dim + i] : 1.f;
+      if (DELTA) rgt[r] = ok ? g[(row * heads + h) * dim + i] : 1.f;
     }
 #pragma unroll
     for (int r = 0; r < NLV; r++) {
@@ -112,7 +110,6 @@ k_recurrence(const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k, int ld
       rv[r] = (tt < nt && col0 + cc < vdim) ? v[(size_t)(first + t0 + tt) * ldv + (size_t)h * vdim + col0 + cc] : zero_v;
     }
     if (DELTA) rb = (int)threadIdx.x < nt ? beta[(size_t)(first + t0 + threadIdx.x) * heads + h] : 0.f;
-    if (HEAD) rd = (int)threadIdx.x < nt ? g[(size_t)(first + t0 + threadIdx.x) * heads + h] : 1.f;
   };
   if (n > 0) fetch(0);
 
@@ -126,16 +123,15 @@ k_recurrence(const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k, int ld
       const float fk = cima_to_f32<TQ>(rk[r]), fq = cima_to_f32<TQ>(rq[r]);
       if (!GATE) sk[tt][i] = DELTA ? fk : rec_silu(fk);
       sq[tt][i] = DELTA ? fq : rec_silu(fq);
-      if (CHANNEL && DELTA) sg[tt][i] = rgt[r];
+      if (DELTA) sg[tt][i] = rgt[r];
       if (GATE) sg[tt][i] = glow[r] + (1.0f - glow[r]) / (1.0f + expf(-(fk + gbias[r])));
     }
 #pragma unroll
     for (int r = 0; r < NLV; r++) {
       const int idx = threadIdx.x + r * REC_THREADS;
-      if (idx < CH * COLS) sv[idx / COLS][idx % COLS] = MODE != 0 ? cima_to_f32<TV>(rv[r]) : rec_silu(cima_to_f32<TV>(rv[r]));
+      if (idx < CH * COLS) sv[idx / COLS][idx % COLS] = CHANNEL ? cima_to_f32<TV>(rv[r]) : rec_silu(cima_to_f32<TV>(rv[r]));
     }
     if (DELTA && threadIdx.x < CH) sb[threadIdx.x] = rb;
-    if (HEAD && threadIdx.x < CH) sd[threadIdx.x] = rd;
     __syncthreads();
     if (t0 + CH < n) fetch(t0 + CH);
     if constexpr (GATE) {
@@ -183,25 +179,7 @@ k_recurrence(const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k, int ld
       float u[CPT];
 #pragma unroll
       for (int x = 0; x < CPT; x++) u[x] = sv[tt][lc + 32 * x];
-      float keep = dh;                                  // what the token leaves of the state, where that is one number
-      if constexpr (HEAD) {
-        float p0[CPT], p1[CPT];
-#pragma unroll
-        for (int x = 0; x < CPT; x++) p0[x] = p1[x] = 0.f;
-#pragma unroll
-        for (int j = 0; j < RP; j += 4) {
-          const float4 k4 = *reinterpret_cast<const float4*>(&sk[tt][(j >> 2) * 32 + rg * 4]);
-#pragma unroll
-          for (int x = 0; x < CPT; x++) {
-            p0[x] = fmaf(S[x][j], k4.x, p0[x]); p1[x] = fmaf(S[x][j + 1], k4.y, p1[x]);
-            p0[x] = fmaf(S[x][j + 2], k4.z, p0[x]); p1[x] = fmaf(S[x][j + 3], k4.w, p1[x]);
-          }
-        }
-        keep = sd[tt];
-        const float b = sb[tt];
-#pragma unroll
-        for (int x = 0; x < CPT; x++) u[x] = b * (u[x] - keep * rec_sum_over_lanes(p0[x] + p1[x]));
-      } else if (DELTA) {
+      if (DELTA) {
         float p0[CPT], p1[CPT];
 #pragma unroll
         for (int x = 0; x < CPT; x++) p0[x] = p1[x] = 0.f;
@@ -224,7 +202,7 @@ k_recurrence(const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k, int ld
 #pragma unroll
         for (int x = 0; x < CPT; x++)
 #pragma unroll
-          for (int j = 0; j < RP; j++) S[x][j] *= keep;
+          for (int j = 0; j < RP; j++) S[x][j] *= dh;
       }
       float o0[CPT], o1[CPT];
 #pragma unroll
@@ -236,7 +214,6 @@ k_recurrence(const TQ* __restrict__ q, int ldq, const TQ* __restrict__ k, int ld
         const float4 q4 = *reinterpret_cast<const float4*>(&sq[tt][i]);
 #pragma unroll
         for (int x = 0; x < CPT; x++) {
-          if (HEAD) { S[x][j] *= keep; S[x][j + 1] *= keep; S[x][j + 2] *= keep; S[x][j + 3] *= keep; }
           S[x][j] = fmaf(k4.x, u[x], S[x][j]); S[x][j + 1] = fmaf(k4.y, u[x], S[x][j + 1]);
           S[x][j + 2] = fmaf(k4.z, u[x], S[x][j + 2]); S[x][j + 3] = fmaf(k4.w, u[x], S[x][j + 3]);
           o0[x] = fmaf(S[x][j], q4.x, o0[x]); o1[x] = fmaf(S[x][j + 1], q4.y, o1[x]);
@@ -285,7 +262,7 @@ int launch_recurrence(const void* q, int ldq, const void* k, int ldk, const void
 
 // Everything of the delta rule that is computed per token before the recurrence, in float32:
 //   qn = q / sqrt(sum q^2 + 1e-6) * dim^(-1/2),  kn = k / sqrt(sum k^2 + 1e-6)            per head of q and k
-//   g  = exp(-exp(A_log[h]) * softplus(a + dt_bias)),  beta = sigmoid(b)                 gdim values of g a head (dim, or one)
+//   g  = exp(-exp(A_log[h]) * softplus(a + dt_bias)),  beta = sigmoid(b)
 // A warp takes one unit of a row: a head of q, a head of k, or a head's decays with its beta; a block four units.  (One
 // block a row, its warps walking the row's units one after another, took 17 us for the 8 rows of a decode step: a chain of
 // some dozen trips to memory on 8 SMs.)
@@ -293,7 +270,7 @@ template <typename TA>
 __global__ void __launch_bounds__(128)
 k_delta_prepare(const TA* __restrict__ qk, int ldqk, const TA* __restrict__ a, int lda, const TA* __restrict__ b, int ldb,
                 const float* __restrict__ A_log, const float* __restrict__ dt_bias, float* __restrict__ qn, float* __restrict__ kn,
-                float* __restrict__ g, float* __restrict__ beta, int heads, int kv_heads, int dim, int gdim) {
+                float* __restrict__ g, float* __restrict__ beta, int heads, int kv_heads, int dim) {
   cima_pdl_wait();
   cima_pdl_trigger();        // the next kernel may be set up while this one runs (it waits for this one's end itself)
   const size_t row = blockIdx.y;
@@ -325,14 +302,14 @@ k_delta_prepare(const TA* __restrict__ qk, int ldqk, const TA* __restrict__ a, i
 #pragma unroll
     for (int j = 0; j < 8; j++) {
       const int i = lane + 32 * j;
-      z[j] = i < gdim ? cima_to_f32<TA>(a[row * lda + (size_t)h * gdim + i]) + dt_bias[h * gdim + i] : 0.f;
+      z[j] = i < dim ? cima_to_f32<TA>(a[row * lda + (size_t)h * dim + i]) + dt_bias[h * dim + i] : 0.f;
     }
 #pragma unroll
     for (int j = 0; j < 8; j++) {
       const int i = lane + 32 * j;
-      if (i < gdim) {
+      if (i < dim) {
         const float sp = z[j] > 20.f ? z[j] : log1pf(expf(z[j]));
-        g[(row * heads + h) * gdim + i] = expf(-rate * sp);
+        g[(row * heads + h) * dim + i] = expf(-rate * sp);
       }
     }
     if (lane == 0) beta[row * heads + h] = 1.0f / (1.0f + expf(-cima_to_f32<TA>(b[row * ldb + h])));
@@ -341,7 +318,6 @@ k_delta_prepare(const TA* __restrict__ qk, int ldqk, const TA* __restrict__ a, i
 }  // namespace
 
 // delta != 0: q, k float32 [T, kv_heads * dim] (prepared), v (vdtype) [T, ldv], g [T, heads * dim], beta [T, heads].
-// delta == 3: the same with one decay a head, g [T, heads].
 // delta == 0: q, k, v of one dtype (vdtype), SiLU applied here; decay [heads].  out [T, heads * vdim] float32.
 // delta == 2 (the gate rule): q and k of v's dtype, k holding the gate's projection; g its bias and decay its lower bound,
 // both [heads * dim] and shared by all tokens.
@@ -365,11 +341,7 @@ extern "C" int cima_recurrence(const void* q, int ldq, const void* k, int ldk, c
   if (delta && (!g || !beta)) return cima_fail(CIMA_E_ARG, "recurrence: the delta rule needs the tokens' decays and step sizes");
   if (!delta && !decay) return cima_fail(CIMA_E_ARG, "recurrence: the decay rule needs the heads' decays");
   int rc;
-  if (delta == 3) {
-    if (vdtype == CIMA_F32) rc = launch_recurrence<float, float, 3>(q, ldq, k, ldk, v, ldv, g, beta, decay, state, seq_slot, seq_first_row, out, n_seqs, heads, kv_heads, dim, vdim, stream);
-    else if (vdtype == CIMA_BF16) rc = launch_recurrence<float, __nv_bfloat16, 3>(q, ldq, k, ldk, v, ldv, g, beta, decay, state, seq_slot, seq_first_row, out, n_seqs, heads, kv_heads, dim, vdim, stream);
-    else return cima_fail(CIMA_E_DTYPE, "recurrence: dtype code %d is neither float32 nor bfloat16", vdtype);
-  } else if (delta) {
+  if (delta) {
     if (vdtype == CIMA_F32) rc = launch_recurrence<float, float, 1>(q, ldq, k, ldk, v, ldv, g, beta, decay, state, seq_slot, seq_first_row, out, n_seqs, heads, kv_heads, dim, vdim, stream);
     else if (vdtype == CIMA_BF16) rc = launch_recurrence<float, __nv_bfloat16, 1>(q, ldq, k, ldk, v, ldv, g, beta, decay, state, seq_slot, seq_first_row, out, n_seqs, heads, kv_heads, dim, vdim, stream);
     else return cima_fail(CIMA_E_DTYPE, "recurrence: dtype code %d is neither float32 nor bfloat16", vdtype);
@@ -381,18 +353,17 @@ extern "C" int cima_recurrence(const void* q, int ldq, const void* k, int ldk, c
   return rc ? rc : cima_launch_result();
 }
 
-// qk [T, ldqk]: q's heads then k's (2 * kv_heads * dim values of a row); a [T, lda]: heads * gdim (gdim = dim or 1); b [T, ldb]: heads.
+// qk [T, ldqk]: q's heads then k's (2 * kv_heads * dim values of a row); a [T, lda]: heads * dim; b [T, ldb]: heads.
 extern "C" int cima_delta_prepare(const void* qk, int ldqk, const void* a, int lda, const void* b, int ldb, int dtype,
                                   const float* A_log, const float* dt_bias, float* qn, float* kn, float* g, float* beta,
-                                  int T, int heads, int kv_heads, int dim, int gdim, cudaStream_t stream) {
+                                  int T, int heads, int kv_heads, int dim, cudaStream_t stream) {
   if (T <= 0) return 0;
   if (heads <= 0 || kv_heads <= 0 || dim <= 0 || dim > 256) return cima_fail(CIMA_E_SIZE, "delta_prepare: heads %d and key heads %d must be positive, the key size %d in 1..256", heads, kv_heads, dim);
-  if (gdim != dim && gdim != 1) return cima_fail(CIMA_E_SIZE, "delta_prepare: %d decays a head are neither one nor one a key channel (%d)", gdim, dim);
   if (T > 65535) return cima_fail(CIMA_E_SIZE, "delta_prepare: %d rows exceed one launch; the caller cuts them", T);
   const dim3 grid((unsigned)((2 * kv_heads + heads + 3) / 4), (unsigned)T);
   int rc;
-  if (dtype == CIMA_F32) rc = cima_launch(k_delta_prepare<float>, grid, dim3(128), (size_t)0, stream, 1, (const float*)qk, ldqk, (const float*)a, lda, (const float*)b, ldb, A_log, dt_bias, qn, kn, g, beta, heads, kv_heads, dim, gdim);
-  else if (dtype == CIMA_BF16) rc = cima_launch(k_delta_prepare<__nv_bfloat16>, grid, dim3(128), (size_t)0, stream, 1, (const __nv_bfloat16*)qk, ldqk, (const __nv_bfloat16*)a, lda, (const __nv_bfloat16*)b, ldb, A_log, dt_bias, qn, kn, g, beta, heads, kv_heads, dim, gdim);
+  if (dtype == CIMA_F32) rc = cima_launch(k_delta_prepare<float>, grid, dim3(128), (size_t)0, stream, 1, (const float*)qk, ldqk, (const float*)a, lda, (const float*)b, ldb, A_log, dt_bias, qn, kn, g, beta, heads, kv_heads, dim);
+  else if (dtype == CIMA_BF16) rc = cima_launch(k_delta_prepare<__nv_bfloat16>, grid, dim3(128), (size_t)0, stream, 1, (const __nv_bfloat16*)qk, ldqk, (const __nv_bfloat16*)a, lda, (const __nv_bfloat16*)b, ldb, A_log, dt_bias, qn, kn, g, beta, heads, kv_heads, dim);
   else return cima_fail(CIMA_E_DTYPE, "delta_prepare: dtype code %d is neither float32 nor bfloat16", dtype);
   return rc ? rc : cima_launch_result();
 }

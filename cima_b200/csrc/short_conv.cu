@@ -12,6 +12,17 @@
 // launch does both, each thread owning its (sequence, channel).
 #include "common.cuh"
 
+// What the sum passes through, chosen at compile time in the kernels of many rows (with the choice inside, their unrolled loops
+// held every activation and took 67 us for 2,048 rows of 4,608 channels): nothing, SiLU, or an entry of CIMA_ACT_* at run time.
+// The kernels of bfloat16 rows take SiLU with the fast exponential and division: a few ulp of float32 in front of the rounding.
+enum { CONV_ACT_NONE = 0, CONV_ACT_SILU = 1, CONV_ACT_ANY = 2 };
+template <typename TA, int ACT>
+__device__ __forceinline__ float conv_act(float v, int act) {
+  if (ACT == CONV_ACT_NONE) return v;
+  if (ACT == CONV_ACT_SILU) return sizeof(TA) == 2 ? v * cima_sigmoid_fast(v) : v / (1.0f + expf(-v));
+  return cima_gate_act(v, act);
+}
+
 constexpr int CONV_MAX_TAPS = 16;
 constexpr int CONV_THREADS = 256;
 
@@ -42,7 +53,8 @@ k_short_conv(const TA* __restrict__ h, const float* __restrict__ w, TA* __restri
     old[j] = v;
     acc = fmaf(w[(size_t)j * C + c], v, acc);
   }
-  if (act >= 0) acc = cima_gate_act(acc, act);
+  if (act == CIMA_ACT_SILU) acc = conv_act<TA, CONV_ACT_SILU>(acc, act);
+  else if (act >= 0) acc = cima_gate_act(acc, act);
   u[(size_t)row * C + c] = cima_from_f32<TA>(acc);
   if (ONE_ROW) {
     // the state moves on by one position: entries 1 .. taps - 2 go down, the row's input comes last
@@ -61,7 +73,7 @@ template <typename TA> struct ConvVec;
 template <> struct ConvVec<float> { static constexpr int N = 4; };
 template <> struct ConvVec<__nv_bfloat16> { static constexpr int N = 8; };
 
-template <typename TA>
+template <typename TA, int ACT>
 __global__ void __launch_bounds__(CONV_THREADS)
 k_short_conv_wide(const TA* __restrict__ h, const float* __restrict__ w, const TA* __restrict__ state,
                   const int* __restrict__ row_seq, const int* __restrict__ seq_slot, const int* __restrict__ seq_first_row,
@@ -106,7 +118,7 @@ k_short_conv_wide(const TA* __restrict__ h, const float* __restrict__ w, const T
   uint4 outv;
   TA* o = reinterpret_cast<TA*>(&outv);
 #pragma unroll
-  for (int i = 0; i < V; i++) o[i] = cima_from_f32<TA>(act >= 0 ? cima_gate_act(acc[i], act) : acc[i]);
+  for (int i = 0; i < V; i++) o[i] = cima_from_f32<TA>(conv_act<TA, ACT>(acc[i], act));
   *reinterpret_cast<uint4*>(u + (size_t)row * C + c) = outv;
 }
 
@@ -117,7 +129,7 @@ k_short_conv_wide(const TA* __restrict__ h, const float* __restrict__ w, const T
 // kernel above.  Same products in the same order: the same bits.
 constexpr int CONV_FEW_TAPS = 4;
 
-template <typename TA, int CONV_ROWS>
+template <typename TA, int CONV_ROWS, int ACT>
 __global__ void __launch_bounds__(CONV_THREADS)
 k_short_conv_rows(const TA* __restrict__ h, const float* __restrict__ w, const TA* __restrict__ state,
                   const int* __restrict__ row_seq, const int* __restrict__ seq_slot, const int* __restrict__ seq_first_row,
@@ -198,7 +210,7 @@ k_short_conv_rows(const TA* __restrict__ h, const float* __restrict__ w, const T
     uint4 outv;
     TA* o = reinterpret_cast<TA*>(&outv);
 #pragma unroll
-    for (int i = 0; i < V; i++) o[i] = cima_from_f32<TA>(act >= 0 ? cima_gate_act(acc[i], act) : acc[i]);
+    for (int i = 0; i < V; i++) o[i] = cima_from_f32<TA>(conv_act<TA, ACT>(acc[i], act));
     *reinterpret_cast<uint4*>(u + (size_t)row * C + c) = outv;
     // this row becomes the next one's nearest past
 #pragma unroll
@@ -259,19 +271,30 @@ extern "C" int cima_short_conv(const void* h, int dtype, int ldh, const float* w
   int rows_each = cells >= 2ll * 148 * 2048 ? 8 : 1;
   if (rows_per_thread == 1 || rows_per_thread == 2 || rows_per_thread == 4 || rows_per_thread == 8) rows_each = rows_per_thread;
   else if (rows_per_thread != 0) return cima_fail(CIMA_E_ARG, "short_conv: %d rows a thread; 0 (chosen here), 1, 2, 4 or 8 are possible", rows_per_thread);
+#define ARGS(TA) (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u
+#define WIDE_Y(TA) (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)
+#define ROWS(TA, N, ACT) rc_ = cima_launch(k_short_conv_rows<TA, N, ACT>, dim3((T + N - 1) / N, WIDE_Y(TA)), block, (size_t)0, stream, 1, ARGS(TA), T, ldh, C, taps, add_input, act)
+#define MANY(TA, ACT) { \
+    if (taps <= CONV_FEW_TAPS && rows_each == 8) ROWS(TA, 8, ACT); \
+    else if (taps <= CONV_FEW_TAPS && rows_each == 4) ROWS(TA, 4, ACT); \
+    else if (taps <= CONV_FEW_TAPS && rows_each == 2) ROWS(TA, 2, ACT); \
+    else rc_ = cima_launch(k_short_conv_wide<TA, ACT>, dim3(T, WIDE_Y(TA)), block, (size_t)0, stream, 1, ARGS(TA), ldh, C, taps, add_input, act); }
 #define RUN(TA) { \
     int rc_; \
     if (one_row) rc_ = cima_launch(k_short_conv<TA, true>, dim3(T, cy), block, (size_t)0, stream, 1, (const TA*)h, w, (TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, ldh, C, taps, add_input, act); \
-    else if (wide && taps <= CONV_FEW_TAPS && rows_each == 8) rc_ = cima_launch(k_short_conv_rows<TA, 8>, dim3((T + 7) / 8, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, T, ldh, C, taps, add_input, act); \
-    else if (wide && taps <= CONV_FEW_TAPS && rows_each == 4) rc_ = cima_launch(k_short_conv_rows<TA, 4>, dim3((T + 3) / 4, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, T, ldh, C, taps, add_input, act); \
-    else if (wide && taps <= CONV_FEW_TAPS && rows_each == 2) rc_ = cima_launch(k_short_conv_rows<TA, 2>, dim3((T + 1) / 2, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, T, ldh, C, taps, add_input, act); \
-    else if (wide) rc_ = cima_launch(k_short_conv_wide<TA>, dim3(T, (unsigned)((C / ConvVec<TA>::N + CONV_THREADS - 1) / CONV_THREADS)), block, (size_t)0, stream, 1, (const TA*)h, w, (const TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, ldh, C, taps, add_input, act); \
-    else rc_ = cima_launch(k_short_conv<TA, false>, dim3(T, cy), block, (size_t)0, stream, 1, (const TA*)h, w, (TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, ldh, C, taps, add_input, act); \
+    else if (!wide) rc_ = cima_launch(k_short_conv<TA, false>, dim3(T, cy), block, (size_t)0, stream, 1, (const TA*)h, w, (TA*)state, row_seq, seq_slot, seq_first_row, (TA*)u, ldh, C, taps, add_input, act); \
+    else if (act < 0) MANY(TA, CONV_ACT_NONE) \
+    else if (act == CIMA_ACT_SILU) MANY(TA, CONV_ACT_SILU) \
+    else MANY(TA, CONV_ACT_ANY) \
     if (rc_) return rc_; \
     if (!one_row && taps > 1) { rc_ = cima_launch(k_short_conv_state<TA>, dim3(n_seqs, cy), block, (size_t)0, stream, 1, (const TA*)h, (TA*)state, seq_slot, seq_first_row, ldh, C, taps); if (rc_) return rc_; } }
   if (dtype == CIMA_F32) RUN(float)
   else if (dtype == CIMA_BF16) RUN(__nv_bfloat16)
   else return cima_fail(CIMA_E_DTYPE, "short_conv: dtype code %d is neither float32 nor bfloat16", dtype);
 #undef RUN
+#undef MANY
+#undef ROWS
+#undef WIDE_Y
+#undef ARGS
   return cima_launch_result();
 }

@@ -1,93 +1,103 @@
 // A token's own input to a layer: z[t, j] = act(sum_k x[t, k] W[j, k]) * D[tok_t, col + j], D the model's side table.
 //
-// token_side_few    the whole of it for the few rows of a decode step, straight from the float32 stream: a warp takes two
-//                   outputs j, its lanes stride the two rows of W by 16 bytes and hold the sums of all rows (at most 8); a fixed
-//                   shuffle tree adds the lanes.  A row's sum does not depend on what else is in the step.
+// token_side_few    the whole of it for the few rows of a decode step, straight from the float32 stream: a block takes four
+//                   outputs j, its eight warps share k in interleaved pieces of 16 bytes a lane and hold the sums of all rows (at
+//                   most 8); the lanes are added by a shuffle tree, the warps in their order.  A row's sum does not depend on what
+//                   else is in the step.
 // token_side_apply  behind a product of many rows: z <- act(z) * D[tok, col + j] in place
 #include "common.cuh"
 
 namespace {
-constexpr int TS_ROWS = 8, TS_OUTS = 2, TS_WARPS = 4;
+constexpr int TS_ROWS = 8, TS_OUTS = 4, TS_WARPS = 8;
 
 template <typename TW> struct TsVec;                          // weights of one 16-byte load
 template <> struct TsVec<float> { static constexpr int N = 4; };
 template <> struct TsVec<__nv_bfloat16> { static constexpr int N = 8; };
 
-template <typename TW, typename TA>
+// VEC false: one value a lane at a time (any width, any alignment).
+template <typename TW, typename TA, bool VEC>
 __global__ void __launch_bounds__(TS_WARPS * 32)
 k_token_side_few(const float* __restrict__ x, const TW* __restrict__ w, const TA* __restrict__ table, int ldt, const int* __restrict__ tokens,
-                 int col, TA* __restrict__ z, int T, int dim, int W, int vocab, int act, int vec) {
+                 int col, TA* __restrict__ z, int T, int dim, int W, int vocab, int act) {
+  constexpr int V = VEC ? TsVec<TW>::N : 1;
+  constexpr int STEP = TS_WARPS * 32 * V;
+  __shared__ float part[TS_WARPS][TS_OUTS * TS_ROWS];
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int j0 = (blockIdx.x * TS_WARPS + warp) * TS_OUTS;
-  if (j0 >= dim) return;
-  const int j1 = min(j0 + 1, dim - 1);                        // (an odd last output is computed twice and stored once)
-  const TW *w0 = w + (size_t)j0 * W, *w1 = w + (size_t)j1 * W;
-  constexpr int V = TsVec<TW>::N;
+  const int j0 = blockIdx.x * TS_OUTS;
+  struct __align__(VEC ? 16 : sizeof(TW)) Piece { TW e[V]; };
+  const TW* wr[TS_OUTS];
+#pragma unroll
+  for (int o = 0; o < TS_OUTS; o++) wr[o] = w + (size_t)min(j0 + o, dim - 1) * W;      // (outputs beyond the last are not stored)
   float acc[TS_OUTS][TS_ROWS];
 #pragma unroll
   for (int o = 0; o < TS_OUTS; o++)
 #pragma unroll
     for (int r = 0; r < TS_ROWS; r++) acc[o][r] = 0.f;
-  if (vec) {
-    // the first weights depend on no kernel: they are requested before the wait
-    uint4 n0 = make_uint4(0u, 0u, 0u, 0u), n1 = n0;
-    if (lane * V < W) { n0 = *reinterpret_cast<const uint4*>(w0 + lane * V); n1 = *reinterpret_cast<const uint4*>(w1 + lane * V); }
-    cima_pdl_wait();
-    for (int k = lane * V; k < W; k += 32 * V) {
-      const uint4 c0 = n0, c1 = n1;
-      const int kn = k + 32 * V;
-      if (kn < W) { n0 = *reinterpret_cast<const uint4*>(w0 + kn); n1 = *reinterpret_cast<const uint4*>(w1 + kn); }
-      const TW *a = reinterpret_cast<const TW*>(&c0), *b = reinterpret_cast<const TW*>(&c1);
-      float4 xv[TS_ROWS][V / 4];
+  // the first weights depend on no kernel: they are requested before the wait
+  const int k0 = (warp * 32 + lane) * V;
+  Piece c[TS_OUTS];
 #pragma unroll
-      for (int r = 0; r < TS_ROWS; r++)
+  for (int o = 0; o < TS_OUTS; o++)
+    if (k0 < W) c[o] = *reinterpret_cast<const Piece*>(wr[o] + k0);
+  cima_pdl_wait();
+  for (int k = k0; k < W; k += STEP) {
+    float xv[TS_ROWS][V];
 #pragma unroll
-        for (int q = 0; q < V / 4; q++)
-          xv[r][q] = r < T ? *reinterpret_cast<const float4*>(x + (size_t)r * W + k + 4 * q) : make_float4(0.f, 0.f, 0.f, 0.f);
+    for (int r = 0; r < TS_ROWS; r++) {
+      if constexpr (VEC) {
 #pragma unroll
-      for (int q = 0; q < V / 4; q++) {
-        const float a0 = cima_to_f32<TW>(a[4 * q]), a1 = cima_to_f32<TW>(a[4 * q + 1]), a2 = cima_to_f32<TW>(a[4 * q + 2]), a3 = cima_to_f32<TW>(a[4 * q + 3]);
-        const float b0 = cima_to_f32<TW>(b[4 * q]), b1 = cima_to_f32<TW>(b[4 * q + 1]), b2 = cima_to_f32<TW>(b[4 * q + 2]), b3 = cima_to_f32<TW>(b[4 * q + 3]);
-#pragma unroll
-        for (int r = 0; r < TS_ROWS; r++) {
-          const float4 f = xv[r][q];
-          acc[0][r] = fmaf(f.x, a0, acc[0][r]); acc[0][r] = fmaf(f.y, a1, acc[0][r]);
-          acc[0][r] = fmaf(f.z, a2, acc[0][r]); acc[0][r] = fmaf(f.w, a3, acc[0][r]);
-          acc[1][r] = fmaf(f.x, b0, acc[1][r]); acc[1][r] = fmaf(f.y, b1, acc[1][r]);
-          acc[1][r] = fmaf(f.z, b2, acc[1][r]); acc[1][r] = fmaf(f.w, b3, acc[1][r]);
+        for (int q = 0; q < V; q += 4) {
+          const float4 f = r < T ? *reinterpret_cast<const float4*>(x + (size_t)r * W + k + q) : make_float4(0.f, 0.f, 0.f, 0.f);
+          xv[r][q] = f.x; xv[r][q + 1] = f.y; xv[r][q + 2] = f.z; xv[r][q + 3] = f.w;
         }
+      } else {
+        xv[r][0] = r < T ? x[(size_t)r * W + k] : 0.f;
       }
     }
-  } else {
-    cima_pdl_wait();
-    for (int k = lane; k < W; k += 32) {
-      const float a = cima_to_f32<TW>(w0[k]), b = cima_to_f32<TW>(w1[k]);
 #pragma unroll
-      for (int r = 0; r < TS_ROWS; r++) {
-        const float f = r < T ? x[(size_t)r * W + k] : 0.f;
-        acc[0][r] = fmaf(f, a, acc[0][r]);
-        acc[1][r] = fmaf(f, b, acc[1][r]);
+    for (int o = 0; o < TS_OUTS; o++)
+#pragma unroll
+      for (int q = 0; q < V; q++) {
+        const float wv = cima_to_f32<TW>(c[o].e[q]);
+#pragma unroll
+        for (int r = 0; r < TS_ROWS; r++) acc[o][r] = fmaf(xv[r][q], wv, acc[o][r]);
       }
+    if (k + STEP < W) {
+#pragma unroll
+      for (int o = 0; o < TS_OUTS; o++) c[o] = *reinterpret_cast<const Piece*>(wr[o] + k + STEP);
     }
   }
   cima_pdl_trigger();
+  // 32 sums over the 32 lanes, handed over by halves: after the step of distance d a lane holds half as many sums, of its half
+  // of the pairs; in the end lane l holds sum number l, added up over all lanes in a fixed order
+  float s[TS_OUTS * TS_ROWS];
 #pragma unroll
-  for (int o = 16; o > 0; o >>= 1)
+  for (int o = 0; o < TS_OUTS; o++)
 #pragma unroll
-    for (int q = 0; q < TS_OUTS; q++)
+    for (int r = 0; r < TS_ROWS; r++) s[o * TS_ROWS + r] = acc[o][r];
 #pragma unroll
-      for (int r = 0; r < TS_ROWS; r++) acc[q][r] += __shfl_xor_sync(0xffffffffu, acc[q][r], o);
-  // lane (q, r) = q * TS_ROWS + r finishes output j0 + q of row r
+  for (int d = 16; d > 0; d >>= 1) {
+    const bool upper = lane & d;
 #pragma unroll
-  for (int q = 0; q < TS_OUTS; q++)
+    for (int i = 0; i < d; i++) {
+      const float mine = upper ? s[i + d] : s[i], other = upper ? s[i] : s[i + d];
+      s[i] = mine + __shfl_xor_sync(0xffffffffu, other, d);
+    }
+  }
+  part[warp][lane] = s[0];
+  __syncthreads();
+  if (warp == 0) {
+    float v = 0.f;
 #pragma unroll
-    for (int r = 0; r < TS_ROWS; r++)
-      if (lane == q * TS_ROWS + r && r < T && j0 + q < dim) {
-        int tok = tokens[r];
-        tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);
-        const float e = cima_to_f32<TA>(table[(size_t)tok * ldt + col + j0 + q]);
-        z[(size_t)r * dim + j0 + q] = cima_from_f32<TA>(cima_gate_act(acc[q][r], act) * e);
-      }
+    for (int q = 0; q < TS_WARPS; q++) v += part[q][lane];
+    const int o = lane / TS_ROWS, r = lane % TS_ROWS;
+    if (r < T && j0 + o < dim) {
+      int tok = tokens[r];
+      tok = tok < 0 ? 0 : (tok >= vocab ? vocab - 1 : tok);
+      const float e = cima_to_f32<TA>(table[(size_t)tok * ldt + col + j0 + o]);
+      z[(size_t)r * dim + j0 + o] = cima_from_f32<TA>(cima_gate_act(v, act) * e);
+    }
+  }
 }
 
 template <typename TA>
@@ -138,15 +148,17 @@ extern "C" int cima_token_side_few(const float* x, const void* w, int wdtype, co
   if (T > TS_ROWS) return cima_fail(CIMA_E_SIZE, "token_side_few: %d rows; this kernel takes at most %d", T, TS_ROWS);
   if (dim <= 0 || W <= 0 || vocab <= 0 || col < 0 || ldt < col + dim) return cima_fail(CIMA_E_SIZE, "token_side_few: %d values from column %d on exceed a table's rows of %d (width %d)", dim, col, ldt, W);
   if (act < 0 || act >= CIMA_ACT_COUNT) return cima_fail(CIMA_E_ARG, "token_side_few: activation code %d is unknown", act);
-  const int vec = W % (wdtype == CIMA_F32 ? 4 : 8) == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
-  const dim3 grid((unsigned)((dim + TS_OUTS * TS_WARPS - 1) / (TS_OUTS * TS_WARPS)));
+  const bool vec = W % (wdtype == CIMA_F32 ? 4 : 8) == 0 && (((uintptr_t)x | (uintptr_t)w) & 15) == 0;
+  const dim3 grid((unsigned)((dim + TS_OUTS - 1) / TS_OUTS));
   int rc;
-#define RUN(TW, TA) rc = cima_launch(k_token_side_few<TW, TA>, grid, dim3(TS_WARPS * 32), (size_t)0, stream, 1, x, (const TW*)w, (const TA*)table, ldt, tokens, col, (TA*)z, T, dim, W, vocab, act, vec)
+#define RUN_V(TW, TA, VEC) cima_launch(k_token_side_few<TW, TA, VEC>, grid, dim3(TS_WARPS * 32), (size_t)0, stream, 1, x, (const TW*)w, (const TA*)table, ldt, tokens, col, (TA*)z, T, dim, W, vocab, act)
+#define RUN(TW, TA) rc = vec ? RUN_V(TW, TA, true) : RUN_V(TW, TA, false)
   if (wdtype == CIMA_F32 && dtype == CIMA_F32) RUN(float, float);
   else if (wdtype == CIMA_BF16 && dtype == CIMA_BF16) RUN(__nv_bfloat16, __nv_bfloat16);
   else if (wdtype == CIMA_F32 && dtype == CIMA_BF16) RUN(float, __nv_bfloat16);
   else return cima_fail(CIMA_E_DTYPE, "token_side_few: weights of dtype code %d with rows of %d are not accepted", wdtype, dtype);
 #undef RUN
+#undef RUN_V
   return rc ? rc : cima_launch_result();
 }
 

@@ -89,7 +89,8 @@ _SIGNATURES = {
     "cima_embed_bigram": [_vp, _vp, _vp, _i, _vp, _i, _i, _i, _f, _i, ctypes.c_longlong, ctypes.c_longlong, _vp, _vp, _vp, _vp, _vp,
                           _i, _vp],
     "cima_recurrence": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
-    "cima_delta_prepare": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _vp],
+    "cima_delta_prepare": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _vp],
+    "cima_delta_rule": [_vp, _i, _vp, _i, _vp, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _i, _i, _i, _i, _i, _i, _i, _vp],
     "cima_group_rmsnorm_gate": [_vp, _vp, _vp, _i, _i, _vp, _i, _i, _i, _i, _i, _f, _i, _vp, _vp, _f, _vp],
     "cima_rms_mean": [_vp, _vp, _i, _vp, _i, _i, _f, _i, _vp],
     "cima_moe_route": [_vp, _i, _i, _i, _i, _i, _i, _f, _i, _i, _i, _i, _vp, _vp, _vp, _vp, _vp, _vp, _vp],
@@ -1013,7 +1014,7 @@ class Kernels:
                    beta: Optional[torch.Tensor] = None, decay: Optional[torch.Tensor] = None, gate=None) -> None:
         """A linear recurrence over the step's rows, sequence by sequence, with the state S [slots, heads, dim, vdim]
         (float32) carried on.  With ``decay`` [heads]: S <- d S + k v^T, o = S^T q, and q, k, v (one dtype) pass SiLU.
-        With ``g`` [T, heads * dim] (a decay a key channel) or [T, heads] (one a head) and ``beta`` [T, heads]: the gated delta rule on prepared float32 q and k
+        With ``g`` [T, heads * dim] and ``beta`` [T, heads]: the gated delta rule on prepared float32 q and k
         ([T, kv_heads * dim]).  With ``gate`` = (bias, lower), both float32 [heads * dim]: the gate rule, S <- diag(f) S +
         (1 - f) v^T with f = lower + (1 - lower) * sigmoid(k + bias) made from the projection that ``k`` holds, o = S^T silu(q),
         v as it is (q, k, v of one dtype, kv_heads = heads).  q, k, v may be column slices of wider matrices; out
@@ -1032,22 +1033,20 @@ class Kernels:
                               f"out {tuple(out.shape)} do not agree with {heads} heads on {kv_heads} of {dim} x {vdim}")
         if delta:
             self._need(g, "g", torch.float32, 2); self._need(beta, "beta", torch.float32, 2)
-            if q.dtype is not torch.float32 or tuple(g.shape) not in ((T, heads * dim), (T, heads)) or tuple(beta.shape) != (T, heads):
-                raise KernelError("recurrence: the delta rule takes float32 q and k, g [T, heads * dim] or [T, heads], and beta [T, heads]")
-            per_head = g.shape[1] == heads and dim > 1
+            if q.dtype is not torch.float32 or tuple(g.shape) != (T, heads * dim) or tuple(beta.shape) != (T, heads):
+                raise KernelError("recurrence: the delta rule takes float32 q and k, g [T, heads * dim] and beta [T, heads]")
         else:
             self._need(decay, "decay", torch.float32, 1)
             if decay.numel() != heads or q.dtype is not v.dtype:
                 raise KernelError("recurrence: the decay rule takes q, k, v of one dtype and one decay a head")
-        mode = 0 if not delta else (3 if per_head else 1)
-        if not self._admit(("recurrence[delta, a decay a head]" if mode == 3 else "recurrence[delta]") if delta else "recurrence[decay]",
+        if not self._admit("recurrence[delta]" if delta else "recurrence[decay]",
                            batch.n_seqs * heads * dim * vdim * 8 + T * (2 * kv_heads * dim * q.element_size() + heads * vdim * (4 + v.element_size())
-                                                                        + (g.shape[1] * 4 if delta else 0)),
+                                                                        + (heads * dim * 4 if delta else 0)),
                            (8.0 if delta else 5.0) * T * heads * dim * vdim): return
         self._check(self.lib.cima_recurrence(q.data_ptr(), q.stride(0), k.data_ptr(), k.stride(0), v.data_ptr(), v.stride(0),
                                              dtype_code(v.dtype), _ptr(g), _ptr(beta), _ptr(decay), state.data_ptr(),
                                              batch.seq_slot.data_ptr(), batch.seq_first_row.data_ptr(), out.data_ptr(), T,
-                                             batch.n_seqs, heads, kv_heads, dim, vdim, mode, self._stream()), "recurrence")
+                                             batch.n_seqs, heads, kv_heads, dim, vdim, int(delta), self._stream()), "recurrence")
 
     def _recurrence_gate(self, q, k, v, state, batch, out, heads, kv_heads, dim, vdim, bias, lower) -> None:
         self._need(state, "state", torch.float32, 4); self._need(out, "out", torch.float32, 2)
@@ -1072,30 +1071,54 @@ class Kernels:
                       qn: torch.Tensor, kn: torch.Tensor, g: torch.Tensor, beta: torch.Tensor, heads: int, kv_heads: int,
                       dim: int) -> None:
         """What the gated delta rule needs of a token besides v, in float32: q and k as unit vectors per head (q also
-        times dim^-1/2), g = exp(-exp(A_log[h]) * softplus(a + dt_bias)) per head and key channel (or, with a [T, heads] and
-        as many biases, per head), beta = sigmoid(b).
+        times dim^-1/2), g = exp(-exp(A_log[h]) * softplus(a + dt_bias)) per head and key channel, beta = sigmoid(b).
         ``qk`` [T, >= 2 * kv_heads * dim] holds q's heads and then k's; qk, a, b of one dtype, rows may be slices."""
         T = qk.shape[0]
         for n, t in (("qk", qk), ("a", a), ("b", b)):
             if t.dim() != 2 or t.stride(1) != 1 or t.shape[0] != T or t.dtype is not qk.dtype or not t.is_cuda:
                 raise KernelError(f"delta_prepare: {n} {tuple(t.shape)} {t.dtype} must be GPU rows of one dtype with unit column stride")
-        gdim = 1 if a.shape[1] == heads else dim                  # decays a head
-        for n, t, shape in (("qn", qn, (T, kv_heads * dim)), ("kn", kn, (T, kv_heads * dim)), ("g", g, (T, heads * gdim)),
+        for n, t, shape in (("qn", qn, (T, kv_heads * dim)), ("kn", kn, (T, kv_heads * dim)), ("g", g, (T, heads * dim)),
                             ("beta", beta, (T, heads))):
             self._need(t, n, torch.float32, 2)
             if tuple(t.shape) != shape:
                 raise KernelError(f"delta_prepare: {n} is {tuple(t.shape)}, expected {shape}")
         self._need(A_log, "A_log", torch.float32, 1); self._need(dt_bias, "dt_bias", torch.float32, 1)
-        if (qk.shape[1] < 2 * kv_heads * dim or a.shape[1] != heads * gdim or b.shape[1] != heads or A_log.numel() != heads
-                or dt_bias.numel() != heads * gdim):
+        if (qk.shape[1] < 2 * kv_heads * dim or a.shape[1] != heads * dim or b.shape[1] != heads or A_log.numel() != heads
+                or dt_bias.numel() != heads * dim):
             raise KernelError("delta_prepare: the inputs' widths do not agree with the heads and the key size")
-        if not self._admit("delta_prepare", T * (2 * kv_heads * dim + heads * gdim + heads) * (4 + qk.element_size())): return
-        for r0 in range(0, T, 65535):                             # a row a block of grid.y
-            r1 = min(T, r0 + 65535)
-            self._check(self.lib.cima_delta_prepare(qk[r0:r1].data_ptr(), qk.stride(0), a[r0:r1].data_ptr(), a.stride(0), b[r0:r1].data_ptr(),
-                                                    b.stride(0), dtype_code(qk.dtype), A_log.data_ptr(), dt_bias.data_ptr(), qn[r0:r1].data_ptr(),
-                                                    kn[r0:r1].data_ptr(), g[r0:r1].data_ptr(), beta[r0:r1].data_ptr(), r1 - r0, heads, kv_heads,
-                                                    dim, gdim, self._stream()), "delta_prepare")
+        if not self._admit("delta_prepare", T * (2 * kv_heads * dim + heads * dim + heads) * (4 + qk.element_size())): return
+        self._check(self.lib.cima_delta_prepare(qk.data_ptr(), qk.stride(0), a.data_ptr(), a.stride(0), b.data_ptr(), b.stride(0),
+                                                dtype_code(qk.dtype), A_log.data_ptr(), dt_bias.data_ptr(), qn.data_ptr(),
+                                                kn.data_ptr(), g.data_ptr(), beta.data_ptr(), T, heads, kv_heads, dim,
+                                                self._stream()), "delta_prepare")
+
+    DELTA_CHUNK_ROWS = 32       # a step that brings a sequence at least this many rows takes 16 tokens at a time (bfloat16)
+
+    def delta_rule(self, c: torch.Tensor, a: torch.Tensor, b: torch.Tensor, A_log: torch.Tensor, dt_bias: torch.Tensor, state: torch.Tensor, batch,
+                   out: torch.Tensor, heads: int, kv_heads: int, dim: int, vdim: int) -> None:
+        """The gated delta rule with one decay a head over the step's rows, the state S [slots, heads, dim, vdim] (float32) carried on:
+        with c's row = [q heads | k heads | v heads], q and k made unit vectors (q also times dim^-1/2), g = exp(-exp(A_log) softplus(a +
+        dt_bias)) and beta = sigmoid(b) of the row's numbers a and b, one of each a head,
+            S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+        everything behind the loads in float32 (the chunked form forms its products from exact bfloat16 rows and three-term splits of
+        float32).  c, a, b of one dtype (rows may be slices); out [T, heads * vdim] float32."""
+        self._need(state, "state", torch.float32, 4); self._need(out, "out", torch.float32, 2)
+        self._need(A_log, "A_log", torch.float32, 1); self._need(dt_bias, "dt_bias", torch.float32, 1)
+        T = batch.n_rows
+        for n, t, w in (("c", c, 2 * kv_heads * dim + heads * vdim), ("a", a, heads), ("b", b, heads)):
+            if t.dim() != 2 or t.stride(1) != 1 or tuple(t.shape) != (T, w) or not t.is_cuda or t.dtype is not c.dtype:
+                raise KernelError(f"delta_rule: {n} {tuple(t.shape)} {t.dtype} must be GPU rows of the step, {w} values wide, one dtype, unit column stride")
+        if tuple(state.shape[1:]) != (heads, dim, vdim) or tuple(out.shape) != (T, heads * vdim) or A_log.numel() != heads or dt_bias.numel() != heads:
+            raise KernelError(f"delta_rule: state {tuple(state.shape)}, out {tuple(out.shape)} and the heads' numbers do not agree with {heads} heads on "
+                              f"{kv_heads} of {dim} x {vdim}")
+        chunked = (c.dtype is torch.bfloat16 and int(getattr(batch, "max_rows", 0) or 0) >= self.DELTA_CHUNK_ROWS and dim <= 128 and dim % 8 == 0
+                   and vdim % 8 == 0 and c.stride(0) % 8 == 0 and c.data_ptr() % 16 == 0)
+        if not self._admit("delta_rule[16 tokens at a time]" if chunked else "delta_rule", batch.n_seqs * heads * dim * vdim * 8 + T * ((2 * kv_heads * dim + heads * (vdim + 2)) * c.element_size() + heads * vdim * 4),
+                           8.0 * T * heads * dim * vdim): return
+        self._check(self.lib.cima_delta_rule(c.data_ptr(), c.stride(0), a.data_ptr(), a.stride(0), b.data_ptr(), b.stride(0), dtype_code(c.dtype),
+                                             A_log.data_ptr(), dt_bias.data_ptr(), state.data_ptr(), batch.seq_slot.data_ptr(),
+                                             batch.seq_first_row.data_ptr(), out.data_ptr(), T, batch.n_seqs, heads, kv_heads, dim, vdim, int(chunked),
+                                             self._stream()), "delta_rule")
 
     def group_rmsnorm_gate(self, o: torch.Tensor, w: torch.Tensor, gate: Optional[torch.Tensor], out: torch.Tensor, groups: int,
                            eps: float, silu: bool = False, divisor=None) -> None:

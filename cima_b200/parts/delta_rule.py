@@ -17,7 +17,8 @@ with its activation run in the activations' dtype.  The ranks of the two low-ran
 Kind ``delta`` is the same but for two lines,
     g     = exp(-exp(A_log[h]) * softplus(W_a h + dt_bias))               one a head
     y     = W_o ( rms(o over a head's values) * w * silu(W_g h) )
-and its projections q | k | v | g | b | a are one product.
+and its projections q | k | v | g | b | a are one product; unit norms, decays, step sizes and the rule are one kernel behind the
+convolution.
 """
 from __future__ import annotations
 
@@ -207,7 +208,7 @@ class HeadDelta:
         return self.proj.nbytes() + self.out.nbytes() + self.conv.nbytes() + (2 * self.heads + self.vdim) * 4
 
     def scratch_row(self) -> int:
-        return 2 * self.channels + 4 * self.kd + 4 * self.vd + 8 * self.heads
+        return 2 * self.channels + 5 * self.vd + 2 * self.heads
 
     graph_safe = True
     takes_pending_norm = True
@@ -229,18 +230,14 @@ class HeadDelta:
 
     def _gated(self, h, batch, cache, site: int) -> torch.Tensor:
         K_, rt = self.rt.kernels, self.rt
-        rows, kd, C, H = h.shape[0], self.kd, self.channels, self.heads
+        rows, C, H = h.shape[0], self.channels, self.heads
         p = self.proj.store(h)                                        # [rows, q | k | v | g | b | a]
         gate, b, a = p[:, C:C + self.vd], p[:, C + self.vd:C + self.vd + H], p[:, C + self.vd + H:C + self.vd + 2 * H]
         c = rt.empty(rows, C)
         K_.short_conv(p[:, :C], self.conv.weight, cache.state[self.conv.state_name(site)] if self.taps > 1 else None, batch, c,
                       add_input=False, act=self.silu)
-        f32 = torch.float32
-        qn, kn = rt.empty(rows, kd, dtype=f32), rt.empty(rows, kd, dtype=f32)
-        g, beta = rt.empty(rows, H, dtype=f32), rt.empty(rows, H, dtype=f32)
-        K_.delta_prepare(c, a, b, self.A_log, self.dt_bias, qn, kn, g, beta, H, self.kv_heads, self.dim)
-        o = rt.empty(rows, self.vd, dtype=f32)
-        K_.recurrence(qn, kn, c[:, 2 * kd:], cache.state[self.state_name(site)], batch, o, H, self.kv_heads, self.dim, self.vdim, g=g, beta=beta)
+        o = rt.empty(rows, self.vd, dtype=torch.float32)
+        K_.delta_rule(c, a, b, self.A_log, self.dt_bias, cache.state[self.state_name(site)], batch, o, H, self.kv_heads, self.dim, self.vdim)
         gated = rt.empty(rows, self.vd)
         K_.group_rmsnorm_gate(o, self.norm, gate, gated, H, self.eps, silu=True)
         return gated

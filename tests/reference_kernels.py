@@ -460,7 +460,7 @@ def _recurrence(self, q, k, v, state, batch, out, heads, kv_heads, dim, vdim, g=
             S = state[slot, h].clone()
             for t in range(lo, hi):
                 if delta:
-                    S = (g[t].view(heads, dim)[h][:, None] if g.shape[1] == heads * dim else g[t, h]) * S
+                    S = g[t].view(heads, dim)[h][:, None] * S
                     u = beta[t, h] * (vf[t, h] - S.T @ kf[t, c])
                 else:
                     S = decay[h] * S
@@ -476,9 +476,18 @@ def _delta_prepare(self, qk, a, b, A_log, dt_bias, qn, kn, g, beta, heads, kv_he
     qf, kf = qk[:, :kd].float().view(T, kv_heads, dim), qk[:, kd:2 * kd].float().view(T, kv_heads, dim)
     qn.copy_((qf / torch.sqrt((qf * qf).sum(-1, keepdim=True) + 1e-6) * dim ** -0.5).view(T, kd))
     kn.copy_((kf / torch.sqrt((kf * kf).sum(-1, keepdim=True) + 1e-6)).view(T, kd))
-    step = torch.nn.functional.softplus(a.float() + dt_bias).view(T, heads, -1)         # a decay a key channel, or one a head
-    g.copy_(torch.exp(-torch.exp(A_log)[None, :, None] * step).view(T, -1))
+    step = torch.nn.functional.softplus(a.float() + dt_bias).view(T, heads, dim)
+    g.copy_(torch.exp(-torch.exp(A_log)[None, :, None] * step).view(T, heads * dim))
     beta.copy_(torch.sigmoid(b.float()))
+
+
+def _delta_rule(self, c, a, b, A_log, dt_bias, state, batch, out, heads, kv_heads, dim, vdim):
+    """By way of the two steps above, with the head's decay in every key channel."""
+    T, kd = c.shape[0], kv_heads * dim
+    qn, kn, g, beta = torch.empty(T, kd), torch.empty(T, kd), torch.empty(T, heads * dim), torch.empty(T, heads)
+    wide = lambda t: t.float().repeat_interleave(dim, dim=-1)
+    self.delta_prepare(c.float(), wide(a), b.float(), A_log, wide(dt_bias), qn, kn, g, beta, heads, kv_heads, dim)
+    self.recurrence(qn, kn, c[:, 2 * kd:], state, batch, out, heads, kv_heads, dim, vdim, g=g, beta=beta)
 
 
 def _group_rmsnorm_gate(self, o, w, gate, out, groups, eps, silu=False, divisor=None):
@@ -638,7 +647,7 @@ for _name, _fn in (("diff_combine", _diff_combine), ("scale_add_group_rmsnorm", 
     setattr(ReferenceKernels, _name, _fn)
 
 for _name, _fn in (("dyt", _dyt), ("dyt_add", _dyt_add), ("embed_bigram", _embed_bigram), ("recurrence", _recurrence),
-                   ("delta_prepare", _delta_prepare), ("group_rmsnorm_gate", _group_rmsnorm_gate), ("rms_mean", _rms_mean),
+                   ("delta_prepare", _delta_prepare), ("delta_rule", _delta_rule), ("group_rmsnorm_gate", _group_rmsnorm_gate), ("rms_mean", _rms_mean),
                    ("moe_route", _moe_route), ("moe_experts", _moe_experts)):
     setattr(ReferenceKernels, _name, _fn)
 

@@ -230,61 +230,114 @@ def test_head_products_with_a_gate(T, heads, N, Kd, ha, ho, dtype):
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 16, 24), (2, 1, 128, 64), (3, 3, 40, 8), (2, 2, 200, 33), (6, 2, 64, 65)])
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 16, 24), (2, 1, 128, 64), (3, 3, 40, 8), (2, 2, 200, 33), (6, 2, 64, 65), (2, 1, 1, 5), (1, 1, 13, 16)])
 def test_delta_rule_with_one_decay_a_head_in_every_cutting(heads, kv_heads, dim, vdim, dtype):
+    """From the convolved rows and slices of the projection on, against the rule in float64; whole, in pieces and token by token
+    from the carried state and beside another sequence: the same bits."""
     torch.manual_seed(dim)
-    T = 75
-    q, k = torch.randn(T, kv_heads, dim), torch.randn(T, kv_heads, dim)
-    q, k = q / q.norm(dim=-1, keepdim=True) * dim ** -0.5, k / k.norm(dim=-1, keepdim=True)
-    k[50] = k[3]                                                                     # a key that is written again
-    v = torch.randn(T, heads * vdim + 5).to(DT[dtype])
-    g, beta = torch.rand(T, heads) ** 0.3, torch.rand(T, heads)
-    g[20], beta[30] = 0.0, 1.0                                                       # a token that forgets all, one that writes all
-    want = plain_delta_rule(q.double(), k.double(), v[:, :heads * vdim].double().view(T, heads, vdim), beta.double(), g.double()).reshape(T, -1)
-    qd, kd, vd, gd, bd = (t.to(DEV) for t in (q.reshape(T, -1), k.reshape(T, -1), v, g, beta))
+    T, kd = 75, kv_heads * dim
+    c = torch.randn(T, 2 * kd + heads * vdim)
+    c[50, kd:2 * kd] = c[3, kd:2 * kd]                                               # a key that is written again
+    c[60, :2 * kd] = 0.0                                                             # rows without a direction
+    c = c.to(DT[dtype])
+    p = (torch.randn(T, 2 * heads + 7) * 2).to(DT[dtype])                            # b | a among other columns
+    p[20, 3 + heads:3 + 2 * heads], p[30, 3:3 + heads] = 60.0, 40.0                  # a token that forgets all, one that writes all
+    A, d = torch.randn(heads) * 1.5 - 1.0, torch.randn(heads)
+    x = c.double()
+    unit = lambda t: t / torch.sqrt((t * t).sum(-1, keepdim=True) + 1e-6)
+    z = p[:, 3 + heads:3 + 2 * heads].double() + d.double()
+    g = torch.exp(-torch.exp(A.double()) * (torch.clamp(z, min=0) + torch.log1p(torch.exp(-z.abs()))))
+    want = plain_delta_rule(unit(x[:, :kd].view(T, kv_heads, dim)) * dim ** -0.5, unit(x[:, kd:2 * kd].view(T, kv_heads, dim)),
+                            x[:, 2 * kd:].view(T, heads, vdim), torch.sigmoid(p[:, 3:3 + heads].double()), g).reshape(T, -1)
+    cd, pd, Ad, dd = c.to(DEV), p.to(DEV), A.to(DEV), d.to(DEV)
+
+    def call(rows, st, batch):
+        o = torch.empty(rows.stop - rows.start, heads * vdim, device=DEV)
+        K().delta_rule(cd[rows], pd[rows, 3 + heads:3 + 2 * heads], pd[rows, 3:3 + heads], Ad, dd, st, batch, o, heads, kv_heads, dim, vdim)
+        return o
 
     def run(counts):
-        st, out, r = torch.zeros(4, heads, dim, vdim, device=DEV), torch.empty(T, heads * vdim, device=DEV), 0
-        for c in counts:
-            o = torch.empty(c, heads * vdim, device=DEV)
-            K().recurrence(qd[r:r + c], kd[r:r + c], vd[r:r + c, :heads * vdim], st, entries_batch([c], [r], [2]), o, heads, kv_heads, dim, vdim,
-                           g=gd[r:r + c].contiguous(), beta=bd[r:r + c].contiguous())
-            out[r:r + c] = o
-            r += c
+        st, out, r = torch.zeros(4, heads, dim, vdim, device=DEV), [], 0
+        for n in counts:
+            out.append(call(slice(r, r + n), st, entries_batch([n], [r], [2])))
+            r += n
         assert float(st[[0, 1, 3]].abs().max()) == 0.0
-        return out, st
+        return torch.cat(out), st
 
     out, st = run([T])
     assert close(out, want, 5e-6)
+    bits = torch.equal if dtype == "float32" else lambda x, y: close(x, y, 5e-6)      # (long bfloat16 steps take 16 tokens at a time)
     for counts in ([2, 5, 33, 35], [1] * T, [16, 1, 58]):
         o2, s2 = run(counts)
-        assert torch.equal(o2, out) and torch.equal(s2, st)                          # the same bits in every cutting
-    # a decay a key channel that is the same in every channel says the same
-    st3, o3 = torch.zeros(4, heads, dim, vdim, device=DEV), torch.empty(T, heads * vdim, device=DEV)
-    K().recurrence(qd, kd, vd[:, :heads * vdim], st3, entries_batch([T], [0], [1]), o3, heads, kv_heads, dim, vdim,
-                   g=gd[:, :, None].expand(T, heads, dim).reshape(T, -1).contiguous(), beta=bd)
-    assert close(o3, out, 3e-6) and close(st3[1], st[2], 3e-6)
+        assert bits(o2, out) and bits(s2, st)
+    if dtype == "bfloat16":
+        (o1, s1), (o2, s2) = run([1] * T), run([31, 13, 31])
+        assert torch.equal(o1, o2) and torch.equal(s1, s2)
+    cd, pd = torch.cat([cd[:40], cd]), torch.cat([pd[:40], pd])
+    st2 = torch.zeros(4, heads, dim, vdim, device=DEV)
+    both = call(slice(0, 40 + T), st2, entries_batch([40, T], [0, 0], [3, 0]))
+    assert torch.equal(both[40:], out) and bits(both[:40], out[:40]) and torch.equal(st2[0], st[2])
 
 
-@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
-@pytest.mark.parametrize("T,heads,kv_heads,dim", [(1, 4, 2, 16), (70, 2, 1, 128), (9, 3, 3, 40), (300, 6, 2, 200)])
-def test_decays_a_head_from_slices_of_one_product(T, heads, kv_heads, dim, dtype):
-    torch.manual_seed(T)
-    p = (torch.randn(T, 2 * kv_heads * dim + 2 * heads + 6) * 2).to(DT[dtype])
-    A, d = torch.randn(heads), torch.randn(heads)
-    kd = kv_heads * dim
-    p[0, 2 * kd + heads:2 * kd + 2 * heads] = 60.0                                   # softplus' straight end
-    pd = p.to(DEV)
-    f = lambda n: torch.empty(T, n, device=DEV)
-    qn, kn, g, beta = f(kd), f(kd), f(heads), f(heads)
-    K().delta_prepare(pd[:, :2 * kd], pd[:, 2 * kd + heads:2 * kd + 2 * heads], pd[:, 2 * kd:2 * kd + heads], A.to(DEV), d.to(DEV), qn, kn, g, beta,
-                      heads, kv_heads, dim)
-    x = p.double()
-    z = x[:, 2 * kd + heads:2 * kd + 2 * heads] + d.double()
-    assert close(g, torch.exp(-torch.exp(A.double()) * (torch.clamp(z, min=0) + torch.log1p(torch.exp(-z.abs())))), 2e-6)
-    assert close(beta, torch.sigmoid(x[:, 2 * kd:2 * kd + heads]), 2e-6)
-    q = x[:, :kd].view(T, kv_heads, dim)
-    assert close(qn.view(T, kv_heads, dim), q / torch.sqrt((q * q).sum(-1, keepdim=True) + 1e-6) * dim ** -0.5, 2e-6)
+@pytest.mark.parametrize("heads,kv_heads,dim,vdim", [(4, 2, 16, 24), (2, 1, 128, 64), (3, 3, 40, 8), (6, 2, 64, 72), (1, 1, 8, 16), (12, 12, 128, 128), (2, 2, 96, 200)])
+def test_delta_rule_of_long_steps_sixteen_tokens_at_a_time(heads, kv_heads, dim, vdim):
+    """Ragged sequences of whole and broken chunks from used states against the rule in float64 and the token kernel: decays from
+    none to complete inside a chunk, keys written again, rows without a direction, alike keys one after another."""
+    torch.manual_seed(dim + vdim)
+    counts, slots = [33, 1, 160, 16, 47, 5], [3, 0, 5, 1, 7, 4]
+    T, kd, H = sum(counts), kv_heads * dim, heads
+    c = torch.randn(T, 2 * kd + H * vdim)
+    c[45:50, kd:2 * kd] = c[44, kd:2 * kd]
+    c[60, :2 * kd] = 0.0
+    c[70, kd:2 * kd] *= 30.0
+    c = c.bfloat16()
+    p = torch.randn(T, 2 * H) * 2
+    p[50:54, H:] = 80.0                                           # forget all, four tokens running
+    p[90:110, H:] = -30.0                                         # forget nothing
+    p[90:110, :H] = 30.0                                          # and write all
+    p = p.bfloat16()
+    A, d = torch.randn(H) * 1.5 - 1.0, torch.randn(H)
+    st0 = torch.randn(8, H, dim, vdim)
+    x = c.double()
+    unit = lambda t: t / torch.sqrt((t * t).sum(-1, keepdim=True) + 1e-6)
+    q, k, v = unit(x[:, :kd].view(T, kv_heads, dim)) * dim ** -0.5, unit(x[:, kd:2 * kd].view(T, kv_heads, dim)), x[:, 2 * kd:].view(T, H, vdim)
+    z = p[:, H:].double() + d.double()
+    g = torch.exp(-torch.exp(A.double()) * (torch.clamp(z, min=0) + torch.log1p(torch.exp(-z.abs()))))
+    beta = torch.sigmoid(p[:, :H].double())
+    want, want_st, r = torch.empty(T, H, vdim, dtype=torch.float64), st0.double(), 0
+    share = torch.arange(H) // (H // kv_heads)
+    for n, s in zip(counts, slots):
+        S = want_st[s]
+        for t in range(r, r + n):
+            kt, qt = k[t][share], q[t][share]
+            S = g[t][:, None, None] * S
+            u = beta[t][:, None] * (v[t] - torch.einsum("hdv,hd->hv", S, kt))
+            S = S + kt[:, :, None] * u[:, None, :]
+            want[t] = torch.einsum("hdv,hd->hv", S, qt)
+        want_st[s] = S
+        r += n
+    cd, pd, Ad, dd = c.to(DEV), p.to(DEV), A.to(DEV), d.to(DEV)
+    batch = entries_batch(counts, [9] * 6, slots)
+    assert batch.max_rows >= K().DELTA_CHUNK_ROWS
+    st, out = st0.to(DEV), torch.full((T, H * vdim), float("nan"), device=DEV)
+    K().delta_rule(cd, pd[:, H:], pd[:, :H], Ad, dd, st, batch, out, H, kv_heads, dim, vdim)
+    assert close(out, want.reshape(T, -1), 1e-5) and close(st, want_st, 1e-5)
+    assert torch.equal(st[[2, 6]].cpu(), st0[[2, 6]])
+    # token by token: the same but for rounding
+    few, out2, r = st0.to(DEV), torch.empty(T, H * vdim, device=DEV), 0
+    for n, s in zip(counts, slots):
+        for lo in range(r, r + n, 20):
+            hi = min(lo + 20, r + n)
+            o = torch.empty(hi - lo, H * vdim, device=DEV)
+            K().delta_rule(cd[lo:hi], pd[lo:hi, H:], pd[lo:hi, :H], Ad, dd, few, entries_batch([hi - lo], [9], [s]), o, H, kv_heads, dim, vdim)
+            out2[lo:hi] = o
+        r += n
+    assert close(out2, out, 1e-5) and close(few, st, 1e-5)
+    # beside others or alone: the same bits
+    alone = st0.to(DEV)
+    o = torch.empty(160, H * vdim, device=DEV)
+    K().delta_rule(cd[34:194], pd[34:194, H:], pd[34:194, :H], Ad, dd, alone, entries_batch([160], [9], [5]), o, H, kv_heads, dim, vdim)
+    assert torch.equal(o, out[34:194]) and torch.equal(alone[5], st[5])
 
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
