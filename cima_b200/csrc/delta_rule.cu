@@ -1,13 +1,13 @@
 // The gated delta rule with one decay a head, from the convolved rows to the read-out in one launch:
 //   q, k -> unit vectors, x / sqrt(sum x^2 + 1e-6);  q also times dim^(-1/2)
 //   g = exp(-exp(A_log[h]) * softplus(a + dt_bias[h])),  beta = sigmoid(b)
-//   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+//   S' = g S + k u^T  with  u = beta (v - g S^T k);  the read-out is S'^T q
 // S [dim, vdim] a head in float32, carried from token to token and from step to step (state [slots, heads, dim, vdim]).
 //
 // With raw rows q, k, their factors rq and rk, and P = S^T k, R = S^T q taken of the state as the token finds it:
 //   u = beta (v - g rk P);   o = g rq R + (rk rq k.q) u;   S <- g S + k (rk u)
 // so one pass over the state gives both sums, the read-out waits for no second pass, and the chain from token to token is one
-// product, a reduction over eight lanes and one update.
+// product, a reduction over sixteen lanes and one update.
 //
 // k_delta_rule walks the tokens one by one (a decode step; 32-bit rows; any size).  A block of four warps owns 32 neighbouring
 // value channels (columns of S) of one (sequence, head).  Sixteen lanes share four columns, each lane keeping a sixteenth of

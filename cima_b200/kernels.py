@@ -1099,7 +1099,7 @@ class Kernels:
         """The gated delta rule with one decay a head over the step's rows, the state S [slots, heads, dim, vdim] (float32) carried on:
         with c's row = [q heads | k heads | v heads], q and k made unit vectors (q also times dim^-1/2), g = exp(-exp(A_log) softplus(a +
         dt_bias)) and beta = sigmoid(b) of the row's numbers a and b, one of each a head,
-            S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+            S' = g S + k u^T  with  u = beta (v - g S^T k);  the read-out is S'^T q
         everything behind the loads in float32 (the chunked form forms its products from exact bfloat16 rows and three-term splits of
         float32).  c, a, b of one dtype (rows may be slices); out [T, heads * vdim] float32."""
         self._need(state, "state", torch.float32, 4); self._need(out, "out", torch.float32, 2)

@@ -12,11 +12,11 @@ The design in this file's notation (T tokens of one sequence, width W, t a posit
   x   <- x + rms(V (gelu_tanh(U x) * D_i[tok])) w3             D_i[tok]: layer i's part of the token's row of a side table
   logits = H (rms(x) w_f)
 
-  "latent_attention":  q = W_uq (rms(W_dq h) w_q);  c = rms(W_dkv h) w_c;  per head k = W_uk c, v = W_uv c;
+  "latent_attention":  q = W_uq (rms(W_dq h) w_q);  c = rms(W_dkv h) w_c;  keys W_uk c and values W_uv c, head by head;
         softmax over all earlier positions of q . k * scale;  heads concatenated times sigmoid(W_g h), then W_o
   "delta":  q, k, v = silu(taps(W h)) per channel over time;  q, k to unit length per head, q also times dim^(-1/2);
         beta = sigmoid(W_b h);  g = exp(-exp(A) softplus(W_a h + d)), one of each a head;
-        S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q;  rms(o) w per head times silu(W_g h), then W_o
+        S' = g S + k (beta (v - g S^T k))^T, read out as o = S'^T q;  rms(o) w per head times silu(W_g h), then W_o
   "attention":  q, k, v = W h + b;  q and k each rms-normed over all their heads at once, with a weight;
         score(i, j) = q_i . k_j * scale - m_h (i - j), m_h = 2^(-8 (h + 1) / H);  j within the window;
         v <- (1 - l) v + l v1 in every mixing layer but the first, v1 the first one's values;  then W_o
